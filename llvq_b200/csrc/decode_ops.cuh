@@ -16,24 +16,9 @@
 #include <cuda_fp16.h>
 
 #include "attn_splitkv.cuh"
+#include "warp_reduce.cuh"
 
 namespace llvq {
-
-__device__ __forceinline__ float warp_sum_f(float v) {
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-    return v;
-}
-__device__ __forceinline__ float warp_max_f(float v) {
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
-    return v;
-}
-__device__ __forceinline__ float warp_min_f(float v) {
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) v = fminf(v, __shfl_xor_sync(0xffffffffu, v, o));
-    return v;
-}
 
 // One CTA of 1024 threads, two f16 per thread and step (n even). x: residual stream, updated in
 // place when delta != nullptr; each thread keeps its elements in registers between the two passes.

@@ -14,6 +14,7 @@
 #include <cuda_fp16.h>
 
 #include "decode_tab.cuh"
+#include "head_pick.cuh"
 #include "kernels_generic.cuh"
 
 namespace llvq {
@@ -77,17 +78,6 @@ dequant_dense_kernel(const unsigned char* __restrict__ blob_g, const OffEntry* _
         }
     }
 }
-
-constexpr int kHeadThreads = 256;   // 8 warps, one embedding row per warp and step
-constexpr int kHeadMaxGrid = 1024;  // partial (value, row) pairs the pick kernel merges
-constexpr int kHeadMaxHidden = 8192;
-
-struct HeadBest {
-    float val;
-    int row;
-};
-
-__device__ __forceinline__ bool head_better(float v, int r, float bv, int br) { return v > bv || (v == bv && r < br); }
 
 // embed: [rows, hidden] f16 (16-byte aligned rows: hidden % 8 == 0); h: [hidden] f16.
 __global__ void __launch_bounds__(kHeadThreads)
@@ -202,37 +192,6 @@ __global__ void embed_gather_q8_kernel(const unsigned char* __restrict__ wq, con
         const size_t g = (size_t)row * gpr + (c >> 6);
         y[(size_t)blockIdx.x * hidden + c] =
             __float2half_rn(q8_deq(wq[(size_t)row * hidden + c], __half2float(scales[g]), __half2float(biases[g])));
-    }
-}
-
-// One CTA: merge the partials; the row index is reported with `row_offset` added (a vocabulary shard).
-__global__ void __launch_bounds__(kHeadMaxGrid)
-lm_head_pick_kernel(const HeadBest* __restrict__ partial, int n, long long row_offset, float* __restrict__ val_out,
-                    long long* __restrict__ idx_out) {
-    llvq_dependent_enter();
-    __shared__ HeadBest red[32];
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    HeadBest b = threadIdx.x < n ? partial[threadIdx.x] : HeadBest{-INFINITY, 0x7fffffff};
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-        const float v = __shfl_xor_sync(0xffffffffu, b.val, o);
-        const int r = __shfl_xor_sync(0xffffffffu, b.row, o);
-        if (head_better(v, r, b.val, b.row)) b = HeadBest{v, r};
-    }
-    if (lane == 0) red[warp] = b;
-    __syncthreads();
-    if (warp == 0) {
-        b = red[lane];
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            const float v = __shfl_xor_sync(0xffffffffu, b.val, o);
-            const int r = __shfl_xor_sync(0xffffffffu, b.row, o);
-            if (head_better(v, r, b.val, b.row)) b = HeadBest{v, r};
-        }
-        if (lane == 0) {
-            *val_out = b.val;
-            *idx_out = row_offset + (b.row == 0x7fffffff ? 0 : b.row);  // all-NaN logits: row 0
-        }
     }
 }
 

@@ -20,11 +20,13 @@ so it can be captured once in a CUDA graph and replayed.
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import Callable, List, Optional, Sequence
+from typing import Callable, Optional, Sequence
 
 import numpy as np
 
-KV_GROUP = 64  # llvq-llm/src/kvq.rs: groups of 64 along head_dim
+from .cache import KV_GROUP, Int8KvCache, kv_dequantize, kv_quantize  # noqa: F401
+from .registry import register
+from .token_loop import TokenLoop
 
 
 @dataclass
@@ -46,55 +48,9 @@ class Qwen3Config:
         return Qwen3Config(h, inter, qh, kvh, hd, layers, vocab)
 
 
-def kv_quantize(x):
-    """[..., head_dim] f16 -> (u8 codes, f16 scale, f16 bias), groups of 64 (kvq.rs:110-165)."""
-    import torch
-    g = x.float().unflatten(-1, (-1, KV_GROUP))
-    mn = g.amin(-1, keepdim=True)
-    mx = g.amax(-1, keepdim=True)
-    s = ((mx - mn) / 255.0).half()
-    mn = mn.half()
-    sf = s.float()
-    safe = torch.where(sf > 0, sf, torch.ones_like(sf))
-    t = (g - mn.float()) / safe
-    # candle's round() rounds halves away from zero (kvq.rs:149-152); torch.round would round them to even
-    q = torch.where(t >= 0, torch.floor(t + 0.5), -torch.floor(0.5 - t)).clamp_(0, 255)
-    q = torch.where(sf > 0, q, torch.zeros_like(q)).to(torch.uint8)
-    return q.flatten(-2), s.squeeze(-1), mn.squeeze(-1)
-
-
-def kv_dequantize(q, s, mn):
-    g = q.unflatten(-1, (-1, KV_GROUP)).float()
-    return (g * s.float().unsqueeze(-1) + mn.float().unsqueeze(-1)).half().flatten(-2)
-
-
 def _silu(x):
     import torch
     return torch.nn.functional.silu(x)
-
-
-class Int8KvCache:
-    """Fixed-capacity int8 KV cache of one block: [capacity, n_kv, head_dim] codes + per-group f16 scale/bias."""
-
-    def __init__(self, capacity: int, n_kv: int, head_dim: int, device):
-        import torch
-        ng = head_dim // KV_GROUP
-        self.q = [torch.zeros(capacity, n_kv, head_dim, dtype=torch.uint8, device=device) for _ in range(2)]
-        self.s = [torch.zeros(capacity, n_kv, ng, dtype=torch.float16, device=device) for _ in range(2)]
-        self.b = [torch.zeros(capacity, n_kv, ng, dtype=torch.float16, device=device) for _ in range(2)]
-
-    def write(self, which: int, pos, x):
-        """pos: int64 device tensor [L]; x: [L, n_kv, head_dim] f16."""
-        q, s, b = kv_quantize(x)
-        self.q[which].index_copy_(0, pos, q)
-        self.s[which].index_copy_(0, pos, s)
-        self.b[which].index_copy_(0, pos, b)
-
-    def read(self, which: int, end: Optional[int] = None):
-        return kv_dequantize(self.q[which][:end], self.s[which][:end], self.b[which][:end])
-
-    def bytes_per_position(self) -> int:
-        return 2 * (self.q[0][0].numel() + 2 * 2 * self.s[0][0].numel())
 
 
 class F16Embedding:
@@ -223,7 +179,7 @@ class TpGroup:
         return buf.view(self.world, L, n).permute(1, 0, 2).reshape(L, self.world * n)
 
 
-class FusedQwen3:
+class FusedQwen3(TokenLoop):
     """`gemv` / `gemm` / `head` hooks let the same loop run on fused projections or on a dense stand-in.
     With a `TpGroup` the handles in `blocks` are this rank's row shards and `embed_head` its vocabulary rows."""
 
@@ -240,7 +196,7 @@ class FusedQwen3:
         forward_rotated are in the reference (llvq-llm/src/fused_cuda.rs:362-402)."""
         import torch
         self.cfg, self.blocks, self.embed, self.final_norm = cfg, list(blocks), embed, final_norm
-        self.gemv, self.gemm, self.head, self.capacity, self.kv_int8 = gemv, gemm, head, capacity, kv_int8
+        self.gemv, self.gemm, self.head, self.kv_int8 = gemv, gemm, head, kv_int8
         self.rotate, self.gemv_rotated = rotate, gemv_rotated
         self.tp = tp if tp is not None and tp.world > 1 else None
         self.world = self.tp.world if self.tp else 1
@@ -248,32 +204,30 @@ class FusedQwen3:
         if self.tp:
             self.tp.check(cfg)
         self.h_loc, self.kv_loc, self.inter_loc = cfg.n_heads // self.world, cfg.n_kv // self.world, cfg.inter // self.world
-        self.prefill_chunk = prefill_chunk
         self.sdpa_from = 1 << 28  # bytes of f32 scores above which the prompt attention is the library's fused kernel
         # `embed`: the tied f16 embedding as a tensor, or an embedding object (F16Embedding, Q8Embedding)
         self.emb = embed if hasattr(embed, "lookup") else F16Embedding(embed, head)
         dev = self.emb.device
-        self.device = dev
+        self._init_loop(dev, capacity, prefill_chunk)
         v_loc = cfg.vocab // self.world
         self.emb_head = self.emb.shard(self.rank * v_loc, (self.rank + 1) * v_loc)
         self.head_offset = self.rank * v_loc
         inv = 1.0 / (cfg.rope_theta ** (torch.arange(0, cfg.head_dim, 2, device=dev, dtype=torch.float32) / cfg.head_dim))
         ang = torch.arange(capacity, device=dev, dtype=torch.float32)[:, None] * inv[None, :]
         self.cos, self.sin = ang.cos(), ang.sin()
-        self.positions = torch.arange(capacity, device=dev)
         if kv_int8:
             self.caches = [Int8KvCache(capacity, self.kv_loc, cfg.head_dim, dev) for _ in blocks]
         else:
             self.caches = [[torch.zeros(capacity, self.kv_loc, cfg.head_dim, dtype=torch.float16, device=dev) for _ in range(2)]
                            for _ in blocks]
-        self._graph = None
+        self._h = torch.zeros(cfg.hidden, dtype=torch.float16, device=dev)  # normalised state behind the last pick
         # `ops`: the C library (llvq_op_* kernels). With it and an int8 cache the token step runs the fused
         # decode kernels; without it every non-projection step is a torch op (the prefill always is).
         self.ops = ops if kv_int8 else None
         if self.ops is not None:
             f16 = dict(dtype=torch.float16, device=dev)
             hd, w = cfg.head_dim, self.world
-            self._x, self._h = torch.zeros(cfg.hidden, **f16), torch.zeros(cfg.hidden, **f16)
+            self._x = torch.zeros(cfg.hidden, **f16)
             # a projection that follows a norm or the SwiGLU product computes that step in its own staging
             # (llvq_gemv_norm_h / llvq_gemv_silu_h); the residual stream then alternates between _x and _x2
             self._x2 = torch.zeros(cfg.hidden, **f16)
@@ -297,9 +251,6 @@ class FusedQwen3:
             sms = torch.cuda.get_device_properties(dev).multi_processor_count
             self.attn_splits = max(1, min(-(-capacity // 256), (2 * sms) // self.kv_loc))
             self._attn_ws = torch.zeros(self.h_loc * self.attn_splits * (hd + 2), dtype=torch.float32, device=dev)
-        # the token and its position live in fixed device tensors: a captured graph keeps their addresses
-        self._tok = torch.zeros(1, dtype=torch.long, device=dev)
-        self._pos = torch.zeros(1, dtype=torch.long, device=dev)
         self._best = torch.zeros(2, dtype=torch.long, device=dev)        # (logit bits, row) of this rank's shard
         if self.ops is None:
             self._best_all = torch.zeros(2 * self.world, dtype=torch.long, device=dev)
@@ -381,17 +332,6 @@ class FusedQwen3:
             x = self._block(i, x, pos, end)
         return x
 
-    def prefill(self, prompt: Sequence[int]):
-        """Run the prompt through the blocks in chunks of `prefill_chunk` tokens (each chunk attends to the
-        cache written so far); returns the hidden state of the last prompt token, [1, hidden]."""
-        import torch
-        toks = torch.tensor(list(prompt), device=self.device, dtype=torch.long)
-        x = None
-        for lo in range(0, len(prompt), self.prefill_chunk):
-            hi = min(len(prompt), lo + self.prefill_chunk)
-            x = self.hidden(toks[lo:hi], self.positions[lo:hi], end=hi)
-        return x[-1:]
-
     def pick(self, h):
         """Greedy token of the normalised hidden state h [hidden] -> int64 [1] (device)."""
         val, idx = self.emb_head.pick(h, self.head_offset)
@@ -404,38 +344,25 @@ class FusedQwen3:
         vals = pairs[:, 0:1].contiguous().view(val.dtype)[:, 0]
         return pairs[:, 1].index_select(0, vals.argmax().reshape(1))  # first rank on ties = lowest row
 
+    def pick_last(self, x):
+        return self.pick(self._rms(x[-1:], self.final_norm)[0])
+
+    def logits(self, x):
+        """Full logits of hidden states (given tokens and diagnostics; the greedy loop uses `pick`)."""
+        return (self._rms(x, self.final_norm) @ self.emb.dense().t()).float()
+
+    def step_logits(self):
+        return (self._h[None] @ self.emb.dense().t()).float()[0]
+
     def logits_last(self, x):
-        """Full logits of the last row (diagnostics; the loop itself uses `pick`)."""
-        h = self._rms(x[-1:], self.final_norm)
-        return (h @ self.emb.dense().t()).float()[0]
+        return self.logits(x[-1:])[0]
 
-    # ---- the loop ----------------------------------------------------------------
-    def generate(self, prompt: Sequence[int], max_new: int, use_graph: bool = False) -> List[int]:
-        """Greedy continuation, `Qwen3::generate` (model.rs:1041-1073): prefill, then one token at a time."""
-        if max_new == 0:
-            return []
-        n = len(prompt)
-        if n + max_new > self.capacity:
-            raise ValueError(f"{n} prompt + {max_new} new tokens exceed the cache capacity {self.capacity}")
-        nxt = self.pick(self._rms(self.prefill(prompt), self.final_norm)[0])
-        out = [int(nxt)]
-        self.start_decode(nxt, n)
-        step = self._graph_step if use_graph else self._eager_step
-        while len(out) < max_new:
-            step()
-            out.append(int(self._tok))  # one scalar read-back per token, as model.rs:1064
-        return out
-
-    def start_decode(self, first_token, position: int) -> None:
-        """Point the token step at `first_token` (device scalar) sitting at `position` (in place: graph-safe)."""
-        self._tok.copy_(first_token.reshape(1))
-        self._pos.fill_(position)
-
+    # ---- the token step ----------------------------------------------------------
     def _eager_step(self):
         if self.ops is not None:
             return self._fused_step()
-        x = self.hidden(self._tok, self._pos)
-        self._tok.copy_(self.pick(self._rms(x[-1:], self.final_norm)[0]))
+        self._h.copy_(self._rms(self.hidden(self._tok, self._pos)[-1], self.final_norm))
+        self._tok.copy_(self.pick(self._h))
         self._pos += 1
 
     def _gemv(self, blk, name, x, out):
@@ -459,7 +386,7 @@ class FusedQwen3:
         L, cfg, tp = self.ops, self.cfg, self.tp
         st = C.c_void_p(torch.cuda.current_stream().cuda_stream)
         p = lambda t: C.c_void_p(t.data_ptr())
-        only = getattr(self, "_only", None)
+        only = self._only
         on = lambda phase: only is None or only == phase
         if on("embed"):
             self._x.copy_(self.emb.lookup(self._tok)[0])
@@ -537,66 +464,6 @@ class FusedQwen3:
             self._pos += 1
 
     PHASES = ("embed", "norm", "projections", "rope_kv_write", "attention", "swiglu", "gathers", "head")
-
-    def phase_split(self, reps: int = 10) -> dict:
-        """Device time of one token step by phase, in ms: every phase's launches (all layers) captured as a graph
-        of their own and replayed `reps` times between two events, at the current position and token. The
-        phases run apart here, so their sum leaves out what the whole step gains by overlapping a kernel's
-        preamble with its predecessor and adds nothing for the gaps between kernels of different phases. The
-        counterpart of the reference's per-phase token timing (llvq-llm/tests/phase_timing.rs). Not for a
-        tensor-parallel model under NCCL gathers (a collective inside a partial graph needs every rank)."""
-        import warnings
-        import torch
-        out = {}
-        tok0 = self._tok.clone()
-        for phase in self.PHASES:
-            if phase == "gathers" and not self.tp:
-                continue
-            self._only = phase
-            try:
-                side = torch.cuda.Stream()
-                side.wait_stream(torch.cuda.current_stream())
-                with torch.cuda.stream(side):
-                    self._fused_step()
-                torch.cuda.current_stream().wait_stream(side)
-                g = torch.cuda.CUDAGraph()
-                with warnings.catch_warnings():
-                    # a phase whose work the projections' kernels have absorbed captures nothing
-                    warnings.filterwarnings("ignore", message="The CUDA Graph is empty")
-                    with torch.cuda.graph(g):
-                        self._fused_step()
-                g.replay()
-                e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-                torch.cuda.synchronize()
-                e0.record()
-                for _ in range(reps):
-                    g.replay()
-                e1.record()
-                torch.cuda.synchronize()
-                out[phase] = e0.elapsed_time(e1) / reps
-            finally:
-                self._only = None
-                self._tok.copy_(tok0)
-        out["sum"] = sum(out.values())
-        return out
-
-    def _graph_step(self):
-        import torch
-        if self._graph is None:
-            tok0, pos0 = self._tok.clone(), self._pos.clone()
-            side = torch.cuda.Stream()
-            side.wait_stream(torch.cuda.current_stream())
-            with torch.cuda.stream(side):  # warm-up outside the capture (lazy initialisations)
-                self._eager_step()
-            torch.cuda.current_stream().wait_stream(side)
-            self._tok.copy_(tok0)
-            self._pos.copy_(pos0)
-            self._graph = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(self._graph):
-                self._eager_step()
-            self._tok.copy_(tok0)
-            self._pos.copy_(pos0)
-        self._graph.replay()
 
 
 def kernel_head(lib):
@@ -704,7 +571,8 @@ def synthetic_model(rt, cfg: Qwen3Config, config_id: int, capacity: int, seed: i
     return model, mats
 
 
-def load_archive_model(rt, ar, capacity: int, kv_int8: bool = True, fused_ops: bool = True, dense_prefill_from: int = 1024):
+def load_archive_model(rt, ar, capacity: int, kv_int8: bool = True, fused_ops: bool = True, dense_prefill_from: int = 1024,
+                       prefill_chunk: int = 2048):
     """A decode loop over a sealed container (`llvq_b200.archive.LvqArchive`): what the reference's fusedrun does
     with a `.llvq` file (llvq-llm/src/bin/fusedrun.rs, fused::load at llvq-llm/src/fused.rs:1147). The projections
     `model.layers.{i}.self_attn.{q,k,v,o}_proj.weight` / `mlp.{gate,up,down}_proj.weight` are uploaded straight
@@ -770,4 +638,10 @@ def load_archive_model(rt, ar, capacity: int, kv_int8: bool = True, fused_ops: b
     emb = raws["model.embed_tokens.weight"]
     return FusedQwen3(cfg, blocks, emb if isinstance(emb, Q8Embedding) else emb.contiguous(), raws["model.norm.weight"], capacity,
                       gemv=rt.forward, gemm=gemm, head=kernel_head(rt.lib), kv_int8=kv_int8, ops=rt.lib if fused_ops else None,
-                      rotate=rt.rotate, gemv_rotated=rt.forward_rotated)
+                      rotate=rt.rotate, gemv_rotated=rt.forward_rotated, prefill_chunk=prefill_chunk)
+
+
+@register("qwen3", "archive", ("float16",), aliases=("Qwen3ForCausalLM",))
+def _load_qwen3(config, ar, dtype, capacity, device, **options):
+    from .runtime import FusedRuntime
+    return load_archive_model(FusedRuntime(device), ar, capacity, **options)
