@@ -1,4 +1,5 @@
-"""ctypes binding of libllvq_b200.so — the same declarations as include/llvq_b200.h."""
+"""ctypes bindings of libllvq_b200.so and libllvq_dense.so — the same declarations as include/llvq_b200.h and
+include/llvq_dense.h."""
 from __future__ import annotations
 
 import ctypes as C
@@ -36,6 +37,24 @@ class ArchiveRawInfo(C.Structure):
     _fields_ = [("name", C.c_char_p), ("tag", C.c_int32), ("rank", C.c_int32), ("bits", C.c_int32), ("group", C.c_int32),
                 ("dims", C.POINTER(C.c_uint64)), ("data", C.POINTER(C.c_uint8)), ("data_bytes", C.c_uint64),
                 ("scales", C.POINTER(C.c_uint8)), ("biases", C.POINTER(C.c_uint8)), ("groups", C.c_uint64)]
+
+
+DN_F32, DN_BF16 = 0, 1
+DN_PLAIN, DN_EMBED, DN_NORM, DN_GLU = 0, 1, 2, 3
+
+
+class DenseGemv(C.Structure):
+    """llvq_dn_gemv_desc of include/llvq_dense.h."""
+    _fields_ = ([(n, C.c_int32) for n in ("dtype", "prologue", "n_out", "k", "ldw", "ld_table", "table_rows")] +
+                [(n, C.c_float) for n in ("alpha", "eps", "scale", "limit", "gain", "shift", "softcap")] +
+                [(n, C.c_void_p) for n in ("w", "bias", "y", "x", "delta", "norm_w", "a_out", "table", "token")])
+
+
+class DenseLatent(C.Structure):
+    """llvq_dn_latent of include/llvq_dense.h."""
+    _fields_ = ([(n, C.c_int32) for n in ("dtype", "heads", "dim", "rot_dim", "vdim", "kv_rank", "ldk", "slots", "ld", "rot_dims", "window", "splits")] +
+                [(n, C.c_float) for n in ("scale", "eps")] +
+                [(n, C.c_void_p) for n in ("ring", "cos_t", "sin_t", "uk", "uv", "kv_norm", "sink", "qlat", "part")])
 
 
 class LlvqError(RuntimeError):
@@ -119,25 +138,57 @@ _SIGNATURES = {
     "llvq_decode_indices": (C.c_int, [C.c_void_p, C.c_void_p, C.c_size_t, C.c_void_p, C.c_void_p, C.c_void_p]),
 }
 
-_lib = None
+_DENSE_SIGNATURES = {
+    "llvq_dn_last_error": (C.c_char_p, []),
+    "llvq_dn_launch_count": (C.c_uint64, []),
+    "llvq_dn_set_overlap": (C.c_int, [C.c_int32]),
+    "llvq_dn_gemv": (C.c_int, [C.POINTER(DenseGemv), C.c_void_p]),
+    "llvq_dn_head": (C.c_int, [C.POINTER(DenseGemv)] + [C.c_void_p] * 4),
+    "llvq_dn_latent_query": (C.c_int, [C.POINTER(DenseLatent)] + [C.c_void_p] * 4),
+    "llvq_dn_latent_decode": (C.c_int, [C.POINTER(DenseLatent)] + [C.c_void_p] * 2),
+    "llvq_dn_latent_value": (C.c_int, [C.POINTER(DenseLatent)] + [C.c_void_p] * 2),
+    "llvq_dn_latent_prefill": (C.c_int, [C.POINTER(DenseLatent), C.c_void_p, C.c_void_p, C.c_int32, C.c_void_p, C.c_int32, C.c_int32, C.c_int32,
+                                         C.c_int64, C.c_int64, C.c_void_p, C.c_int32, C.c_void_p]),
+    "llvq_dn_embed_rows": (C.c_int, [C.c_int32, C.c_void_p, C.c_int32, C.c_int32, C.c_void_p, C.c_int32, C.c_int32, C.c_float] + [C.c_void_p] * 3),
+    "llvq_dn_postnorm_rows": (C.c_int, [C.c_int32] + [C.c_void_p] * 4 + [C.c_float] * 2 + [C.c_void_p] * 2 + [C.c_int32] * 2 + [C.c_void_p]),
+    "llvq_dn_latent_rows": (C.c_int, [C.POINTER(DenseLatent), C.c_void_p, C.c_int32, C.c_int32, C.c_void_p, C.c_void_p, C.c_int64, C.c_int32, C.c_int32,
+                                      C.c_void_p]),
+    "llvq_dn_glu_rows": (C.c_int, [C.c_int32] + [C.c_void_p] * 3 + [C.c_int32] * 2 + [C.c_float] * 3 + [C.c_void_p]),
+    "llvq_dn_softcap": (C.c_int, [C.c_void_p, C.c_size_t, C.c_float, C.c_void_p]),
+}
+
+_loaded = {}
+
+
+def _load(lib: str, signatures: dict, build: bool) -> C.CDLL:
+    if lib not in _loaded:
+        path = _build.build(lib=lib) if build else lib
+        if not os.path.exists(path):
+            raise RuntimeError(f"{path} is missing: the CUDA library was not built; there is no fallback")
+        L = C.CDLL(path)
+        for name, (res, args) in signatures.items():
+            f = getattr(L, name)
+            f.restype = res
+            f.argtypes = args
+        _loaded[lib] = L
+    return _loaded[lib]
 
 
 def load(build: bool = True) -> C.CDLL:
     """Load the library (building it first when asked and stale). Fails loudly when it is missing."""
-    global _lib
-    if _lib is None:
-        path = _build.build() if build else _build.LIB
-        if not os.path.exists(path):
-            raise RuntimeError(f"{path} is missing: the CUDA library was not built; there is no fallback")
-        L = C.CDLL(path)
-        for name, (res, args) in _SIGNATURES.items():
-            f = getattr(L, name)
-            f.restype = res
-            f.argtypes = args
-        _lib = L
-    return _lib
+    return _load(_build.LIB, _SIGNATURES, build)
+
+
+def load_dense(build: bool = True) -> C.CDLL:
+    """The same for the dense-weight library."""
+    return _load(_build.DENSE_LIB, _DENSE_SIGNATURES, build)
 
 
 def check(status: int) -> None:
     if status != OK:
         raise LlvqError(status, load().llvq_last_error().decode())
+
+
+def check_dense(status: int) -> None:
+    if status != OK:
+        raise LlvqError(status, load_dense().llvq_dn_last_error().decode())

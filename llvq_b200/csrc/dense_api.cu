@@ -1,0 +1,314 @@
+// C ABI of libllvq_dense.so (include/llvq_dense.h): models with dense bf16 or f32 weights.
+#include <cuda_runtime.h>
+
+#include <algorithm>
+
+#include "../../include/llvq_dense.h"
+#include "dense_gemv.cuh"
+#include "dense_rows.cuh"
+#include "host_util.cuh"
+#include "latent_attn.cuh"
+#include "latent_prefill.cuh"
+
+using namespace llvq;
+
+static_assert(kHeadMaxGrid * sizeof(HeadBest) == 8192, "scratch of llvq_dn_head");
+
+namespace {
+
+constexpr size_t kMaxSmem = 227 * 1024;
+
+bool bad_dtype(int dt) { return dt != LLVQ_DN_F32 && dt != LLVQ_DN_BF16; }
+int elem_size(int dt) { return dt == LLVQ_DN_BF16 ? 2 : 4; }
+
+int sm_count() {
+    static std::atomic<int> cached{0};
+    int n = cached.load();
+    if (!n) {
+        int dev = 0;
+        cudaGetDevice(&dev);
+        if (cudaDeviceGetAttribute(&n, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess) n = 148;
+        cached = n;
+    }
+    return n;
+}
+
+int check_gemv(const llvq_dn_gemv_desc* d, const char* who) {
+    if (!d || bad_dtype(d->dtype)) return fail(kStatusInvalid, "%s: null descriptor or element type", who);
+    const int vn = 16 / elem_size(d->dtype);
+    if (!d->w || d->n_out <= 0 || d->k <= 0 || d->ldw < d->k || d->ldw % vn || ((uintptr_t)d->w & 15))
+        return fail(kStatusInvalid, "%s: matrix of %d x %d, row stride %d (a multiple of %d, 16-byte aligned)", who, d->n_out, d->k, d->ldw, vn);
+    switch (d->prologue) {
+        case LLVQ_DN_PLAIN:
+        case LLVQ_DN_GLU:
+            if (!d->x) return fail(kStatusInvalid, "%s: null activation", who);
+            break;
+        case LLVQ_DN_NORM:
+            if (!d->x || !d->norm_w || d->a_out == d->x) return fail(kStatusInvalid, "%s: norm needs x, norm_w and another buffer to store to", who);
+            break;
+        case LLVQ_DN_EMBED:
+            if (!d->table || !d->token || d->ld_table < d->k || d->table_rows <= 0) return fail(kStatusInvalid, "%s: embed needs a table and a token", who);
+            break;
+        default: return fail(kStatusInvalid, "%s: prologue %d", who, d->prologue);
+    }
+    return kStatusOk;
+}
+
+template <typename T, int PRO, bool HEAD>
+int launch_gemv(const DenseGemvArgs& a, int grid, cudaStream_t s) {
+    const int rows = a.n_out / grid + 1;
+    const size_t smem = ((size_t)a.ldw + (size_t)rows * a.kslices) * sizeof(float);
+    if (smem > kMaxSmem) return fail(kStatusUnsupported, "dn_gemv: %d columns need %zu bytes of shared memory", a.k, smem);
+    if (smem > 40 * 1024) {
+        const int st = ensure_dyn_smem((const void*)dense_gemv_kernel<T, PRO, HEAD>, smem);
+        if (st) return st;
+    }
+    CUDA_TRY(launch_dep(dense_gemv_kernel<T, PRO, HEAD>, dim3(grid), dim3(kGvThreads), smem, s, a));
+    g_launches++;
+    return kStatusOk;
+}
+
+template <typename T>
+int gemv_t(const llvq_dn_gemv_desc* d, HeadBest* best, int* grid_out, cudaStream_t s) {
+    DenseGemvArgs a{};
+    a.w = d->w, a.bias = d->bias, a.y = d->y, a.x = d->x, a.delta = d->delta, a.norm_w = d->norm_w, a.a_out = d->a_out;
+    a.table = d->table, a.token = (const long long*)d->token, a.best = best;
+    a.n_out = d->n_out, a.k = d->k, a.ldw = d->ldw, a.ld_table = d->ld_table, a.table_rows = d->table_rows;
+    a.alpha = d->alpha, a.eps = d->eps, a.scale = d->scale, a.limit = d->limit, a.gain = d->gain, a.shift = d->shift, a.cap = d->softcap;
+    // column slices: enough lanes for a row's vectors; rows of a CTA are shared by the row groups that are left
+    const int vecs = d->ldw / Vec16<T>::N;
+    a.kslices = vecs > 128 ? 8 : vecs > 64 ? 4 : vecs > 32 ? 2 : 1;
+    const int rows_step = kGvWarps / a.kslices * kGvRows;
+    int grid = std::min((d->n_out + rows_step - 1) / rows_step, 4 * sm_count());
+    if (best) grid = std::min(grid, kHeadMaxGrid);
+    if (grid_out) *grid_out = grid;
+    if (best) {
+        if (d->prologue == LLVQ_DN_NORM) return launch_gemv<T, kGvNorm, true>(a, grid, s);
+        if (d->prologue == LLVQ_DN_PLAIN) return launch_gemv<T, kGvPlain, true>(a, grid, s);
+        return fail(kStatusUnsupported, "dn_head: prologue %d (plain or norm)", d->prologue);
+    }
+    switch (d->prologue) {
+        case LLVQ_DN_PLAIN: return launch_gemv<T, kGvPlain, false>(a, grid, s);
+        case LLVQ_DN_EMBED: return launch_gemv<T, kGvEmbed, false>(a, grid, s);
+        case LLVQ_DN_NORM: return launch_gemv<T, kGvNorm, false>(a, grid, s);
+        default: return launch_gemv<T, kGvGlu, false>(a, grid, s);
+    }
+}
+
+int check_latent(const llvq_dn_latent* a, const char* who) {
+    if (!a || bad_dtype(a->dtype)) return fail(kStatusInvalid, "%s: null descriptor or element type", who);
+    const int vn = 16 / elem_size(a->dtype);
+    if (a->heads <= 0 || a->dim <= 0 || a->rot_dim < 0 || a->vdim <= 0 || a->kv_rank <= 0 || a->window <= 0)
+        return fail(kStatusInvalid, "%s: a size is not positive", who);
+    if (a->rot_dims < 0 || a->rot_dims > a->rot_dim || a->rot_dims % 2 || (a->rot_dims && (!a->cos_t || !a->sin_t)))
+        return fail(kStatusInvalid, "%s: %d rotated of %d dimensions", who, a->rot_dims, a->rot_dim);
+    if (a->ld % vn || a->ld < a->kv_rank + a->rot_dim || a->slots <= 0 || !a->ring || ((uintptr_t)a->ring & 15))
+        return fail(kStatusInvalid, "%s: cache rows of %d elements, %d slots", who, a->ld, a->slots);
+    if (a->ldk % vn || a->ldk < a->kv_rank) return fail(kStatusInvalid, "%s: row stride %d of the up projections", who, a->ldk);
+    return kStatusOk;
+}
+
+LatentRing ring_of(const llvq_dn_latent* a) { return LatentRing{a->ring, a->slots, a->ld}; }
+RotaryTable rot_of(const llvq_dn_latent* a) { return RotaryTable{a->cos_t, a->sin_t, a->rot_dims}; }
+
+template <typename T>
+int latent_query_t(const llvq_dn_latent* a, const float* q, const float* y_kv, const int64_t* pos, cudaStream_t s) {
+    LatentQueryArgs k{q, a->uk, a->qlat, y_kv, a->kv_norm, (const long long*)pos, ring_of(a), rot_of(a),
+                      a->heads, a->dim, a->rot_dim, a->kv_rank, a->ldk, a->eps};
+    const int slices = (a->ldk / Vec16<T>::N + 31) / 32;
+    CUDA_TRY(launch_dep(latent_query_kernel<T>, dim3(a->heads + (y_kv ? 1 : 0), slices), dim3(256), 0, s, k));
+    g_launches++;
+    return kStatusOk;
+}
+
+template <typename T>
+int latent_decode_t(const llvq_dn_latent* a, const int64_t* pos, cudaStream_t s) {
+    LatentDecodeArgs k{a->qlat, (const long long*)pos, a->part, a->part + (size_t)a->heads * a->splits * 2, ring_of(a), a->heads, a->kv_rank,
+                       a->window, a->scale};
+    const size_t smem = latent_decode_smem<T>(a->ld, a->kv_rank);
+    if (smem > kMaxSmem) return fail(kStatusUnsupported, "dn_latent_decode: cache rows of %d elements need %zu bytes of shared memory", a->ld, smem);
+    const int st = ensure_dyn_smem((const void*)latent_decode_kernel<T>, smem);
+    if (st) return st;
+    CUDA_TRY(launch_dep(latent_decode_kernel<T>, dim3((a->heads + kLdHeads - 1) / kLdHeads, a->splits), dim3(256), smem, s, k));
+    g_launches++;
+    return kStatusOk;
+}
+
+template <typename T>
+int latent_value_t(const llvq_dn_latent* a, float* ctx, cudaStream_t s) {
+    LatentValueArgs k{a->part, a->part + (size_t)a->heads * a->splits * 2, a->sink, a->uv, ctx, a->heads, a->vdim, a->kv_rank, a->ldk, a->splits};
+    const size_t smem = ((size_t)a->ldk + a->splits) * sizeof(float);
+    if (smem > kMaxSmem) return fail(kStatusUnsupported, "dn_latent_value: %d latent dimensions, %d splits", a->kv_rank, a->splits);
+    const int st = ensure_dyn_smem((const void*)latent_value_kernel<T>, smem);
+    if (st) return st;
+    CUDA_TRY(launch_dep(latent_value_kernel<T>, dim3(a->heads, (a->vdim + kLvRows - 1) / kLvRows), dim3(256), smem, s, k));
+    g_launches++;
+    return kStatusOk;
+}
+
+template <int NV, bool VEC>
+int prefill_mma(const LatentPrefillArgs& p, size_t smem, cudaStream_t s) {
+    const int st = ensure_dyn_smem((const void*)latent_prefill_mma_kernel<NV, VEC>, smem);
+    if (st) return st;
+    CUDA_TRY(launch_dep(latent_prefill_mma_kernel<NV, VEC>, dim3((p.n_q + kLpM - 1) / kLpM, p.heads, (p.vdim + NV * 8 - 1) / (NV * 8)),
+                        dim3(kLpThreads), smem, s, p));
+    g_launches++;
+    return kStatusOk;
+}
+
+template <typename T>
+int prefill_simt(const LatentPrefillArgs& p, cudaStream_t s) {
+    const size_t smem = (size_t)kLsWarps * (p.dim + p.rot_dim + p.vdim) * sizeof(float);
+    if (smem > kMaxSmem) return fail(kStatusUnsupported, "dn_latent_prefill: head sizes %d + %d, %d", p.dim, p.rot_dim, p.vdim);
+    const int st = ensure_dyn_smem((const void*)latent_prefill_simt_kernel<T>, smem);
+    if (st) return st;
+    CUDA_TRY(launch_dep(latent_prefill_simt_kernel<T>, dim3((p.n_q + kLsWarps - 1) / kLsWarps, p.heads), dim3(kLsWarps * 32), smem, s, p));
+    g_launches++;
+    return kStatusOk;
+}
+
+}  // namespace
+
+extern "C" {
+
+const char* llvq_dn_last_error(void) { return g_error.c_str(); }
+uint64_t llvq_dn_launch_count(void) { return g_launches.load(); }
+int llvq_dn_set_overlap(int32_t on) {
+    g_overlap_ops = on ? 1 : 0;
+    return kStatusOk;
+}
+
+int llvq_dn_gemv(const llvq_dn_gemv_desc* d, llvq_dn_stream stream) {
+    const int st = check_gemv(d, "dn_gemv");
+    if (st) return st;
+    if (!d->y) return fail(kStatusInvalid, "dn_gemv: null result");
+    return d->dtype == LLVQ_DN_BF16 ? gemv_t<bf16>(d, nullptr, nullptr, (cudaStream_t)stream) : gemv_t<float>(d, nullptr, nullptr, (cudaStream_t)stream);
+}
+
+int llvq_dn_head(const llvq_dn_gemv_desc* d, void* scratch, float* val_out, int64_t* idx_out, llvq_dn_stream stream) {
+    int st = check_gemv(d, "dn_head");
+    if (st) return st;
+    if (!scratch || !val_out || !idx_out) return fail(kStatusInvalid, "dn_head: null argument");
+    cudaStream_t s = (cudaStream_t)stream;
+    int grid = 0;
+    st = d->dtype == LLVQ_DN_BF16 ? gemv_t<bf16>(d, (HeadBest*)scratch, &grid, s) : gemv_t<float>(d, (HeadBest*)scratch, &grid, s);
+    if (st) return st;
+    CUDA_TRY(launch_dep(lm_head_pick_kernel, dim3(1), dim3(kHeadMaxGrid), 0, s, (const HeadBest*)scratch, grid, 0ll, val_out, (long long*)idx_out));
+    g_launches++;
+    return kStatusOk;
+}
+
+int llvq_dn_latent_query(const llvq_dn_latent* a, const float* q, const float* y_kv, const int64_t* pos, llvq_dn_stream stream) {
+    const int st = check_latent(a, "dn_latent_query");
+    if (st) return st;
+    if (!q || !pos || !a->uk || !a->qlat || (y_kv && !a->kv_norm)) return fail(kStatusInvalid, "dn_latent_query: null argument");
+    return a->dtype == LLVQ_DN_BF16 ? latent_query_t<bf16>(a, q, y_kv, pos, (cudaStream_t)stream) : latent_query_t<float>(a, q, y_kv, pos, (cudaStream_t)stream);
+}
+
+int llvq_dn_latent_decode(const llvq_dn_latent* a, const int64_t* pos, llvq_dn_stream stream) {
+    const int st = check_latent(a, "dn_latent_decode");
+    if (st) return st;
+    if (!pos || !a->qlat || !a->part || a->splits < 1 || a->splits > 4096) return fail(kStatusInvalid, "dn_latent_decode: null argument or %d splits", a->splits);
+    if (a->window > a->slots) return fail(kStatusInvalid, "dn_latent_decode: a window of %d over %d slots", a->window, a->slots);
+    return a->dtype == LLVQ_DN_BF16 ? latent_decode_t<bf16>(a, pos, (cudaStream_t)stream) : latent_decode_t<float>(a, pos, (cudaStream_t)stream);
+}
+
+int llvq_dn_latent_value(const llvq_dn_latent* a, float* ctx, llvq_dn_stream stream) {
+    const int st = check_latent(a, "dn_latent_value");
+    if (st) return st;
+    if (!ctx || !a->part || !a->uv || a->splits < 1 || a->splits > 4096) return fail(kStatusInvalid, "dn_latent_value: null argument or %d splits", a->splits);
+    return a->dtype == LLVQ_DN_BF16 ? latent_value_t<bf16>(a, ctx, (cudaStream_t)stream) : latent_value_t<float>(a, ctx, (cudaStream_t)stream);
+}
+
+int llvq_dn_latent_prefill(const llvq_dn_latent* a, const void* q, const void* kv, int32_t ld_kv, const void* kr, int32_t ld_kr,
+                           int32_t n_q, int32_t n_k, int64_t pos0, int64_t key0, void* out, int32_t kernel, llvq_dn_stream stream) {
+    const int st = check_latent(a, "dn_latent_prefill");
+    if (st) return st;
+    if (!q || !kv || !kr || !out) return fail(kStatusInvalid, "dn_latent_prefill: null argument");
+    if (n_q <= 0 || n_k <= 0 || pos0 < 0 || key0 < 0 || key0 > pos0 || pos0 + n_q > key0 + n_k || ld_kv < a->heads * (a->dim + a->vdim) || ld_kr < a->rot_dim)
+        return fail(kStatusInvalid, "dn_latent_prefill: %d queries at %lld over %d keys at %lld", n_q, (long long)pos0, n_k, (long long)key0);
+    LatentPrefillArgs p{q, kv, kr, a->sink, out, rot_of(a), pos0, key0, n_q, n_k, a->heads, a->dim, a->rot_dim, a->vdim, ld_kv, ld_kr,
+                        a->window, a->scale};
+    cudaStream_t s = (cudaStream_t)stream;
+    if (a->dtype == LLVQ_DN_F32) return prefill_simt<float>(p, s);
+    const int nv = a->vdim <= 64 ? 8 : a->vdim <= 128 ? 16 : 32;
+    const size_t smem = latent_prefill_smem(a->dim, a->rot_dim, nv);
+    if (kernel == 1 || smem > kMaxSmem) return prefill_simt<bf16>(p, s);
+    const bool vec = !((a->dim | a->rot_dim | a->vdim | ld_kv | ld_kr) & 7) && !(((uintptr_t)q | (uintptr_t)kv | (uintptr_t)kr | (uintptr_t)out) & 15);
+    if (nv == 8) return vec ? prefill_mma<8, true>(p, smem, s) : prefill_mma<8, false>(p, smem, s);
+    if (nv == 16) return vec ? prefill_mma<16, true>(p, smem, s) : prefill_mma<16, false>(p, smem, s);
+    return vec ? prefill_mma<32, true>(p, smem, s) : prefill_mma<32, false>(p, smem, s);
+}
+
+int llvq_dn_embed_rows(int32_t dtype, const void* table, int32_t ld, int32_t table_rows, const int64_t* tokens, int32_t rows, int32_t n,
+                       float scale, float* x, void* xt, llvq_dn_stream stream) {
+    if (bad_dtype(dtype) || !table || !tokens || !x || rows <= 0 || n <= 0 || ld < n || table_rows <= 0) return fail(kStatusInvalid, "dn_embed_rows: bad argument");
+    cudaStream_t s = (cudaStream_t)stream;
+    if (dtype == LLVQ_DN_BF16)
+        CUDA_TRY(launch_dep(embed_rows_kernel<bf16>, dim3(rows), dim3(kRowThreads), 0, s, (const bf16*)table, ld, table_rows, (const long long*)tokens, scale, x, (bf16*)xt, n));
+    else
+        CUDA_TRY(launch_dep(embed_rows_kernel<float>, dim3(rows), dim3(kRowThreads), 0, s, (const float*)table, ld, table_rows, (const long long*)tokens, scale, x, (float*)xt, n));
+    g_launches++;
+    return kStatusOk;
+}
+
+int llvq_dn_postnorm_rows(int32_t dtype, const float* x, const void* y, const float* bias, const float* w, float alpha, float eps,
+                          void* xt, float* out, int32_t rows, int32_t n, llvq_dn_stream stream) {
+    if (bad_dtype(dtype) || !x || !w || rows <= 0 || n <= 0 || (size_t)n * 4 > kMaxSmem - 1024) return fail(kStatusInvalid, "dn_postnorm_rows: bad argument");
+    cudaStream_t s = (cudaStream_t)stream;
+    const size_t smem = (size_t)n * 4;
+    const void* f = dtype == LLVQ_DN_BF16 ? (const void*)postnorm_rows_kernel<bf16> : (const void*)postnorm_rows_kernel<float>;
+    if (smem > 40 * 1024) {
+        const int st = ensure_dyn_smem(f, smem);
+        if (st) return st;
+    }
+    if (dtype == LLVQ_DN_BF16)
+        CUDA_TRY(launch_dep(postnorm_rows_kernel<bf16>, dim3(rows), dim3(kRowThreads), smem, s, x, (const bf16*)y, bias, w, alpha, eps, (bf16*)xt, out, n));
+    else
+        CUDA_TRY(launch_dep(postnorm_rows_kernel<float>, dim3(rows), dim3(kRowThreads), smem, s, x, (const float*)y, bias, w, alpha, eps, (float*)xt, out, n));
+    g_launches++;
+    return kStatusOk;
+}
+
+int llvq_dn_latent_rows(const llvq_dn_latent* a, const void* y, int32_t ldy, int32_t q_rank, const float* q_norm, void* cq,
+                        int64_t pos0, int32_t rows, int32_t store_kv, llvq_dn_stream stream) {
+    const int st = check_latent(a, "dn_latent_rows");
+    if (st) return st;
+    if (!y || !q_norm || !cq || q_rank <= 0 || rows <= 0 || rows > a->slots || pos0 < 0 || (store_kv && !a->kv_norm) ||
+        ldy < q_rank + (store_kv ? a->kv_rank + a->rot_dim : 0))
+        return fail(kStatusInvalid, "dn_latent_rows: %d rows into %d slots, row stride %d", rows, a->slots, ldy);
+    LatentRing ring = ring_of(a);
+    if (!store_kv) ring.rows = nullptr;
+    cudaStream_t s = (cudaStream_t)stream;
+    if (a->dtype == LLVQ_DN_BF16)
+        CUDA_TRY(launch_dep(latent_rows_kernel<bf16>, dim3(rows), dim3(kRowThreads), 0, s, (const bf16*)y, ldy, q_rank, q_norm, (bf16*)cq, a->kv_norm, a->kv_rank,
+                            a->rot_dim, rot_of(a), (long long)pos0, ring, a->eps));
+    else
+        CUDA_TRY(launch_dep(latent_rows_kernel<float>, dim3(rows), dim3(kRowThreads), 0, s, (const float*)y, ldy, q_rank, q_norm, (float*)cq, a->kv_norm, a->kv_rank,
+                            a->rot_dim, rot_of(a), (long long)pos0, ring, a->eps));
+    g_launches++;
+    return kStatusOk;
+}
+
+int llvq_dn_glu_rows(int32_t dtype, const void* gate_up, const float* bias, void* out, int32_t rows, int32_t n, float limit, float gain,
+                     float shift, llvq_dn_stream stream) {
+    if (bad_dtype(dtype) || !gate_up || !out || rows <= 0 || n <= 0) return fail(kStatusInvalid, "dn_glu_rows: bad argument");
+    cudaStream_t s = (cudaStream_t)stream;
+    const dim3 grid(rows, std::max(1, std::min(8, n / (4 * kRowThreads))));
+    if (dtype == LLVQ_DN_BF16)
+        CUDA_TRY(launch_dep(glu_rows_kernel<bf16>, grid, dim3(kRowThreads), 0, s, (const bf16*)gate_up, bias, (bf16*)out, n, limit, gain, shift));
+    else
+        CUDA_TRY(launch_dep(glu_rows_kernel<float>, grid, dim3(kRowThreads), 0, s, (const float*)gate_up, bias, (float*)out, n, limit, gain, shift));
+    g_launches++;
+    return kStatusOk;
+}
+
+int llvq_dn_softcap(float* y, size_t n, float cap, llvq_dn_stream stream) {
+    if (!y || !n || !(cap > 0.0f)) return fail(kStatusInvalid, "dn_softcap: bad argument");
+    const int grid = (int)std::min<size_t>((n + kRowThreads - 1) / kRowThreads, 4096);
+    CUDA_TRY(launch_dep(softcap_kernel, dim3(grid), dim3(kRowThreads), 0, (cudaStream_t)stream, y, n, cap));
+    g_launches++;
+    return kStatusOk;
+}
+
+}  // extern "C"
