@@ -69,9 +69,19 @@ def latent_queries(h, w, p, mx, eps, positions):
     return q[..., :dim], rotate(q[..., dim:], positions, mx["rot"]["dims"], mx["rot"]["base"])
 
 
+def attend(qn, qr, c, kr, uk, uv, scale, visible, sink):
+    """Queries [I, H, dim] and [I, H, rot_dim], cached latents [J, kv_rank] and rotated key parts [J, rot_dim], one
+    visible[i, j] per pair -> [I, H, vdim]. uk: [H dim, kv_rank], uv: [H vdim, kv_rank], both head by head."""
+    H, n = qn.shape[1], c.shape[0]
+    k = (c @ uk.T).reshape(n, H, -1)
+    v = (c @ uv.T).reshape(n, H, -1)
+    scores = (torch.einsum("ihd,jhd->hij", qn, k) + torch.einsum("ihd,jd->hij", qr, kr)) * scale
+    return torch.einsum("hij,jhd->ihd", softmax_with_sink(scores, visible, sink), v)
+
+
 def latent_attention(h, latents, layer, w, p, mx, eps):
     """h [T, D]; `latents` keeps every layer's (latent, rotated key part) for the layers that read them again."""
-    n, H = h.shape[0], mx["heads"]
+    n = h.shape[0]
     positions = torch.arange(n)
     src = mx.get("kv_from")
     if src is None:
@@ -79,12 +89,9 @@ def latent_attention(h, latents, layer, w, p, mx, eps):
         src = layer
     c, kr = latents[src]
     qn, qr = latent_queries(h, w, p, mx, eps, positions)
-    k = (c @ w[p + ".uk"].T).reshape(n, H, mx["dim"])
-    v = (c @ w[p + ".uv"].T).reshape(n, H, mx["vdim"])
-    scores = (torch.einsum("ihd,jhd->hij", qn, k) + torch.einsum("ihd,jd->hij", qr, kr)) * mx["scale"]
     mask = mx.get("mask")
-    a = softmax_with_sink(scores, window_mask(n, mask["size"] if mask else None), w.get(p + ".sink"))
-    return torch.einsum("hij,jhd->ihd", a, v).reshape(n, -1) @ w[p + ".o"].T
+    y = attend(qn, qr, c, kr, w[p + ".uk"], w[p + ".uv"], mx["scale"], window_mask(n, mask["size"] if mask else None), w.get(p + ".sink"))
+    return y.reshape(n, -1) @ w[p + ".o"].T
 
 
 def clamped_gated_mlp(h, w, p, limit):
@@ -129,7 +136,7 @@ def random_model(cfg, seed=0, weight_scale=1.0):
     def vec(name, n, mean=0.0, std=0.3):
         w[name] = (mean + std * torch.randn(n, generator=g)).bfloat16()
 
-    w["embed"] = torch.randn(cfg["vocab"], D, generator=g).bfloat16()
+    w["embed"] = (0.3 * torch.randn(cfg["vocab"], D, generator=g)).bfloat16()  # logits of a few units
     for i, layer in enumerate(cfg["layers"]):
         mx, p = layer["mixer"], f"l{i}.mix"
         H = mx["heads"]
