@@ -733,6 +733,189 @@ def tp_block(args, rt, torch, dist, world, rank, local_rank):
                                        "gathered_rows_bit_exact": gathered_ok}}
 
 
+def latent_config(shape: str, layers: int, window: int):
+    """A latent-attention model of the named model's width, feed-forward, heads and vocabulary; every third layer reads
+    the cache of the layer before it."""
+    from llvq_b200 import latent, synth
+    h, inter, qh, _, hd, _, vocab = synth.MODEL_SHAPES[shape]
+    dim, rot, q_rank, kv_rank = hd, 64, 1536, 512
+
+    def layer(i):
+        a = latent.LatentAttentionConfig(qh, dim, rot, hd, q_rank, kv_rank, (dim + rot) ** -0.5, 10000.0, rot, window, i - 1 if i % 3 == 2 else None)
+        return latent.LatentLayerConfig(a, latent.GatedMlpConfig(inter, 7.0))
+    return latent.LatentConfig(vocab, h, 1e-5, 2.0, 1.0, 30.0, [layer(i) for i in range(layers)])
+
+
+def latent_model(torch, cfg, capacity, seed=1):
+    """Random bf16 weights drawn on the device, fan-in scaled."""
+    from llvq_b200 import latent
+    g = torch.Generator(device="cuda").manual_seed(seed)
+    shapes = {"embed": (cfg.vocab, cfg.width), "final.norm": (cfg.width,)}
+    for i, l in enumerate(cfg.layers):
+        a, p, m = l.attn, f"l{i}.mix", f"l{i}.mlp"
+        shapes.update({f"l{i}.norm1": (cfg.width,), f"l{i}.norm2": (cfg.width,), p + ".dq": (a.q_rank, cfg.width), p + ".dq.norm": (a.q_rank,),
+                       p + ".uq": (a.heads * (a.dim + a.rot_dim), a.q_rank), p + ".dkv": (a.kv_rank + a.rot_dim, cfg.width),
+                       p + ".dkv.norm": (a.kv_rank,), p + ".uk": (a.heads * a.dim, a.kv_rank), p + ".uv": (a.heads * a.vdim, a.kv_rank),
+                       p + ".sink": (a.heads,), p + ".o": (cfg.width, a.heads * a.vdim), m + ".gate": (l.mlp.ff, cfg.width), m + ".gate.b": (l.mlp.ff,),
+                       m + ".up": (l.mlp.ff, cfg.width), m + ".up.b": (l.mlp.ff,), m + ".down": (cfg.width, l.mlp.ff), m + ".down.b": (cfg.width,)})
+
+    def tensor(name):
+        s = shapes[name]
+        w = torch.randn(*s, generator=g, device="cuda", dtype=torch.float32)
+        if name.endswith((".dq.norm", ".dkv.norm")):
+            return (1 + 0.02 * w).bfloat16()
+        return (w * (s[1] ** -0.5 if len(s) == 2 else 0.02)).bfloat16()
+    return latent.LatentLM(cfg, tensor, "bfloat16", capacity, torch.device("cuda"))
+
+
+def run_latent(args):
+    """--latent: prefill and greedy decode of latent-attention models (bf16, random weights) at the layer sizes of
+    qwen3-4b / 8b / 14b, beside the archive-code Qwen3 model of the same size on the same tokens, with the time of each
+    kernel against its roofline: bytes over the measured copy bandwidth, for the prompt attention and the matrix
+    products FLOPs over the measured bf16 throughput. Token-step phases are replayed apart (all layers; the weights of a
+    phase exceed L2 where `l2` says so); prompt kernels rotate over operand sets larger than L2. Device-timed."""
+    import ctypes as C
+    import gc
+    import torch
+    from llvq_b200 import FusedRuntime, _lib
+    from llvq_b200.model import Qwen3Config, synthetic_model
+    peak = measured_peaks()[0]
+    tflops = 1590.0
+    if os.path.exists(os.path.join(ROOT, "MEASURED_PEAKS.json")):
+        tflops = float(json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))["bf16_tflops"])
+    n_layers, window, prompt_len, new_tokens = args.latent_layers, args.window, 2048, 96
+    torch.cuda.set_device(0)
+    sampler = ClockSampler(0)
+    sampler.start()
+
+    def event_ms(fn, reps):
+        for _ in range(3):
+            fn(0)
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        e0.record()
+        for k in range(reps):
+            fn(k)
+        e1.record()
+        torch.cuda.synchronize()
+        return e0.elapsed_time(e1) / reps
+
+    def loop_times(model):
+        prompt = np.random.default_rng(5).integers(0, model.cfg.vocab, prompt_len).tolist()
+        model.generate(prompt, 4, use_graph=True)
+        pre = event_ms(lambda k: model.prefill(prompt), max(args.steps // 2, 3))
+        model.start_decode(model.pick_last(model.prefill(prompt)), prompt_len)
+        dec = event_ms(lambda k: model._graph_step(), new_tokens - 8)
+        return {"prefill_ms": round(pre, 3), "prefill_tok_per_s": round(prompt_len / pre * 1e3), "decode_ms_per_token": round(dec, 4),
+                "decode_tok_per_s": round(1e3 / dec, 1)}
+
+    def phases(model, sizes):
+        model._pos.fill_(window - 1)  # `window` positions are read by both models' attention
+        out = {}
+        for name, ms in model.phase_split(reps=20).items():
+            b = sizes.get(name)
+            out[name] = {"us_per_layer": round(ms * 1e3 / n_layers, 2)} if name != "head" else {"us": round(ms * 1e3, 2)}
+            if b:
+                out[name].update(GBps=round(b / ms / 1e6, 1), frac=round(b / ms / 1e6 / peak, 4), l2="weights exceed L2" if b > 126e6 else "fits L2")
+        return out
+
+    results = []
+    for shape in args.latent_shapes.split(","):
+        cfg = latent_config(shape, n_layers, window)
+        m = latent_model(torch, cfg, prompt_len + 128)
+        lib, a, L, lat = m.lib, cfg.layers[0].attn, m.layers[0], m._lat[0]
+        launches = lib.llvq_dn_launch_count()
+        r = {"shape": shape, "layers": n_layers, "width": cfg.width, "ff": cfg.layers[0].mlp.ff, "heads": a.heads, "window": window,
+             "head_dims": [a.dim, a.rot_dim, a.vdim], "ranks": [a.q_rank, a.kv_rank], "latent": loop_times(m)}
+        wb = lambda *names: sum(x[n].w.numel() * 2 for x in m.layers for n in names)
+        up = [(x["ukv"].ld * 2 * c.attn.heads * c.attn.dim, x["ukv"].ld * 2 * c.attn.heads * c.attn.vdim) for x, c in zip(m.layers, cfg.layers)]
+        r["latent"]["token_step"] = phases(m, {"projections": wb("dq_dkv", "uq", "o", "gate_up", "down"), "latent_query": sum(u for u, _ in up),
+                                               "attention": sum(min(window, x.slots) * x.ld * 2 for x in m.rings), "latent_value": sum(v for _, v in up),
+                                               "head": m.embed.w.numel() * 2})
+        # kernels of one prompt portion: 2048 queries behind a full window
+        n, T = prompt_len, prompt_len + window - 1
+        new = lambda *s: torch.randn(*s, device="cuda").bfloat16()
+        sets = [dict(q=new(n, L["uq"].n), kv=new(T, L["ukv"].n), kr=new(T, a.rot_dim), out=new(n, a.heads * a.vdim), x=torch.randn(n, cfg.width, device="cuda"),
+                     xt=new(n, cfg.width), y=new(n, cfg.width), gu=new(n, L["gate_up"].n), act=new(n, cfg.layers[0].mlp.ff),
+                     yd=new(n, L["dq_dkv"].n), cq=new(n, a.q_rank)) for _ in range(3)]
+        st, check = m._cuda_stream, _lib.check_dense
+        pairs = n * window
+
+        def attend(k):
+            s = sets[k % 3]
+            check(lib.llvq_dn_latent_prefill(C.byref(lat), s["q"].data_ptr(), s["kv"].data_ptr(), s["kv"].shape[1], s["kr"].data_ptr(), a.rot_dim, n, T,
+                                             window - 1, 0, s["out"].data_ptr(), 0, st()))
+
+        def norm(k):
+            s = sets[k % 3]
+            check(lib.llvq_dn_postnorm_rows(m.dt, s["x"].data_ptr(), s["y"].data_ptr(), None, L["norm1"].data_ptr(), 2.0, 1e-5, s["xt"].data_ptr(),
+                                            s["x"].data_ptr(), n, cfg.width, st()))
+
+        def glu(k):
+            s = sets[k % 3]
+            check(lib.llvq_dn_glu_rows(m.dt, s["gu"].data_ptr(), L["gate_up_b"].data_ptr(), s["act"].data_ptr(), n, cfg.layers[0].mlp.ff, 7.0, 1.702, 1.0, st()))
+
+        def rows(k):
+            s = sets[k % 3]
+            check(lib.llvq_dn_latent_rows(C.byref(lat), s["yd"].data_ptr(), s["yd"].shape[1], a.q_rank, L["dq_norm"].data_ptr(), s["cq"].data_ptr(), 0, n, 1, st()))
+        pk = {}
+        ms = event_ms(attend, 12)
+        fl = 2.0 * pairs * a.heads * (a.dim + a.rot_dim + a.vdim)
+        pk["attention"] = {"us": round(ms * 1e3, 1), "TFLOPs": round(fl / ms / 1e9, 1), "frac": round(fl / ms / 1e9 / tflops, 4)}
+        for name, fn, b in (("add_norm", norm, n * cfg.width * 12), ("gated_unit", glu, n * cfg.layers[0].mlp.ff * 6),
+                            ("latent_rows", rows, 2 * n * (2 * a.q_rank + 2 * a.kv_rank + 2 * a.rot_dim))):
+            ms = event_ms(fn, 24)
+            pk[name] = {"us": round(ms * 1e3, 1), "GBps": round(b / ms / 1e6, 1), "frac": round(b / ms / 1e6 / peak, 4)}
+
+        def products(k):
+            s = sets[k % 3]
+            for x, w in ((s["xt"], L["dq_dkv"]), (s["cq"], L["uq"]), (s["out"], L["o"]), (s["xt"], L["gate_up"]), (s["act"], L["down"])):
+                m._mm(x, w.rows(0))
+        ms = event_ms(products, 12)
+        fl = 2.0 * n * sum(L[k].n * L[k].k for k in ("dq_dkv", "uq", "o", "gate_up", "down"))
+        pk["library products"] = {"us": round(ms * 1e3, 1), "TFLOPs": round(fl / ms / 1e9, 1), "frac": round(fl / ms / 1e9 / tflops, 4)}
+        r["latent"]["prompt_kernels"] = pk
+        r["latent"]["launches"] = int(lib.llvq_dn_launch_count() - launches)
+        r["latent"]["weight_bytes_per_layer"] = wb("dq_dkv", "uq", "o", "gate_up", "down", "ukv") // n_layers
+        r["latent"]["cache_bytes"] = m.cache_bytes()
+        del m, sets, L, lat
+        gc.collect()
+        torch.cuda.empty_cache()
+
+        # the archive-code model of the same size
+        rt = FusedRuntime(0)
+        qc = Qwen3Config.named(shape)
+        q, _ = synthetic_model(rt, qc, config_id=2, capacity=prompt_len + 128, layers=n_layers, keep_host=False, device_codes=True)
+        r["qwen3"] = loop_times(q)
+        pb = sum(blk[k].algorithmic_bytes(2, 2) for blk in q.blocks for k in ("qkv", "o", "gate_up", "down"))
+        r["qwen3"]["token_step"] = phases(q, {"projections": pb, "attention": sum(c.bytes_per_position() * window for c in q.caches),
+                                              "head": qc.vocab * qc.hidden * 2})
+        # its prompt attention over as many keys (full causal, through the library), and its norm and gated unit
+        half = lambda *s: torch.randn(*s, device="cuda").half()
+        q.positions = torch.arange(T, device="cuda")
+        qs = [(half(n, qc.n_heads, qc.head_dim), half(T, qc.n_kv, qc.head_dim), half(T, qc.n_kv, qc.head_dim)) for _ in range(3)]
+        xs = [(half(n, qc.hidden), half(n, qc.hidden), half(n, 2 * qc.inter)) for _ in range(3)]
+        ms = event_ms(lambda k: q._attend(*qs[k % 3], q.positions[T - n:], T), 6)
+        fl = 4.0 * (n * (T - n) + n * (n + 1) / 2) * qc.n_heads * qc.head_dim
+        pk = {"attention": {"us": round(ms * 1e3, 1), "TFLOPs": round(fl / ms / 1e9, 1), "frac": round(fl / ms / 1e9 / tflops, 4)}}
+        from llvq_b200.model import _silu
+        ms = event_ms(lambda k: q._rms(xs[k % 3][0] + xs[k % 3][1], q.final_norm), 24)
+        pk["add_norm"] = {"us": round(ms * 1e3, 1), "frac": round(n * qc.hidden * 8 / ms / 1e6 / peak, 4)}
+        ms = event_ms(lambda k: (_silu(xs[k % 3][2][:, :qc.inter].float()) * xs[k % 3][2][:, qc.inter:].float()).half(), 24)
+        pk["gated_unit"] = {"us": round(ms * 1e3, 1), "frac": round(n * qc.inter * 6 / ms / 1e6 / peak, 4)}
+        r["qwen3"]["prompt_kernels"] = pk
+        results.append(r)
+        del q, qs, xs
+        rt.close()
+        gc.collect()
+        torch.cuda.empty_cache()
+    clocks = sampler.stop()
+    emit({"metric": "latent_decode_tok_per_s", "value": results[0]["latent"]["decode_tok_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": new_tokens - 8,
+          "warmup": 3, "ms_per_step": results[0]["latent"]["decode_ms_per_token"], "higher_is_better": True, "vs_baseline": None, "dtype": "bf16",
+          "data": "synthetic (random weights and tokens)", "clocks": clocks, "peaks": {"hbm_gbs": peak, "bf16_tflops": tflops},
+          "config": {"prompt_tokens": prompt_len, "window": window, "layers": n_layers}, "results": results})
+
+
 _RESULT_FD = None
 
 
@@ -786,7 +969,14 @@ def main():
                     help="skip the tensor-parallel block (configuration 4: Qwen3-14B sharded over the ranks of this run)")
     ap.add_argument("--no-groups", action="store_true",
                     help="launch q, k, v and gate, up separately instead of row-concatenated")
+    ap.add_argument("--latent", action="store_true",
+                    help="instead of the headline workload: latent-attention models beside the Qwen3 model of equal size")
+    ap.add_argument("--latent-shapes", default="qwen3-4b,qwen3-8b,qwen3-14b", help="--latent: layer sizes, by model name")
+    ap.add_argument("--latent-layers", type=int, default=8, help="--latent: layers of both models")
+    ap.add_argument("--window", type=int, default=1024, help="--latent: sliding window of the latent layers")
     args = ap.parse_args()
+    if args.latent:
+        return run_latent(args)
     if args.impl == "reference":
         return run_reference(args)
     if args.tp_decode:
