@@ -20,6 +20,8 @@ typedef void* llvq_dn_stream;
 
 const char* llvq_dn_last_error(void);
 uint64_t llvq_dn_launch_count(void);
+/* Read and clear the error word of the current device (synchronises): bit 0 = a kernel's bounded wait ran out. */
+int llvq_dn_poll_error(int32_t* out);
 /* Programmatic overlap of consecutive launches (on by default). */
 int llvq_dn_set_overlap(int32_t on);
 

@@ -141,6 +141,7 @@ _SIGNATURES = {
 _DENSE_SIGNATURES = {
     "llvq_dn_last_error": (C.c_char_p, []),
     "llvq_dn_launch_count": (C.c_uint64, []),
+    "llvq_dn_poll_error": (C.c_int, [C.POINTER(C.c_int32)]),
     "llvq_dn_set_overlap": (C.c_int, [C.c_int32]),
     "llvq_dn_gemv": (C.c_int, [C.POINTER(DenseGemv), C.c_void_p]),
     "llvq_dn_head": (C.c_int, [C.POINTER(DenseGemv)] + [C.c_void_p] * 4),

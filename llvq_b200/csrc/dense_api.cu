@@ -54,6 +54,50 @@ int check_gemv(const llvq_dn_gemv_desc* d, const char* who) {
     return kStatusOk;
 }
 
+__device__ unsigned int g_device_error;  // bits set by kernels whose bounded wait ran out
+
+unsigned int* device_error() {
+    static std::atomic<unsigned int*> cached[64];
+    int dev = 0;
+    if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) return nullptr;
+    if (!cached[dev].load()) {
+        void* p = nullptr;
+        if (cudaGetSymbolAddress(&p, g_device_error) != cudaSuccess) return nullptr;
+        cached[dev] = (unsigned int*)p;
+    }
+    return cached[dev].load();
+}
+
+template <int VPL, int PRO, bool HEAD>
+int launch_stream_vpl(const DenseGemvArgs& a, int grid, size_t smem, cudaStream_t s) {
+    const int st = ensure_dyn_smem((const void*)dense_gemv_stream_kernel<VPL, PRO, HEAD>, smem);
+    if (st) return st;
+    CUDA_TRY(launch_dep(dense_gemv_stream_kernel<VPL, PRO, HEAD>, dim3(grid), dim3(kGvThreads), smem, s, a));
+    g_launches++;
+    return kStatusOk;
+}
+
+template <int PRO, bool HEAD>
+int launch_stream(const DenseGemvArgs& a, int grid, size_t smem, cudaStream_t s) {
+    if (a.segv <= 3 * 32) return launch_stream_vpl<3, PRO, HEAD>(a, grid, smem, s);
+    if (a.segv <= 6 * 32) return launch_stream_vpl<6, PRO, HEAD>(a, grid, smem, s);
+    return launch_stream_vpl<kGsMaxVpl, PRO, HEAD>(a, grid, smem, s);
+}
+
+// Column segments, ring and grid of the stream kernel; false when a row is too long for it.
+bool plan_stream(DenseGemvArgs& a, int* grid, size_t* smem) {
+    const int vecs = a.ldw / 8;
+    a.nseg = 1;
+    while (a.nseg < kGvWarps && (vecs + a.nseg - 1) / a.nseg > 6 * 32) a.nseg *= 2;
+    a.segv = (vecs + a.nseg - 1) / a.nseg;
+    if (a.segv > kGsMaxVpl * 32 || (a.nseg - 1) * a.segv >= vecs) return false;
+    a.slots = std::max(2, std::min(kGsMaxSlots, kGsRingBytes / (a.segv * 16)));
+    const int groups = kGvWarps / a.nseg;
+    *grid = std::min((a.n_out + groups - 1) / groups, sm_count());
+    *smem = (size_t)kGvWarps * a.slots * a.segv * 16 + (size_t)(a.n_out / *grid + 1) * a.nseg * sizeof(float);
+    return *smem <= kMaxSmem - 2048;
+}
+
 template <typename T, int PRO, bool HEAD>
 int launch_gemv(const DenseGemvArgs& a, int grid, cudaStream_t s) {
     const int rows = a.n_out / grid + 1;
@@ -76,6 +120,26 @@ int gemv_t(const llvq_dn_gemv_desc* d, HeadBest* best, int* grid_out, cudaStream
     a.n_out = d->n_out, a.k = d->k, a.ldw = d->ldw, a.ld_table = d->ld_table, a.table_rows = d->table_rows;
     a.alpha = d->alpha, a.eps = d->eps, a.scale = d->scale, a.limit = d->limit, a.gain = d->gain, a.shift = d->shift, a.cap = d->softcap;
     // column slices: enough lanes for a row's vectors; rows of a CTA are shared by the row groups that are left
+    if constexpr (sizeof(T) == 2) {
+        size_t smem = 0;
+        int grid = 0;
+        a.err = device_error();
+        a.vec_x = !(((uintptr_t)a.x | (uintptr_t)a.delta | (uintptr_t)a.norm_w) & 15) && (d->prologue != LLVQ_DN_GLU || a.k % 4 == 0);
+        if (a.err && plan_stream(a, &grid, &smem)) {
+            if (grid_out) *grid_out = grid;
+            if (best) {
+                if (d->prologue == LLVQ_DN_NORM) return launch_stream<kGvNorm, true>(a, grid, smem, s);
+                if (d->prologue == LLVQ_DN_PLAIN) return launch_stream<kGvPlain, true>(a, grid, smem, s);
+                return fail(kStatusUnsupported, "dn_head: prologue %d (plain or norm)", d->prologue);
+            }
+            switch (d->prologue) {
+                case LLVQ_DN_PLAIN: return launch_stream<kGvPlain, false>(a, grid, smem, s);
+                case LLVQ_DN_EMBED: return launch_stream<kGvEmbed, false>(a, grid, smem, s);
+                case LLVQ_DN_NORM: return launch_stream<kGvNorm, false>(a, grid, smem, s);
+                default: return launch_stream<kGvGlu, false>(a, grid, smem, s);
+            }
+        }
+    }
     const int vecs = d->ldw / Vec16<T>::N;
     a.kslices = vecs > 128 ? 8 : vecs > 64 ? 4 : vecs > 32 ? 2 : 1;
     const int rows_step = kGvWarps / a.kslices * kGvRows;
@@ -111,25 +175,43 @@ int check_latent(const llvq_dn_latent* a, const char* who) {
 LatentRing ring_of(const llvq_dn_latent* a) { return LatentRing{a->ring, a->slots, a->ld}; }
 RotaryTable rot_of(const llvq_dn_latent* a) { return RotaryTable{a->cos_t, a->sin_t, a->rot_dims}; }
 
-template <typename T>
+// Whether the token's attention runs on the tensor cores (bf16 rows of a size that fits one tile in shared memory).
+bool decode_on_mma(const llvq_dn_latent* a) {
+    return a->dtype == LLVQ_DN_BF16 && a->kv_rank <= 1024 && latent_decode_mma_smem(a->ld) <= kMaxSmem;
+}
+
+template <typename T, typename Q>
 int latent_query_t(const llvq_dn_latent* a, const float* q, const float* y_kv, const int64_t* pos, cudaStream_t s) {
     LatentQueryArgs k{q, a->uk, a->qlat, y_kv, a->kv_norm, (const long long*)pos, ring_of(a), rot_of(a),
                       a->heads, a->dim, a->rot_dim, a->kv_rank, a->ldk, a->eps};
     const int slices = (a->ldk / Vec16<T>::N + 31) / 32;
-    CUDA_TRY(launch_dep(latent_query_kernel<T>, dim3(a->heads + (y_kv ? 1 : 0), slices), dim3(256), 0, s, k));
+    CUDA_TRY(launch_dep(latent_query_kernel<T, Q>, dim3(a->heads + (y_kv ? 1 : 0), slices), dim3(256), 0, s, k));
+    g_launches++;
+    return kStatusOk;
+}
+
+LatentDecodeArgs decode_args(const llvq_dn_latent* a, const int64_t* pos) {
+    return LatentDecodeArgs{a->qlat, (const long long*)pos, a->part, a->part + (size_t)a->heads * a->splits * 2, ring_of(a), a->heads, a->kv_rank,
+                            a->window, a->scale};
+}
+
+template <int CH>
+int latent_decode_mma(const llvq_dn_latent* a, const int64_t* pos, cudaStream_t s) {
+    const size_t smem = latent_decode_mma_smem(a->ld);
+    const int st = ensure_dyn_smem((const void*)latent_decode_mma_kernel<CH>, smem);
+    if (st) return st;
+    CUDA_TRY(launch_dep(latent_decode_mma_kernel<CH>, dim3((a->heads + kLmHeads - 1) / kLmHeads, a->splits), dim3(256), smem, s, decode_args(a, pos)));
     g_launches++;
     return kStatusOk;
 }
 
 template <typename T>
 int latent_decode_t(const llvq_dn_latent* a, const int64_t* pos, cudaStream_t s) {
-    LatentDecodeArgs k{a->qlat, (const long long*)pos, a->part, a->part + (size_t)a->heads * a->splits * 2, ring_of(a), a->heads, a->kv_rank,
-                       a->window, a->scale};
     const size_t smem = latent_decode_smem<T>(a->ld, a->kv_rank);
     if (smem > kMaxSmem) return fail(kStatusUnsupported, "dn_latent_decode: cache rows of %d elements need %zu bytes of shared memory", a->ld, smem);
     const int st = ensure_dyn_smem((const void*)latent_decode_kernel<T>, smem);
     if (st) return st;
-    CUDA_TRY(launch_dep(latent_decode_kernel<T>, dim3((a->heads + kLdHeads - 1) / kLdHeads, a->splits), dim3(256), smem, s, k));
+    CUDA_TRY(launch_dep(latent_decode_kernel<T>, dim3((a->heads + kLdHeads - 1) / kLdHeads, a->splits), dim3(256), smem, s, decode_args(a, pos)));
     g_launches++;
     return kStatusOk;
 }
@@ -173,6 +255,14 @@ extern "C" {
 
 const char* llvq_dn_last_error(void) { return g_error.c_str(); }
 uint64_t llvq_dn_launch_count(void) { return g_launches.load(); }
+int llvq_dn_poll_error(int32_t* out) {
+    if (!out) return fail(kStatusInvalid, "dn_poll_error: null argument");
+    unsigned int v = 0, zero = 0;
+    CUDA_TRY(cudaMemcpyFromSymbol(&v, g_device_error, sizeof v));
+    if (v) CUDA_TRY(cudaMemcpyToSymbol(g_device_error, &zero, sizeof zero));
+    *out = (int32_t)v;
+    return kStatusOk;
+}
 int llvq_dn_set_overlap(int32_t on) {
     g_overlap_ops = on ? 1 : 0;
     return kStatusOk;
@@ -202,7 +292,9 @@ int llvq_dn_latent_query(const llvq_dn_latent* a, const float* q, const float* y
     const int st = check_latent(a, "dn_latent_query");
     if (st) return st;
     if (!q || !pos || !a->uk || !a->qlat || (y_kv && !a->kv_norm)) return fail(kStatusInvalid, "dn_latent_query: null argument");
-    return a->dtype == LLVQ_DN_BF16 ? latent_query_t<bf16>(a, q, y_kv, pos, (cudaStream_t)stream) : latent_query_t<float>(a, q, y_kv, pos, (cudaStream_t)stream);
+    cudaStream_t s = (cudaStream_t)stream;
+    if (a->dtype == LLVQ_DN_F32) return latent_query_t<float, float>(a, q, y_kv, pos, s);
+    return decode_on_mma(a) ? latent_query_t<bf16, bf16>(a, q, y_kv, pos, s) : latent_query_t<bf16, float>(a, q, y_kv, pos, s);
 }
 
 int llvq_dn_latent_decode(const llvq_dn_latent* a, const int64_t* pos, llvq_dn_stream stream) {
@@ -210,7 +302,12 @@ int llvq_dn_latent_decode(const llvq_dn_latent* a, const int64_t* pos, llvq_dn_s
     if (st) return st;
     if (!pos || !a->qlat || !a->part || a->splits < 1 || a->splits > 4096) return fail(kStatusInvalid, "dn_latent_decode: null argument or %d splits", a->splits);
     if (a->window > a->slots) return fail(kStatusInvalid, "dn_latent_decode: a window of %d over %d slots", a->window, a->slots);
-    return a->dtype == LLVQ_DN_BF16 ? latent_decode_t<bf16>(a, pos, (cudaStream_t)stream) : latent_decode_t<float>(a, pos, (cudaStream_t)stream);
+    cudaStream_t s = (cudaStream_t)stream;
+    if (a->dtype == LLVQ_DN_F32) return latent_decode_t<float>(a, pos, s);
+    if (!decode_on_mma(a)) return latent_decode_t<bf16>(a, pos, s);
+    if (a->kv_rank <= 128) return latent_decode_mma<1>(a, pos, s);
+    if (a->kv_rank <= 256) return latent_decode_mma<2>(a, pos, s);
+    return a->kv_rank <= 512 ? latent_decode_mma<4>(a, pos, s) : latent_decode_mma<8>(a, pos, s);
 }
 
 int llvq_dn_latent_value(const llvq_dn_latent* a, float* ctx, llvq_dn_stream stream) {

@@ -8,7 +8,16 @@
 //   epilogue  y = W a + bias, f32; the head variant caps the logits (cap * tanh(y / cap)), stores them and
 //             keeps the best (logit, row) of the CTA for lm_head_pick_kernel.
 //
-// The work is one pass over W. A CTA owns a contiguous range of rows, its warps are split into row groups and
+// The work is one pass over W. Two kernels:
+//
+//   dense_gemv_stream_kernel (bf16)  one CTA per SM owns a contiguous range of rows; every warp is bound to one
+//       column segment, keeps the activation of that segment in registers and walks the CTA's rows with a ring of
+//       bulk copies of its own (row segment -> shared memory, one mbarrier per slot). The ring is filled before the
+//       dependency wait: W does not depend on the kernel before, so a small matrix is on the chip by the time its
+//       activation exists. No warp waits for another until the row sums are added.
+//   dense_gemv_kernel (f32, and rows too long for the ring)  loads straight into registers.
+//
+// In the second, a CTA owns a contiguous range of rows, its warps are split into row groups and
 // `kslices` column slices per group; a warp takes kGvRows rows at a time with 16-byte loads. The first loads
 // are issued before the dependency wait: W does not depend on the kernel before. Partial sums of the column
 // slices meet in shared memory and are added in slice order, so a row's result depends on nothing but the
@@ -16,6 +25,7 @@
 #pragma once
 #include "dense_elem.cuh"
 #include "head_pick.cuh"
+#include "mbarrier.cuh"
 
 namespace llvq {
 
@@ -42,7 +52,45 @@ struct DenseGemvArgs {
     float scale;          // embed
     float limit, gain, shift;  // glu
     float cap;            // head: 0 = no cap
+    // stream kernel: column segments (1, 2, 4 or 8), vectors of a segment, ring slots of a warp
+    int nseg, segv, slots;
+    int vec_x;            // x, delta, norm_w (glu: both halves of x) may be read 16 bytes at a time
+    unsigned int* err;    // bit 0: a copy did not land in time
 };
+
+// y, bias, soft cap and the greedy candidate of the rows [r0, r1) of a CTA, from the partial sums of their segments.
+template <bool HEAD>
+__device__ __forceinline__ void gemv_finish(const DenseGemvArgs& A, const float* part, int segments, int r0, int r1, HeadBest* best_s) {
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    HeadBest b{-INFINITY, 0x7fffffff};
+    for (int r = r0 + tid; r < r1; r += kGvThreads) {
+        float s = 0.0f;
+        for (int k = 0; k < segments; ++k) s += part[(r - r0) * segments + k];
+        if (A.bias) s += A.bias[r];
+        if constexpr (HEAD) {
+            if (A.cap > 0.0f) s = A.cap * tanhf(s / A.cap);
+            if (head_better(s, r, b.val, b.row)) b = HeadBest{s, r};
+            if (A.y) A.y[r] = s;
+        } else {
+            A.y[r] = s;
+        }
+    }
+    if constexpr (HEAD) {
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float v = __shfl_xor_sync(0xffffffffu, b.val, o);
+            const int r = __shfl_xor_sync(0xffffffffu, b.row, o);
+            if (head_better(v, r, b.val, b.row)) b = HeadBest{v, r};
+        }
+        if (lane == 0) best_s[warp] = b;
+        __syncthreads();
+        if (tid == 0) {
+            for (int k = 1; k < kGvWarps; ++k)
+                if (head_better(best_s[k].val, best_s[k].row, b.val, b.row)) b = best_s[k];
+            A.best[blockIdx.x] = b;
+        }
+    }
+}
 
 template <typename T, int PRO, bool HEAD>
 __global__ void __launch_bounds__(kGvThreads)
@@ -135,34 +183,155 @@ dense_gemv_kernel(DenseGemvArgs A) {
         }
     }
     __syncthreads();
-    HeadBest b{-INFINITY, 0x7fffffff};
-    for (int r = r0 + tid; r < r1; r += kGvThreads) {
-        float s = 0.0f;
-        for (int k = 0; k < A.kslices; ++k) s += part[(r - r0) * A.kslices + k];
-        if (A.bias) s += A.bias[r];
-        if constexpr (HEAD) {
-            if (A.cap > 0.0f) s = A.cap * tanhf(s / A.cap);
-            if (head_better(s, r, b.val, b.row)) b = HeadBest{s, r};
-            if (A.y) A.y[r] = s;
-        } else {
-            A.y[r] = s;
-        }
-    }
-    if constexpr (HEAD) {
+    gemv_finish<HEAD>(A, part, A.kslices, r0, r1, best_s);
+}
+
+constexpr int kGsRingBytes = 11 * 1024;  // of a warp: two CTAs (this launch's and the next one's) fit an SM together
+constexpr int kGsMaxSlots = 8;
+constexpr int kGsMaxVpl = 10;            // activation vectors a lane can keep
+
+// Eight consecutive activation values from column c on; zeros beyond k.
+__device__ __forceinline__ void gs_load8(const float* p, int c, int k, int vec, float (&f)[8]) {
+    if (vec && c + 8 <= k) {
+        const float4 u = *reinterpret_cast<const float4*>(p + c), v = *reinterpret_cast<const float4*>(p + c + 4);
+        f[0] = u.x, f[1] = u.y, f[2] = u.z, f[3] = u.w, f[4] = v.x, f[5] = v.y, f[6] = v.z, f[7] = v.w;
+    } else {
 #pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            const float v = __shfl_xor_sync(0xffffffffu, b.val, o);
-            const int r = __shfl_xor_sync(0xffffffffu, b.row, o);
-            if (head_better(v, r, b.val, b.row)) b = HeadBest{v, r};
-        }
-        if (lane == 0) best_s[warp] = b;
-        __syncthreads();
-        if (tid == 0) {
-            for (int k = 1; k < kGvWarps; ++k)
-                if (head_better(best_s[k].val, best_s[k].row, b.val, b.row)) b = best_s[k];
-            A.best[blockIdx.x] = b;
+        for (int j = 0; j < 8; ++j) f[j] = c + j < k ? p[c + j] : 0.0f;
+    }
+}
+
+template <int VPL, int PRO, bool HEAD>
+__global__ void __launch_bounds__(kGvThreads, 2)
+dense_gemv_stream_kernel(DenseGemvArgs A) {
+    extern __shared__ __align__(128) unsigned char gs_raw[];
+    __shared__ __align__(8) unsigned long long bars[kGvWarps][kGsMaxSlots];
+    __shared__ float red[kGvWarps];
+    __shared__ HeadBest best_s[kGvWarps];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int r0 = (int)((long long)A.n_out * blockIdx.x / gridDim.x), r1 = (int)((long long)A.n_out * (blockIdx.x + 1) / gridDim.x);
+    const int seg = warp % A.nseg, group = warp / A.nseg, groups = kGvWarps / A.nseg;
+    const int nv = min(A.segv, A.ldw / 8 - seg * A.segv);  // vectors of this warp's segment
+    const int mine = (r1 - r0 - group + groups - 1) / groups;  // rows of this warp: r0 + group, + groups, ...
+    const unsigned int slot_bytes = (unsigned int)A.segv * 16u, bytes = (unsigned int)nv * 16u;
+    unsigned char* ring = gs_raw + (size_t)warp * A.slots * slot_bytes;
+    const unsigned int ring_s = pipe_smem_addr(ring), bar0 = pipe_smem_addr(&bars[warp][0]);
+    float* part = reinterpret_cast<float*>(gs_raw + (size_t)kGvWarps * A.slots * slot_bytes);  // [rows of the CTA][nseg]
+    const unsigned char* src = reinterpret_cast<const unsigned char*>(A.w) + ((size_t)(r0 + group) * A.ldw + (size_t)seg * A.segv * 8) * 2;
+    const size_t src_step = (size_t)groups * A.ldw * 2;
+    if (lane == 0) {
+        for (int i = 0; i < A.slots; ++i) mbar_init(bar0 + 8 * i, 1);
+        mbar_init_fence();
+        for (int i = 0; i < min(A.slots, mine); ++i) {
+            pipe_expect_tx(bar0 + 8 * i, bytes);
+            pipe_bulk_copy(ring_s + i * slot_bytes, src + i * src_step, bytes, bar0 + 8 * i);
         }
     }
+    __syncwarp();
+    llvq_dependent_enter();
+
+    // ---- the activation of this warp's segment, in registers ----
+    float a[VPL][8];
+    float ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < VPL; ++i) {
+        const int v = lane + 32 * i, c = (seg * A.segv + v) * 8;
+        if (v >= nv) {
+#pragma unroll
+            for (int j = 0; j < 8; ++j) a[i][j] = 0.0f;
+            continue;
+        }
+        if constexpr (PRO == kGvPlain) {
+            gs_load8(A.x, c, A.k, A.vec_x, a[i]);
+        } else if constexpr (PRO == kGvEmbed) {
+            long long t = *A.token;
+            if (t < 0 || t >= A.table_rows) t = 0;
+            const bf16* row = reinterpret_cast<const bf16*>(A.table) + (size_t)t * A.ld_table;
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                a[i][j] = c + j < A.k ? A.scale * to_f32(row[c + j]) : 0.0f;
+                if (blockIdx.x == 0 && group == 0 && A.a_out && c + j < A.k) A.a_out[c + j] = a[i][j];
+            }
+        } else if constexpr (PRO == kGvNorm) {
+            gs_load8(A.x, c, A.k, A.vec_x, a[i]);
+            float d[8];
+#pragma unroll
+            for (int j = 0; j < 8; ++j) d[j] = 0.0f;
+            if (A.delta) gs_load8(A.delta, c, A.k, A.vec_x, d);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                a[i][j] = fmaf(A.alpha, a[i][j], d[j]);
+                ss = fmaf(a[i][j], a[i][j], ss);
+            }
+        } else {
+            float u[8];
+            gs_load8(A.x, c, A.k, A.vec_x, a[i]);
+            gs_load8(A.x + A.k, c, A.k, A.vec_x, u);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) a[i][j] = c + j < A.k ? clamped_glu(a[i][j], u[j], A.limit, A.gain, A.shift) : 0.0f;
+        }
+    }
+    if constexpr (PRO == kGvNorm) {
+        ss = warp_sum_f(ss);
+        if (lane == 0) red[warp] = ss;
+        __syncthreads();
+        float tot = 0.0f;
+        for (int s = 0; s < A.nseg; ++s) tot += red[s];  // the first row group's warps hold every segment once
+        const float r = 1.0f / sqrtf(tot / (float)A.k + A.eps);
+#pragma unroll
+        for (int i = 0; i < VPL; ++i) {
+            const int v = lane + 32 * i, c = (seg * A.segv + v) * 8;
+            if (v >= nv) continue;
+            float w[8];
+            gs_load8(A.norm_w, c, A.k, A.vec_x, w);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                a[i][j] *= r * w[j];
+                if (blockIdx.x == 0 && group == 0 && A.a_out && c + j < A.k) A.a_out[c + j] = a[i][j];
+            }
+        }
+    }
+
+    // ---- the rows ----
+    bool ok = true;
+    int slot = 0;
+    unsigned int parity = 0;
+    for (int i = 0; i < mine; ++i) {
+        ok = pipe_mbar_wait(bar0 + 8 * slot, parity);
+        if (!ok) break;
+        const uint4* w_s = reinterpret_cast<const uint4*>(ring + (size_t)slot * slot_bytes);
+        float acc0 = 0.0f, acc1 = 0.0f;
+#pragma unroll
+        for (int k = 0; k < VPL; ++k) {
+            const int v = lane + 32 * k;
+            if (v < nv) {
+                float f[8];
+                Vec16<bf16>::widen(w_s[v], f);
+#pragma unroll
+                for (int j = 0; j < 8; j += 2) {
+                    acc0 = fmaf(f[j], a[k][j], acc0);
+                    acc1 = fmaf(f[j + 1], a[k][j + 1], acc1);
+                }
+            }
+        }
+        __syncwarp();  // the slot is read: it takes the row `slots` further on
+        if (lane == 0 && i + A.slots < mine) {
+            pipe_expect_tx(bar0 + 8 * slot, bytes);
+            pipe_bulk_copy(ring_s + slot * slot_bytes, src + (size_t)(i + A.slots) * src_step, bytes, bar0 + 8 * slot);
+        }
+        const float s = warp_sum_f(acc0 + acc1);
+        if (lane == 0) part[(group + i * groups) * A.nseg + seg] = s;
+        if (++slot == A.slots) {
+            slot = 0;
+            parity ^= 1u;
+        }
+    }
+    if (!ok) {  // give the copies in flight one more bounded chance to land before the CTA's memory is given up
+        for (int i = 0; i < A.slots; ++i) pipe_mbar_wait(bar0 + 8 * i, parity);
+        if (lane == 0) atomicOr(A.err, 1u);
+    }
+    __syncthreads();
+    gemv_finish<HEAD>(A, part, A.nseg, r0, r1, best_s);
 }
 
 }  // namespace llvq

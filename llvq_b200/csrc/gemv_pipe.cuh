@@ -42,6 +42,7 @@
 
 #include "decode_tab.cuh"
 #include "kernels_generic.cuh"
+#include "mbarrier.cuh"
 
 namespace llvq {
 
@@ -60,7 +61,6 @@ constexpr int kGroupWarps = kGroupThreads / 32;
 constexpr int kDigitBytes = 24576;    // shared memory given to the activation digits
 constexpr int kTileRowsMax = 128;     // rows per tile
 constexpr int kStageWarps = 4 / kPipeGroups > 0 ? 4 / kPipeGroups : 1;  // warps of a group that stage the next tile's digits and row data
-constexpr unsigned int kPipeSpinLimit = 1u << 22;
 #ifndef LLVQ_CLS_GROUPS
 #define LLVQ_CLS_GROUPS 2
 #endif
@@ -180,34 +180,6 @@ __device__ __forceinline__ unsigned long long pipe_now_ns() {
     unsigned long long t;
     asm volatile("mov.u64 %0, %globaltimer;" : "=l"(t));
     return t;
-}
-
-__device__ __forceinline__ unsigned int pipe_smem_addr(const void* p) {
-    return (unsigned int)__cvta_generic_to_shared(p);
-}
-
-// Bounded wait for the phase of the given parity of an mbarrier; false when the spin limit ran out.
-__device__ __forceinline__ bool pipe_mbar_wait(unsigned int bar, unsigned int parity = 0) {
-    unsigned int done = 0;
-    for (unsigned int spin = 0; spin < kPipeSpinLimit && !done; ++spin) {
-        asm volatile(
-            "{\n\t.reg .pred p;\n\t"
-            "mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
-            "selp.u32 %0, 1, 0, p;\n\t}"
-            : "=r"(done)
-            : "r"(bar), "r"(parity)
-            : "memory");
-    }
-    return done != 0;
-}
-
-__device__ __forceinline__ void pipe_expect_tx(unsigned int bar, unsigned int bytes) {
-    asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ void pipe_bulk_copy(unsigned int dst, const void* src, unsigned int bytes, unsigned int bar) {
-    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst),
-                 "l"(src), "r"(bytes), "r"(bar)
-                 : "memory");
 }
 
 __device__ __forceinline__ int dp4a_ss(unsigned int a, unsigned int b, int c) {

@@ -38,28 +38,6 @@ inline size_t latent_prefill_smem(int dim, int rot_dim, int nv) {
     return (kLpM * qk + 2 * kLpN * (qk + v)) * sizeof(bf16);
 }
 
-__device__ __forceinline__ void lp_ldmatrix4(unsigned int (&r)[4], const bf16* p) {
-    const unsigned int a = (unsigned int)__cvta_generic_to_shared(p);
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
-}
-__device__ __forceinline__ void lp_ldmatrix4_trans(unsigned int (&r)[4], const bf16* p) {
-    const unsigned int a = (unsigned int)__cvta_generic_to_shared(p);
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
-}
-__device__ __forceinline__ void lp_mma(float (&d)[4], const unsigned int (&a)[4], unsigned int b0, unsigned int b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void lp_copy16(bf16* dst, const bf16* src, bool valid) {
-    const unsigned int d = (unsigned int)__cvta_generic_to_shared(dst);
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d), "l"(src), "r"(valid ? 16 : 0) : "memory");
-}
-__device__ __forceinline__ unsigned int lp_pack(float lo, float hi) {
-    const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
-    return *reinterpret_cast<const unsigned int*>(&v);
-}
-
 // NV: 8-column tiles of the value slice a CTA accumulates (even). VEC: every row piece is a whole number of aligned
 // 16-byte vectors; otherwise tiles are staged element by element.
 template <int NV, bool VEC>
@@ -96,12 +74,12 @@ latent_prefill_mma_kernel(LatentPrefillArgs A) {
                 const int r = i / ct, c = i - r * ct, j = base + r;
                 const bool in = j < k_end && c < cn + cr;
                 const bf16* src = !in ? KV : c < cn ? KV + (size_t)j * A.ld_kv + (size_t)h * A.dim + 8 * c : KR + (size_t)j * A.ld_kr + 8 * (c - cn);
-                lp_copy16(dk + r * pitch + 8 * c, src, in);
+                copy16_async(dk + r * pitch + 8 * c, src, in);
             }
             for (int i = tid; i < kLpN * NV; i += kLpThreads) {
                 const int r = i / NV, c = i - r * NV, j = base + r;
                 const bool in = j < k_end && 8 * c < v_n;
-                lp_copy16(dv + r * vp + 8 * c, in ? KV + (size_t)j * A.ld_kv + (size_t)A.heads * A.dim + (size_t)h * A.vdim + v_lo + 8 * c : KV, in);
+                copy16_async(dv + r * vp + 8 * c, in ? KV + (size_t)j * A.ld_kv + (size_t)A.heads * A.dim + (size_t)h * A.vdim + v_lo + 8 * c : KV, in);
             }
         } else {
             for (int i = tid; i < kLpN * (pitch - 8); i += kLpThreads) {
@@ -129,7 +107,7 @@ latent_prefill_mma_kernel(LatentPrefillArgs A) {
             const int cn = A.dim / 8;
             for (int i = tid; i < kLpM * cn; i += kLpThreads) {
                 const int r = i / cn, c = i - r * cn;
-                lp_copy16(sq + r * pitch + 8 * c, r < q_n ? Q + (size_t)(q_lo + r) * qrow + (size_t)h * qk + 8 * c : Q, r < q_n);
+                copy16_async(sq + r * pitch + 8 * c, r < q_n ? Q + (size_t)(q_lo + r) * qrow + (size_t)h * qk + 8 * c : Q, r < q_n);
             }
             asm volatile("cp.async.commit_group;" ::: "memory");
         } else {
@@ -188,13 +166,13 @@ latent_prefill_mma_kernel(LatentPrefillArgs A) {
 #pragma unroll 2
         for (int k = 0; k < ksteps; ++k) {
             unsigned int a[4];
-            lp_ldmatrix4(a, sq + (warp * 16 + (lane & 15)) * pitch + k * 16 + (lane >> 4) * 8);
+            ldmatrix4(a, sq + (warp * 16 + (lane & 15)) * pitch + k * 16 + (lane >> 4) * 8);
 #pragma unroll
             for (int n = 0; n < 8; n += 2) {
                 unsigned int b[4];
-                lp_ldmatrix4(b, tk + (n * 8 + (lane & 7) + (lane >> 4) * 8) * pitch + k * 16 + ((lane >> 3) & 1) * 8);
-                lp_mma(s[n], a, b[0], b[1]);
-                lp_mma(s[n + 1], a, b[2], b[3]);
+                ldmatrix4(b, tk + (n * 8 + (lane & 7) + (lane >> 4) * 8) * pitch + k * 16 + ((lane >> 3) & 1) * 8);
+                mma_bf16(s[n], a, b[0], b[1]);
+                mma_bf16(s[n + 1], a, b[2], b[3]);
             }
         }
         const bool edge = base + kLpN - 1 > qa || base < qa + 15 - A.window + 1 || base + kLpN > k_end;
@@ -231,8 +209,8 @@ latent_prefill_mma_kernel(LatentPrefillArgs A) {
                 e[j] = exp2f(s[n][j] - base_m[j >> 1]);
                 l[j >> 1] += e[j];
             }
-            p[n][0] = lp_pack(e[0], e[1]);
-            p[n][1] = lp_pack(e[2], e[3]);
+            p[n][0] = pack_bf16(e[0], e[1]);
+            p[n][1] = pack_bf16(e[2], e[3]);
         }
 #pragma unroll
         for (int n = 0; n < NV; ++n)
@@ -245,9 +223,9 @@ latent_prefill_mma_kernel(LatentPrefillArgs A) {
             for (int n = 0; n < NV; n += 2) {
                 if (n >= nv_used) break;
                 unsigned int b[4];
-                lp_ldmatrix4_trans(b, tv + (k * 16 + (lane & 15)) * vp + n * 8 + (lane >> 4) * 8);
-                lp_mma(o[n], a, b[0], b[1]);
-                lp_mma(o[n + 1], a, b[2], b[3]);
+                ldmatrix4_trans(b, tv + (k * 16 + (lane & 15)) * vp + n * 8 + (lane >> 4) * 8);
+                mma_bf16(o[n], a, b[0], b[1]);
+                mma_bf16(o[n + 1], a, b[2], b[3]);
             }
         }
     }
@@ -272,7 +250,7 @@ latent_prefill_mma_kernel(LatentPrefillArgs A) {
         for (int n = 0; n < NV; ++n) {
             const int c = n * 8 + (lane & 3) * 2;
             if constexpr (VEC) {
-                if (c < v_n) *reinterpret_cast<unsigned int*>(dst + c) = lp_pack(o[n][2 * r] * f, o[n][2 * r + 1] * f);
+                if (c < v_n) *reinterpret_cast<unsigned int*>(dst + c) = pack_bf16(o[n][2 * r] * f, o[n][2 * r + 1] * f);
             } else {
                 if (c < v_n) dst[c] = from_f32<bf16>(o[n][2 * r] * f);
                 if (c + 1 < v_n) dst[c + 1] = from_f32<bf16>(o[n][2 * r + 1] * f);

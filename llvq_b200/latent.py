@@ -213,8 +213,9 @@ class LatentLM(TokenLoop):
         sms = torch.cuda.get_device_properties(dev).multi_processor_count
 
         def splits(a):
-            groups = -(-a.heads // 8)
-            return max(1, min(-(-min(a.window or self.capacity, self.capacity) // 32), max(1, 2 * sms // groups), 64))
+            heads, tile = (16, 64) if self.dtype == torch.bfloat16 else (8, 32)  # per CTA and step of the attention kernel
+            groups = -(-a.heads // heads)
+            return max(1, min(-(-min(a.window or self.capacity, self.capacity) // tile), 2 * sms // groups, 128))
 
         buf = lambda n: torch.zeros(n, **f32)
         self._stream = [buf(cfg.width), buf(cfg.width)]  # a norm reads one and stores the other
