@@ -29,18 +29,18 @@ int llvq_dn_set_overlap(int32_t on);
 enum {
     LLVQ_DN_PLAIN = 0, /* a = x */
     LLVQ_DN_EMBED = 1, /* a = scale * table[*token] */
-    LLVQ_DN_NORM = 2,  /* t = alpha x + delta; a = t / sqrt(mean(t^2) + eps) * norm_w */
-    LLVQ_DN_GLU = 3    /* x = [gate k | up k]; g = min(gate, limit), u = clamp(up, +-limit); a = g sigmoid(gain g) (u + shift) */
+    LLVQ_DN_NORM = 2   /* t = alpha x + delta; a = t / sqrt(mean(t^2) + eps) * norm_w */
 };
 typedef struct {
     int32_t dtype, prologue;
+    int32_t glu;            /* rows are (gate, up) pairs: y[i] = g sigmoid(gain g) (u + shift), g = min(gate_i, limit), u = clamp(up_i, +-limit) */
     int32_t n_out, k, ldw;
     int32_t ld_table, table_rows;
     float alpha, eps, scale, limit, gain, shift;
     float softcap;          /* llvq_dn_head only: logits <- softcap * tanh(logits / softcap); 0 = none */
     const void* w;
     const float* bias;      /* or NULL */
-    float* y;               /* llvq_dn_head: the logits, may be NULL */
+    float* y;               /* [n_out], or [n_out / 2] with glu; llvq_dn_head: the logits, may be NULL */
     const float* x;
     const float* delta;     /* or NULL */
     const float* norm_w;
@@ -98,6 +98,7 @@ int llvq_dn_postnorm_rows(int32_t dtype, const float* x, const void* y, const fl
  * rows of positions pos0 .. pos0 + rows - 1 (rows <= slots). */
 int llvq_dn_latent_rows(const llvq_dn_latent* a, const void* y, int32_t ldy, int32_t q_rank, const float* q_norm, void* cq,
                         int64_t pos0, int32_t rows, int32_t store_kv, llvq_dn_stream stream);
+/* gate_up and bias in (gate, up) pairs: [rows, n, 2] and [n, 2] -> [rows, n]. */
 int llvq_dn_glu_rows(int32_t dtype, const void* gate_up, const float* bias, void* out, int32_t rows, int32_t n, float limit, float gain,
                      float shift, llvq_dn_stream stream);
 int llvq_dn_softcap(float* y, size_t n, float cap, llvq_dn_stream stream);

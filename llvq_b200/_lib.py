@@ -40,12 +40,12 @@ class ArchiveRawInfo(C.Structure):
 
 
 DN_F32, DN_BF16 = 0, 1
-DN_PLAIN, DN_EMBED, DN_NORM, DN_GLU = 0, 1, 2, 3
+DN_PLAIN, DN_EMBED, DN_NORM = 0, 1, 2
 
 
 class DenseGemv(C.Structure):
     """llvq_dn_gemv_desc of include/llvq_dense.h."""
-    _fields_ = ([(n, C.c_int32) for n in ("dtype", "prologue", "n_out", "k", "ldw", "ld_table", "table_rows")] +
+    _fields_ = ([(n, C.c_int32) for n in ("dtype", "prologue", "glu", "n_out", "k", "ldw", "ld_table", "table_rows")] +
                 [(n, C.c_float) for n in ("alpha", "eps", "scale", "limit", "gain", "shift", "softcap")] +
                 [(n, C.c_void_p) for n in ("w", "bias", "y", "x", "delta", "norm_w", "a_out", "table", "token")])
 

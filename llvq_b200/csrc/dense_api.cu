@@ -38,9 +38,9 @@ int check_gemv(const llvq_dn_gemv_desc* d, const char* who) {
     const int vn = 16 / elem_size(d->dtype);
     if (!d->w || d->n_out <= 0 || d->k <= 0 || d->ldw < d->k || d->ldw % vn || ((uintptr_t)d->w & 15))
         return fail(kStatusInvalid, "%s: matrix of %d x %d, row stride %d (a multiple of %d, 16-byte aligned)", who, d->n_out, d->k, d->ldw, vn);
+    if (d->glu && d->n_out % 2) return fail(kStatusInvalid, "%s: %d rows are not (gate, up) pairs", who, d->n_out);
     switch (d->prologue) {
         case LLVQ_DN_PLAIN:
-        case LLVQ_DN_GLU:
             if (!d->x) return fail(kStatusInvalid, "%s: null activation", who);
             break;
         case LLVQ_DN_NORM:
@@ -94,13 +94,13 @@ bool plan_stream(DenseGemvArgs& a, int* grid, size_t* smem) {
     a.slots = std::max(2, std::min(kGsMaxSlots, kGsRingBytes / (a.segv * 16)));
     const int groups = kGvWarps / a.nseg;
     *grid = std::min((a.n_out + groups - 1) / groups, sm_count());
-    *smem = (size_t)kGvWarps * a.slots * a.segv * 16 + (size_t)(a.n_out / *grid + 1) * a.nseg * sizeof(float);
+    *smem = (size_t)kGvWarps * a.slots * a.segv * 16 + (size_t)(a.n_out / *grid + 2) * a.nseg * sizeof(float);
     return *smem <= kMaxSmem - 2048;
 }
 
 template <typename T, int PRO, bool HEAD>
 int launch_gemv(const DenseGemvArgs& a, int grid, cudaStream_t s) {
-    const int rows = a.n_out / grid + 1;
+    const int rows = a.n_out / grid + 2;  // pairs stay together
     const size_t smem = ((size_t)a.ldw + (size_t)rows * a.kslices) * sizeof(float);
     if (smem > kMaxSmem) return fail(kStatusUnsupported, "dn_gemv: %d columns need %zu bytes of shared memory", a.k, smem);
     if (smem > 40 * 1024) {
@@ -118,13 +118,14 @@ int gemv_t(const llvq_dn_gemv_desc* d, HeadBest* best, int* grid_out, cudaStream
     a.w = d->w, a.bias = d->bias, a.y = d->y, a.x = d->x, a.delta = d->delta, a.norm_w = d->norm_w, a.a_out = d->a_out;
     a.table = d->table, a.token = (const long long*)d->token, a.best = best;
     a.n_out = d->n_out, a.k = d->k, a.ldw = d->ldw, a.ld_table = d->ld_table, a.table_rows = d->table_rows;
+    a.glu = d->glu;
     a.alpha = d->alpha, a.eps = d->eps, a.scale = d->scale, a.limit = d->limit, a.gain = d->gain, a.shift = d->shift, a.cap = d->softcap;
     // column slices: enough lanes for a row's vectors; rows of a CTA are shared by the row groups that are left
     if constexpr (sizeof(T) == 2) {
         size_t smem = 0;
         int grid = 0;
         a.err = device_error();
-        a.vec_x = !(((uintptr_t)a.x | (uintptr_t)a.delta | (uintptr_t)a.norm_w) & 15) && (d->prologue != LLVQ_DN_GLU || a.k % 4 == 0);
+        a.vec_x = !(((uintptr_t)a.x | (uintptr_t)a.delta | (uintptr_t)a.norm_w) & 15);
         if (a.err && plan_stream(a, &grid, &smem)) {
             if (grid_out) *grid_out = grid;
             if (best) {
@@ -135,8 +136,7 @@ int gemv_t(const llvq_dn_gemv_desc* d, HeadBest* best, int* grid_out, cudaStream
             switch (d->prologue) {
                 case LLVQ_DN_PLAIN: return launch_stream<kGvPlain, false>(a, grid, smem, s);
                 case LLVQ_DN_EMBED: return launch_stream<kGvEmbed, false>(a, grid, smem, s);
-                case LLVQ_DN_NORM: return launch_stream<kGvNorm, false>(a, grid, smem, s);
-                default: return launch_stream<kGvGlu, false>(a, grid, smem, s);
+                default: return launch_stream<kGvNorm, false>(a, grid, smem, s);
             }
         }
     }
@@ -154,8 +154,7 @@ int gemv_t(const llvq_dn_gemv_desc* d, HeadBest* best, int* grid_out, cudaStream
     switch (d->prologue) {
         case LLVQ_DN_PLAIN: return launch_gemv<T, kGvPlain, false>(a, grid, s);
         case LLVQ_DN_EMBED: return launch_gemv<T, kGvEmbed, false>(a, grid, s);
-        case LLVQ_DN_NORM: return launch_gemv<T, kGvNorm, false>(a, grid, s);
-        default: return launch_gemv<T, kGvGlu, false>(a, grid, s);
+        default: return launch_gemv<T, kGvNorm, false>(a, grid, s);
     }
 }
 
@@ -278,6 +277,7 @@ int llvq_dn_gemv(const llvq_dn_gemv_desc* d, llvq_dn_stream stream) {
 int llvq_dn_head(const llvq_dn_gemv_desc* d, void* scratch, float* val_out, int64_t* idx_out, llvq_dn_stream stream) {
     int st = check_gemv(d, "dn_head");
     if (st) return st;
+    if (d->glu) return fail(kStatusUnsupported, "dn_head: rows in pairs");
     if (!scratch || !val_out || !idx_out) return fail(kStatusInvalid, "dn_head: null argument");
     cudaStream_t s = (cudaStream_t)stream;
     int grid = 0;
@@ -353,6 +353,7 @@ int llvq_dn_postnorm_rows(int32_t dtype, const float* x, const void* y, const fl
                           void* xt, float* out, int32_t rows, int32_t n, llvq_dn_stream stream) {
     if (bad_dtype(dtype) || !x || !w || rows <= 0 || n <= 0 || (size_t)n * 4 > kMaxSmem - 1024) return fail(kStatusInvalid, "dn_postnorm_rows: bad argument");
     cudaStream_t s = (cudaStream_t)stream;
+    const int vec = n % 4 == 0 && !(((uintptr_t)x | (uintptr_t)y | (uintptr_t)bias | (uintptr_t)w | (uintptr_t)xt | (uintptr_t)out) & 15);
     const size_t smem = (size_t)n * 4;
     const void* f = dtype == LLVQ_DN_BF16 ? (const void*)postnorm_rows_kernel<bf16> : (const void*)postnorm_rows_kernel<float>;
     if (smem > 40 * 1024) {
@@ -360,9 +361,9 @@ int llvq_dn_postnorm_rows(int32_t dtype, const float* x, const void* y, const fl
         if (st) return st;
     }
     if (dtype == LLVQ_DN_BF16)
-        CUDA_TRY(launch_dep(postnorm_rows_kernel<bf16>, dim3(rows), dim3(kRowThreads), smem, s, x, (const bf16*)y, bias, w, alpha, eps, (bf16*)xt, out, n));
+        CUDA_TRY(launch_dep(postnorm_rows_kernel<bf16>, dim3(rows), dim3(kRowThreads), smem, s, x, (const bf16*)y, bias, w, alpha, eps, (bf16*)xt, out, n, vec));
     else
-        CUDA_TRY(launch_dep(postnorm_rows_kernel<float>, dim3(rows), dim3(kRowThreads), smem, s, x, (const float*)y, bias, w, alpha, eps, (float*)xt, out, n));
+        CUDA_TRY(launch_dep(postnorm_rows_kernel<float>, dim3(rows), dim3(kRowThreads), smem, s, x, (const float*)y, bias, w, alpha, eps, (float*)xt, out, n, vec));
     g_launches++;
     return kStatusOk;
 }
@@ -391,11 +392,12 @@ int llvq_dn_glu_rows(int32_t dtype, const void* gate_up, const float* bias, void
                      float shift, llvq_dn_stream stream) {
     if (bad_dtype(dtype) || !gate_up || !out || rows <= 0 || n <= 0) return fail(kStatusInvalid, "dn_glu_rows: bad argument");
     cudaStream_t s = (cudaStream_t)stream;
-    const dim3 grid(rows, std::max(1, std::min(8, n / (4 * kRowThreads))));
+    const int vec = n % 4 == 0 && !(((uintptr_t)gate_up | (uintptr_t)bias | (uintptr_t)out) & 15);
+    const dim3 grid(rows, (n + 8 * kRowThreads - 1) / (8 * kRowThreads));
     if (dtype == LLVQ_DN_BF16)
-        CUDA_TRY(launch_dep(glu_rows_kernel<bf16>, grid, dim3(kRowThreads), 0, s, (const bf16*)gate_up, bias, (bf16*)out, n, limit, gain, shift));
+        CUDA_TRY(launch_dep(glu_rows_kernel<bf16>, grid, dim3(kRowThreads), 0, s, (const bf16*)gate_up, bias, (bf16*)out, n, limit, gain, shift, vec));
     else
-        CUDA_TRY(launch_dep(glu_rows_kernel<float>, grid, dim3(kRowThreads), 0, s, (const float*)gate_up, bias, (float*)out, n, limit, gain, shift));
+        CUDA_TRY(launch_dep(glu_rows_kernel<float>, grid, dim3(kRowThreads), 0, s, (const float*)gate_up, bias, (float*)out, n, limit, gain, shift, vec));
     g_launches++;
     return kStatusOk;
 }

@@ -4,7 +4,7 @@
 //   postnorm_rows_kernel  t = alpha * x + y (+ bias); x = t / sqrt(mean(t^2) + eps) * w, and its T copy
 //   latent_rows_kernel  the down projections of a latent-attention layer: the query latent normed into cq, the
 //                       token's cache row normed, rotated and stored into the ring
-//   glu_rows_kernel     clamped gated unit of [gate | up] with their biases
+//   glu_rows_kernel     clamped gated unit of (gate, up) pairs with their biases
 //   softcap_kernel      logits <- cap * tanh(logits / cap)
 #pragma once
 #include "latent_attn.cuh"
@@ -29,27 +29,72 @@ embed_rows_kernel(const T* __restrict__ table, int ld, int table_rows, const lon
     }
 }
 
-// Dynamic shared memory: n floats. out may be x: a CTA has read its row before it writes; y may be null (alpha = 1: a plain norm).
+// Four consecutive values as f32 and back.
+template <typename T>
+__device__ __forceinline__ float4 load4(const T* p) {
+    if constexpr (sizeof(T) == 4) {
+        return *reinterpret_cast<const float4*>(p);
+    } else {
+        const uint2 u = *reinterpret_cast<const uint2*>(p);
+        return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xffff0000u));
+    }
+}
+template <typename T>
+__device__ __forceinline__ void store4(T* p, float4 v) {
+    if constexpr (sizeof(T) == 4) {
+        *reinterpret_cast<float4*>(p) = v;
+    } else {
+        __align__(16) const T r[4] = {from_f32<T>(v.x), from_f32<T>(v.y), from_f32<T>(v.z), from_f32<T>(v.w)};
+        *reinterpret_cast<uint2*>(p) = *reinterpret_cast<const uint2*>(r);
+    }
+}
+
+// Dynamic shared memory: n floats. out may be x: a CTA has read its row before it writes; y may be null (alpha = 1: a
+// plain norm). vec: n % 4 == 0 and every row on a 16-byte boundary.
 template <typename T>
 __global__ void __launch_bounds__(kRowThreads)
 postnorm_rows_kernel(const float* x, const T* __restrict__ y, const float* __restrict__ bias, const float* __restrict__ w,
-                     float alpha, float eps, T* __restrict__ xt, float* out, int n) {
+                     float alpha, float eps, T* __restrict__ xt, float* out, int n, int vec) {
     extern __shared__ __align__(16) float row_s[];
     __shared__ float red[kRowThreads / 32];
     llvq_dependent_enter();
     const size_t o = (size_t)blockIdx.x * n;
     float ss = 0.0f;
-    for (int i = threadIdx.x; i < n; i += kRowThreads) {
-        float t = alpha * x[o + i];
-        if (y) t += to_f32(y[o + i]) + (bias ? bias[i] : 0.0f);
-        row_s[i] = t;
-        ss = fmaf(t, t, ss);
+    if (vec) {
+        for (int i = 4 * threadIdx.x; i < n; i += 4 * kRowThreads) {
+            float4 t = load4(x + o + i);
+            t.x *= alpha, t.y *= alpha, t.z *= alpha, t.w *= alpha;
+            if (y) {
+                const float4 d = load4(y + o + i);
+                const float4 b = bias ? load4(bias + i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                t.x += d.x + b.x, t.y += d.y + b.y, t.z += d.z + b.z, t.w += d.w + b.w;
+            }
+            *reinterpret_cast<float4*>(row_s + i) = t;
+            ss = fmaf(t.x, t.x, fmaf(t.y, t.y, fmaf(t.z, t.z, fmaf(t.w, t.w, ss))));
+        }
+    } else {
+        for (int i = threadIdx.x; i < n; i += kRowThreads) {
+            float t = alpha * x[o + i];
+            if (y) t += to_f32(y[o + i]) + (bias ? bias[i] : 0.0f);
+            row_s[i] = t;
+            ss = fmaf(t, t, ss);
+        }
     }
     const float r = 1.0f / sqrtf(block_sum_f(ss, red) / (float)n + eps);
-    for (int i = threadIdx.x; i < n; i += kRowThreads) {
-        const float v = row_s[i] * r * w[i];
-        if (out) out[o + i] = v;
-        if (xt) xt[o + i] = from_f32<T>(v);
+    if (vec) {
+        for (int i = 4 * threadIdx.x; i < n; i += 4 * kRowThreads) {
+            float4 t = *reinterpret_cast<const float4*>(row_s + i);
+            const float4 f = load4(w + i);
+            t.x *= r * f.x, t.y *= r * f.y, t.z *= r * f.z, t.w *= r * f.w;
+            if (out) store4(out + o + i, t);
+            if (xt) store4(xt + o + i, t);
+        }
+    } else {
+        for (int i = threadIdx.x; i < n; i += kRowThreads) {
+            const float v = row_s[i] * r * w[i];
+            if (out) out[o + i] = v;
+            if (xt) xt[o + i] = from_f32<T>(v);
+        }
     }
 }
 
@@ -72,14 +117,48 @@ latent_rows_kernel(const T* __restrict__ y, int ldy, int q_rank, const float* __
     if (ring.rows) store_latent_row<T>(row + q_rank, kv_norm, eps, kv_rank, rot_dim, rt, pos0 + blockIdx.x, ring, red);
 }
 
+// gu: [rows, n, 2] (gate, up) pairs, bias: [n, 2] or null. grid = (rows, ceil(n / (8 threads))); a thread takes four
+// neighbouring outputs at a time where the row allows 16-byte loads (vec).
 template <typename T>
 __global__ void __launch_bounds__(kRowThreads)
-glu_rows_kernel(const T* __restrict__ gu, const float* __restrict__ bias, T* __restrict__ out, int n, float limit, float gain, float shift) {
+glu_rows_kernel(const T* __restrict__ gu, const float* __restrict__ bias, T* __restrict__ out, int n, float limit, float gain, float shift, int vec) {
     llvq_dependent_enter();
     const T* g = gu + (size_t)blockIdx.x * 2 * n;
-    for (int i = threadIdx.x + blockIdx.y * kRowThreads; i < n; i += kRowThreads * gridDim.y) {
-        const float bg = bias ? bias[i] : 0.0f, bu = bias ? bias[n + i] : 0.0f;
-        out[(size_t)blockIdx.x * n + i] = from_f32<T>(clamped_glu(to_f32(g[i]) + bg, to_f32(g[n + i]) + bu, limit, gain, shift));
+    T* o = out + (size_t)blockIdx.x * n;
+    const int lo = blockIdx.y * 8 * kRowThreads, hi = min(n, lo + 8 * kRowThreads);
+    if (vec) {  // n % 4 == 0, rows on 16-byte boundaries
+        constexpr int LV = 8 * sizeof(T) / 16;  // 16-byte loads of four pairs
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            const int i = lo + 4 * (threadIdx.x + k * kRowThreads);
+            if (i >= hi) break;
+            float f[8], b[8];
+#pragma unroll
+            for (int j = 0; j < LV; ++j) {
+                float t[Vec16<T>::N];
+                Vec16<T>::widen(__ldg(reinterpret_cast<const uint4*>(g + 2 * i) + j), t);
+#pragma unroll
+                for (int e = 0; e < Vec16<T>::N; ++e) f[j * Vec16<T>::N + e] = t[e];
+            }
+#pragma unroll
+            for (int j = 0; j < 8; ++j) b[j] = 0.0f;
+            if (bias) {
+                const float4 u = __ldg(reinterpret_cast<const float4*>(bias + 2 * i)), v = __ldg(reinterpret_cast<const float4*>(bias + 2 * i) + 1);
+                b[0] = u.x, b[1] = u.y, b[2] = u.z, b[3] = u.w, b[4] = v.x, b[5] = v.y, b[6] = v.z, b[7] = v.w;
+            }
+            __align__(16) T r[4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) r[j] = from_f32<T>(clamped_glu(f[2 * j] + b[2 * j], f[2 * j + 1] + b[2 * j + 1], limit, gain, shift));
+            if constexpr (sizeof(T) == 2)
+                *reinterpret_cast<uint2*>(o + i) = *reinterpret_cast<const uint2*>(r);
+            else
+                *reinterpret_cast<uint4*>(o + i) = *reinterpret_cast<const uint4*>(r);
+        }
+        return;
+    }
+    for (int i = lo + threadIdx.x; i < hi; i += kRowThreads) {
+        const float bg = bias ? bias[2 * i] : 0.0f, bu = bias ? bias[2 * i + 1] : 0.0f;
+        o[i] = from_f32<T>(clamped_glu(to_f32(g[2 * i]) + bg, to_f32(g[2 * i + 1]) + bu, limit, gain, shift));
     }
 }
 

@@ -14,8 +14,8 @@ the rest in row kernels and one attention kernel). The token step keeps everythi
                 attention over the ring, split over positions      (llvq_dn_latent_decode)
                 merge, sink, value expansion                       (llvq_dn_latent_value)
                 o                                               (plain)
-                [gate | up] with the norm of the sum before it  (norm prologue)
-                down with the gated unit                        (glu prologue)
+                gate and up with the norm of the sum before it, the gated unit of their sums (norm prologue, glu epilogue)
+                down                                            (plain)
     then        the last norm, and the head with the final norm, soft cap and greedy pick
 
 The residual stream, norms, rotations, scores, softmax and the token step's activations are f32 in both element
@@ -116,14 +116,21 @@ class LatentConfig:
 
 
 class DenseMatrix:
-    """Row-concatenated [out, in] matrices on the device, rows padded with zeros to whole 16-byte vectors."""
+    """Row-concatenated (or row-interleaved) [out, in] matrices on the device, rows padded with zeros to whole 16-byte
+    vectors."""
 
-    def __init__(self, parts, dtype, device):
+    def __init__(self, parts, dtype, device, interleave: bool = False):
         import torch
         self.n, self.k = sum(p.shape[0] for p in parts), parts[0].shape[1]
         vec = 16 // torch.empty(0, dtype=dtype).element_size()
         self.ld = -(-self.k // vec) * vec
         self.w = torch.zeros(self.n, self.ld, dtype=dtype, device=device)
+        if interleave:
+            if len({p.shape[0] for p in parts}) != 1:
+                raise ValueError(f"interleaved matrices of {[p.shape[0] for p in parts]} rows")
+            for i, p in enumerate(parts):
+                self.w[i::len(parts), :self.k].copy_(p)
+            return
         at = 0
         for p in parts:
             self.w[at:at + p.shape[0], :self.k].copy_(p)
@@ -149,9 +156,8 @@ class LatentLM(TokenLoop):
         self._init_loop(device, capacity, prefill_chunk)
         f32 = dict(dtype=torch.float32, device=device)
 
-        def mat(*names):
-            m = DenseMatrix([tensor(n) for n in names], self.dtype, device)
-            return m
+        def mat(*names, interleave: bool = False):
+            return DenseMatrix([tensor(n) for n in names], self.dtype, device, interleave)
 
         def vec(*names, base: float = 0.0):
             return torch.cat([tensor(n).to(**f32) for n in names]) + base
@@ -175,7 +181,8 @@ class LatentLM(TokenLoop):
                 self.rings.append(self.rings[a.kv_from])
             if lc.mlp is not None:
                 m = f"l{i}.mlp"
-                L.update(norm2=vec(f"l{i}.norm2", base=1.0), gate_up=mat(m + ".gate", m + ".up"), gate_up_b=vec(m + ".gate.b", m + ".up.b"),
+                L.update(norm2=vec(f"l{i}.norm2", base=1.0), gate_up=mat(m + ".gate", m + ".up", interleave=True),  # (gate, up) pairs
+                         gate_up_b=vec(m + ".gate.b", m + ".up.b").reshape(2, -1).t().reshape(-1).contiguous(),
                          down=mat(m + ".down"), down_b=vec(m + ".down.b"))
             self._check_layer(i, lc, L)
             if (a.rot_base, a.rot_dims) not in tables:  # angles in double, rounded once
@@ -224,7 +231,7 @@ class LatentLM(TokenLoop):
         self._q = buf(max(L["uq"].n for L in self.layers))
         self._ctx = buf(max(L["o"].k for L in self.layers))
         self._o, self._down = buf(cfg.width), buf(cfg.width)
-        self._gu = buf(max([L["gate_up"].n for L in self.layers if "gate_up" in L] or [1]))
+        self._act = buf(max([lc.mlp.ff for lc in cfg.layers if lc.mlp is not None] or [1]))
         self._qlat = buf(max(a.heads * r.ld for a, r in zip(attn, self.rings)))
         self._part = buf(max(a.heads * splits(a) * (a.kv_rank + 2) for a in attn))
         self._logits = buf(cfg.vocab)
@@ -269,8 +276,8 @@ class LatentLM(TokenLoop):
             gemv(L["o"], self._o, prologue=_lib.DN_PLAIN, x=ptr(self._ctx))
             pending = (self._o, L["norm1"])
             if lc.mlp is not None:
-                gemv(L["gate_up"], self._gu, L["gate_up_b"], **normed(*pending))
-                gemv(L["down"], self._down, L["down_b"], prologue=_lib.DN_GLU, x=ptr(self._gu), limit=lc.mlp.limit, gain=GLU_GAIN, shift=GLU_SHIFT)
+                gemv(L["gate_up"], self._act, L["gate_up_b"], glu=1, limit=lc.mlp.limit, gain=GLU_GAIN, shift=GLU_SHIFT, **normed(*pending))
+                gemv(L["down"], self._down, L["down_b"], prologue=_lib.DN_PLAIN, x=ptr(self._act))
                 pending = (self._down, L["norm2"])
         last, (delta, w) = self._stream[0], pending
         steps.append(("norm", lambda st: _lib.check_dense(lib.llvq_dn_postnorm_rows(

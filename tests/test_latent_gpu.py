@@ -86,7 +86,7 @@ def test_token_projection_and_its_prologues(dtype, n, k):
     w, x, delta, bias, nw = rnd(1, n, k), rnd(2, k), rnd(3, k), rnd(4, n), 1 + 0.3 * rnd(5, k)
     m = padded(w, dtype)
     y, a_out = torch.full((n,), 9.0, device="cuda"), torch.zeros(k, device="cuda")
-    g, bg = torch.cat([rnd(6, k), 2 * rnd(7, k)]).cuda(), bias.cuda()
+    bg = bias.cuda()
     xg, dg, nwg = x.cuda(), delta.cuda(), nw.cuda()
 
     def go(**kw):
@@ -107,9 +107,13 @@ def test_token_projection_and_its_prologues(dtype, n, k):
     close(go(prologue=_lib.DN_NORM, x=P(xg), delta=P(dg), alpha=1.7, norm_w=P(nwg), a_out=P(a_out)), plain.plain_norm(t, nw.double(), 1e-3))
     assert rel(a_out, plain.plain_norm(t, nw.double(), 1e-3)) < 1e-6 and torch.equal(xg.cpu(), x)
     close(go(prologue=_lib.DN_NORM, x=P(xg), alpha=1.0, norm_w=P(nwg)), plain.plain_norm(X, nw.double(), 1e-3))
-    gd = g.double().cpu()
-    gate, up = gd[:k].clamp(max=0.9), gd[k:].clamp(-0.9, 0.9)
-    close(go(prologue=_lib.DN_GLU, x=P(g), limit=0.9, gain=1.3, shift=0.5), gate * torch.sigmoid(1.3 * gate) * (up + 0.5))
+    if n % 2 == 0:  # rows in (gate, up) pairs
+        y = torch.full((n // 2,), 9.0, device="cuda")
+        s = (W @ plain.plain_norm(t, nw.double(), 1e-3) + bias.double()).reshape(-1, 2)
+        gate, up = s[:, 0].clamp(max=2.0), s[:, 1].clamp(-2.0, 2.0)
+        pairs = go(prologue=_lib.DN_NORM, x=P(xg), delta=P(dg), alpha=1.7, norm_w=P(nwg), bias=P(bg), glu=1, limit=2.0, gain=1.3, shift=0.5)
+        assert rel(pairs, gate * torch.sigmoid(1.3 * gate) * (up + 0.5)) < 1e-5
+        y = torch.full((n,), 9.0, device="cuda")
     table = rnd(8, 6, k)
     tm = padded(table, dtype)
     tok = torch.tensor([4], device="cuda")
@@ -164,11 +168,11 @@ def test_row_kernels(dtype, n):
     _lib.check_dense(L.llvq_dn_embed_rows(dn(dtype), tm.ptr(), tm.ld, 11, P(ids), rows, n, 0.3, P(out), P(xt), stream()))
     want = 0.3 * table[torch.tensor([3, 0, 10, 3, 0, 0, 7])].double()
     assert rel(out, want) < 1e-6 and rel(xt, want) < tol
-    gu, gb = 2 * rnd(26, rows, 2 * n), rnd(27, 2 * n)
+    gu, gb = 2 * rnd(26, rows, 2 * n), rnd(27, 2 * n)  # (gate, up) pairs
     gug, gbg, act = gu.to(T).cuda(), gb.cuda(), torch.zeros(rows, n, dtype=T, device="cuda")
     _lib.check_dense(L.llvq_dn_glu_rows(dn(dtype), P(gug), P(gbg), P(act), rows, n, 1.1, 1.702, 1.0, stream()))
     s = gu.double() + gb.double()
-    g, u = s[:, :n].clamp(max=1.1), s[:, n:].clamp(-1.1, 1.1)
+    g, u = s[:, 0::2].clamp(max=1.1), s[:, 1::2].clamp(-1.1, 1.1)
     assert rel(act, g * torch.sigmoid(1.702 * g) * (u + 1)) < tol
     v = 30 * rnd(28, 1000)
     vg = v.cuda()
