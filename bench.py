@@ -835,7 +835,7 @@ def run_latent(args):
         # kernels of one prompt portion: 2048 queries behind a full window
         n, T = prompt_len, prompt_len + window - 1
         new = lambda *s: torch.randn(*s, device="cuda").bfloat16()
-        sets = [dict(q=new(n, L["uq"].n), kv=new(T, L["ukv"].n), kr=new(T, a.rot_dim), out=new(n, a.heads * a.vdim), x=torch.randn(n, cfg.width, device="cuda"),
+        sets = [dict(q=new(n, L["uq"].n), k=new(T, a.heads * a.dim), vt=new(a.heads * a.vdim, T + 1), kr=new(T, a.rot_dim), out=new(n, a.heads * a.vdim), x=torch.randn(n, cfg.width, device="cuda"),
                      xt=new(n, cfg.width), y=new(n, cfg.width), gu=new(n, L["gate_up"].n), act=new(n, cfg.layers[0].mlp.ff),
                      yd=new(n, L["dq_dkv"].n), cq=new(n, a.q_rank)) for _ in range(3)]
         st, check = m._cuda_stream, _lib.check_dense
@@ -843,8 +843,8 @@ def run_latent(args):
 
         def attend(k):
             s = sets[k % 3]
-            check(lib.llvq_dn_latent_prefill(C.byref(lat), s["q"].data_ptr(), s["kv"].data_ptr(), s["kv"].shape[1], s["kr"].data_ptr(), a.rot_dim, n, T,
-                                             window - 1, 0, s["out"].data_ptr(), 0, st()))
+            check(lib.llvq_dn_latent_prefill(C.byref(lat), s["q"].data_ptr(), s["k"].data_ptr(), s["k"].shape[1], s["kr"].data_ptr(), a.rot_dim,
+                                             s["vt"].data_ptr(), s["vt"].shape[1], n, T, window - 1, 0, s["out"].data_ptr(), 0, st()))
 
         def norm(k):
             s = sets[k % 3]

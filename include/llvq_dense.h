@@ -84,9 +84,13 @@ int llvq_dn_latent_value(const llvq_dn_latent* a, float* ctx, llvq_dn_stream str
 /* Attention of a prompt portion: q [n_q, heads * (dim + rot_dim)] before rotation, kv [n_k, ld_kv] = expanded
  * [heads * dim keys | heads * vdim values], kr [n_k, ld_kr] rotated key parts; query i is position pos0 + i, key j
  * position key0 + j. out [n_q, heads * vdim]. Reads window, scale, sink, rot_dims, tables and sizes of `a`.
+ * vt: NULL, or, where llvq_dn_latent_prefill_transposes says 1 (the tcgen05 kernel serves the portion), the values apart
+ * and transposed, [heads * vdim, ld_vt], ld_vt a multiple of 8 and zeros from n_k to the next one; kv then holds keys only.
  * kernel: 0 = by size and type, 1 = the generic one. */
+int llvq_dn_latent_prefill_transposes(const llvq_dn_latent* a, int32_t n_q);
 int llvq_dn_latent_prefill(const llvq_dn_latent* a, const void* q, const void* kv, int32_t ld_kv, const void* kr, int32_t ld_kr,
-                           int32_t n_q, int32_t n_k, int64_t pos0, int64_t key0, void* out, int32_t kernel, llvq_dn_stream stream);
+                           const void* vt, int32_t ld_vt, int32_t n_q, int32_t n_k, int64_t pos0, int64_t key0, void* out, int32_t kernel,
+                           llvq_dn_stream stream);
 
 /* ---- rows of a prompt portion ---- */
 int llvq_dn_embed_rows(int32_t dtype, const void* table, int32_t ld, int32_t table_rows, const int64_t* tokens, int32_t rows, int32_t n,

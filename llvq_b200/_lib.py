@@ -148,7 +148,8 @@ _DENSE_SIGNATURES = {
     "llvq_dn_latent_query": (C.c_int, [C.POINTER(DenseLatent)] + [C.c_void_p] * 4),
     "llvq_dn_latent_decode": (C.c_int, [C.POINTER(DenseLatent)] + [C.c_void_p] * 2),
     "llvq_dn_latent_value": (C.c_int, [C.POINTER(DenseLatent)] + [C.c_void_p] * 2),
-    "llvq_dn_latent_prefill": (C.c_int, [C.POINTER(DenseLatent), C.c_void_p, C.c_void_p, C.c_int32, C.c_void_p, C.c_int32, C.c_int32, C.c_int32,
+    "llvq_dn_latent_prefill_transposes": (C.c_int, [C.POINTER(DenseLatent), C.c_int32]),
+    "llvq_dn_latent_prefill": (C.c_int, [C.POINTER(DenseLatent)] + [C.c_void_p, C.c_void_p, C.c_int32, C.c_void_p, C.c_int32] + [C.c_void_p, C.c_int32, C.c_int32, C.c_int32,
                                          C.c_int64, C.c_int64, C.c_void_p, C.c_int32, C.c_void_p]),
     "llvq_dn_embed_rows": (C.c_int, [C.c_int32, C.c_void_p, C.c_int32, C.c_int32, C.c_void_p, C.c_int32, C.c_int32, C.c_float] + [C.c_void_p] * 3),
     "llvq_dn_postnorm_rows": (C.c_int, [C.c_int32] + [C.c_void_p] * 4 + [C.c_float] * 2 + [C.c_void_p] * 2 + [C.c_int32] * 2 + [C.c_void_p]),

@@ -9,6 +9,7 @@
 #include "host_util.cuh"
 #include "latent_attn.cuh"
 #include "latent_prefill.cuh"
+#include "latent_prefill_tc.cuh"
 
 using namespace llvq;
 
@@ -248,6 +249,14 @@ int prefill_simt(const LatentPrefillArgs& p, cudaStream_t s) {
     return kStatusOk;
 }
 
+// The tcgen05 kernel takes heads of whole 16-byte vectors whose tiles fit shared memory and TMEM, and portions that
+// fill a good part of its query tiles.
+bool prefill_on_tc(const llvq_dn_latent* a, int n_q) {
+    const int qk = a->dim + a->rot_dim;
+    return a->dtype == LLVQ_DN_BF16 && n_q >= 64 && a->scale > 0.0f && !((a->dim | a->rot_dim | a->vdim | a->kv_rank) & 7) && tc_v_rows(a->vdim) <= 192 &&
+           latent_prefill_tc_smem(qk, a->vdim) <= kMaxSmem - 1024;
+}
+
 }  // namespace
 
 extern "C" {
@@ -317,16 +326,33 @@ int llvq_dn_latent_value(const llvq_dn_latent* a, float* ctx, llvq_dn_stream str
     return a->dtype == LLVQ_DN_BF16 ? latent_value_t<bf16>(a, ctx, (cudaStream_t)stream) : latent_value_t<float>(a, ctx, (cudaStream_t)stream);
 }
 
+int llvq_dn_latent_prefill_transposes(const llvq_dn_latent* a, int32_t n_q) {
+    return check_latent(a, "dn_latent_prefill_transposes") == kStatusOk && prefill_on_tc(a, n_q) ? 1 : 0;
+}
+
 int llvq_dn_latent_prefill(const llvq_dn_latent* a, const void* q, const void* kv, int32_t ld_kv, const void* kr, int32_t ld_kr,
-                           int32_t n_q, int32_t n_k, int64_t pos0, int64_t key0, void* out, int32_t kernel, llvq_dn_stream stream) {
+                           const void* vt, int32_t ld_vt, int32_t n_q, int32_t n_k, int64_t pos0, int64_t key0, void* out, int32_t kernel, llvq_dn_stream stream) {
     const int st = check_latent(a, "dn_latent_prefill");
     if (st) return st;
     if (!q || !kv || !kr || !out) return fail(kStatusInvalid, "dn_latent_prefill: null argument");
-    if (n_q <= 0 || n_k <= 0 || pos0 < 0 || key0 < 0 || key0 > pos0 || pos0 + n_q > key0 + n_k || ld_kv < a->heads * (a->dim + a->vdim) || ld_kr < a->rot_dim)
+    if (n_q <= 0 || n_k <= 0 || pos0 < 0 || key0 < 0 || key0 > pos0 || pos0 + n_q > key0 + n_k || ld_kv < a->heads * (a->dim + (vt ? 0 : a->vdim)) ||
+        ld_kr < a->rot_dim || (vt && ld_vt < n_k))
         return fail(kStatusInvalid, "dn_latent_prefill: %d queries at %lld over %d keys at %lld", n_q, (long long)pos0, n_k, (long long)key0);
     LatentPrefillArgs p{q, kv, kr, a->sink, out, rot_of(a), pos0, key0, n_q, n_k, a->heads, a->dim, a->rot_dim, a->vdim, ld_kv, ld_kr,
                         a->window, a->scale};
     cudaStream_t s = (cudaStream_t)stream;
+    if (vt) {
+        if (!prefill_on_tc(a, n_q) || ((ld_kv | ld_kr | ld_vt) & 7) || (((uintptr_t)q | (uintptr_t)kv | (uintptr_t)kr | (uintptr_t)vt | (uintptr_t)out) & 15))
+            return fail(kStatusInvalid, "dn_latent_prefill: transposed values where llvq_dn_latent_prefill_transposes says no, or rows not on 16 bytes");
+        LatentPrefillTcArgs tc{p, vt, ld_vt, device_error()};
+        if (!tc.err) return fail(kStatusCuda, "dn_latent_prefill: no error word");
+        const size_t smem = latent_prefill_tc_smem(a->dim + a->rot_dim, a->vdim);
+        const int st2 = ensure_dyn_smem((const void*)latent_prefill_tc_kernel, smem);
+        if (st2) return st2;
+        CUDA_TRY(launch_dep(latent_prefill_tc_kernel, dim3((n_q + 2 * kTcM - 1) / (2 * kTcM), a->heads), dim3(kTcThreads), smem, s, tc));
+        g_launches++;
+        return kStatusOk;
+    }
     if (a->dtype == LLVQ_DN_F32) return prefill_simt<float>(p, s);
     const int nv = a->vdim <= 64 ? 8 : a->vdim <= 128 ? 16 : 32;
     const size_t smem = latent_prefill_smem(a->dim, a->rot_dim, nv);

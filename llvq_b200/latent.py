@@ -322,6 +322,19 @@ class LatentLM(TokenLoop):
                 m.allow_tf32 = held
         return torch.mm(x, w.t()) if out_dtype is None else torch.mm(x, w.t(), out_dtype=out_dtype)
 
+    def _expand(self, c, ukv, a, transposed: bool):
+        """Keys and values of cached latents c [n, kv_rank]: ([n, keys | values], None), or ([n, keys], [values, n to a
+        multiple of 8]) for the attention kernel that reads the values along the positions."""
+        import torch
+        if not transposed:
+            return self._mm(c, ukv.rows(0)), None
+        n, split = c.shape[0], a.heads * a.dim
+        vt = torch.empty(a.heads * a.vdim, -(-n // 8) * 8, dtype=self.dtype, device=self.device)
+        if n % 8:
+            vt[:, n:].zero_()
+        torch.mm(ukv.rows(split), c.t(), out=vt[:, :n])
+        return self._mm(c, ukv.rows(0, split)), vt
+
     def hidden(self, tokens, pos, end: int, layers_out: Optional[list] = None):
         """tokens, pos: int64 [L], positions [end - L, end); returns the f32 stream [L, width] behind the last layer.
         `layers_out` collects a copy of the stream behind every layer."""
@@ -351,10 +364,11 @@ class LatentLM(TokenLoop):
             q = self._mm(cq, L["uq"].rows(0))
             lo = max(0, start - lat.window + 1)  # the first position any query of the portion sees
             rows = ring.read(lo, end)
-            kv = self._mm(rows[:, :a.kv_rank], L["ukv"].rows(0))
+            kv, vt = self._expand(rows[:, :a.kv_rank], L["ukv"], a, lib.llvq_dn_latent_prefill_transposes(C.byref(lat), n))
             ctx = new(n, a.heads * a.vdim)
             check(lib.llvq_dn_latent_prefill(C.byref(lat), q.data_ptr(), kv.data_ptr(), kv.shape[1],
-                                             rows.data_ptr() + a.kv_rank * rows.element_size(), ring.ld, n, end - lo, start, lo, ctx.data_ptr(), 0, st))
+                                             rows.data_ptr() + a.kv_rank * rows.element_size(), ring.ld, vt.data_ptr() if vt is not None else None,
+                                             vt.shape[1] if vt is not None else 0, n, end - lo, start, lo, ctx.data_ptr(), 0, st))
             add_norm(self._mm(ctx, L["o"].rows(0)), None, L["norm1"])
             if lc.mlp is not None:
                 gu = self._mm(xt, L["gate_up"].rows(0))

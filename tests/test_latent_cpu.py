@@ -43,7 +43,9 @@ def test_bad_arguments_are_refused_without_a_gpu():
     assert L.llvq_dn_latent_decode(C.byref(a), 16, None) == bad and b"rotated" in L.llvq_dn_last_error()
     a.rot_dims = 4
     assert L.llvq_dn_latent_decode(C.byref(a), 16, None) == bad and b"window of 9 over 8" in L.llvq_dn_last_error()
-    assert L.llvq_dn_latent_prefill(C.byref(a), 16, 16, 32, 16, 4, 4, 4, 5, 2, 16, 0, None) == bad  # query 8 has no key
+    assert L.llvq_dn_latent_prefill(C.byref(a), 16, 16, 32, 16, 4, None, 0, 4, 4, 5, 2, 16, 0, None) == bad  # query 8 has no key
+    assert L.llvq_dn_latent_prefill(C.byref(a), 16, 16, 32, 16, 4, 16, 8, 4, 4, 2, 2, 16, 0, None) == bad  # no transposed values in f32
+    assert L.llvq_dn_latent_prefill_transposes(C.byref(a), 500) == 0
     assert L.llvq_dn_latent_rows(C.byref(a), 16, 64, 8, 16, 16, 0, 9, 0, None) == bad  # nine rows into eight slots
     assert L.llvq_dn_softcap(16, 4, 0.0, None) == bad
     with pytest.raises(_lib.LlvqError):

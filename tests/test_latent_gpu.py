@@ -122,9 +122,7 @@ def test_token_projection_and_its_prologues(dtype, n, k):
     assert rel(a_out, 0.6 * table[4]) < 1e-6
     tok.fill_(6)  # outside the table: row 0, not foreign memory
     close(go(**emb), 0.6 * table[0].double())
-    err = C.c_int32(7)
-    _lib.check_dense(L.llvq_dn_poll_error(C.byref(err)))
-    assert err.value == 0
+    no_time_out()
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -180,6 +178,13 @@ def test_row_kernels(dtype, n):
     assert rel(vg, 5 * torch.tanh(v.double() / 5)) < 1e-6
 
 
+def no_time_out():
+    _lib, L = lib()
+    err = C.c_int32(7)
+    _lib.check_dense(L.llvq_dn_poll_error(C.byref(err)))
+    assert err.value == 0
+
+
 class Attention:
     """One latent-attention layer's operands: random latents, keys and queries of n positions, and the descriptor."""
 
@@ -232,7 +237,9 @@ class Attention:
         return ctx.cpu()
 
     def prefill(self, lo, hi, kernel=0, key0=None):
-        """Queries lo .. hi - 1 over keys key0 (by default the first one any of them sees) .. hi - 1."""
+        """Queries lo .. hi - 1 over keys key0 (by default the first one any of them sees) .. hi - 1. kernel: 0 = the one
+        the library picks, 1 = the generic one, 2 = the one for values along the keys where the library prefers them
+        transposed."""
         _lib, L = lib()
         T = TYPES[self.dtype]
         key0 = max(0, lo - self.window + 1) if key0 is None else key0
@@ -242,14 +249,21 @@ class Attention:
         rows = torch.zeros(hi - key0, self.ring.ld, dtype=T, device="cuda")
         rows[:, self.rank:self.rank + self.rot] = self.kr[key0:hi].to(T).cuda()
         out = torch.full((hi - lo, self.H, self.vdim), 7.0, dtype=T, device="cuda")
+        vt, split = None, self.H * self.dim
+        if kernel == 0 and L.llvq_dn_latent_prefill_transposes(C.byref(self.d), hi - lo):
+            vt = torch.zeros(self.H * self.vdim, -(-kv.shape[0] // 8) * 8, dtype=T, device="cuda")
+            vt[:, :kv.shape[0]] = kv[:, split:].t()
+            kv = kv[:, :split].contiguous()
+        self.transposed = vt is not None
         _lib.check_dense(L.llvq_dn_latent_prefill(C.byref(self.d), P(q), P(kv), kv.shape[1], P(rows) + self.rank * rows.element_size(), self.ring.ld,
-                                                  hi - lo, hi - key0, lo, key0, P(out), kernel, stream()))
+                                                  P(vt), vt.shape[1] if vt is not None else 0, hi - lo, hi - key0, lo, key0, P(out), 1 if kernel == 1 else 0, stream()))
         return out.float().cpu()
 
 
 HEADS = [  # heads, dim, rot, vdim, kv_rank, rot_dims
     (3, 24, 8, 40, 56, None), (5, 17, 6, 9, 30, None), (9, 32, 16, 48, 128, None), (2, 128, 64, 128, 512, None), (1, 192, 32, 200, 96, None),
-    (1, 700, 40, 300, 64, None), (2, 16, 12, 20, 24, 6), (17, 8, 2, 8, 8, None), (2, 3, 2, 17, 5, None)]
+    (1, 700, 40, 300, 64, None), (2, 16, 12, 20, 24, 6), (17, 8, 2, 8, 8, None), (2, 3, 2, 17, 5, None),
+    (2, 64, 32, 80, 24, None), (1, 8, 8, 8, 8, None), (3, 40, 8, 184, 32, 4), (1, 120, 56, 192, 16, None)]
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -266,8 +280,31 @@ def test_prompt_attention(dtype, shape, window):
         worst = (got.double() - want[lo:hi]).flatten(1).norm(dim=1) / want[lo:hi].flatten(1).norm(dim=1)
         assert worst.max() < 4 * tol, (lo, hi, int(worst.argmax()))
     if dtype == "bfloat16":
-        assert rel(a.prefill(37, 140, kernel=1), want[37:140]) < tol
+        for kernel in (1, 2):
+            assert rel(a.prefill(37, 140, kernel=kernel), want[37:140]) < tol
     assert rel(a.prefill(200, 290, key0=0), want[200:290]) < tol  # keys ahead of every window are ignored
+    no_time_out()
+
+
+@pytest.mark.parametrize("window", [1, 64, 129, 700, 5000])
+def test_prompt_attention_of_long_portions_on_the_tensor_cores(window):
+    """Several query tiles of 128 and pairs of them, ragged ends, scores that grow along the keys (the running maximum is
+    raised again and again, and by more than the rescaling threshold)."""
+    a = Attention("bfloat16", 2, 128, 64, 128, 64, 900, window, 900, seed=2, scale=4.0 * 192 ** -0.5)
+    for grow in (False, True):
+        if grow:
+            u = torch.randn(64, generator=gen(9))
+            a.c = (a.c * 0.05 + torch.linspace(0, 3, 900)[:, None] * u / u.norm() * 2).bfloat16().float()
+            k = (u.double() @ a.uk.double().T).reshape(1, 2, 128)
+            a.qn = (a.qn * 0.1 + (k / k.norm(dim=-1, keepdim=True)).float() * 6).bfloat16().float()
+        want = a.want()
+        for lo, hi in ((0, 900), (0, 129), (100, 228), (131, 700), (640, 900), (0, 64)):
+            got = a.prefill(lo, hi)
+            assert a.transposed
+            assert rel(got, want[lo:hi]) < 1.2e-2, (grow, lo, hi)
+            worst = (got.double() - want[lo:hi]).flatten(1).norm(dim=1) / want[lo:hi].flatten(1).norm(dim=1)
+            assert worst.max() < 4e-2, (grow, lo, hi, int(worst.argmax()))
+    no_time_out()
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
