@@ -154,42 +154,77 @@ latent_prefill_tc_kernel(LatentPrefillTcArgs T) {
     }
     llvq_dependent_enter();
 
-    // ---- query tiles, rotated: rows beyond the portion and columns beyond qk are zero ----
+    // ---- query tiles, rotated: rows beyond the portion and columns beyond qk are zero. Eight lanes bring the 128 bytes of
+    // a row's panel, a warp four rows at a time ----
     {
-        const bf16* Q = reinterpret_cast<const bf16*>(A.q);
+        const bf16* Q = reinterpret_cast<const bf16*>(A.q) + (size_t)h * qk;
         const size_t qrow = (size_t)A.heads * qk;
-        const int cn = A.dim / 8, half = A.rt.dims / 2, pieces = panels * 8;
-        const int rows = two ? 2 * kTcM : kTcM;
-        for (int i = tid; i < rows * pieces; i += kTcThreads) {
-            const int r = i / pieces, c = i - r * pieces;
+        const int cn = A.dim / 8, half = A.rt.dims / 2, rows = two ? 2 * kTcM : kTcM;
+        for (int p = 0; p < panels; ++p) {
+            const int c = p * 8 + (lane & 7);
             if (c >= cn && 8 * c < qk) continue;  // the rotated part comes below
-            unsigned char* dst = base0 + (r >= kTcM ? q_bytes : 0) + (c >> 3) * (kTcM * 128) + tc_swz(r & (kTcM - 1), c & 7);
-            const bool in = c < cn && q_lo + r < A.n_q;
-            *reinterpret_cast<uint4*>(dst) = in ? *reinterpret_cast<const uint4*>(Q + (size_t)(q_lo + r) * qrow + (size_t)h * qk + 8 * c) : make_uint4(0, 0, 0, 0);
-        }
-        const int rest = A.rot_dim - half;  // pairs, then what passes
-        auto put = [&](int r, int c, bf16 v) {
-            const int col = A.dim + c;
-            *reinterpret_cast<bf16*>(base0 + (r >= kTcM ? q_bytes : 0) + (col >> 6) * (kTcM * 128) + tc_swz(r & (kTcM - 1), (col & 63) >> 3) + 2 * (col & 7)) = v;
-        };
-        for (int i = tid; i < rows * rest; i += kTcThreads) {
-            const int r = i / rest, c = i - r * rest;
-            const bool in = q_lo + r < A.n_q;
-            const bf16* src = Q + (size_t)(q_lo + r) * qrow + (size_t)h * qk + A.dim;
-            if (c < half) {
-                float a = 0.0f, b = 0.0f;
-                if (in) {
-                    const size_t p = (size_t)(A.pos0 + q_lo + r) * half + c;
-                    const float cs = A.rt.cos_t[p], sn = A.rt.sin_t[p], u = to_f32(src[c]), v = to_f32(src[c + half]);
-                    a = u * cs - v * sn;
-                    b = v * cs + u * sn;
-                }
-                put(r, c, from_f32<bf16>(a));
-                put(r, c + half, from_f32<bf16>(b));
-            } else {
-                put(r, c + half, in ? src[c + half] : __float2bfloat16_rn(0.0f));
+#pragma unroll 4
+            for (int r = warp * 4 + (lane >> 3); r < rows; r += kTcThreads / 8) {
+                const bool in = c < cn && q_lo + r < A.n_q;
+                copy16_async(reinterpret_cast<bf16*>(base0 + (r >= kTcM ? q_bytes : 0) + p * (kTcM * 128) + tc_swz(r & (kTcM - 1), lane & 7)),
+                             in ? Q + (size_t)(q_lo + r) * qrow + 8 * c : Q, in);
             }
         }
+        auto at = [&](int r, int col) {
+            return base0 + (r >= kTcM ? q_bytes : 0) + (col >> 6) * (kTcM * 128) + tc_swz(r & (kTcM - 1), (col & 63) >> 3) + 2 * (col & 7);
+        };
+        if (half % 8 == 0) {  // whole vectors of pairs
+            const int hp = half / 8, per = hp + (A.rot_dim - 2 * half) / 8;
+#pragma unroll 2
+            for (int i = tid; i < rows * per; i += kTcThreads) {
+                const int r = i / per, c = i - r * per;
+                const bool in = q_lo + r < A.n_q;
+                const bf16* src = Q + (size_t)(q_lo + r) * qrow + A.dim;
+                const uint4 zero = make_uint4(0, 0, 0, 0);
+                if (c >= hp) {
+                    *reinterpret_cast<uint4*>(at(r, A.dim + half + 8 * c)) = in ? *reinterpret_cast<const uint4*>(src + half + 8 * c) : zero;
+                    continue;
+                }
+                uint4 a = zero, b = zero;
+                if (in) {
+                    float u[8], v[8], x[8], y[8];
+                    Vec16<bf16>::widen(*reinterpret_cast<const uint4*>(src + 8 * c), u);
+                    Vec16<bf16>::widen(*reinterpret_cast<const uint4*>(src + half + 8 * c), v);
+                    const size_t p = (size_t)(A.pos0 + q_lo + r) * half + 8 * c;
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) {
+                        const float cs = A.rt.cos_t[p + j], sn = A.rt.sin_t[p + j];
+                        x[j] = u[j] * cs - v[j] * sn;
+                        y[j] = v[j] * cs + u[j] * sn;
+                    }
+                    a = make_uint4(pack_bf16(x[0], x[1]), pack_bf16(x[2], x[3]), pack_bf16(x[4], x[5]), pack_bf16(x[6], x[7]));
+                    b = make_uint4(pack_bf16(y[0], y[1]), pack_bf16(y[2], y[3]), pack_bf16(y[4], y[5]), pack_bf16(y[6], y[7]));
+                }
+                *reinterpret_cast<uint4*>(at(r, A.dim + 8 * c)) = a;
+                *reinterpret_cast<uint4*>(at(r, A.dim + half + 8 * c)) = b;
+            }
+        } else {
+            const int rest = A.rot_dim - half;  // pairs, then what passes
+            for (int i = tid; i < rows * rest; i += kTcThreads) {
+                const int r = i / rest, c = i - r * rest;
+                const bool in = q_lo + r < A.n_q;
+                const bf16* src = Q + (size_t)(q_lo + r) * qrow + A.dim;
+                if (c < half) {
+                    float x = 0.0f, y = 0.0f;
+                    if (in) {
+                        const size_t p = (size_t)(A.pos0 + q_lo + r) * half + c;
+                        const float cs = A.rt.cos_t[p], sn = A.rt.sin_t[p], u = to_f32(src[c]), v = to_f32(src[c + half]);
+                        x = u * cs - v * sn;
+                        y = v * cs + u * sn;
+                    }
+                    *reinterpret_cast<bf16*>(at(r, A.dim + c)) = from_f32<bf16>(x);
+                    *reinterpret_cast<bf16*>(at(r, A.dim + c + half)) = from_f32<bf16>(y);
+                } else {
+                    *reinterpret_cast<bf16*>(at(r, A.dim + c + half)) = in ? src[c + half] : __float2bfloat16_rn(0.0f);
+                }
+            }
+        }
+        asm volatile("cp.async.wait_all;" ::: "memory");
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
     }
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -359,27 +394,39 @@ latent_prefill_tc_kernel(LatentPrefillTcArgs T) {
         const bf16* KR = reinterpret_cast<const bf16*>(A.kr);
         const bf16* VT = reinterpret_cast<const bf16*>(T.vt);
         const bool keys = warp < 11;
-        const int me = keys ? tid - 9 * 32 : tid - 11 * 32;
         const unsigned int full = keys ? kfull : vfull, free_ = keys ? kfree : vfree;
-        const int cn = A.dim / 8, cq = qk / 8, pieces = ksteps * 2;
+        const int cn = A.dim / 8, cq = qk / 8, sub = lane >> 3, c8 = lane & 7;  // a warp brings 128 bytes of four rows at a time
         for (int t = 0; t < tiles; ++t) {
             if (t >= 2) ok = pipe_mbar_wait(free_ + 8 * (t & 1), ((t >> 1) - 1) & 1);
             if (!ok) break;
             const int base = k_begin + t * kTcN;
             if (keys) {
-                unsigned char* dst = base0 + off_k + (t & 1) * k_bytes;
-                for (int i = me; i < kTcN * pieces; i += kTcKeyLoaders) {
-                    const int r = i / pieces, c = i - r * pieces, j = base + r;
-                    const bool in = j < k_end && c < cq;
-                    const bf16* src = !in ? K : c < cn ? K + (size_t)j * A.ld_kv + (size_t)h * A.dim + 8 * c : KR + (size_t)j * A.ld_kr + 8 * (c - cn);
-                    copy16_async(reinterpret_cast<bf16*>(dst + (c >> 3) * (kTcN * 128) + tc_swz(r, c & 7)), src, in);
+                const int r0 = (warp - 9) * 32 + sub, n_in = k_end - base - r0;  // rows r0, r0 + 4, ...: row 4 i is there for 4 i < n_in
+                for (int p = 0; p < panels; ++p) {
+                    const int c = p * 8 + c8;
+                    if (c >= 2 * ksteps) continue;
+                    const bool own = c < cn, in_c = c < cq;
+                    const size_t step = 4 * (size_t)(own ? A.ld_kv : A.ld_kr);
+                    const bf16* src = own ? K + (size_t)(base + r0) * A.ld_kv + (size_t)h * A.dim + 8 * c : KR + (size_t)(base + r0) * A.ld_kr + 8 * (c - cn);
+                    unsigned char* dst = base0 + off_k + (t & 1) * k_bytes + p * (kTcN * 128) + r0 * 128;
+                    const int even = (c8 ^ (r0 & 7)) << 4, odd = (c8 ^ ((r0 + 4) & 7)) << 4;
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) {
+                        const bool in = in_c && 4 * i < n_in;
+                        copy16_async(reinterpret_cast<bf16*>(dst + i * 512 + (i & 1 ? odd : even)), in ? src + i * step : K, in);
+                    }
                 }
             } else {
-                unsigned char* dst = base0 + off_v + (t & 1) * v_bytes;
-                for (int i = me; i < vrows * 8; i += kTcValueLoaders) {
-                    const int r = i >> 3, c = i & 7, j = base + 8 * c;
-                    const bool in = r < A.vdim && j < A.n_k;
-                    copy16_async(reinterpret_cast<bf16*>(dst + tc_swz(r, c)), in ? VT + ((size_t)h * A.vdim + r) * T.ld_vt + j : VT, in);
+                const int j = base + 8 * c8;
+                const bool in_j = j < A.n_k;
+                const size_t step = 4 * (size_t)T.ld_vt;
+                const bf16* src = VT + ((size_t)h * A.vdim + sub) * T.ld_vt + j;
+                unsigned char* dst = base0 + off_v + (t & 1) * v_bytes + sub * 128;
+                const int even = (c8 ^ sub) << 4, odd = (c8 ^ (sub + 4)) << 4;
+#pragma unroll 4
+                for (int i = 0; i < vrows / 4; ++i) {
+                    const bool in = in_j && 4 * i + sub < A.vdim;
+                    copy16_async(reinterpret_cast<bf16*>(dst + i * 512 + (i & 1 ? odd : even)), in ? src + i * step : VT, in);
                 }
             }
             asm volatile("cp.async.commit_group;\n\tcp.async.wait_group 0;" ::: "memory");
