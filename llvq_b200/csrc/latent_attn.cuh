@@ -313,20 +313,21 @@ latent_decode_mma_kernel(LatentDecodeArgs A) {
 #pragma unroll
             for (int j = 0; j < 4; ++j) o[c][k][j] = 0.0f;
     if (t0 < t1) {
-        for (int i = tid; i < kLmHeads * vecs; i += 256) {
-            const int r = i / vecs, c = i - r * vecs;
+        for (int r = warp; r < kLmHeads; r += 8) {
             const bool in = head0 + r < A.heads;
-            copy16_async(sq + r * pitch + 8 * c, in ? qlat + (size_t)(head0 + r) * ld + 8 * c : qlat, in);
+            for (int c = lane; c < vecs; c += 32) copy16_async(sq + r * pitch + 8 * c, in ? qlat + (size_t)(head0 + r) * ld + 8 * c : qlat, in);
         }
     }
     const float s2 = A.scale * kLog2e;
     for (int base = t0; base < t1; base += kLmKeys) {
         const int here = min(kLmKeys, t1 - base);
-        for (int i = tid; i < kLmKeys * vecs; i += 256) {  // rows beyond the split are zero
-            const int r = i / vecs, c = i - r * vecs;
+#pragma unroll 4
+        for (int r = warp; r < kLmKeys; r += 8) {  // rows beyond the split are zero
             int slot = slot0 + base + r;
             if (slot >= A.ring.slots) slot -= A.ring.slots;
-            copy16_async(sk + r * pitch + 8 * c, r < here ? rows + (size_t)slot * ld + 8 * c : rows, r < here);
+            const bool in = r < here;
+            const bf16* src = in ? rows + (size_t)slot * ld : rows;
+            for (int c = lane; c < vecs; c += 32) copy16_async(sk + r * pitch + 8 * c, src + 8 * c, in);
         }
         asm volatile("cp.async.commit_group;\n\tcp.async.wait_group 0;" ::: "memory");
         __syncthreads();
