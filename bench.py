@@ -20,7 +20,8 @@ GEMM), `decode` = configuration 2 (greedy decode, with the token step split by p
 `tp` = configuration 4 on the ranks of the run (row-sharded GEMV pass and tensor-parallel
 decode; tp1 figures at N = 1). `--impl reference` times the CPU path alone, as the
 reference arm, and adds as a side measurement the reference's own serving kernel on its
-transcoded layout where that kernel was built from the reference's sources.
+transcoded layout where that kernel was built from the reference's sources. `--latent` leaves this workload aside
+and times latent-attention models (dense bf16 weights) beside the Qwen3 model of equal size.
 """
 from __future__ import annotations
 
