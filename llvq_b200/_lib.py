@@ -47,7 +47,9 @@ class DenseGemv(C.Structure):
     """llvq_dn_gemv_desc of include/llvq_dense.h."""
     _fields_ = ([(n, C.c_int32) for n in ("dtype", "prologue", "glu", "n_out", "k", "ldw", "ld_table", "table_rows")] +
                 [(n, C.c_float) for n in ("alpha", "eps", "scale", "limit", "gain", "shift", "softcap")] +
-                [(n, C.c_void_p) for n in ("w", "bias", "y", "x", "delta", "norm_w", "a_out", "table", "token")])
+                [(n, C.c_void_p) for n in ("w", "bias", "y", "x", "delta", "norm_w", "a_out", "table", "token")] +
+                [("glu_scale", C.c_float)] + [(n, C.c_int32) for n in ("rows2", "glu2", "k_r", "ld_r", "route_rows", "top", "matrices")] +
+                [(n, C.c_void_p) for n in ("residual", "t_out", "w2", "norm_w2", "y2", "w_r", "route")])
 
 
 class DenseLatent(C.Structure):

@@ -5,11 +5,14 @@
 
 #include "../../include/llvq_dense.h"
 #include "dense_gemv.cuh"
+#include "delta_rule.cuh"
 #include "dense_rows.cuh"
+#include "gqa_attn.cuh"
 #include "host_util.cuh"
 #include "latent_attn.cuh"
 #include "latent_prefill.cuh"
 #include "latent_prefill_tc.cuh"
+#include "linear_recurrence.cuh"
 
 using namespace llvq;
 
@@ -45,13 +48,26 @@ int check_gemv(const llvq_dn_gemv_desc* d, const char* who) {
             if (!d->x) return fail(kStatusInvalid, "%s: null activation", who);
             break;
         case LLVQ_DN_NORM:
-            if (!d->x || !d->norm_w || d->a_out == d->x) return fail(kStatusInvalid, "%s: norm needs x, norm_w and another buffer to store to", who);
+            if ((!d->x && !d->table) || !d->norm_w || (d->x && (d->a_out == d->x || d->t_out == d->x)))
+                return fail(kStatusInvalid, "%s: norm needs x, norm_w and another buffer to store to", who);
+            if (d->table && (!d->token || d->ld_table < d->ldw || d->ld_table % vn || ((uintptr_t)d->table & 15) || d->table_rows <= 0))
+                return fail(kStatusInvalid, "%s: norm of a table row needs a token and rows of %d", who, d->ldw);
             break;
         case LLVQ_DN_EMBED:
             if (!d->table || !d->token || d->ld_table < d->k || d->table_rows <= 0) return fail(kStatusInvalid, "%s: embed needs a table and a token", who);
             break;
         default: return fail(kStatusInvalid, "%s: prologue %d", who, d->prologue);
     }
+    if (d->route && (!d->token || d->route_rows <= 0 || d->top <= 0 || d->matrices <= 0 || !(d->rows2 || d->w_r)))
+        return fail(kStatusInvalid, "%s: a route of %d matrices of %d", who, d->top, d->matrices);
+    if (d->rows2) {
+        const int unit = (d->route ? d->top : 1) * (d->glu2 ? 2 : 1);
+        if (d->prologue != LLVQ_DN_NORM || d->rows2 < 0 || d->rows2 % unit || !d->w2 || ((uintptr_t)d->w2 & 15) || !d->norm_w2 || !d->y2)
+            return fail(kStatusInvalid, "%s: %d second rows", who, d->rows2);
+    }
+    if (d->w_r && (d->prologue != LLVQ_DN_PLAIN || !d->route || d->k_r <= 0 || d->ld_r < d->k_r || d->ld_r % vn || ((uintptr_t)d->w_r & 15)))
+        return fail(kStatusInvalid, "%s: routed columns of %d, row stride %d", who, d->k_r, d->ld_r);
+    if (d->residual && d->glu) return fail(kStatusInvalid, "%s: a residual beside a gated unit", who);
     return kStatusOk;
 }
 
@@ -85,24 +101,46 @@ int launch_stream(const DenseGemvArgs& a, int grid, size_t smem, cudaStream_t s)
     return launch_stream_vpl<kGsMaxVpl, PRO, HEAD>(a, grid, smem, s);
 }
 
+// Deals the CTAs of a grid to the two sets of rows; returns the most rows a CTA gets (pairs stay together).
+int deal_rows(DenseGemvArgs& a, int grid) {
+    a.cta2 = grid;
+    if (!a.rows2) return a.n_out / grid + 2;
+    a.cta2 = std::max(1, std::min(grid - 1, (int)((long long)grid * a.n_out / (a.n_out + a.rows2))));
+    return std::max(a.n_out / a.cta2, a.rows2 / (grid - a.cta2)) + 2;
+}
+
 // Column segments, ring and grid of the stream kernel; false when a row is too long for it.
 bool plan_stream(DenseGemvArgs& a, int* grid, size_t* smem) {
     const int vecs = a.ldw / 8;
-    a.nseg = 1;
-    while (a.nseg < kGvWarps && (vecs + a.nseg - 1) / a.nseg > 6 * 32) a.nseg *= 2;
-    a.segv = (vecs + a.nseg - 1) / a.nseg;
-    if (a.segv > kGsMaxVpl * 32 || (a.nseg - 1) * a.segv >= vecs) return false;
+    if (a.w_r) {  // segments of one length for the matrix and for each routed one
+        const int vecs_r = a.ld_r / 8, total = vecs + a.top * vecs_r;
+        bool found = false;
+        for (int n = (total + 6 * 32 - 1) / (6 * 32); n <= kGvWarps && !found; ++n) {
+            a.segv = (total + n - 1) / n - 1;
+            while (!found && ++a.segv <= kGsMaxVpl * 32) {
+                a.seg_r = (vecs_r + a.segv - 1) / a.segv;
+                a.nseg = (vecs + a.segv - 1) / a.segv + a.top * a.seg_r;
+                found = a.nseg <= n;
+            }
+        }
+        if (!found) return false;
+    } else {
+        a.nseg = 1;
+        while (a.nseg < kGvWarps && (vecs + a.nseg - 1) / a.nseg > 6 * 32) a.nseg *= 2;
+        a.segv = (vecs + a.nseg - 1) / a.nseg;
+        if (a.segv > kGsMaxVpl * 32 || (a.nseg - 1) * a.segv >= vecs) return false;
+    }
     a.slots = std::max(2, std::min(kGsMaxSlots, kGsRingBytes / (a.segv * 16)));
     const int groups = kGvWarps / a.nseg;
-    *grid = std::min((a.n_out + groups - 1) / groups, sm_count());
-    *smem = (size_t)kGvWarps * a.slots * a.segv * 16 + (size_t)(a.n_out / *grid + 2) * a.nseg * sizeof(float);
+    *grid = std::max(a.rows2 ? 2 : 1, std::min((a.n_out + a.rows2 + groups - 1) / groups, sm_count()));
+    *smem = (size_t)kGvWarps * a.slots * a.segv * 16 + (size_t)deal_rows(a, *grid) * a.nseg * sizeof(float);
     return *smem <= kMaxSmem - 2048;
 }
 
 template <typename T, int PRO, bool HEAD>
-int launch_gemv(const DenseGemvArgs& a, int grid, cudaStream_t s) {
-    const int rows = a.n_out / grid + 2;  // pairs stay together
-    const size_t smem = ((size_t)a.ldw + (size_t)rows * a.kslices) * sizeof(float);
+int launch_gemv(DenseGemvArgs a, int grid, cudaStream_t s) {
+    const int rows = deal_rows(a, grid);
+    const size_t smem = ((size_t)a.ldw + (a.w_r ? (size_t)a.top * a.ld_r : 0) + (size_t)rows * a.kslices) * sizeof(float);
     if (smem > kMaxSmem) return fail(kStatusUnsupported, "dn_gemv: %d columns need %zu bytes of shared memory", a.k, smem);
     if (smem > 40 * 1024) {
         const int st = ensure_dyn_smem((const void*)dense_gemv_kernel<T, PRO, HEAD>, smem);
@@ -120,13 +158,18 @@ int gemv_t(const llvq_dn_gemv_desc* d, HeadBest* best, int* grid_out, cudaStream
     a.table = d->table, a.token = (const long long*)d->token, a.best = best;
     a.n_out = d->n_out, a.k = d->k, a.ldw = d->ldw, a.ld_table = d->ld_table, a.table_rows = d->table_rows;
     a.glu = d->glu;
+    a.glu_scale = d->glu_scale == 0.0f ? 1.0f : d->glu_scale;
+    a.residual = d->residual, a.t_out = d->t_out;
+    a.w2 = d->w2, a.norm_w2 = d->norm_w2, a.y2 = d->y2, a.rows2 = d->rows2, a.glu2 = d->glu2;
+    a.w_r = d->w_r, a.k_r = d->k_r, a.ld_r = d->ld_r;
+    if (d->route) a.route = d->route, a.route_rows = d->route_rows, a.top = d->top, a.matrices = d->matrices, a.rows_m = d->rows2 / d->top;
     a.alpha = d->alpha, a.eps = d->eps, a.scale = d->scale, a.limit = d->limit, a.gain = d->gain, a.shift = d->shift, a.cap = d->softcap;
     // column slices: enough lanes for a row's vectors; rows of a CTA are shared by the row groups that are left
     if constexpr (sizeof(T) == 2) {
         size_t smem = 0;
         int grid = 0;
         a.err = device_error();
-        a.vec_x = !(((uintptr_t)a.x | (uintptr_t)a.delta | (uintptr_t)a.norm_w) & 15);
+        a.vec_x = !(((uintptr_t)a.x | (uintptr_t)a.delta | (uintptr_t)a.norm_w | (uintptr_t)a.norm_w2) & 15);
         if (a.err && plan_stream(a, &grid, &smem)) {
             if (grid_out) *grid_out = grid;
             if (best) {
@@ -141,10 +184,10 @@ int gemv_t(const llvq_dn_gemv_desc* d, HeadBest* best, int* grid_out, cudaStream
             }
         }
     }
-    const int vecs = d->ldw / Vec16<T>::N;
+    const int vecs = (d->ldw + (d->w_r ? d->top * d->ld_r : 0)) / Vec16<T>::N;
     a.kslices = vecs > 128 ? 8 : vecs > 64 ? 4 : vecs > 32 ? 2 : 1;
     const int rows_step = kGvWarps / a.kslices * kGvRows;
-    int grid = std::min((d->n_out + rows_step - 1) / rows_step, 4 * sm_count());
+    int grid = std::max(d->rows2 ? 2 : 1, std::min((d->n_out + d->rows2 + rows_step - 1) / rows_step, 4 * sm_count()));
     if (best) grid = std::min(grid, kHeadMaxGrid);
     if (grid_out) *grid_out = grid;
     if (best) {
@@ -251,10 +294,36 @@ int prefill_simt(const LatentPrefillArgs& p, cudaStream_t s) {
 
 // The tcgen05 kernel takes heads of whole 16-byte vectors whose tiles fit shared memory and TMEM, and portions that
 // fill a good part of its query tiles.
+bool prefill_fits_tc(int dtype, int n_q, int dim, int rot_dim, int vdim, float scale) {
+    return dtype == LLVQ_DN_BF16 && n_q >= 64 && scale > 0.0f && !((dim | rot_dim | vdim) & 7) && tc_v_rows(vdim) <= 192 &&
+           latent_prefill_tc_smem(dim + rot_dim, vdim) <= kMaxSmem - 1024;
+}
 bool prefill_on_tc(const llvq_dn_latent* a, int n_q) {
-    const int qk = a->dim + a->rot_dim;
-    return a->dtype == LLVQ_DN_BF16 && n_q >= 64 && a->scale > 0.0f && !((a->dim | a->rot_dim | a->vdim | a->kv_rank) & 7) && tc_v_rows(a->vdim) <= 192 &&
-           latent_prefill_tc_smem(qk, a->vdim) <= kMaxSmem - 1024;
+    return !(a->kv_rank & 7) && prefill_fits_tc(a->dtype, n_q, a->dim, a->rot_dim, a->vdim, a->scale);
+}
+
+int prefill_tc(const LatentPrefillArgs& p, const void* vt, int ld_vt, cudaStream_t s) {
+    LatentPrefillTcArgs tc{p, vt, ld_vt, device_error()};
+    if (!tc.err) return fail(kStatusCuda, "prompt attention: no error word");
+    const size_t smem = latent_prefill_tc_smem(p.dim + p.rot_dim, p.vdim);
+    const int st = ensure_dyn_smem((const void*)latent_prefill_tc_kernel, smem);
+    if (st) return st;
+    CUDA_TRY(launch_dep(latent_prefill_tc_kernel, dim3((p.n_q + 2 * kTcM - 1) / (2 * kTcM), p.heads), dim3(kTcThreads), smem, s, tc));
+    g_launches++;
+    return kStatusOk;
+}
+
+// Values along the positions. kernel: 0 = by size and type, 1 = the generic one.
+int prefill_plain(int dtype, const LatentPrefillArgs& p, int kernel, cudaStream_t s) {
+    if (dtype == LLVQ_DN_F32) return prefill_simt<float>(p, s);
+    const int nv = p.vdim <= 64 ? 8 : p.vdim <= 128 ? 16 : 32;
+    const size_t smem = latent_prefill_smem(p.dim, p.rot_dim, nv);
+    if (kernel == 1 || smem > kMaxSmem) return prefill_simt<bf16>(p, s);
+    const bool vec = !((p.dim | p.rot_dim | p.vdim | p.ld_kv | p.ld_kr | p.k_head | p.v_head | p.v_off) & 7) &&
+                     !(((uintptr_t)p.q | (uintptr_t)p.kv | (uintptr_t)p.kr | (uintptr_t)p.out) & 15);
+    if (nv == 8) return vec ? prefill_mma<8, true>(p, smem, s) : prefill_mma<8, false>(p, smem, s);
+    if (nv == 16) return vec ? prefill_mma<16, true>(p, smem, s) : prefill_mma<16, false>(p, smem, s);
+    return vec ? prefill_mma<32, true>(p, smem, s) : prefill_mma<32, false>(p, smem, s);
 }
 
 }  // namespace
@@ -286,7 +355,7 @@ int llvq_dn_gemv(const llvq_dn_gemv_desc* d, llvq_dn_stream stream) {
 int llvq_dn_head(const llvq_dn_gemv_desc* d, void* scratch, float* val_out, int64_t* idx_out, llvq_dn_stream stream) {
     int st = check_gemv(d, "dn_head");
     if (st) return st;
-    if (d->glu) return fail(kStatusUnsupported, "dn_head: rows in pairs");
+    if (d->glu || d->rows2 || d->residual) return fail(kStatusUnsupported, "dn_head: rows in pairs, second rows or a residual");
     if (!scratch || !val_out || !idx_out) return fail(kStatusInvalid, "dn_head: null argument");
     cudaStream_t s = (cudaStream_t)stream;
     int grid = 0;
@@ -339,28 +408,14 @@ int llvq_dn_latent_prefill(const llvq_dn_latent* a, const void* q, const void* k
         ld_kr < a->rot_dim || (vt && ld_vt < n_k))
         return fail(kStatusInvalid, "dn_latent_prefill: %d queries at %lld over %d keys at %lld", n_q, (long long)pos0, n_k, (long long)key0);
     LatentPrefillArgs p{q, kv, kr, a->sink, out, rot_of(a), pos0, key0, n_q, n_k, a->heads, a->dim, a->rot_dim, a->vdim, ld_kv, ld_kr,
-                        a->window, a->scale};
+                        a->window, a->scale, 1, a->dim, a->vdim, a->heads * a->dim};
     cudaStream_t s = (cudaStream_t)stream;
     if (vt) {
         if (!prefill_on_tc(a, n_q) || ((ld_kv | ld_kr | ld_vt) & 7) || (((uintptr_t)q | (uintptr_t)kv | (uintptr_t)kr | (uintptr_t)vt | (uintptr_t)out) & 15))
             return fail(kStatusInvalid, "dn_latent_prefill: transposed values where llvq_dn_latent_prefill_transposes says no, or rows not on 16 bytes");
-        LatentPrefillTcArgs tc{p, vt, ld_vt, device_error()};
-        if (!tc.err) return fail(kStatusCuda, "dn_latent_prefill: no error word");
-        const size_t smem = latent_prefill_tc_smem(a->dim + a->rot_dim, a->vdim);
-        const int st2 = ensure_dyn_smem((const void*)latent_prefill_tc_kernel, smem);
-        if (st2) return st2;
-        CUDA_TRY(launch_dep(latent_prefill_tc_kernel, dim3((n_q + 2 * kTcM - 1) / (2 * kTcM), a->heads), dim3(kTcThreads), smem, s, tc));
-        g_launches++;
-        return kStatusOk;
+        return prefill_tc(p, vt, ld_vt, s);
     }
-    if (a->dtype == LLVQ_DN_F32) return prefill_simt<float>(p, s);
-    const int nv = a->vdim <= 64 ? 8 : a->vdim <= 128 ? 16 : 32;
-    const size_t smem = latent_prefill_smem(a->dim, a->rot_dim, nv);
-    if (kernel == 1 || smem > kMaxSmem) return prefill_simt<bf16>(p, s);
-    const bool vec = !((a->dim | a->rot_dim | a->vdim | ld_kv | ld_kr) & 7) && !(((uintptr_t)q | (uintptr_t)kv | (uintptr_t)kr | (uintptr_t)out) & 15);
-    if (nv == 8) return vec ? prefill_mma<8, true>(p, smem, s) : prefill_mma<8, false>(p, smem, s);
-    if (nv == 16) return vec ? prefill_mma<16, true>(p, smem, s) : prefill_mma<16, false>(p, smem, s);
-    return vec ? prefill_mma<32, true>(p, smem, s) : prefill_mma<32, false>(p, smem, s);
+    return prefill_plain(a->dtype, p, kernel, s);
 }
 
 int llvq_dn_embed_rows(int32_t dtype, const void* table, int32_t ld, int32_t table_rows, const int64_t* tokens, int32_t rows, int32_t n,
@@ -414,16 +469,39 @@ int llvq_dn_latent_rows(const llvq_dn_latent* a, const void* y, int32_t ldy, int
     return kStatusOk;
 }
 
-int llvq_dn_glu_rows(int32_t dtype, const void* gate_up, const float* bias, void* out, int32_t rows, int32_t n, float limit, float gain,
-                     float shift, llvq_dn_stream stream) {
-    if (bad_dtype(dtype) || !gate_up || !out || rows <= 0 || n <= 0) return fail(kStatusInvalid, "dn_glu_rows: bad argument");
+int llvq_dn_gated_rows(int32_t dtype, const void* gate_up, const float* bias, void* out, int32_t ld_out, int32_t rows, int32_t n, float limit, float gain,
+                       float shift, float scale, llvq_dn_stream stream) {
+    if (bad_dtype(dtype) || !gate_up || !out || rows <= 0 || n <= 0 || ld_out < n) return fail(kStatusInvalid, "dn_gated_rows: bad argument");
     cudaStream_t s = (cudaStream_t)stream;
-    const int vec = n % 4 == 0 && !(((uintptr_t)gate_up | (uintptr_t)bias | (uintptr_t)out) & 15);
+    const int vec = n % 4 == 0 && ld_out % 4 == 0 && !(((uintptr_t)gate_up | (uintptr_t)bias | (uintptr_t)out) & 15);
     const dim3 grid(rows, (n + 8 * kRowThreads - 1) / (8 * kRowThreads));
     if (dtype == LLVQ_DN_BF16)
-        CUDA_TRY(launch_dep(glu_rows_kernel<bf16>, grid, dim3(kRowThreads), 0, s, (const bf16*)gate_up, bias, (bf16*)out, n, limit, gain, shift, vec));
+        CUDA_TRY(launch_dep(glu_rows_kernel<bf16>, grid, dim3(kRowThreads), 0, s, (const bf16*)gate_up, bias, (bf16*)out, ld_out, n, limit, gain, shift, scale, vec));
     else
-        CUDA_TRY(launch_dep(glu_rows_kernel<float>, grid, dim3(kRowThreads), 0, s, (const float*)gate_up, bias, (float*)out, n, limit, gain, shift, vec));
+        CUDA_TRY(launch_dep(glu_rows_kernel<float>, grid, dim3(kRowThreads), 0, s, (const float*)gate_up, bias, (float*)out, ld_out, n, limit, gain, shift, scale, vec));
+    g_launches++;
+    return kStatusOk;
+}
+int llvq_dn_glu_rows(int32_t dtype, const void* gate_up, const float* bias, void* out, int32_t rows, int32_t n, float limit, float gain,
+                     float shift, llvq_dn_stream stream) {
+    return llvq_dn_gated_rows(dtype, gate_up, bias, out, n, rows, n, limit, gain, shift, 1.0f, stream);
+}
+
+int llvq_dn_add_norms_rows(int32_t dtype, float* x, const void* y, const void* routed, const int32_t* places, int32_t top, const float* w1, void* h1,
+                           const float* w2, void* h2, float eps, int32_t rows, int32_t n, llvq_dn_stream stream) {
+    if (bad_dtype(dtype) || !x || rows <= 0 || n <= 0 || (size_t)n * 4 > kMaxSmem - 1024 || (routed && (!places || top <= 0)) || (w1 && !h1) || (w2 && !h2))
+        return fail(kStatusInvalid, "dn_add_norms_rows: bad argument");
+    const int vec = n % 4 == 0 && !(((uintptr_t)x | (uintptr_t)y | (uintptr_t)routed | (uintptr_t)w1 | (uintptr_t)w2 | (uintptr_t)h1 | (uintptr_t)h2) & 15);
+    AddNormsArgs k{x, y, routed, places, w1, w2, h1, h2, n, routed ? top : 0, vec, eps};
+    const size_t smem = (size_t)n * 4;
+    if (smem > 40 * 1024) {
+        const int st = ensure_dyn_smem(dtype == LLVQ_DN_BF16 ? (const void*)add_norms_rows_kernel<bf16> : (const void*)add_norms_rows_kernel<float>, smem);
+        if (st) return st;
+    }
+    if (dtype == LLVQ_DN_BF16)
+        CUDA_TRY(launch_dep(add_norms_rows_kernel<bf16>, dim3(rows), dim3(kRowThreads), smem, (cudaStream_t)stream, k));
+    else
+        CUDA_TRY(launch_dep(add_norms_rows_kernel<float>, dim3(rows), dim3(kRowThreads), smem, (cudaStream_t)stream, k));
     g_launches++;
     return kStatusOk;
 }
@@ -437,3 +515,5 @@ int llvq_dn_softcap(float* y, size_t n, float cap, llvq_dn_stream stream) {
 }
 
 }  // extern "C"
+
+#include "mixer_api.cuh"

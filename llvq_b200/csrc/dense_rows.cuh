@@ -4,6 +4,7 @@
 //   postnorm_rows_kernel  t = alpha * x + y (+ bias); x = t / sqrt(mean(t^2) + eps) * w, and its T copy
 //   latent_rows_kernel  the down projections of a latent-attention layer: the query latent normed into cq, the
 //                       token's cache row normed, rotated and stored into the ring
+//   add_norms_rows_kernel  x += y (+ the token's rows of a routed product); two norms of the sum for two sublayers
 //   glu_rows_kernel     clamped gated unit of (gate, up) pairs with their biases
 //   softcap_kernel      logits <- cap * tanh(logits / cap)
 #pragma once
@@ -98,6 +99,85 @@ postnorm_rows_kernel(const float* x, const T* __restrict__ y, const float* __res
     }
 }
 
+struct AddNormsArgs {
+    float* x;            // [rows, n], the residual stream
+    const void* y;       // [rows, n] of T, or null
+    const void* routed;  // [rows * top, n] of T, or null: row t takes places[t * top ..]
+    const int* places;
+    const float* w1;     // norm weights as applied, or null: no such norm
+    const float* w2;
+    void* h1;            // [rows, n] of T
+    void* h2;
+    int n, top, vec;
+    float eps;
+};
+
+// Dynamic shared memory: n floats. vec: n % 4 == 0 and every row on a 16-byte boundary.
+template <typename T>
+__global__ void __launch_bounds__(kRowThreads)
+add_norms_rows_kernel(AddNormsArgs A) {
+    extern __shared__ __align__(16) float row_s[];
+    __shared__ float red[kRowThreads / 32];
+    llvq_dependent_enter();
+    const size_t o = (size_t)blockIdx.x * A.n;
+    const T* Y = reinterpret_cast<const T*>(A.y);
+    const T* P = reinterpret_cast<const T*>(A.routed);
+    const int* place = A.places + (size_t)blockIdx.x * A.top;
+    const bool change = Y || P;
+    float ss = 0.0f;
+    if (A.vec) {
+        for (int i = 4 * threadIdx.x; i < A.n; i += 4 * kRowThreads) {
+            float4 t = load4(A.x + o + i);
+            if (Y) {
+                const float4 d = load4(Y + o + i);
+                t.x += d.x, t.y += d.y, t.z += d.z, t.w += d.w;
+            }
+            if (P) {
+                float4 d = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                for (int j = 0; j < A.top; ++j) {
+                    const float4 e = load4(P + (size_t)place[j] * A.n + i);
+                    d.x += e.x, d.y += e.y, d.z += e.z, d.w += e.w;
+                }
+                t.x += d.x, t.y += d.y, t.z += d.z, t.w += d.w;
+            }
+            if (change) store4(A.x + o + i, t);
+            *reinterpret_cast<float4*>(row_s + i) = t;
+            ss = fmaf(t.x, t.x, fmaf(t.y, t.y, fmaf(t.z, t.z, fmaf(t.w, t.w, ss))));
+        }
+    } else {
+        for (int i = threadIdx.x; i < A.n; i += kRowThreads) {
+            float t = A.x[o + i];
+            if (Y) t += to_f32(Y[o + i]);
+            if (P) {
+                float d = 0.0f;
+                for (int j = 0; j < A.top; ++j) d += to_f32(P[(size_t)place[j] * A.n + i]);
+                t += d;
+            }
+            if (change) A.x[o + i] = t;
+            row_s[i] = t;
+            ss = fmaf(t, t, ss);
+        }
+    }
+    if (!A.w1 && !A.w2) return;
+    const float r = 1.0f / sqrtf(block_sum_f(ss, red) / (float)A.n + A.eps);
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+        const float* w = k ? A.w2 : A.w1;
+        T* h = reinterpret_cast<T*>(k ? A.h2 : A.h1);
+        if (!w) continue;
+        if (A.vec) {
+            for (int i = 4 * threadIdx.x; i < A.n; i += 4 * kRowThreads) {
+                float4 t = *reinterpret_cast<const float4*>(row_s + i);
+                const float4 f = load4(w + i);
+                t.x *= r * f.x, t.y *= r * f.y, t.z *= r * f.z, t.w *= r * f.w;
+                store4(h + o + i, t);
+            }
+        } else {
+            for (int i = threadIdx.x; i < A.n; i += kRowThreads) h[o + i] = from_f32<T>(row_s[i] * r * w[i]);
+        }
+    }
+}
+
 // y: [rows, q_rank + kv_rank + rot_dim] (q_rank only when the layer reads another layer's ring: ring.rows null).
 template <typename T>
 __global__ void __launch_bounds__(kRowThreads)
@@ -117,14 +197,15 @@ latent_rows_kernel(const T* __restrict__ y, int ldy, int q_rank, const float* __
     if (ring.rows) store_latent_row<T>(row + q_rank, kv_norm, eps, kv_rank, rot_dim, rt, pos0 + blockIdx.x, ring, red);
 }
 
-// gu: [rows, n, 2] (gate, up) pairs, bias: [n, 2] or null. grid = (rows, ceil(n / (8 threads))); a thread takes four
+// gu: [rows, n, 2] (gate, up) pairs, bias: [n, 2] or null; the unit times `scale` into rows of stride ldo. grid = (rows, ceil(n / (8 threads))); a thread takes four
 // neighbouring outputs at a time where the row allows 16-byte loads (vec).
 template <typename T>
 __global__ void __launch_bounds__(kRowThreads)
-glu_rows_kernel(const T* __restrict__ gu, const float* __restrict__ bias, T* __restrict__ out, int n, float limit, float gain, float shift, int vec) {
+glu_rows_kernel(const T* __restrict__ gu, const float* __restrict__ bias, T* __restrict__ out, int ldo, int n, float limit, float gain, float shift,
+                float scale, int vec) {
     llvq_dependent_enter();
     const T* g = gu + (size_t)blockIdx.x * 2 * n;
-    T* o = out + (size_t)blockIdx.x * n;
+    T* o = out + (size_t)blockIdx.x * ldo;
     const int lo = blockIdx.y * 8 * kRowThreads, hi = min(n, lo + 8 * kRowThreads);
     if (vec) {  // n % 4 == 0, rows on 16-byte boundaries
         constexpr int LV = 8 * sizeof(T) / 16;  // 16-byte loads of four pairs
@@ -148,7 +229,7 @@ glu_rows_kernel(const T* __restrict__ gu, const float* __restrict__ bias, T* __r
             }
             __align__(16) T r[4];
 #pragma unroll
-            for (int j = 0; j < 4; ++j) r[j] = from_f32<T>(clamped_glu(f[2 * j] + b[2 * j], f[2 * j + 1] + b[2 * j + 1], limit, gain, shift));
+            for (int j = 0; j < 4; ++j) r[j] = from_f32<T>(scale * clamped_glu(f[2 * j] + b[2 * j], f[2 * j + 1] + b[2 * j + 1], limit, gain, shift));
             if constexpr (sizeof(T) == 2)
                 *reinterpret_cast<uint2*>(o + i) = *reinterpret_cast<const uint2*>(r);
             else
@@ -158,7 +239,7 @@ glu_rows_kernel(const T* __restrict__ gu, const float* __restrict__ bias, T* __r
     }
     for (int i = lo + threadIdx.x; i < hi; i += kRowThreads) {
         const float bg = bias ? bias[2 * i] : 0.0f, bu = bias ? bias[2 * i + 1] : 0.0f;
-        o[i] = from_f32<T>(clamped_glu(to_f32(g[2 * i]) + bg, to_f32(g[2 * i + 1]) + bu, limit, gain, shift));
+        o[i] = from_f32<T>(scale * clamped_glu(to_f32(g[2 * i]) + bg, to_f32(g[2 * i + 1]) + bu, limit, gain, shift));
     }
 }
 

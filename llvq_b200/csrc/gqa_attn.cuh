@@ -1,0 +1,316 @@
+// Grouped-query attention over a ring of cached rows, the token step, and the row kernels of a prompt portion around
+// its attention (whose kernels are those of latent_prefill*.cuh: keys and values of a head apart, nothing rotated).
+//
+// A cached row is [kv_heads keys | kv_heads values], every head padded with zeros to whole 16-byte vectors; position p
+// sits in slot p % slots. Queries and keys are RMS normed per head with weights of their own before they meet.
+//
+//   gqa_token            a CTA takes four query heads of one key/value head and one split of the visible positions, in
+//                        tiles of 64: thread = (position, quarter of the key) for the scores, (position group, value
+//                        vector) for the sums; online softmax in base 2, f32. The CTA whose split holds the token itself
+//                        norms its key; the first of a group stores the cache row. The last split to arrive merges them
+//                        all in order, gates the heads and scales them: no CTA waits for another.
+//   gqa_rows_kernel      a portion: queries normed, cache rows stored.
+//   gate_rows_kernel     out = x * sigmoid(gate) * scale.
+#pragma once
+#include "latent_attn.cuh"
+
+namespace llvq {
+
+constexpr int kGqHeads = 4, kGqTile = 64, kGqThreads = 256, kGqMaxSplits = 128;
+
+struct GqaRing {
+    void* rows;  // [slots, ld] of T
+    int slots, ld;
+    int kd, vd;  // a head's key and value, padded; the values start at kv_heads * kd
+};
+
+struct GqaArgs {
+    const float* q;       // [heads, dim]
+    const float* k;       // [kv_heads, dim]
+    const float* v;       // [kv_heads, vdim]
+    const float* gate;    // [heads, vdim] before the sigmoid, or null
+    const float* q_norm;  // [dim], as applied
+    const float* k_norm;
+    const long long* pos;
+    float* part_ml;       // [heads, splits, 2]
+    float* part_o;        // [heads, splits, vdim]
+    unsigned int* arrived; // [units], zero before the first launch and after every one
+    float* out;           // [heads, vdim]
+    GqaRing ring;
+    int heads, kv_heads, dim, vdim, window, splits;
+    float scale, eps, out_scale;
+};
+
+__host__ __device__ inline int gqa_chunks(int heads, int kv_heads) { return (heads / kv_heads + kGqHeads - 1) / kGqHeads; }
+inline int gqa_ctas(int heads, int kv_heads, int splits) { return kv_heads * gqa_chunks(heads, kv_heads) * splits; }
+// Shared memory of one CTA: queries, the token's own key and value, quarter scores, weights, split factors, sums.
+template <typename T>
+inline size_t gqa_token_smem(int kd, int vd) {
+    return (size_t)kGqHeads * kd * 4 + (size_t)(kd + vd) * sizeof(T) + (size_t)4 * kGqHeads * kGqTile * 4 + (size_t)kGqHeads * kGqTile * 4 +
+           (size_t)kGqHeads * kGqMaxSplits * 4 + (size_t)kGqThreads * Vec16<T>::N * 4 + 64;
+}
+
+__device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
+
+// 1 / rms of a row by one warp, the same value in every lane.
+template <typename X>
+__device__ __forceinline__ float warp_inv_rms(const X* x, int n, float eps) {
+    float ss = 0.0f;
+    for (int i = threadIdx.x & 31; i < n; i += 32) {
+        const float v = to_f32(x[i]);
+        ss = fmaf(v, v, ss);
+    }
+    return 1.0f / sqrtf(warp_sum_f(ss) / (float)n + eps);
+}
+
+// One CTA's part of the token step. `smem` holds gqa_token_smem bytes. The caller has passed the dependency wait.
+template <typename T>
+__device__ __forceinline__ void gqa_token(const GqaArgs& A, int cta, unsigned char* smem) {
+    constexpr int VN = Vec16<T>::N;
+    __shared__ float corr_s[kGqHeads], inv_s[kGqHeads];
+    __shared__ int last_s;
+    const int kd = A.ring.kd, vd = A.ring.vd, kvecs = kd / VN, vvecs = vd / VN;
+    float* red = reinterpret_cast<float*>(smem);                                 // [256][VN]
+    float* q_s = red + kGqThreads * VN;                                          // [4][kd]
+    T* k_new = reinterpret_cast<T*>(q_s + kGqHeads * kd);                        // [kd]
+    T* v_new = k_new + kd;                                                       // [vd]
+    float* s_s = reinterpret_cast<float*>(v_new + vd);                           // [quarter][4][64]
+    float* p_s = s_s + 4 * kGqHeads * kGqTile;                                   // [4][64]
+    float* f_s = p_s + kGqHeads * kGqTile;                                       // [4][splits]
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int unit = cta / A.splits, split = cta - unit * A.splits, chunks = gqa_chunks(A.heads, A.kv_heads);
+    const int g = unit / chunks, chunk = unit - g * chunks, rep = A.heads / A.kv_heads;
+    const int head0 = g * rep + chunk * kGqHeads, nh = min(kGqHeads, rep - chunk * kGqHeads);
+    const long long pos = *A.pos;
+    const int n = (int)min((long long)A.window, pos + 1);  // visible positions pos - n + 1 .. pos
+    int per = (n + A.splits - 1) / A.splits;
+    per = (per + kGqTile - 1) / kGqTile * kGqTile;
+    const int t0 = split * per, t1 = min(n, t0 + per);
+    const bool own = t0 < n && t1 == n;  // this split holds the token itself
+    const int slot0 = (int)((pos - n + 1) % A.ring.slots);  // n <= slots: at most one wrap below
+    T* row_new = reinterpret_cast<T*>(A.ring.rows) + (size_t)(pos % A.ring.slots) * A.ring.ld;
+
+    if (warp < nh && t0 < t1) {
+        const float* q = A.q + (size_t)(head0 + warp) * A.dim;
+        const float f = warp_inv_rms(q, A.dim, A.eps) * A.scale * kLog2e;
+        for (int i = lane; i < kd; i += 32) q_s[warp * kd + i] = i < A.dim ? q[i] * f * A.q_norm[i] : 0.0f;
+    } else if (warp < kGqHeads) {
+        for (int i = lane; i < kd; i += 32) q_s[warp * kd + i] = 0.0f;
+    } else if (own && warp == kGqHeads) {
+        const float* k = A.k + (size_t)g * A.dim;
+        const float f = warp_inv_rms(k, A.dim, A.eps);
+        for (int i = lane; i < kd; i += 32) {
+            const T t = from_f32<T>(i < A.dim ? k[i] * f * A.k_norm[i] : 0.0f);
+            k_new[i] = t;
+            if (chunk == 0) row_new[(size_t)g * kd + i] = t;
+        }
+    } else if (own && warp == kGqHeads + 1) {
+        const float* v = A.v + (size_t)g * A.vdim;
+        for (int i = lane; i < vd; i += 32) {
+            const T t = from_f32<T>(i < A.vdim ? v[i] : 0.0f);
+            v_new[i] = t;
+            if (chunk == 0) row_new[(size_t)A.kv_heads * kd + (size_t)g * vd + i] = t;
+        }
+    }
+    __syncthreads();
+
+    float m = -INFINITY, l = 0.0f;  // of head `warp`, in warps below nh
+    int vl = 1;                     // threads along the value vectors
+    while (vl < vvecs) vl *= 2;
+    const int vi = tid % vl, grp = tid / vl, grps = kGqThreads / vl;
+    float acc[kGqHeads][VN];
+#pragma unroll
+    for (int h = 0; h < kGqHeads; ++h)
+#pragma unroll
+        for (int j = 0; j < VN; ++j) acc[h][j] = 0.0f;
+    auto row_at = [&](int idx) {
+        int slot = slot0 + idx;
+        if (slot >= A.ring.slots) slot -= A.ring.slots;
+        return reinterpret_cast<const T*>(A.ring.rows) + (size_t)slot * A.ring.ld;
+    };
+    for (int base = t0; base < t1; base += kGqTile) {
+        const int here = min(kGqTile, t1 - base);
+        {  // scores: thread = (position, quarter of the key's vectors)
+            const int p = tid & (kGqTile - 1), quarter = tid / kGqTile, idx = base + p;
+            float s[kGqHeads] = {0.0f, 0.0f, 0.0f, 0.0f};
+            if (p < here) {
+                const uint4* kr = reinterpret_cast<const uint4*>(idx == n - 1 ? k_new : row_at(idx) + (size_t)g * kd);
+#pragma unroll 4
+                for (int c = quarter; c < kvecs; c += 4) {
+                    float f[VN];
+                    Vec16<T>::widen(kr[c], f);
+#pragma unroll
+                    for (int h = 0; h < kGqHeads; ++h)
+#pragma unroll
+                        for (int j = 0; j < VN; j += 4) {
+                            const float4 qv = *reinterpret_cast<const float4*>(q_s + h * kd + c * VN + j);
+                            s[h] = fmaf(f[j], qv.x, s[h]);
+                            s[h] = fmaf(f[j + 1], qv.y, s[h]);
+                            s[h] = fmaf(f[j + 2], qv.z, s[h]);
+                            s[h] = fmaf(f[j + 3], qv.w, s[h]);
+                        }
+                }
+            }
+#pragma unroll
+            for (int h = 0; h < kGqHeads; ++h) s_s[(quarter * kGqHeads + h) * kGqTile + p] = s[h];
+        }
+        __syncthreads();
+        if (warp < nh) {
+            float s[2];
+#pragma unroll
+            for (int k = 0; k < 2; ++k) {
+                const int p = lane + 32 * k;
+                s[k] = -INFINITY;
+                if (p < here) {
+                    s[k] = 0.0f;
+#pragma unroll
+                    for (int quarter = 0; quarter < 4; ++quarter) s[k] += s_s[(quarter * kGqHeads + warp) * kGqTile + p];
+                }
+            }
+            const float mn = fmaxf(m, warp_max_f(fmaxf(s[0], s[1])));  // finite: a tile holds a visible position
+            const float corr = exp2f(m - mn), e0 = exp2f(s[0] - mn), e1 = exp2f(s[1] - mn);
+            l = l * corr + warp_sum_f(e0 + e1);
+            m = mn;
+            p_s[warp * kGqTile + lane] = e0;
+            p_s[warp * kGqTile + lane + 32] = e1;
+            if (lane == 0) corr_s[warp] = corr;
+        } else if (warp < kGqHeads) {
+            p_s[warp * kGqTile + lane] = 0.0f;
+            p_s[warp * kGqTile + lane + 32] = 0.0f;
+            if (lane == 0) corr_s[warp] = 1.0f;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int h = 0; h < kGqHeads; ++h)
+#pragma unroll
+            for (int j = 0; j < VN; ++j) acc[h][j] *= corr_s[h];
+        if (vi < vvecs) {
+#pragma unroll 4
+            for (int p = grp; p < here; p += grps) {
+                const int idx = base + p;
+                const T* vr = idx == n - 1 ? v_new : row_at(idx) + (size_t)A.kv_heads * kd + (size_t)g * vd;
+                float f[VN];
+                Vec16<T>::widen(reinterpret_cast<const uint4*>(vr)[vi], f);
+#pragma unroll
+                for (int h = 0; h < kGqHeads; ++h) {
+                    const float w = p_s[h * kGqTile + p];
+#pragma unroll
+                    for (int j = 0; j < VN; ++j) acc[h][j] = fmaf(w, f[j], acc[h][j]);
+                }
+            }
+        }
+    }
+    if (warp < nh && lane == 0) {
+        float* ml = A.part_ml + ((size_t)(head0 + warp) * A.splits + split) * 2;
+        ml[0] = m;  // -inf for a split beyond the visible positions
+        ml[1] = l;
+    }
+    for (int h = 0; h < nh && t0 < t1; ++h) {
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < kGqHeads; ++k)
+            if (k == h) {
+#pragma unroll
+                for (int j = 0; j < VN; ++j) red[(grp * vl + vi) * VN + j] = acc[k][j];
+            }
+        __syncthreads();
+        for (int d = tid; d < A.vdim; d += kGqThreads) {
+            float o = 0.0f;
+            for (int k = 0; k < grps; ++k) o += red[k * vl * VN + d];
+            A.part_o[((size_t)(head0 + h) * A.splits + split) * A.vdim + d] = o;
+        }
+    }
+    // ---- the last split to arrive merges ----
+    __threadfence();
+    __syncthreads();
+    if (tid == 0) last_s = atomicAdd(A.arrived + unit, 1u) == (unsigned int)A.splits - 1u;
+    __syncthreads();
+    if (!last_s) return;
+    __threadfence();
+    if (tid == 0) A.arrived[unit] = 0;
+    if (warp < nh) {
+        const float* ml = A.part_ml + (size_t)(head0 + warp) * A.splits * 2;
+        float mt = -INFINITY, lt = 0.0f;
+        for (int s = lane; s < A.splits; s += 32) mt = fmaxf(mt, __ldcg(ml + 2 * s));
+        mt = warp_max_f(mt);
+        for (int s = lane; s < A.splits; s += 32) {
+            const float ms = __ldcg(ml + 2 * s), f = ms == -INFINITY ? 0.0f : exp2f(ms - mt);
+            f_s[warp * kGqMaxSplits + s] = f;
+            lt = fmaf(__ldcg(ml + 2 * s + 1), f, lt);
+        }
+        lt = warp_sum_f(lt);
+        if (lane == 0) inv_s[warp] = A.out_scale / lt;
+    }
+    __syncthreads();
+    for (int e = tid; e < nh * A.vdim; e += kGqThreads) {
+        const int h = e / A.vdim, d = e - h * A.vdim;
+        const size_t at = (size_t)(head0 + h) * A.vdim + d;
+        const float* po = A.part_o + (size_t)(head0 + h) * A.splits * A.vdim + d;
+        float o = 0.0f;
+#pragma unroll 8
+        for (int s = 0; s < A.splits; ++s) {
+            const float f = f_s[h * kGqMaxSplits + s];
+            if (f != 0.0f) o = fmaf(__ldcg(po + (size_t)s * A.vdim), f, o);  // the sums of an empty split are not written
+        }
+        o *= inv_s[h];
+        A.out[at] = A.gate ? o * sigmoid_f(A.gate[at]) : o;
+    }
+}
+
+// ---- prompt portions ----
+
+struct GqaRowsArgs {
+    const void* q;  // rows of one product, stride ldy: [heads, dim], [kv_heads, dim], [kv_heads, vdim]
+    const void* k;
+    const void* v;
+    void* qn;       // [rows, heads * dim] of T
+    const float* q_norm;
+    const float* k_norm;
+    GqaRing ring;
+    long long pos0;
+    int ldy, heads, kv_heads, dim, vdim;
+    float eps;
+};
+
+// grid = rows, 256 threads: a warp takes a head at a time.
+template <typename T>
+__global__ void __launch_bounds__(256)
+gqa_rows_kernel(GqaRowsArgs A) {
+    llvq_dependent_enter();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const size_t o = (size_t)blockIdx.x * A.ldy;
+    const long long pos = A.pos0 + blockIdx.x;
+    T* row = reinterpret_cast<T*>(A.ring.rows) + (size_t)(pos % A.ring.slots) * A.ring.ld;
+    for (int u = warp; u < A.heads + 2 * A.kv_heads; u += 8) {
+        if (u < A.heads) {
+            const T* q = reinterpret_cast<const T*>(A.q) + o + (size_t)u * A.dim;
+            T* dst = reinterpret_cast<T*>(A.qn) + ((size_t)blockIdx.x * A.heads + u) * A.dim;
+            const float f = warp_inv_rms(q, A.dim, A.eps);
+            for (int i = lane; i < A.dim; i += 32) dst[i] = from_f32<T>(to_f32(q[i]) * f * A.q_norm[i]);
+        } else if (u < A.heads + A.kv_heads) {
+            const int g = u - A.heads;
+            const T* k = reinterpret_cast<const T*>(A.k) + o + (size_t)g * A.dim;
+            const float f = warp_inv_rms(k, A.dim, A.eps);
+            for (int i = lane; i < A.dim; i += 32) row[(size_t)g * A.ring.kd + i] = from_f32<T>(to_f32(k[i]) * f * A.k_norm[i]);
+        } else {
+            const int g = u - A.heads - A.kv_heads;
+            const T* v = reinterpret_cast<const T*>(A.v) + o + (size_t)g * A.vdim;
+            for (int i = lane; i < A.vdim; i += 32) row[(size_t)A.kv_heads * A.ring.kd + (size_t)g * A.ring.vd + i] = v[i];
+        }
+    }
+}
+
+// out[r, c] = x[r, c] * sigmoid(gate[r, c]) * scale; grid = (rows, ceil(n / 1024)).
+template <typename T>
+__global__ void __launch_bounds__(256)
+gate_rows_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ gate, int ldg, T* __restrict__ out, int ldo, int n, float scale) {
+    llvq_dependent_enter();
+    const size_t r = blockIdx.x;
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+        const int c = (blockIdx.y * 4 + k) * 256 + threadIdx.x;
+        if (c < n) out[r * ldo + c] = from_f32<T>(to_f32(x[r * ldx + c]) * scale * sigmoid_f(to_f32(gate[r * ldg + c])));
+    }
+}
+
+}  // namespace llvq

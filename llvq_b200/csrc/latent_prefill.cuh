@@ -1,6 +1,7 @@
-// Latent attention of a prompt portion, keys and values expanded (k = W_uk c, v = W_uv c by a matrix product
-// ahead of it): causal, windowed, with a sink in the denominator. Queries are laid out head by head as
-// [dim unrotated | rot_dim to be rotated], kv rows as [heads * dim keys | heads * vdim values], the rotated key
+// Attention of a prompt portion over keys and values laid out per position, causal, windowed, with a sink in the
+// denominator: latent attention (expanded by a matrix product ahead of it, k = W_uk c, v = W_uv c) and, with nothing to
+// rotate, grouped-query attention (query head h reads key/value head h / rep; heads may be padded). Queries are laid out head by head as
+// [dim unrotated | rot_dim to be rotated], kv rows as [keys, k_head apart | values from v_off on, v_head apart], the rotated key
 // part is read from the cached rows (one for all heads). Key j of the operands is position key0 + j, query i is
 // position pos0 + i.
 //
@@ -27,6 +28,7 @@ struct LatentPrefillArgs {
     int n_q, n_k, heads, dim, rot_dim, vdim, ld_kv, ld_kr;
     int window;
     float scale;
+    int rep, k_head, v_head, v_off;
 };
 
 constexpr int kLpM = 128, kLpN = 64, kLpThreads = 256;
@@ -53,7 +55,7 @@ latent_prefill_mma_kernel(LatentPrefillArgs A) {
     const bf16* KV = reinterpret_cast<const bf16*>(A.kv);
     const bf16* KR = reinterpret_cast<const bf16*>(A.kr);
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int h = blockIdx.y, v_lo = blockIdx.z * NV * 8, v_n = min(NV * 8, A.vdim - v_lo);
+    const int h = blockIdx.y, hk = h / A.rep, v_lo = blockIdx.z * NV * 8, v_n = min(NV * 8, A.vdim - v_lo);
     // long rows first: the last CTAs of a portion see the most keys
     const int q_lo = ((int)gridDim.x - 1 - (int)blockIdx.x) * kLpM, q_n = min(kLpM, A.n_q - q_lo);
     llvq_dependent_enter();
@@ -73,25 +75,25 @@ latent_prefill_mma_kernel(LatentPrefillArgs A) {
             for (int i = tid; i < kLpN * ct; i += kLpThreads) {
                 const int r = i / ct, c = i - r * ct, j = base + r;
                 const bool in = j < k_end && c < cn + cr;
-                const bf16* src = !in ? KV : c < cn ? KV + (size_t)j * A.ld_kv + (size_t)h * A.dim + 8 * c : KR + (size_t)j * A.ld_kr + 8 * (c - cn);
+                const bf16* src = !in ? KV : c < cn ? KV + (size_t)j * A.ld_kv + (size_t)hk * A.k_head + 8 * c : KR + (size_t)j * A.ld_kr + 8 * (c - cn);
                 copy16_async(dk + r * pitch + 8 * c, src, in);
             }
             for (int i = tid; i < kLpN * NV; i += kLpThreads) {
                 const int r = i / NV, c = i - r * NV, j = base + r;
                 const bool in = j < k_end && 8 * c < v_n;
-                copy16_async(dv + r * vp + 8 * c, in ? KV + (size_t)j * A.ld_kv + (size_t)A.heads * A.dim + (size_t)h * A.vdim + v_lo + 8 * c : KV, in);
+                copy16_async(dv + r * vp + 8 * c, in ? KV + (size_t)j * A.ld_kv + A.v_off + (size_t)hk * A.v_head + v_lo + 8 * c : KV, in);
             }
         } else {
             for (int i = tid; i < kLpN * (pitch - 8); i += kLpThreads) {
                 const int r = i / (pitch - 8), c = i - r * (pitch - 8), j = base + r;
                 bf16 v = __float2bfloat16_rn(0.0f);
-                if (j < k_end && c < qk) v = c < A.dim ? KV[(size_t)j * A.ld_kv + (size_t)h * A.dim + c] : KR[(size_t)j * A.ld_kr + c - A.dim];
+                if (j < k_end && c < qk) v = c < A.dim ? KV[(size_t)j * A.ld_kv + (size_t)hk * A.k_head + c] : KR[(size_t)j * A.ld_kr + c - A.dim];
                 dk[r * pitch + c] = v;
             }
             for (int i = tid; i < kLpN * NV * 8; i += kLpThreads) {
                 const int r = i / (NV * 8), c = i - r * (NV * 8), j = base + r;
                 bf16 v = __float2bfloat16_rn(0.0f);
-                if (j < k_end && c < v_n) v = KV[(size_t)j * A.ld_kv + (size_t)A.heads * A.dim + (size_t)h * A.vdim + v_lo + c];
+                if (j < k_end && c < v_n) v = KV[(size_t)j * A.ld_kv + A.v_off + (size_t)hk * A.v_head + v_lo + c];
                 dv[r * vp + c] = v;
             }
         }
@@ -266,7 +268,7 @@ template <typename T>
 __global__ void __launch_bounds__(kLsWarps * 32)
 latent_prefill_simt_kernel(LatentPrefillArgs A) {
     extern __shared__ __align__(16) float ls_smem[];
-    const int qk = A.dim + A.rot_dim, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, h = blockIdx.y;
+    const int qk = A.dim + A.rot_dim, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, h = blockIdx.y, hk = h / A.rep;
     float* q_s = ls_smem + (size_t)warp * (qk + A.vdim);
     float* o_s = q_s + qk;
     llvq_dependent_enter();
@@ -297,7 +299,7 @@ latent_prefill_simt_kernel(LatentPrefillArgs A) {
         const int j = base + lane, here = min(32, last - base + 1);
         float s = -INFINITY;
         if (j <= last) {
-            const T* k = KV + (size_t)j * A.ld_kv + (size_t)h * A.dim;
+            const T* k = KV + (size_t)j * A.ld_kv + (size_t)hk * A.k_head;
             const T* kr = KR + (size_t)j * A.ld_kr;
             float a = 0.0f;
             for (int c = 0; c < A.dim; ++c) a = fmaf(q_s[c], to_f32(k[c]), a);
@@ -307,7 +309,7 @@ latent_prefill_simt_kernel(LatentPrefillArgs A) {
         const float mn = fmaxf(m, warp_max_f(s)), corr = exp2f(m - mn), p = exp2f(s - mn);
         l = l * corr + warp_sum_f(p);
         m = mn;
-        const T* v = KV + (size_t)base * A.ld_kv + (size_t)A.heads * A.dim + (size_t)h * A.vdim;
+        const T* v = KV + (size_t)base * A.ld_kv + A.v_off + (size_t)hk * A.v_head;
         for (int c0 = 0; c0 < A.vdim; c0 += 32) {  // every lane takes part in the shuffles
             const int c = c0 + lane;
             const bool in = c < A.vdim;

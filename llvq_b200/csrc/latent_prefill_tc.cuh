@@ -29,7 +29,7 @@ constexpr int kTcKeyLoaders = 64, kTcValueLoaders = 32;  // threads
 
 struct LatentPrefillTcArgs {
     LatentPrefillArgs p;      // kv = the keys [n_k, ld_kv]
-    const void* vt;           // [heads * vdim, ld_vt], zero from n_k to the next multiple of 8
+    const void* vt;           // [heads / rep * vdim, ld_vt], zero from n_k to the next multiple of 8
     int ld_vt;
     unsigned int* err;
 };
@@ -118,7 +118,7 @@ latent_prefill_tc_kernel(LatentPrefillTcArgs T) {
     unsigned char* base0 = tc_raw + (smem0 - pipe_smem_addr(tc_raw));
     const unsigned int q_bytes = (unsigned int)(kTcM * 128 * panels), k_bytes = (unsigned int)(kTcN * 128 * panels), v_bytes = (unsigned int)(vrows * 128);
     const unsigned int off_k = 2 * q_bytes, off_v = off_k + 2 * k_bytes, off_p = off_v + 2 * v_bytes;
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y, hk = h / A.rep;
     const int q_lo = ((int)gridDim.x - 1 - (int)blockIdx.x) * 2 * kTcM;  // rows with the most keys first
     const int off = (int)(A.pos0 - A.key0);
     const bool two = q_lo + kTcM < A.n_q;
@@ -407,7 +407,7 @@ latent_prefill_tc_kernel(LatentPrefillTcArgs T) {
                     if (c >= 2 * ksteps) continue;
                     const bool own = c < cn, in_c = c < cq;
                     const size_t step = 4 * (size_t)(own ? A.ld_kv : A.ld_kr);
-                    const bf16* src = own ? K + (size_t)(base + r0) * A.ld_kv + (size_t)h * A.dim + 8 * c : KR + (size_t)(base + r0) * A.ld_kr + 8 * (c - cn);
+                    const bf16* src = own ? K + (size_t)(base + r0) * A.ld_kv + (size_t)hk * A.k_head + 8 * c : KR + (size_t)(base + r0) * A.ld_kr + 8 * (c - cn);
                     unsigned char* dst = base0 + off_k + (t & 1) * k_bytes + p * (kTcN * 128) + r0 * 128;
                     const int even = (c8 ^ (r0 & 7)) << 4, odd = (c8 ^ ((r0 + 4) & 7)) << 4;
 #pragma unroll
@@ -420,7 +420,7 @@ latent_prefill_tc_kernel(LatentPrefillTcArgs T) {
                 const int j = base + 8 * c8;
                 const bool in_j = j < A.n_k;
                 const size_t step = 4 * (size_t)T.ld_vt;
-                const bf16* src = VT + ((size_t)h * A.vdim + sub) * T.ld_vt + j;
+                const bf16* src = VT + ((size_t)hk * A.vdim + sub) * T.ld_vt + j;
                 unsigned char* dst = base0 + off_v + (t & 1) * v_bytes + sub * 128;
                 const int even = (c8 ^ sub) << 4, odd = (c8 ^ (sub + 4)) << 4;
 #pragma unroll 4

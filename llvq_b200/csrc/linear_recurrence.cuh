@@ -1,0 +1,259 @@
+// Short causal convolutions over time and the real-gated linear recurrence behind one (per channel):
+//
+//   u = conv(x) + bias;  r = sigmoid(Ra u + ra), i = sigmoid(Ri u + ri)  (block-diagonal matrices)
+//   log a = -c r softplus(lam);  S <- a S + sqrt(1 - a^2) i u;  out = S gelu(y) * scale
+//
+// What a sequence carries from token to token lives in two kinds of store, both addressed by position, so that a step
+// that is run again at its position changes nothing and no CTA reads what another writes:
+//
+//   convolution inputs   f32 [taps, channels]: the input of position p in row p % taps. A step reads the rows of the
+//                        taps - 1 positions before it and writes its own.
+//   recurrent state      f32 [2, ...]: the state before position p in half p % 2; a step reads that half and writes the
+//                        other. Position 0 reads zeros whatever is stored, as convolutions do ahead of the first token.
+//
+//   lru_token            the token step: a CTA takes 32 channels of a block: the block's u, two rows of the gate matrix
+//                        per channel, the recurrence, the gate branch.
+//   conv_rows_kernel     u of a prompt portion; conv_keep_kernel then stores the inputs the next step reads.
+//   lru_scan_kernel      the recurrence of a portion, one pass: a CTA owns 32 channels, a warp 32 tokens at a time in
+//                        registers; the warps' products and sums meet in shared memory, 512 tokens a turn.
+#pragma once
+#include "gqa_attn.cuh"
+
+namespace llvq {
+
+__device__ __forceinline__ float gelu_tanh_f(float z) {
+    return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+__device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
+__device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
+
+constexpr float kLruDecay = 8.0f;  // c
+constexpr int kLruRows = 32;       // channels of a CTA
+
+// Convolution of one channel at `pos` over inputs kept in a ring of `taps` rows; x is the token's own input.
+__device__ __forceinline__ float conv_token(const float* w, int taps, const float* ring, int channels, int ch, long long pos, float x) {
+    float u = w[taps - 1] * x;
+    for (int k = 1; k < taps; ++k)
+        if (pos >= k) u = fmaf(w[taps - 1 - k], ring[(size_t)((pos - k) % taps) * channels + ch], u);
+    return u;
+}
+
+struct LruArgs {
+    const float* x;       // [width] input of the convolution
+    const float* y;       // [width] gate branch before its activation
+    const float* conv_w;  // [width, taps]
+    const float* conv_b;  // [width]
+    const void* w;        // [blocks, 2 n, ldw] of T: the rows of Ra, then those of Ri
+    const float* b;       // [blocks, 2 n]
+    const float* lam;     // [width]: softplus of the stored value
+    const long long* pos;
+    float* conv;          // [taps, width]
+    float* state;         // [2, width]
+    float* out;           // [width]
+    int blocks, n, taps, ldw;
+    float out_scale;
+};
+
+__host__ __device__ inline int lru_tiles(int n) { return (n + kLruRows - 1) / kLruRows; }
+
+// One step of the recurrence of a channel; returns the new state.
+__device__ __forceinline__ float lru_step(float r, float i, float lam, float u, float s) {
+    const float log_a = -kLruDecay * r * lam;
+    return fmaf(expf(log_a), s, sqrtf(-expm1f(2.0f * log_a)) * i * u);
+}
+
+// One CTA's part; `smem` holds ldw floats. Calls the dependency wait itself, behind its first loads of the matrices.
+template <typename T>
+__device__ __forceinline__ void lru_token(const LruArgs& A, int cta, float* u_s) {
+    constexpr int VN = Vec16<T>::N;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int tiles = lru_tiles(A.n), blk = cta / tiles, c0 = (cta - blk * tiles) * kLruRows + warp * 4;  // this warp's first channel of the block
+    const int vecs = A.ldw / VN, width = A.blocks * A.n;
+    const uint4* W = reinterpret_cast<const uint4*>(A.w) + (size_t)blk * 2 * A.n * vecs;
+    auto row = [&](int k) { return W + (size_t)((k >> 2) * A.n + min(c0 + (k & 3), A.n - 1)) * vecs; };  // k: 4 rows of Ra, 4 of Ri
+    uint4 ahead[8];
+    if (c0 < A.n && lane < vecs) {
+#pragma unroll
+        for (int k = 0; k < 8; ++k) ahead[k] = __ldg(row(k) + lane);
+    }
+    llvq_dependent_enter();
+    const long long pos = *A.pos;
+    for (int c = tid; c < A.ldw; c += 256) {
+        const int ch = blk * A.n + c;
+        u_s[c] = c < A.n ? A.conv_b[ch] + conv_token(A.conv_w + (size_t)ch * A.taps, A.taps, A.conv, width, ch, pos, A.x[ch]) : 0.0f;
+    }
+    __syncthreads();
+    if (c0 >= A.n) return;
+    float acc[8];
+#pragma unroll
+    for (int k = 0; k < 8; ++k) acc[k] = 0.0f;
+    for (int v = lane; v < vecs; v += 32) {
+        if (v != lane) {
+#pragma unroll
+            for (int k = 0; k < 8; ++k) ahead[k] = __ldg(row(k) + v);
+        }
+#pragma unroll
+        for (int k = 0; k < 8; ++k) {
+            float f[VN];
+            Vec16<T>::widen(ahead[k], f);
+#pragma unroll
+            for (int j = 0; j < VN; ++j) acc[k] = fmaf(f[j], u_s[v * VN + j], acc[k]);
+        }
+    }
+    float zr = 0.0f, zi = 0.0f;
+#pragma unroll
+    for (int k = 0; k < 8; ++k) {
+        const float s = warp_sum_f(acc[k]);
+        if (lane == (k & 3)) (k < 4 ? zr : zi) = s;
+    }
+    const int c = c0 + lane, ch = blk * A.n + c;
+    if (lane < 4 && c < A.n) {
+        const float r = sigmoid_f(zr + A.b[(size_t)blk * 2 * A.n + c]), i = sigmoid_f(zi + A.b[(size_t)blk * 2 * A.n + A.n + c]);
+        const float s = pos > 0 ? A.state[(size_t)(pos & 1) * width + ch] : 0.0f;
+        const float t = lru_step(r, i, A.lam[ch], u_s[c], s);
+        A.state[(size_t)((pos + 1) & 1) * width + ch] = t;
+        A.conv[(size_t)(pos % A.taps) * width + ch] = A.x[ch];
+        A.out[ch] = t * gelu_tanh_f(A.y[ch]) * A.out_scale;
+    }
+}
+
+// Attention and recurrence that read the same token, side by side in one launch: the first `attn_ctas` CTAs are the attention's.
+template <typename T>
+__global__ void __launch_bounds__(256)
+mixer_token_kernel(GqaArgs A, int attn_ctas, LruArgs R) {
+    extern __shared__ __align__(16) unsigned char mt_smem[];
+    if ((int)blockIdx.x < attn_ctas) {
+        llvq_dependent_enter();
+        gqa_token<T>(A, blockIdx.x, mt_smem);
+    } else {
+        lru_token<T>(R, blockIdx.x - attn_ctas, reinterpret_cast<float*>(mt_smem));
+    }
+}
+
+// ---- prompt portions ----
+
+// Input of channel c at place t of a portion that starts at pos0 (t may be negative), as f32; xb: the channel's input bias.
+template <typename T>
+__device__ __forceinline__ float conv_input(const T* x, int ldx, float xb, const float* ring, int channels, int taps, long long pos0, int t, int c) {
+    if (t >= 0) return to_f32(x[(size_t)t * ldx + c]) + xb;
+    const long long p = pos0 + t;
+    return p >= 0 ? ring[(size_t)(p % taps) * channels + c] : 0.0f;
+}
+
+constexpr int kConvRun = 16;  // tokens of a thread
+
+// grid = (ceil(channels / 256), ceil(n / 16)): a thread slides along 16 tokens of one channel.
+template <typename T>
+__global__ void __launch_bounds__(256)
+conv_rows_kernel(const T* __restrict__ x, int ldx, const float* __restrict__ x_bias, const float* __restrict__ w, const float* __restrict__ bias, const float* __restrict__ ring,
+                 T* __restrict__ out, int channels, int taps, long long pos0, int n) {
+    llvq_dependent_enter();
+    const int c = blockIdx.x * 256 + threadIdx.x, t0 = blockIdx.y * kConvRun, t1 = min(n, t0 + kConvRun);
+    if (c >= channels) return;
+    const float b = bias ? bias[c] : 0.0f, xb = x_bias ? x_bias[c] : 0.0f;
+    const float* wc = w + (size_t)c * taps;
+    if (taps == 4) {
+        const float w0 = wc[0], w1 = wc[1], w2 = wc[2], w3 = wc[3];
+        float x3 = conv_input(x, ldx, xb, ring, channels, 4, pos0, t0 - 3, c), x2 = conv_input(x, ldx, xb, ring, channels, 4, pos0, t0 - 2, c),
+              x1 = conv_input(x, ldx, xb, ring, channels, 4, pos0, t0 - 1, c);
+        float in[kConvRun];
+#pragma unroll
+        for (int k = 0; k < kConvRun; ++k) in[k] = t0 + k < t1 ? to_f32(x[(size_t)(t0 + k) * ldx + c]) + xb : 0.0f;
+#pragma unroll
+        for (int k = 0; k < kConvRun; ++k) {
+            if (t0 + k < t1) out[(size_t)(t0 + k) * channels + c] = from_f32<T>(fmaf(w0, x3, fmaf(w1, x2, fmaf(w2, x1, fmaf(w3, in[k], b)))));
+            x3 = x2, x2 = x1, x1 = in[k];
+        }
+        return;
+    }
+    for (int t = t0; t < t1; ++t) {
+        float u = b;
+        for (int k = 0; k < taps; ++k) u = fmaf(wc[taps - 1 - k], conv_input(x, ldx, xb, ring, channels, taps, pos0, t - k, c), u);
+        out[(size_t)t * channels + c] = from_f32<T>(u);
+    }
+}
+
+// The last taps inputs of the portion into the ring. Runs behind the kernels that read it.
+template <typename T>
+__global__ void __launch_bounds__(256)
+conv_keep_kernel(const T* __restrict__ x, int ldx, const float* __restrict__ x_bias, float* __restrict__ ring, int channels, int taps, long long pos0, int n) {
+    llvq_dependent_enter();
+    const int c = blockIdx.x * 256 + threadIdx.x;
+    if (c >= channels) return;
+    for (int t = max(0, n - taps); t < n; ++t) ring[(size_t)((pos0 + t) % taps) * channels + c] = to_f32(x[(size_t)t * ldx + c]) + (x_bias ? x_bias[c] : 0.0f);
+}
+
+struct LruScanArgs {
+    const void* u;       // [n_tok, width] of T
+    const float* z;      // [blocks, n_tok, 2 n]: Ra u, then Ri u, without their biases
+    const float* b;      // [blocks, 2 n]
+    const float* lam;    // [width]: softplus of the stored value
+    const void* y;       // [n_tok, ldy] of T
+    const float* y_bias; // [width]
+    float* state;        // [2, width]
+    void* out;           // [n_tok, ldo] of T
+    long long pos0;
+    int n_tok, blocks, n, ldy, ldo;
+    float out_scale;
+};
+
+constexpr int kScanTok = 32, kScanWarps = 16;
+
+// grid = ceil(width / 32), 512 threads: lane = channel, warp = 32 tokens of the turn's 512.
+template <typename T>
+__global__ void __launch_bounds__(kScanWarps * 32)
+lru_scan_kernel(LruScanArgs A) {
+    __shared__ float prod_s[kScanWarps][32], sum_s[kScanWarps][32], carry_s[32];
+    llvq_dependent_enter();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, width = A.blocks * A.n;
+    const int ch = blockIdx.x * 32 + lane, cc = min(ch, width - 1), blk = cc / A.n, c = cc - blk * A.n;
+    const float br = A.b[(size_t)blk * 2 * A.n + c], bi = A.b[(size_t)blk * 2 * A.n + A.n + c], lam = A.lam[cc], yb = A.y_bias[cc];
+    const float* z = A.z + (size_t)blk * A.n_tok * 2 * A.n + c;
+    const T* U = reinterpret_cast<const T*>(A.u) + cc;
+    const T* Y = reinterpret_cast<const T*>(A.y) + cc;
+    T* O = reinterpret_cast<T*>(A.out) + cc;
+    if (warp == 0) carry_s[lane] = A.pos0 > 0 ? A.state[(size_t)(A.pos0 & 1) * width + cc] : 0.0f;
+    for (int t0 = 0; t0 < A.n_tok; t0 += kScanWarps * kScanTok) {
+        const int tw = t0 + warp * kScanTok;
+        float a[kScanTok], x[kScanTok];
+#pragma unroll
+        for (int k = 0; k < kScanTok; ++k) {
+            const int t = min(tw + k, A.n_tok - 1);
+            a[k] = z[(size_t)t * 2 * A.n];
+            x[k] = z[(size_t)t * 2 * A.n + A.n];
+        }
+        float prod = 1.0f, sum = 0.0f;
+#pragma unroll
+        for (int k = 0; k < kScanTok; ++k) {
+            const int t = tw + k;
+            if (t < A.n_tok) {
+                const float log_a = -kLruDecay * sigmoid_f(a[k] + br) * lam;
+                a[k] = expf(log_a);
+                x[k] = sqrtf(-expm1f(2.0f * log_a)) * sigmoid_f(x[k] + bi) * to_f32(U[(size_t)t * width]);
+            } else {
+                a[k] = 1.0f;
+                x[k] = 0.0f;
+            }
+            prod *= a[k];
+            sum = fmaf(a[k], sum, x[k]);
+        }
+        prod_s[warp][lane] = prod;
+        sum_s[warp][lane] = sum;
+        __syncthreads();
+        float s = carry_s[lane];
+        for (int w = 0; w < warp; ++w) s = fmaf(prod_s[w][lane], s, sum_s[w][lane]);
+        __syncthreads();  // the carry and the warps' sums are read
+        if (warp == kScanWarps - 1) carry_s[lane] = fmaf(prod, s, sum);
+#pragma unroll
+        for (int k = 0; k < kScanTok; ++k) {
+            const int t = tw + k;
+            s = fmaf(a[k], s, x[k]);
+            if (t < A.n_tok && ch < width)
+                O[(size_t)t * A.ldo] = from_f32<T>(s * gelu_tanh_f(to_f32(Y[(size_t)t * A.ldy]) + yb) * A.out_scale);
+        }
+    }
+    __syncthreads();
+    if (warp == 0 && ch < width) A.state[(size_t)((A.pos0 + A.n_tok) & 1) * width + ch] = carry_s[lane];
+}
+
+}  // namespace llvq
