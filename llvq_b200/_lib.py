@@ -59,6 +59,25 @@ class DenseLatent(C.Structure):
                 [(n, C.c_void_p) for n in ("ring", "cos_t", "sin_t", "uk", "uv", "kv_norm", "sink", "qlat", "part")])
 
 
+class DenseGqa(C.Structure):
+    """llvq_dn_gqa of include/llvq_dense.h."""
+    _fields_ = ([(n, C.c_int32) for n in ("dtype", "heads", "kv_heads", "dim", "vdim", "slots", "ld", "kd", "vd", "window", "splits")] +
+                [(n, C.c_float) for n in ("scale", "eps", "out_scale")] +
+                [(n, C.c_void_p) for n in ("ring", "q_norm", "k_norm", "q", "k", "v", "gate", "part", "arrived", "out")])
+
+
+class DenseLru(C.Structure):
+    """llvq_dn_lru of include/llvq_dense.h."""
+    _fields_ = ([(n, C.c_int32) for n in ("dtype", "blocks", "n", "taps", "ldw")] + [("out_scale", C.c_float)] +
+                [(n, C.c_void_p) for n in ("conv_w", "conv_b", "b", "lam", "conv", "state", "w", "x", "y", "out")])
+
+
+class DenseDelta(C.Structure):
+    """llvq_dn_delta of include/llvq_dense.h."""
+    _fields_ = ([(n, C.c_int32) for n in ("dtype", "heads", "kv_heads", "dim", "vdim", "vp", "taps")] + [("eps", C.c_float)] +
+                [(n, C.c_void_p) for n in ("conv_w", "decay", "dt_bias", "norm", "conv", "state", "x", "gate", "beta", "alpha", "o", "arrived", "out")])
+
+
 class LlvqError(RuntimeError):
     def __init__(self, status: int, message: str):
         super().__init__(f"llvq status {status}: {message}")
@@ -158,6 +177,20 @@ _DENSE_SIGNATURES = {
     "llvq_dn_latent_rows": (C.c_int, [C.POINTER(DenseLatent), C.c_void_p, C.c_int32, C.c_int32, C.c_void_p, C.c_void_p, C.c_int64, C.c_int32, C.c_int32,
                                       C.c_void_p]),
     "llvq_dn_glu_rows": (C.c_int, [C.c_int32] + [C.c_void_p] * 3 + [C.c_int32] * 2 + [C.c_float] * 3 + [C.c_void_p]),
+    "llvq_dn_gated_rows": (C.c_int, [C.c_int32] + [C.c_void_p] * 3 + [C.c_int32] * 3 + [C.c_float] * 4 + [C.c_void_p]),
+    "llvq_dn_add_norms_rows": (C.c_int, [C.c_int32] + [C.c_void_p] * 4 + [C.c_int32] + [C.c_void_p] * 4 + [C.c_float] + [C.c_int32] * 2 + [C.c_void_p]),
+    "llvq_dn_mixer_token": (C.c_int, [C.POINTER(DenseGqa), C.POINTER(DenseLru)] + [C.c_void_p] * 2),
+    "llvq_dn_gqa_rows": (C.c_int, [C.POINTER(DenseGqa)] + [C.c_void_p] * 3 + [C.c_int32, C.c_void_p, C.c_int64, C.c_int32, C.c_void_p]),
+    "llvq_dn_gqa_prefill_transposes": (C.c_int, [C.POINTER(DenseGqa), C.c_int32]),
+    "llvq_dn_gqa_prefill": (C.c_int, [C.POINTER(DenseGqa)] + [C.c_void_p] * 3 + [C.c_int32] * 3 + [C.c_int64] * 2 + [C.c_void_p, C.c_int32, C.c_void_p]),
+    "llvq_dn_gate_rows": (C.c_int, [C.c_int32] + [C.c_void_p, C.c_int32] * 3 + [C.c_int32] * 2 + [C.c_float, C.c_void_p]),
+    "llvq_dn_conv_rows": (C.c_int, [C.c_int32, C.c_void_p, C.c_int32] + [C.c_void_p] * 5 + [C.c_int32] * 2 + [C.c_int64, C.c_int32, C.c_void_p]),
+    "llvq_dn_conv_keep": (C.c_int, [C.c_int32, C.c_void_p, C.c_int32] + [C.c_void_p] * 2 + [C.c_int32] * 2 + [C.c_int64, C.c_int32, C.c_void_p]),
+    "llvq_dn_lru_rows": (C.c_int, [C.POINTER(DenseLru)] + [C.c_void_p] * 3 + [C.c_int32, C.c_void_p, C.c_void_p, C.c_int32, C.c_int64, C.c_int32, C.c_void_p]),
+    "llvq_dn_delta_token": (C.c_int, [C.POINTER(DenseDelta)] + [C.c_void_p] * 2),
+    "llvq_dn_delta_scratch": (C.c_int, [C.POINTER(DenseDelta), C.c_int32, C.POINTER(C.c_size_t)]),
+    "llvq_dn_delta_rows": (C.c_int, [C.POINTER(DenseDelta), C.c_void_p, C.c_int32, C.c_void_p, C.c_void_p, C.c_int32, C.c_void_p, C.c_void_p, C.c_int32, C.c_int64,
+                                     C.c_int32, C.c_void_p]),
     "llvq_dn_softcap": (C.c_int, [C.c_void_p, C.c_size_t, C.c_float, C.c_void_p]),
 }
 

@@ -1,5 +1,5 @@
-"""Caches of one sequence: the int8 key/value cache of grouped-query attention and the ring of latent rows of
-latent attention."""
+"""What one sequence keeps from token to token: the int8 key/value cache of grouped-query attention, rings of cached rows
+(latent rows, or keys and values of a window), the states of recurrent layers and the inputs of short convolutions."""
 from __future__ import annotations
 
 from typing import Optional
@@ -53,17 +53,21 @@ class Int8KvCache:
         return 2 * (self.q[0][0].numel() + 2 * 2 * self.s[0][0].numel())
 
 
-class LatentRing:
-    """Cache of one latent-attention layer: per position one row [latent | rotated key part | zeros] shared by all
-    heads. Position p sits in slot p % slots. `slots` covers the widest window that reads the layer and one prompt
-    portion, so that a portion is stored whole before its first query looks back."""
+def whole_vectors(n: int, dtype) -> int:
+    """n elements up to a whole number of 16-byte vectors."""
+    vec = 16 // dtype.itemsize
+    return -(-n // vec) * vec
 
-    def __init__(self, capacity: int, window: int, portion: int, kv_rank: int, rot_dim: int, dtype, device):
+
+class RowRing:
+    """One row of `width` elements (and zeros to a whole vector) per position; position p sits in slot p % slots. `slots`
+    covers the widest window that reads the layer and one prompt portion, so that a portion is stored whole before its
+    first query looks back."""
+
+    def __init__(self, capacity: int, window: int, portion: int, width: int, dtype, device):
         import torch
-        vec = 16 // torch.empty(0, dtype=dtype).element_size()
         self.slots = min(capacity, window - 1 + portion)
-        self.kv_rank, self.rot_dim = kv_rank, rot_dim
-        self.ld = -(-(kv_rank + rot_dim) // vec) * vec
+        self.ld = whole_vectors(width, dtype)
         self.rows = torch.zeros(self.slots, self.ld, dtype=dtype, device=device)
 
     def read(self, lo: int, hi: int):
@@ -78,3 +82,48 @@ class LatentRing:
 
     def bytes_per_position(self) -> int:
         return self.ld * self.rows.element_size()
+
+
+class LatentRing(RowRing):
+    """Cache of one latent-attention layer: rows [latent | rotated key part], shared by all heads."""
+
+    def __init__(self, capacity: int, window: int, portion: int, kv_rank: int, rot_dim: int, dtype, device):
+        super().__init__(capacity, window, portion, kv_rank + rot_dim, dtype, device)
+        self.kv_rank, self.rot_dim = kv_rank, rot_dim
+
+
+class KvRing(RowRing):
+    """Cache of one grouped-query layer: rows [kv_heads keys | kv_heads values], every head padded to whole vectors."""
+
+    def __init__(self, capacity: int, window: int, portion: int, kv_heads: int, dim: int, vdim: int, dtype, device):
+        self.kv_heads, self.dim, self.vdim = kv_heads, dim, vdim
+        self.kd, self.vd = whole_vectors(dim, dtype), whole_vectors(vdim, dtype)
+        super().__init__(capacity, window, portion, kv_heads * (self.kd + self.vd), dtype, device)
+
+    def values_transposed(self, rows):
+        """[kv_heads * vdim, positions to a multiple of 8] of rows read from the ring, zeros beyond them."""
+        import torch
+        n, k = rows.shape[0], self.kv_heads * self.kd
+        vt = torch.empty(self.kv_heads * self.vdim, -(-n // 8) * 8, dtype=rows.dtype, device=rows.device)
+        vt[:, n:].zero_()
+        v = rows[:, k:k + self.kv_heads * self.vd].unflatten(1, (self.kv_heads, self.vd))[..., :self.vdim]
+        vt.view(self.kv_heads, self.vdim, -1)[..., :n].copy_(v.permute(1, 2, 0))
+        return vt
+
+
+class RecurrentState:
+    """f32 state of one recurrent layer in two halves: the state before position p is half p % 2, so a step reads one
+    half and writes the other, and running it again at its position changes nothing. Nothing needs clearing: position 0
+    starts from zeros whatever is stored."""
+
+    def __init__(self, *shape: int, device):
+        import torch
+        self.halves = torch.zeros(2, *shape, dtype=torch.float32, device=device)
+
+
+class ConvInputs:
+    """The last inputs of a short causal convolution, f32: the input of position p is row p % taps."""
+
+    def __init__(self, taps: int, channels: int, device):
+        import torch
+        self.rows = torch.zeros(taps, channels, dtype=torch.float32, device=device)

@@ -31,8 +31,8 @@ import numpy as np
 
 from . import _lib
 from .cache import LatentRing
+from .dense import DenseLM, DenseMatrix
 from .registry import register
-from .token_loop import TokenLoop
 
 GLU_GAIN, GLU_SHIFT = 1.702, 1.0  # sigmoid(1.702 g), (u + 1)
 
@@ -115,45 +115,14 @@ class LatentConfig:
                             float(c["embedding"]["scale"]), float(cap) if cap else None, layers)
 
 
-class DenseMatrix:
-    """Row-concatenated (or row-interleaved) [out, in] matrices on the device, rows padded with zeros to whole 16-byte
-    vectors."""
-
-    def __init__(self, parts, dtype, device, interleave: bool = False):
-        import torch
-        self.n, self.k = sum(p.shape[0] for p in parts), parts[0].shape[1]
-        vec = 16 // torch.empty(0, dtype=dtype).element_size()
-        self.ld = -(-self.k // vec) * vec
-        self.w = torch.zeros(self.n, self.ld, dtype=dtype, device=device)
-        if interleave:
-            if len({p.shape[0] for p in parts}) != 1:
-                raise ValueError(f"interleaved matrices of {[p.shape[0] for p in parts]} rows")
-            for i, p in enumerate(parts):
-                self.w[i::len(parts), :self.k].copy_(p)
-            return
-        at = 0
-        for p in parts:
-            self.w[at:at + p.shape[0], :self.k].copy_(p)
-            at += p.shape[0]
-
-    def rows(self, lo: int, hi: Optional[int] = None):
-        """The unpadded rows as an operand of a matrix product."""
-        return self.w[lo:hi, :self.k]
-
-    def ptr(self, row: int = 0) -> int:
-        return self.w.data_ptr() + row * self.ld * self.w.element_size()
-
-
-class LatentLM(TokenLoop):
+class LatentLM(DenseLM):
     PHASES = ("embed", "projections", "latent_query", "attention", "latent_value", "norm", "head")
 
     def __init__(self, cfg: LatentConfig, tensor, dtype: str, capacity: int, device, prefill_chunk: int = 2048):
         """`tensor(name)` gives a weight by its name (any device)."""
         import torch
-        self.cfg, self.lib = cfg, _lib.load_dense()
-        self.dtype = {"bfloat16": torch.bfloat16, "float32": torch.float32}[dtype]
-        self.dt = {"bfloat16": _lib.DN_BF16, "float32": _lib.DN_F32}[dtype]
-        self._init_loop(device, capacity, prefill_chunk)
+        self.cfg, self.eps, self.softcap = cfg, cfg.eps, cfg.softcap or 0.0
+        self._init_dense(dtype, device, capacity, prefill_chunk)
         f32 = dict(dtype=torch.float32, device=device)
 
         def mat(*names, interleave: bool = False):
@@ -162,7 +131,7 @@ class LatentLM(TokenLoop):
         def vec(*names, base: float = 0.0):
             return torch.cat([tensor(n).to(**f32) for n in names]) + base
 
-        self.embed = mat("embed")
+        self.embed = self.head = mat("embed")
         if self.embed.w.shape[0] != cfg.vocab or self.embed.k != cfg.width:
             raise ValueError(f"embed is {tuple(tensor('embed').shape)}, config.json says {cfg.vocab} x {cfg.width}")
         self.final_norm = vec("final.norm", base=1.0)  # stored around zero
@@ -234,9 +203,7 @@ class LatentLM(TokenLoop):
         self._act = buf(max([lc.mlp.ff for lc in cfg.layers if lc.mlp is not None] or [1]))
         self._qlat = buf(max(a.heads * r.ld for a, r in zip(attn, self.rings)))
         self._part = buf(max(a.heads * splits(a) * (a.kv_rank + 2) for a in attn))
-        self._logits = buf(cfg.vocab)
-        self._best_val, self._scratch = buf(1), torch.zeros(8192, dtype=torch.uint8, device=dev)
-        self._best_idx = torch.zeros(1, dtype=torch.long, device=dev)
+        self._init_head()
         ptr = lambda t: t.data_ptr() if t is not None else None
         self._lat = []
         for a, L, r in zip(attn, self.layers, self.rings):
@@ -285,43 +252,7 @@ class LatentLM(TokenLoop):
         steps.append(("head", lambda st: self._head(self._x, st)))
         self._steps = steps
 
-    def _head(self, x, st) -> None:
-        """Final norm, capped logits and greedy pick of one f32 hidden state."""
-        E = self.embed
-        d = _lib.DenseGemv(dtype=self.dt, prologue=_lib.DN_NORM, n_out=E.n, k=E.k, ldw=E.ld, alpha=1.0, eps=self.cfg.eps,
-                           softcap=self.cfg.softcap or 0.0, w=E.ptr(), y=self._logits.data_ptr(), x=x.data_ptr(), norm_w=self.final_norm.data_ptr())
-        _lib.check_dense(self.lib.llvq_dn_head(C.byref(d), self._scratch.data_ptr(), self._best_val.data_ptr(), self._best_idx.data_ptr(), st))
-
-    @staticmethod
-    def _cuda_stream():
-        import torch
-        return C.c_void_p(torch.cuda.current_stream().cuda_stream)
-
-    def _eager_step(self) -> None:
-        st, only = self._cuda_stream(), self._only
-        for phase, call in self._steps:
-            if only is None or only == phase:
-                call(st)
-        if only is None:
-            self._tok.copy_(self._best_idx)
-            self._pos += 1
-
-    def step_logits(self):
-        return self._logits.clone()
-
     # ---- prompt portions ---------------------------------------------------------
-    def _mm(self, x, w, out_dtype=None):
-        """x w^T by the library: bf16 with f32 accumulation, or true f32."""
-        import torch
-        m = torch.backends.cuda.matmul
-        if self.dtype == torch.float32:
-            held, m.allow_tf32 = m.allow_tf32, False
-            try:
-                return torch.mm(x, w.t())
-            finally:
-                m.allow_tf32 = held
-        return torch.mm(x, w.t()) if out_dtype is None else torch.mm(x, w.t(), out_dtype=out_dtype)
-
     def _expand(self, c, ukv, a, transposed: bool):
         """Keys and values of cached latents c [n, kv_rank]: ([n, keys | values], None), or ([n, keys], [values, n to a
         multiple of 8]) for the attention kernel that reads the values along the positions."""
@@ -379,22 +310,6 @@ class LatentLM(TokenLoop):
             if layers_out is not None:
                 layers_out.append(x.clone())
         return x
-
-    def pick_last(self, x):
-        self._head(x[-1:].contiguous(), self._cuda_stream())
-        return self._best_idx.clone()
-
-    def logits(self, x):
-        import torch
-        st = self._cuda_stream()
-        x = x.contiguous()
-        h = torch.empty(x.shape, dtype=self.dtype, device=self.device)
-        _lib.check_dense(self.lib.llvq_dn_postnorm_rows(self.dt, x.data_ptr(), None, None, self.final_norm.data_ptr(), 1.0, self.cfg.eps, h.data_ptr(),
-                                                        None, x.shape[0], self.cfg.width, st))
-        y = self._mm(h, self.embed.rows(0), torch.float32)
-        if self.cfg.softcap:
-            _lib.check_dense(self.lib.llvq_dn_softcap(y.data_ptr(), y.numel(), self.cfg.softcap, st))
-        return y
 
     def cache_bytes(self) -> int:
         """Bytes of all rings (a shared one counts once)."""

@@ -38,7 +38,7 @@ def register(name: str, container: str, dtypes: Tuple[str, ...], aliases: Tuple[
 
 
 def architectures() -> Dict[str, Architecture]:
-    from . import latent, model  # noqa: F401  (they register themselves)
+    from . import hybrid, latent, model  # noqa: F401  (they register themselves)
     return dict(_ARCHITECTURES)
 
 
