@@ -5,7 +5,7 @@
 // with unit vectors k and q / sqrt(dim) from short convolutions and a silu, beta = sigmoid(b),
 // g = exp(-exp(A_log) softplus(a + dt_bias)). Both read-outs are taken from the state before the token,
 // S^T k and S^T q, so that one reduction over dim serves them: o = g S^T q + (k q) u. Stores follow
-// linear_recurrence.cuh (convolution inputs by position, the state in two halves by the position's parity);
+// linear_recurrence.cuh (decays less one, convolution inputs by position, the state in two halves by the position's parity);
 // a head's state is [dim, vp] with vp the value size in whole vectors of four, zero beyond vdim.
 //
 //   delta_token_kernel  a CTA takes 32 value columns of a head; the head's last CTA to arrive norms and gates its
@@ -87,7 +87,7 @@ delta_token_kernel(DeltaArgs A) {
     kk = block_sum_f(kk, red);
     kq = block_sum_f(kq, red);
     const float fq = 1.0f / sqrtf(qq + kUnitEps) / sqrtf((float)A.dim), fk = 1.0f / sqrtf(kk + kUnitEps);
-    const float dec = expf(-A.decay[h] * softplus_f(A.a[h] + A.dt_bias[h]));
+    const float dec = expm1f(-A.decay[h] * softplus_f(A.a[h] + A.dt_bias[h]));  // g - 1
 
     // ---- both read-outs of the state before the token ----
     float4 sk = make_float4(0.0f, 0.0f, 0.0f, 0.0f), sq = sk;
@@ -119,17 +119,17 @@ delta_token_kernel(DeltaArgs A) {
             const float xv = A.x[cv];
             const float v = silu_f(conv_token(A.conv_w + (size_t)cv * A.taps, A.taps, A.conv, channels, cv, pos, xv));
             A.conv[(size_t)(pos % A.taps) * channels + cv] = xv;
-            u = sigmoid_f(A.b[h]) * (v - dec * fk * tk);
+            u = sigmoid_f(A.b[h]) * (v - fk * carry(dec, tk, 0.0f));
         }
         u_s[tid] = u * fk;  // the key is scaled where it is used
-        A.o[(size_t)h * A.vp + j] = dec * fq * tq + kq * fk * fq * u;
+        A.o[(size_t)h * A.vp + j] = fq * (carry(dec, tq, 0.0f) + kq * fk * u);
     }
     __syncthreads();
     const float4 u = *reinterpret_cast<const float4*>(u_s + j4);
     auto write = [&](const float4& s, int i) {
         const float k = k_s[i];
         *reinterpret_cast<float4*>(Sn + (size_t)i * A.vp) =
-            make_float4(fmaf(k, u.x, dec * s.x), fmaf(k, u.y, dec * s.y), fmaf(k, u.z, dec * s.z), fmaf(k, u.w, dec * s.w));
+            make_float4(carry(dec, s.x, k * u.x), carry(dec, s.y, k * u.y), carry(dec, s.z, k * u.z), carry(dec, s.w, k * u.w));
     };
     if (in) {
 #pragma unroll
@@ -173,7 +173,7 @@ struct DeltaPrepArgs {
     const float* dt_bias;
     float* qk;       // [n, kv_heads, 2, dp]: unit key, unit query / sqrt(dim)
     float* v;        // [n, heads, vdim]
-    float* sc;       // [n, heads, 4]: g, beta, k q, 0
+    float* sc;       // [n, heads, 4]: g - 1, beta, k q, 0
     long long pos0;
     int ldx, heads, kv_heads, dim, vdim, taps, dp;
 };
@@ -215,7 +215,7 @@ delta_prep_kernel(DeltaPrepArgs A) {
     for (int h = threadIdx.x; h < A.heads; h += 256) {
         const float* ba = A.ba + (size_t)t * 2 * A.heads;
         reinterpret_cast<float4*>(A.sc)[(size_t)t * A.heads + h] =
-            make_float4(expf(-A.decay[h] * softplus_f(ba[A.heads + h] + A.dt_bias[h])), sigmoid_f(ba[h]), kq_s[h / rep], 0.0f);
+            make_float4(expm1f(-A.decay[h] * softplus_f(ba[A.heads + h] + A.dt_bias[h])), sigmoid_f(ba[h]), kq_s[h / rep], 0.0f);
     }
 }
 
@@ -248,11 +248,6 @@ __device__ __forceinline__ float2 unpack2(f32x2 v) {
 __device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
     f32x2 r;
     asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
-    return r;
-}
-__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
-    f32x2 r;
-    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
     return r;
 }
 
@@ -331,14 +326,14 @@ delta_scan_kernel(DeltaScanArgs A) {
                 tk += __shfl_xor_sync(0xffffffffu, tk, o);
                 tq += __shfl_xor_sync(0xffffffffu, tq, o);
             }
-            const float u = sc.y * (v - sc.x * tk);
+            const float u = sc.y * (v - carry(sc.x, tk, 0.0f));
             const f32x2 g2 = pack2(sc.x, sc.x), u2 = pack2(u, u);
 #pragma unroll
             for (int m = 0; m < FOURS; ++m) {
-                S[m][0] = fma2(k[m][0], u2, mul2(g2, S[m][0]));
-                S[m][1] = fma2(k[m][1], u2, mul2(g2, S[m][1]));
+                S[m][0] = fma2(k[m][0], u2, fma2(g2, S[m][0], S[m][0]));
+                S[m][1] = fma2(k[m][1], u2, fma2(g2, S[m][1], S[m][1]));
             }
-            if (l == 0) o_s[t * kDtCols + col] = fmaf(sc.z, u, sc.x * tq);
+            if (l == 0) o_s[t * kDtCols + col] = fmaf(sc.z, u, carry(sc.x, tq, 0.0f));
         }
         __syncthreads();
         for (int i = tid; i < here * kDtCols; i += kThreads) {

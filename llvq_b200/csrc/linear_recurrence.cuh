@@ -56,11 +56,11 @@ struct LruArgs {
 
 __host__ __device__ inline int lru_tiles(int n) { return (n + kLruRows - 1) / kLruRows; }
 
-// One step of the recurrence of a channel; returns the new state.
-__device__ __forceinline__ float lru_step(float r, float i, float lam, float u, float s) {
-    const float log_a = -kLruDecay * r * lam;
-    return fmaf(expf(log_a), s, sqrtf(-expm1f(2.0f * log_a)) * i * u);
-}
+// Decays are kept as d = a - 1: a state is carried by s + (d s + x), which loses nothing where a rounds to a value near
+// one and a sequence is long. 1 - a^2 = -d (2 + d).
+__device__ __forceinline__ float lru_decay(float r, float lam) { return expm1f(-kLruDecay * r * lam); }
+__device__ __forceinline__ float lru_input(float d, float i, float u) { return sqrtf(-d * (2.0f + d)) * i * u; }
+__device__ __forceinline__ float carry(float d, float s, float x) { return s + fmaf(d, s, x); }
 
 // One CTA's part; `smem` holds ldw floats. Calls the dependency wait itself, behind its first loads of the matrices.
 template <typename T>
@@ -110,7 +110,7 @@ __device__ __forceinline__ void lru_token(const LruArgs& A, int cta, float* u_s)
     if (lane < 4 && c < A.n) {
         const float r = sigmoid_f(zr + A.b[(size_t)blk * 2 * A.n + c]), i = sigmoid_f(zi + A.b[(size_t)blk * 2 * A.n + A.n + c]);
         const float s = pos > 0 ? A.state[(size_t)(pos & 1) * width + ch] : 0.0f;
-        const float t = lru_step(r, i, A.lam[ch], u_s[c], s);
+        const float d = lru_decay(r, A.lam[ch]), t = carry(d, s, lru_input(d, i, u_s[c]));
         A.state[(size_t)((pos + 1) & 1) * width + ch] = t;
         A.conv[(size_t)(pos % A.taps) * width + ch] = A.x[ch];
         A.out[ch] = t * gelu_tanh_f(A.y[ch]) * A.out_scale;
@@ -222,20 +222,19 @@ lru_scan_kernel(LruScanArgs A) {
             a[k] = z[(size_t)t * 2 * A.n];
             x[k] = z[(size_t)t * 2 * A.n + A.n];
         }
-        float prod = 1.0f, sum = 0.0f;
+        float prod = 1.0f, sum = 0.0f;  // a[] holds decays less one from here on
 #pragma unroll
         for (int k = 0; k < kScanTok; ++k) {
             const int t = tw + k;
             if (t < A.n_tok) {
-                const float log_a = -kLruDecay * sigmoid_f(a[k] + br) * lam;
-                a[k] = expf(log_a);
-                x[k] = sqrtf(-expm1f(2.0f * log_a)) * sigmoid_f(x[k] + bi) * to_f32(U[(size_t)t * width]);
+                a[k] = lru_decay(sigmoid_f(a[k] + br), lam);
+                x[k] = lru_input(a[k], sigmoid_f(x[k] + bi), to_f32(U[(size_t)t * width]));
             } else {
-                a[k] = 1.0f;
+                a[k] = 0.0f;
                 x[k] = 0.0f;
             }
-            prod *= a[k];
-            sum = fmaf(a[k], sum, x[k]);
+            prod = carry(a[k], prod, 0.0f);
+            sum = carry(a[k], sum, x[k]);
         }
         prod_s[warp][lane] = prod;
         sum_s[warp][lane] = sum;
@@ -247,7 +246,7 @@ lru_scan_kernel(LruScanArgs A) {
 #pragma unroll
         for (int k = 0; k < kScanTok; ++k) {
             const int t = tw + k;
-            s = fmaf(a[k], s, x[k]);
+            s = carry(a[k], s, x[k]);
             if (t < A.n_tok && ch < width)
                 O[(size_t)t * A.ldo] = from_f32<T>(s * gelu_tanh_f(to_f32(Y[(size_t)t * A.ldy]) + yb) * A.out_scale);
         }
