@@ -143,3 +143,135 @@ def test_row_kernels(dtype, n):
     assert rel(act[:, :n], 0.5 * plain.silu(gu.double()[:, 0::2]) * gu.double()[:, 1::2]) < tol and bool((act[:, n:] == 7.0).all())
     ok(L.llvq_dn_gate_rows(dn(dtype), P(yg), n, P(gug), 2 * n, P(act), n + 8, rows, n, 1.5, stream()))
     assert rel(act[:, :n], 1.5 * y.double() * torch.sigmoid(gu.double()[:, :n])) < tol and bool((act[:, n:] == 7.0).all())
+
+
+# ---- windowed grouped-query attention ------------------------------------------------
+class Attention:
+    """One layer's operands: raw queries, keys, values and output gates of n positions, and the descriptor."""
+
+    def __init__(self, dtype, heads, kv_heads, dim, vdim, n, window, slots, seed=0, splits=3, scale=None, chunk=1):
+        from llvq_b200.cache import KvRing
+        _lib, _ = lib()
+        self.dtype, T = dtype, TYPES[dtype]
+        self.n, self.H, self.G, self.dim, self.vdim, self.window = n, heads, kv_heads, dim, vdim, window
+        self.scale = dim ** -0.5 if scale is None else scale
+        self.q, self.k = rnd(seed + 31, n, heads, dim), rnd(seed + 32, n, kv_heads, dim)
+        self.v, self.gate = rnd(seed + 33, n, kv_heads, vdim), rnd(seed + 34, n, heads, vdim)
+        self.qn, self.kn = 1 + 0.3 * rnd(seed + 35, dim), 1 + 0.3 * rnd(seed + 36, dim)
+        self.qn_g, self.kn_g = self.qn.cuda(), self.kn.cuda()
+        self.ring = KvRing(slots, slots, 1, kv_heads, dim, vdim, T, "cuda")
+        self.part = torch.zeros(heads * splits * (vdim + 2), device="cuda")
+        self.arrived = torch.zeros(kv_heads * -(-heads // kv_heads // 4), dtype=torch.int32, device="cuda")
+        self.d = _lib.DenseGqa(dtype=dn(dtype), heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, slots=slots, ld=self.ring.ld, kd=self.ring.kd, vd=self.ring.vd,
+                               window=window, splits=splits, scale=self.scale, eps=1e-4, out_scale=0.7, ring=P(self.ring.rows), q_norm=P(self.qn_g),
+                               k_norm=P(self.kn_g), part=P(self.part), arrived=P(self.arrived))
+
+    def want(self, gated=True):
+        q, k = plain.rms_norm(self.q.double(), self.qn.double(), 1e-4), plain.rms_norm(self.k.double(), self.kn.double(), 1e-4)
+        y = plain.grouped_attention(q, k, self.v.double(), self.scale, plain.window_mask(self.n, self.window))
+        return 0.7 * y * torch.sigmoid(self.gate.double()) if gated else y
+
+    def store(self, lo, hi):
+        """Rows of a portion: the cache rows and the normed queries."""
+        _, L = lib()
+        T = TYPES[self.dtype]
+        y = torch.cat([t[lo:hi].flatten(1) for t in (self.q, self.k, self.v)], dim=1).to(T).cuda()
+        qn = torch.zeros(hi - lo, self.H * self.dim, dtype=T, device="cuda")
+        at = [0, self.H * self.dim, (self.H + self.G) * self.dim]
+        ok(L.llvq_dn_gqa_rows(C.byref(self.d), *(y.data_ptr() + a * y.element_size() for a in at), y.shape[1], P(qn), lo, hi - lo, stream()))
+        return qn
+
+    def decode(self, p):
+        _, L = lib()
+        q, k, v, g = (t[p].cuda().contiguous() for t in (self.q, self.k, self.v, self.gate))
+        out, pos = torch.full((self.H, self.vdim), 7.0, device="cuda"), torch.tensor([p], device="cuda")
+        self.d.q, self.d.k, self.d.v, self.d.gate, self.d.out = P(q), P(k), P(v), P(g), P(out)
+        ok(L.llvq_dn_mixer_token(C.byref(self.d), None, P(pos), stream()))
+        return out.cpu()
+
+    def prefill(self, lo, hi, kernel=0):
+        """Queries lo .. hi - 1; earlier rows are in the ring. kernel 1: the generic one, 2: not the transposed one."""
+        _, L = lib()
+        qn = self.store(lo, hi)
+        key0 = max(0, lo - self.window + 1)
+        rows = self.ring.read(key0, hi)
+        vt = self.ring.values_transposed(rows) if kernel == 0 and L.llvq_dn_gqa_prefill_transposes(C.byref(self.d), hi - lo) else None
+        self.transposed = vt is not None
+        out = torch.full((hi - lo, self.H, self.vdim), 7.0, dtype=TYPES[self.dtype], device="cuda")
+        ok(L.llvq_dn_gqa_prefill(C.byref(self.d), P(qn), P(rows), P(vt), vt.shape[1] if vt is not None else 0, hi - lo, hi - key0, lo, key0, P(out),
+                                 1 if kernel == 1 else 0, stream()))
+        return out.float().cpu()
+
+
+HEADS = [(4, 4, 24, 40), (6, 2, 13, 9), (5, 1, 17, 33), (8, 2, 64, 48), (12, 1, 128, 128), (2, 1, 200, 264), (1, 1, 8, 8), (3, 3, 3, 2), (16, 8, 32, 184)]
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("shape", HEADS, ids=str)
+def test_prompt_attention(dtype, shape):
+    tol = 3e-6 if dtype == "float32" else 1.2e-2
+    for window in (1, 45, 64, 1000):
+        a = Attention(dtype, *shape, 300, window, 300, scale=1.5 * shape[2] ** -0.5)
+        want = a.want(gated=False)
+        for lo, hi in ((0, 300), (0, 1), (0, 2), (37, 140), (127, 129), (299, 300), (64, 256)):
+            if lo:
+                a.store(0, lo)
+            for kernel in (0, 1, 2) if dtype == "bfloat16" and lo == 37 else (0,):
+                got = a.prefill(lo, hi, kernel)
+                assert rel(got, want[lo:hi]) < tol and worst_row(got, want[lo:hi]) < 4 * tol, (window, lo, hi, kernel)
+    assert dtype == "float32" or bool((shape[2] | shape[3]) & 7) or shape[3] > 192 or L_transposes(a)
+    no_time_out()
+
+
+def L_transposes(a):
+    a.prefill(0, 300)
+    return a.transposed
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("shape", HEADS, ids=str)
+def test_token_attention_over_the_ring(dtype, shape):
+    tol = 3e-6 if dtype == "float32" else 6e-3
+    for window, slots, splits in ((1, 40, 1), (33, 40, 2), (64, 64, 3), (65, 70, 1), (150, 160, 3), (400, 400, 7)):
+        a = Attention(dtype, *shape, 260, window, slots, splits=splits, seed=window, scale=1.5 * shape[2] ** -0.5)
+        want, at = a.want(), 0
+        for p in (0, 1, 2, 31, 63, 64, 65, 100, 149, 150, 159, 160, 161, 200, 259):
+            while at < p:
+                hi = min(p, at + slots)
+                a.store(at, hi)
+                at = hi
+            held = a.ring.rows.clone()
+            first = a.decode(p)
+            assert rel(first, want[p]) < tol, (window, slots, p)
+            assert torch.equal(a.decode(p), first)           # again at the same position
+            once = a.ring.rows.clone()
+            a.ring.rows.copy_(held)
+            a.store(p, p + 1)                                  # the row a portion stores
+            assert rel(a.ring.rows, once) < 1e-6 if dtype == "float32" else rel(a.ring.rows, once) < 2e-3
+            at = p + 1
+        assert int(a.arrived.abs().sum()) == 0
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_a_query_that_looks_for_one_key_finds_it_just_inside_the_window_only(dtype):
+    """One key stands out for one query by tens of score units: just inside the window it takes all the weight, just
+    outside it leaves no trace, whatever tile, split or portion its place falls into."""
+    n, window = 330, 130
+    tol = 1e-5 if dtype == "float32" else 1.2e-2
+    for p in (129, 130, 131, 192, 255, 256, 329):
+        for gap in (window - 1, window, 0, 1, 63, 64):
+            if p - gap < 0:
+                continue
+            a = Attention(dtype, 4, 2, 40, 24, n, window, window + 70, seed=7, splits=4, scale=1.0)
+            j = p - gap
+            a.q[p], a.k[j] = a.k[j].repeat_interleave(2, 0), a.k[j]
+            a.qn, a.kn = torch.ones(40), torch.ones(40)
+            a.qn_g.fill_(1.0), a.kn_g.fill_(1.0)
+            want = a.want(gated=False)
+            alone = a.v[j].double().repeat_interleave(2, 0)
+            assert (rel(want[p], alone) < 1e-3) == (gap < window)
+            for lo in (max(0, p - 60), max(0, p - 5), p):
+                a.store(max(0, lo - window - 2), lo) if lo else None
+                assert rel(a.prefill(lo, min(n, p + 9))[p - lo], want[p]) < tol, (p, gap, lo)
+            a.store(max(0, p - window - 2), p)
+            assert rel(a.decode(p), a.want()[p]) < tol, (p, gap)
