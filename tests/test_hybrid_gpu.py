@@ -231,7 +231,7 @@ def L_transposes(a):
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("shape", HEADS, ids=str)
 def test_token_attention_over_the_ring(dtype, shape):
-    tol = 3e-6 if dtype == "float32" else 6e-3
+    tol = 3e-6 if dtype == "float32" else 1.5e-2  # cached keys and values are rounded once
     for window, slots, splits in ((1, 40, 1), (33, 40, 2), (64, 64, 3), (65, 70, 1), (150, 160, 3), (400, 400, 7)):
         a = Attention(dtype, *shape, 260, window, slots, splits=splits, seed=window, scale=1.5 * shape[2] ** -0.5)
         want, at = a.want(), 0
@@ -247,7 +247,7 @@ def test_token_attention_over_the_ring(dtype, shape):
             once = a.ring.rows.clone()
             a.ring.rows.copy_(held)
             a.store(p, p + 1)                                  # the row a portion stores
-            assert rel(a.ring.rows, once) < 1e-6 if dtype == "float32" else rel(a.ring.rows, once) < 2e-3
+            assert rel(a.ring.rows, once) < (1e-6 if dtype == "float32" else 2e-3)
             at = p + 1
         assert int(a.arrived.abs().sum()) == 0
 
@@ -275,3 +275,215 @@ def test_a_query_that_looks_for_one_key_finds_it_just_inside_the_window_only(dty
                 assert rel(a.prefill(lo, min(n, p + 9))[p - lo], want[p]) < tol, (p, gap, lo)
             a.store(max(0, p - window - 2), p)
             assert rel(a.decode(p), a.want()[p]) < tol, (p, gap)
+
+
+# ---- convolutions and the gated linear recurrence --------------------------------------
+PORTIONS = ([200], [2], [1, 2, 3, 70, 1, 5], [64, 65, 63, 8], [33, 1])
+
+
+def portions(n, sizes):
+    at, k = 0, 0
+    while at < n:
+        m = min(sizes[min(k, len(sizes) - 1)], n - at)
+        yield at, at + m
+        at, k = at + m, k + 1
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("channels,taps", [(1, 1), (37, 2), (300, 4), (64, 5), (20, 9)])
+def test_convolution_carries_its_inputs_over_portions(dtype, channels, taps):
+    _, L = lib()
+    T, n, ld = TYPES[dtype], 200, channels + 3
+    x, w, b, xb = rnd(1, n, channels), rnd(2, channels, taps), rnd(3, channels), rnd(4, channels)
+    want = plain.causal_conv(x.double() + xb.double(), w.double()) + b.double()
+    buf = torch.full((n, ld), 50.0, dtype=T, device="cuda")
+    buf[:, :channels] = x.cuda()
+    wg, bg, xbg = w.cuda(), b.cuda(), xb.cuda()
+    ring = torch.full((taps, channels), float("nan"), device="cuda")  # nothing ahead of the first token is read
+    for sizes in PORTIONS:
+        out = torch.zeros(n, channels, dtype=T, device="cuda")
+        for lo, hi in portions(n, sizes):
+            src = buf[lo:].data_ptr()
+            ok(L.llvq_dn_conv_rows(dn(dtype), src, ld, P(xbg), P(wg), P(bg), P(ring), out[lo:].data_ptr(), channels, taps, lo, hi - lo, stream()))
+            ok(L.llvq_dn_conv_keep(dn(dtype), src, ld, P(xbg), P(ring), channels, taps, lo, hi - lo, stream()))
+        assert rel(out, want) < (1e-6 if dtype == "float32" else 3e-3), sizes
+
+
+class Recurrence:
+    """One recurrent block's operands over n tokens, and the descriptor."""
+
+    def __init__(self, dtype, blocks, size, taps, n, seed=0, lam=-4.0):
+        from llvq_b200.cache import ConvInputs, RecurrentState, whole_vectors
+        _lib, _ = lib()
+        T = TYPES[dtype]
+        self.dtype, self.n, self.width, self.blocks, self.size = dtype, n, blocks * size, blocks, size
+        W = self.width
+        self.x, self.y = rnd(seed + 1, n, W), rnd(seed + 2, n, W)
+        self.conv_w, self.conv_b = rnd(seed + 3, W, taps), 0.3 * rnd(seed + 4, W)
+        self.ra, self.ri = ((rnd(seed + k, blocks, size, size) / size ** 0.5).bfloat16().float() for k in (5, 6))
+        self.rab, self.rib, self.lam = rnd(seed + 7, blocks, size), rnd(seed + 8, blocks, size), lam + 1.5 * rnd(seed + 9, W)
+        self.g = torch.zeros(blocks, 2 * size, whole_vectors(size, T), dtype=T, device="cuda")
+        self.g[:, :size, :size], self.g[:, size:, :size] = self.ra.cuda(), self.ri.cuda()
+        self.t = dict(conv_w=self.conv_w.cuda(), conv_b=self.conv_b.cuda(), b=torch.cat([self.rab, self.rib], 1).contiguous().cuda(),
+                      lam=plain.softplus(self.lam.double()).float().cuda(), w=self.g)
+        self.conv, self.state = ConvInputs(taps, W, "cuda"), RecurrentState(W, device="cuda")
+        self.conv.rows.fill_(float("nan")), self.state.halves.fill_(float("nan"))  # nothing is read ahead of the first token
+        self.d = _lib.DenseLru(dtype=dn(dtype), blocks=blocks, n=size, taps=taps, ldw=self.g.shape[2], out_scale=1.3, conv=P(self.conv.rows),
+                               state=P(self.state.halves), **{k: P(v) for k, v in self.t.items()})
+
+    def want(self, rounded=False):
+        u = plain.causal_conv(self.x.double(), self.conv_w.double()) + self.conv_b.double()
+        u = u.bfloat16().double() if rounded else u
+        r, i = (torch.sigmoid(plain.block_diagonal(u, m.double(), b.double())) for m, b in ((self.ra, self.rab), (self.ri, self.rib)))
+        return plain.gated_recurrence(u, r, i, self.lam.double()) * plain.gelu_tanh(self.y.double()) * 1.3
+
+    def token(self, p):
+        _, L = lib()
+        x, y, out, pos = self.x[p].cuda(), self.y[p].cuda(), torch.zeros(self.width, device="cuda"), torch.tensor([p], device="cuda")
+        self.d.x, self.d.y, self.d.out = P(x), P(y), P(out)
+        ok(L.llvq_dn_mixer_token(None, C.byref(self.d), P(pos), stream()))
+        return out.cpu()
+
+    def rows(self, lo, hi):
+        _, L = lib()
+        T, n, W = TYPES[self.dtype], hi - lo, self.width
+        x, y = self.x[lo:hi].to(T).cuda(), self.y[lo:hi].to(T).cuda()
+        u, out = torch.zeros(n, W, dtype=T, device="cuda"), torch.zeros(n, W, dtype=T, device="cuda")
+        zero = torch.zeros(W, device="cuda")
+        ok(L.llvq_dn_conv_rows(self.d.dtype, P(x), W, None, self.d.conv_w, self.d.conv_b, self.d.conv, P(u), W, self.d.taps, lo, n, stream()))
+        ok(L.llvq_dn_conv_keep(self.d.dtype, P(x), W, None, self.d.conv, W, self.d.taps, lo, n, stream()))
+        z = torch.einsum("tbi,boi->bto", u.view(n, self.blocks, self.size).double(), self.g[..., :self.size].double()).float().contiguous()
+        ok(L.llvq_dn_lru_rows(C.byref(self.d), P(u), P(z), P(y), W, P(zero), P(out), W, lo, n, stream()))
+        return out.float().cpu()
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("blocks,size,taps", [(1, 1, 1), (3, 14, 3), (5, 7, 2), (4, 80, 4), (2, 320, 4), (1, 700, 5)])
+def test_linear_recurrence_by_token_and_by_portion(dtype, blocks, size, taps):
+    n = 200
+    a = Recurrence(dtype, blocks, size, taps, n)
+    want, rounded = a.want(), a.want(rounded=dtype == "bfloat16")
+    got = torch.stack([a.token(p) for p in range(n)])
+    assert rel(got, want) < 3e-6 and worst_row(got, want) < 1e-4
+    for sizes in PORTIONS:
+        got = torch.cat([a.rows(lo, hi) for lo, hi in portions(n, sizes)])
+        assert rel(got, rounded) < (3e-6 if dtype == "float32" else 4e-3), sizes
+    # portions and tokens in turn, on the same state; a token run again at its position changes nothing
+    got, at = [], 0
+    for m in (70, 1, 1, 2, 1, 65, 60):
+        if m == 1:
+            first = a.token(at)
+            assert torch.equal(a.token(at), first)
+            got.append(first[None])
+        else:
+            got.append(a.rows(at, at + m))
+        at += m
+    assert at == n and rel(torch.cat(got), want) < (3e-6 if dtype == "float32" else 1e-2)
+
+
+def test_a_state_that_hardly_decays_is_carried_exactly():
+    """Thousands of tokens with decays of 1 - 1e-5 and below: an error in a decay would add up over all of them."""
+    n = 3000
+    a = Recurrence("float32", 2, 24, 2, n, seed=3, lam=-13.0)
+    want = a.want()
+    got = torch.cat([a.rows(lo, hi) for lo, hi in portions(n, [1500, 700, 2, 800])])
+    assert rel(got[-100:], want[-100:]) < 5e-6
+    for p in range(64):
+        a.token(p)
+    got = a.rows(64, n)
+    assert rel(got[-100:], want[-100:]) < 5e-6
+
+
+# ---- gated delta rule --------------------------------------------------------------------
+class Delta:
+    def __init__(self, dtype, heads, kv_heads, dim, vdim, taps, n, seed=0, decay=-2.0):
+        from llvq_b200.cache import ConvInputs, RecurrentState
+        _lib, _ = lib()
+        self.dtype, self.n, self.H, self.G, self.dim, self.vdim = dtype, n, heads, kv_heads, dim, vdim
+        self.ch = 2 * kv_heads * dim + heads * vdim
+        self.x, self.gate = rnd(seed + 1, n, self.ch), rnd(seed + 2, n, heads, vdim)
+        self.b, self.a = rnd(seed + 3, n, heads), rnd(seed + 4, n, heads)
+        self.conv_w, self.A_log, self.dt, self.norm = rnd(seed + 5, self.ch, taps), decay + rnd(seed + 6, heads), rnd(seed + 7, heads), 1 + 0.3 * rnd(seed + 8, vdim)
+        self.t = dict(conv_w=self.conv_w.cuda(), decay=self.A_log.double().exp().float().cuda(), dt_bias=self.dt.cuda(), norm=self.norm.cuda())
+        vp = -(-vdim // 4) * 4
+        self.conv, self.state = ConvInputs(taps, self.ch, "cuda"), RecurrentState(heads, dim, vp, device="cuda")
+        self.conv.rows.fill_(float("nan"))
+        self.state.halves[..., :vdim] = float("nan")  # nothing is read ahead of the first token
+        self.o, self.arrived = torch.zeros(heads * vp, device="cuda"), torch.zeros(heads, dtype=torch.int32, device="cuda")
+        self.d = _lib.DenseDelta(dtype=dn(dtype), heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, vp=vp, taps=taps, eps=1e-4, conv=P(self.conv.rows),
+                                 state=P(self.state.halves), o=P(self.o), arrived=P(self.arrived), **{k: P(v) for k, v in self.t.items()})
+
+    def want(self):
+        n, H, G = self.n, self.H, self.G
+        c = plain.silu(plain.causal_conv(self.x.double(), self.conv_w.double()))
+        q, k, v = c.split([G * self.dim, G * self.dim, H * self.vdim], dim=1)
+        q, k = plain.unit_vector(q.reshape(n, G, -1)) * self.dim ** -0.5, plain.unit_vector(k.reshape(n, G, -1))
+        q, k = q.repeat_interleave(H // G, 1), k.repeat_interleave(H // G, 1)
+        o, _ = plain.delta_rule(q, k, v.reshape(n, H, -1), torch.sigmoid(self.b.double()), plain.delta_decay(self.a.double(), self.A_log.double(), self.dt.double()))
+        return plain.gated_head_norm(o, self.norm.double(), self.gate.double(), 1e-4)
+
+    def token(self, p):
+        _, L = lib()
+        t = [v[p].cuda().contiguous() for v in (self.x, self.gate, self.b, self.a)]
+        out, pos = torch.zeros(self.H, self.vdim, device="cuda"), torch.tensor([p], device="cuda")
+        self.d.x, self.d.gate, self.d.beta, self.d.alpha, self.d.out = *(P(v) for v in t), P(out)
+        ok(L.llvq_dn_delta_token(C.byref(self.d), P(pos), stream()))
+        return out.cpu()
+
+    def rows(self, lo, hi):
+        _, L = lib()
+        T, n, hv = TYPES[self.dtype], hi - lo, self.H * self.vdim
+        x, gate = self.x[lo:hi].to(T).cuda(), self.gate[lo:hi].flatten(1).to(T).cuda()
+        ba = torch.cat([self.b[lo:hi], self.a[lo:hi]], 1).contiguous().cuda()
+        floats = C.c_size_t()
+        ok(L.llvq_dn_delta_scratch(C.byref(self.d), n, C.byref(floats)))
+        scratch, out = torch.zeros(floats.value, device="cuda"), torch.full((n, hv + 5), 7.0, dtype=T, device="cuda")
+        ok(L.llvq_dn_delta_rows(C.byref(self.d), P(x), self.ch, P(ba), P(gate), hv, P(scratch), P(out), hv + 5, lo, n, stream()))
+        assert bool((out[:, hv:] == 7.0).all())
+        return out[:, :hv].float().cpu().view(n, self.H, self.vdim)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("shape", [(1, 1, 1, 1, 1), (3, 1, 11, 7, 2), (4, 4, 6, 18, 5), (4, 2, 64, 96, 4), (2, 1, 128, 128, 4), (1, 1, 256, 33, 3), (2, 1, 300, 36, 4),
+                                   (1, 1, 520, 20, 2), (1, 1, 1000, 9, 2)], ids=str)
+def test_delta_rule_by_token_and_by_portion(dtype, shape):
+    n = 200
+    a = Delta(dtype, *shape, n)
+    want = a.want()
+    got = torch.stack([a.token(p) for p in range(n)])
+    assert rel(got, want) < 1e-5 and worst_row(got, want) < 1e-4
+    assert int(a.arrived.abs().sum()) == 0
+    for sizes in PORTIONS:
+        got = torch.cat([a.rows(lo, hi) for lo, hi in portions(n, sizes)])
+        assert rel(got, want) < (1e-5 if dtype == "float32" else 4e-3), sizes
+    got, at = [], 0
+    for m in (70, 1, 1, 2, 1, 65, 60):
+        if m == 1:
+            first = a.token(at)
+            assert torch.equal(a.token(at), first)
+            got.append(first[None])
+        else:
+            got.append(a.rows(at, at + m))
+        at += m
+    assert at == n and rel(torch.cat(got), want) < (1e-5 if dtype == "float32" else 4e-3)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_delta_state_remembers_a_far_key(dtype):
+    """Hardly any decay, and a query that equals one far key: what was written there is read back hundreds of tokens on."""
+    n, far = 700, 40
+    a = Delta(dtype, 2, 2, 64, 64, 1, n, seed=5, decay=-9.0)
+    qk = 2 * 64
+    a.conv_w[:], a.t["conv_w"][:] = 1.0, 1.0
+    a.b[:] = -4.0                                    # small writes everywhere
+    a.b[far] = 8.0
+    a.x[-1, :qk] = a.x[far, qk:2 * qk]               # the last query is the far key
+    want = a.want()
+    b = copy.copy(a)
+    b.x = a.x.clone()
+    b.x[far, 2 * qk:] = -a.x[far, 2 * qk:]
+    assert ((b.want()[-1] - want[-1]).norm() / want[-1].norm()) > 0.3  # the plain statement depends on it
+    tol = 1e-4 if dtype == "float32" else 6e-3
+    assert rel(a.rows(0, n)[-1], want[-1]) < tol
+    got = torch.cat([a.rows(lo, hi) for lo, hi in portions(n - 1, [333, 64, 2, 300])])
+    assert rel(a.token(n - 1), want[-1]) < tol and rel(got[far:], want[far:-1]) < 6e-3
