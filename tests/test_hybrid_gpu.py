@@ -242,7 +242,7 @@ def test_token_attention_over_the_ring(dtype, shape):
                 at = hi
             held = a.ring.rows.clone()
             first = a.decode(p)
-            assert rel(first, want[p]) < tol, (window, slots, p)
+            assert (first - want[p]).norm() < tol * want.norm() / 260 ** 0.5, (window, slots, p)
             assert torch.equal(a.decode(p), first)           # again at the same position
             once = a.ring.rows.clone()
             a.ring.rows.copy_(held)
@@ -257,7 +257,7 @@ def test_a_query_that_looks_for_one_key_finds_it_just_inside_the_window_only(dty
     """One key stands out for one query by tens of score units: just inside the window it takes all the weight, just
     outside it leaves no trace, whatever tile, split or portion its place falls into."""
     n, window = 330, 130
-    tol = 1e-5 if dtype == "float32" else 1.2e-2
+    tol = 1e-5 if dtype == "float32" else 2.5e-2  # scores of up to 40 from keys and queries of 8 bits
     for p in (129, 130, 131, 192, 255, 256, 329):
         for gap in (window - 1, window, 0, 1, 63, 64):
             if p - gap < 0:
@@ -487,3 +487,188 @@ def test_delta_state_remembers_a_far_key(dtype):
     assert rel(a.rows(0, n)[-1], want[-1]) < tol
     got = torch.cat([a.rows(lo, hi) for lo, hi in portions(n - 1, [333, 64, 2, 300])])
     assert rel(a.token(n - 1), want[-1]) < tol and rel(got[far:], want[far:-1]) < 6e-3
+
+
+# ---- the model ---------------------------------------------------------------------
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", list(cases.ALL))
+def test_prompts_portions_and_tokens_give_the_plain_logits(dtype, name):
+    cfg = cases.ALL[name]
+    m, w = build(cfg, 5, dtype, 400)
+    toks = tokens_of(cfg, 210, 6)
+    layers, want_layers = [], []
+    want = plain.forward(cfg, w, toks, layers_out=want_layers)
+    m.hidden(torch.tensor(toks, device="cuda"), m.positions[:210], end=210, layers_out=layers)
+    assert len(layers) == len(want_layers) == len(m.cfg.runs)
+    for i, (a, b) in enumerate(zip(layers, want_layers)):
+        assert rel(a, b) < (1e-5 if dtype == "float32" else 4e-2), i
+    runs = {"whole": [210], "tokens": [1], "twos": [2], "mixed": [64, 1, 3, 17, 2, 1, 1, 70, 5, 2], "then tokens": [150, 1]}
+    for k, sizes in runs.items():
+        y = run(m, toks, sizes)
+        assert rel(y, want) < TOL[dtype], k
+        worst = (y.double() - want).norm(dim=1) / want.norm(dim=1)
+        assert worst.max() < 4 * TOL[dtype], (k, int(worst.argmax()))
+    assert rel(run(m, toks[:40], [1], use_graph=False), want[:40]) < TOL[dtype]
+    no_time_out()
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_rings_that_wrap_and_states_used_again(dtype):
+    """Portions of at most 16 tokens: the rings are a window and 15 positions long and wrap many times; further sequences
+    start over in the slots and states the ones before have left. Every pass of a looped layer keeps its own."""
+    m, w = build(cases.UNEVEN, 8, dtype, 900, chunk=16)
+    assert [s["ring"].slots for s in m.states if "ring" in s] == [34, 22, 34, 22, 16]
+    stores = [s["state"].halves.data_ptr() for s in m.states] + [s["conv"].rows.data_ptr() for s in m.states]
+    assert len(set(stores)) == 2 * len(cases_runs(m)) and m.cache_bytes() > 0
+    for seed, n, sizes in ((1, 300, [7, 16, 2, 1, 1, 40, 3]), (2, 95, [1]), (3, 1, [1]), (4, 140, [140]), (5, 23, [20, 2])):
+        toks = tokens_of(cases.UNEVEN, n, seed)
+        want = plain.forward(cases.UNEVEN, w, toks)
+        y = run(m, toks, sizes)
+        assert rel(y, want) < TOL[dtype], (seed, n)
+        assert ((y.double() - want).norm(dim=1) / want.norm(dim=1)).max() < 4 * TOL[dtype]
+
+
+def cases_runs(m):
+    return m.cfg.runs
+
+
+def test_logits_do_not_depend_on_what_ran_before():
+    m, w = build(cases.EVEN, 9, "bfloat16", 300, chunk=50)
+    toks = tokens_of(cases.EVEN, 120, 1)
+    first = run(m, toks, [50, 30, 1])
+    run(m, tokens_of(cases.EVEN, 299, 2), [13])
+    m.feed(tokens_of(cases.EVEN, 77, 3), [0])  # left without a release: generate takes the states over
+    m.generate(tokens_of(cases.EVEN, 5, 4), 9, use_graph=True)
+    assert torch.equal(run(m, toks, [50, 30, 1]), first)
+
+
+@pytest.mark.parametrize("odd", [0, 1])
+def test_the_first_replayed_step_does_not_move_the_state_twice(odd):
+    """Capturing the step's graph runs it once ahead of the first replay."""
+    m, w = build(cases.UNEVEN, 19, "float32", 100)
+    toks = tokens_of(cases.UNEVEN, 30 + odd, 2)
+    want = plain.forward(cases.UNEVEN, w, toks)
+    got = torch.cat([m.feed(toks[:20 + odd], [19 + odd])] + [m.feed([t], [0]) for t in toks[20 + odd:]])
+    assert rel(got, want[19 + odd:]) < TOL["float32"]
+
+
+@pytest.mark.parametrize("name,layer", [("uneven", 1), ("uneven", 2), ("even", 0), ("even", 3)])
+def test_every_layers_window_ends_where_it_should(name, layer):
+    """One attention layer alone, its neighbours blind: a token reaches exactly window - 1 positions ahead."""
+    cfg = copy.deepcopy(cases.ALL[name])
+    cfg["layers"], cfg["loop"] = [cfg["layers"][layer]], None
+    m_, mlp = cfg["layers"][0]["mixer"], cfg["layers"][0]["mlp"]
+    m_["right_scale"] = 0.0
+    size = m_["left"]["mask"]["size"]
+    m, w = build(cfg, 10, "float32", 300, chunk=96)
+    at = 21
+    toks = tokens_of(cfg, at + size + 4, 5)
+    other = list(toks)
+    other[at] = (other[at] + 1) % cfg["vocab"]
+    inside, outside = at + size - 1, at + size
+    want = (plain.forward(cfg, w, toks) - plain.forward(cfg, w, other)).norm(dim=1)
+    assert want[inside] > 1e-6 and want[outside] < 1e-12  # the plain statement has the edge there
+    for sizes in ([len(toks)], [at + 1, 2], [30, 1], [1]):
+        d = (run(m, toks, sizes) - run(m, other, sizes)).norm(dim=1)
+        assert abs(float(d[inside]) - float(want[inside])) < 0.2 * float(want[inside]) + 1e-4, sizes
+        assert float(d[outside]) == 0.0 and float(d[at - 1]) == 0.0, sizes
+
+
+def test_long_decoding_stays_on_the_plain_logits():
+    for dtype in DTYPES:
+        m, w = build(cases.UNEVEN, 12, dtype, 700, chunk=8)
+        toks = tokens_of(cases.UNEVEN, 600, 7)
+        want = plain.forward(cases.UNEVEN, w, toks)
+        y = run(m, toks, [5, 1])
+        assert rel(y[-100:], want[-100:]) < TOL[dtype]
+        assert rel(run(m, toks[:64], [1], use_graph=False), want[:64]) < TOL[dtype]
+
+
+def test_output_projections_apart_where_one_would_be_too_long():
+    from llvq_b200.hybrid import HybridLM
+    toks = tokens_of(cases.EVEN, 90, 3)
+    w = cases.random_model(cases.EVEN, 21)
+    want = plain.forward(cases.EVEN, w, toks)
+    held = HybridLM.JOINED_COLUMNS
+    try:
+        HybridLM.JOINED_COLUMNS = {2: 700, 4: 700}
+        for dtype in DTYPES:
+            m, _ = build(cases.EVEN, 21, dtype, 128, weights=w)
+            assert m.layers[0]["down"] is not None
+            for sizes in ([90], [1], [40, 1, 1, 2]):
+                assert rel(run(m, toks, sizes), want) < TOL[dtype], sizes
+    finally:
+        HybridLM.JOINED_COLUMNS = held
+
+
+@pytest.mark.parametrize("name", list(cases.ALL))
+def test_greedy_generation_through_the_entry_point(tmp_path, name):
+    """The command line and load_model on a folder: the tokens are the plain statement's greedy ones (f32), the graph
+    replays the eager tokens, and the bf16 model agrees with its own fed logits."""
+    from llvq_b200.registry import load_model
+    cfg = cases.ALL[name]
+    w = cases.random_model(cfg, 14)
+    path = cases.write_folder(tmp_path / name, cfg, w)
+    prompt = tokens_of(cfg, 20, 8)
+    seq = list(prompt)
+    for _ in range(24):
+        seq.append(int(plain.forward(cfg, w, seq)[-1].argmax()))
+    want = seq[20:]
+    assert len(set(want)) > 4
+    m = load_model(path, 64, "float32", prefill_chunk=7)
+    assert m.generate(prompt, 24) == want and m.generate(prompt, 24, use_graph=True) == want
+    assert m.generate(prompt, 1) == want[:1] and m.generate(prompt, 0) == []
+    with pytest.raises(ValueError):
+        m.generate(prompt, 60)
+    b = load_model(path, 64)
+    assert b.dtype == torch.bfloat16
+    out = b.generate(prompt, 24, use_graph=True)
+    assert b.generate(prompt, 24) == out
+    fed = [b.feed(prompt, [19])] + [b.feed([t], [0]) for t in out[:-1]]
+    assert [int(y[0].argmax()) for y in fed] == out
+    if name == "uneven":
+        res = subprocess.run([sys.executable, "-m", "llvq_b200", "generate", "--model", path, "--tokens", ",".join(map(str, prompt)), "--max-new", "24",
+                              "--dtype", "float32"], cwd=ROOT, capture_output=True, text=True, timeout=300)
+        assert res.returncode == 0 and json.loads(res.stdout)["tokens"] == want, res.stderr
+        steps = [{"step": 0, "entries": [{"id": "a", "tokens": prompt[:9], "want": [8, 1]}], "end": []},
+                 {"step": 1, "entries": [{"id": "a", "tokens": prompt[9:10], "want": [0]}], "end": ["a"]},
+                 {"step": 2, "entries": [{"id": "b", "tokens": prompt[:3], "want": [2]}], "end": ["b"]}]
+        res = subprocess.run([os.path.join(ROOT, "bin", "trace_run"), "--model", path, "--dtype", "float32", "--out", str(tmp_path), "--max-tokens", "32"],
+                             input="".join(json.dumps(s) + "\n" for s in steps), capture_output=True, text=True, timeout=300)
+        assert res.returncode == 0 and res.stdout.split() == "done 0 done 1 done 2".split(), res.stderr
+        full = plain.forward(cfg, w, prompt)
+        for step, rows in ((0, [8, 1]), (1, [9]), (2, [2])):
+            assert rel(torch.from_numpy(np.fromfile(tmp_path / f"{step}.f32", "<f4").reshape(len(rows), -1)), full[rows]) < TOL["float32"]
+
+
+def test_phases_leave_the_tokens_alone():
+    _lib, L = lib()
+    m, _ = build(cases.EVEN, 15, "bfloat16", 96)
+    prompt = tokens_of(cases.EVEN, 12, 3)
+    want = m.generate(prompt, 30, use_graph=True)
+    ph = m.phase_split(reps=2)
+    assert set(ph) == set(m.PHASES) | {"sum"} and all(v >= 0 for v in ph.values())
+    assert m.generate(prompt, 30, use_graph=True) == want
+    try:
+        L.llvq_dn_set_overlap(0)
+        other, _ = build(cases.EVEN, 15, "bfloat16", 96)
+        assert other.generate(prompt, 30, use_graph=True) == want
+    finally:
+        L.llvq_dn_set_overlap(1)
+
+
+def test_weights_that_do_not_fit_the_configuration_are_refused():
+    w = cases.random_model(cases.UNEVEN, 1)
+    for name, shape in (("l0.mix.q", (12, 90)), ("l1.mix.left.q.norm", (12,)), ("embed", (203, 91)), ("l1.mix.right.ra", (3, 14, 13)), ("l0.mlp.e4.up", (20, 90)),
+                        ("l3.mix.v.conv", (72, 4)), ("l2.mix.right.o", (90, 34))):
+        bad = dict(w)
+        bad[name] = torch.zeros(*shape).bfloat16()
+        with pytest.raises(ValueError, match="config.json says"):
+            build(cases.UNEVEN, 1, "bfloat16", 16, weights=bad)
+    bad = dict(w)
+    bad["l0.mlp.table"] = w["l0.mlp.table"] + 3
+    with pytest.raises(ValueError, match="outside"):
+        build(cases.UNEVEN, 1, "bfloat16", 16, weights=bad)
+    del bad["l4.mix.right.lam"]
+    with pytest.raises(KeyError):
+        build(cases.UNEVEN, 1, "bfloat16", 16, weights=bad)
