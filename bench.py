@@ -21,7 +21,8 @@ GEMM), `decode` = configuration 2 (greedy decode, with the token step split by p
 decode; tp1 figures at N = 1). `--impl reference` times the CPU path alone, as the
 reference arm, and adds as a side measurement the reference's own serving kernel on its
 transcoded layout where that kernel was built from the reference's sources. `--latent` leaves this workload aside
-and times latent-attention models (dense bf16 weights) beside the Qwen3 model of equal size.
+and times latent-attention models (dense bf16 weights) beside the Qwen3 model of equal size, `--hybrid` hybrid models beside
+those.
 """
 from __future__ import annotations
 
@@ -769,27 +770,19 @@ def latent_model(torch, cfg, capacity, seed=1):
     return latent.LatentLM(cfg, tensor, "bfloat16", capacity, torch.device("cuda"))
 
 
-def run_latent(args):
-    """--latent: prefill and greedy decode of latent-attention models (bf16, random weights) at the layer sizes of
-    qwen3-4b / 8b / 14b, beside the archive-code Qwen3 model of the same size on the same tokens, with the time of each
-    kernel against its roofline: bytes over the measured copy bandwidth, for the prompt attention and the matrix
-    products FLOPs over the measured bf16 throughput. Token-step phases are replayed apart (all layers; the weights of a
-    phase exceed L2 where `l2` says so); prompt kernels rotate over operand sets larger than L2. Device-timed."""
-    import ctypes as C
-    import gc
-    import torch
-    from llvq_b200 import FusedRuntime, _lib
-    from llvq_b200.model import Qwen3Config, synthetic_model
-    peak = measured_peaks()[0]
-    tflops = 1590.0
-    if os.path.exists(os.path.join(ROOT, "MEASURED_PEAKS.json")):
-        tflops = float(json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))["bf16_tflops"])
-    n_layers, window, prompt_len, new_tokens = args.latent_layers, args.window, 2048, 96
-    torch.cuda.set_device(0)
-    sampler = ClockSampler(0)
-    sampler.start()
+class LayerBench:
+    """Timings of a model at the layer sizes of a named one: prompt and token loop, token-step phases, kernels of a prompt
+    portion. Device-timed; see run_latent for what the figures are taken against."""
 
-    def event_ms(fn, reps):
+    def __init__(self, args):
+        import torch
+        self.torch, self.steps, self.n_layers, self.window, self.prompt_len, self.new_tokens = torch, args.steps, args.latent_layers, args.window, 2048, 96
+        self.peak, self.tflops = measured_peaks()[0], 1590.0
+        if os.path.exists(os.path.join(ROOT, "MEASURED_PEAKS.json")):
+            self.tflops = float(json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))["bf16_tflops"])
+
+    def event_ms(self, fn, reps):
+        torch = self.torch
         for _ in range(3):
             fn(0)
         e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
@@ -801,36 +794,41 @@ def run_latent(args):
         torch.cuda.synchronize()
         return e0.elapsed_time(e1) / reps
 
-    def loop_times(model):
+    def loop_times(self, model):
+        prompt_len, new_tokens, event_ms = self.prompt_len, self.new_tokens, self.event_ms
         prompt = np.random.default_rng(5).integers(0, model.cfg.vocab, prompt_len).tolist()
         model.generate(prompt, 4, use_graph=True)
-        pre = event_ms(lambda k: model.prefill(prompt), max(args.steps // 2, 3))
+        pre = event_ms(lambda k: model.prefill(prompt), max(self.steps // 2, 3))
         model.start_decode(model.pick_last(model.prefill(prompt)), prompt_len)
         dec = event_ms(lambda k: model._graph_step(), new_tokens - 8)
         return {"prefill_ms": round(pre, 3), "prefill_tok_per_s": round(prompt_len / pre * 1e3), "decode_ms_per_token": round(dec, 4),
                 "decode_tok_per_s": round(1e3 / dec, 1)}
 
-    def phases(model, sizes):
-        model._pos.fill_(window - 1)  # `window` positions are read by both models' attention
+    def phases(self, model, sizes, runs=None):
+        """`sizes`: bytes a phase reads (all layers); `runs`: layers a phase runs in, where not all."""
+        model._pos.fill_(self.window - 1)  # `window` positions are read by both models' attention
         out = {}
         for name, ms in model.phase_split(reps=20).items():
             b = sizes.get(name)
-            out[name] = {"us_per_layer": round(ms * 1e3 / n_layers, 2)} if name != "head" else {"us": round(ms * 1e3, 2)}
+            out[name] = {"us_per_layer": round(ms * 1e3 / (runs or {}).get(name, self.n_layers), 2)} if name != "head" else {"us": round(ms * 1e3, 2)}
             if b:
-                out[name].update(GBps=round(b / ms / 1e6, 1), frac=round(b / ms / 1e6 / peak, 4), l2="weights exceed L2" if b > 126e6 else "fits L2")
+                out[name].update(GBps=round(b / ms / 1e6, 1), frac=round(b / ms / 1e6 / self.peak, 4), l2="weights exceed L2" if b > 126e6 else "fits L2")
         return out
 
-    results = []
-    for shape in args.latent_shapes.split(","):
+    def latent(self, shape: str) -> dict:
+        import ctypes as C
+        import gc
+        from llvq_b200 import _lib
+        torch, n_layers, window, prompt_len, peak, tflops = self.torch, self.n_layers, self.window, self.prompt_len, self.peak, self.tflops
         cfg = latent_config(shape, n_layers, window)
         m = latent_model(torch, cfg, prompt_len + 128)
         lib, a, L, lat = m.lib, cfg.layers[0].attn, m.layers[0], m._lat[0]
         launches = lib.llvq_dn_launch_count()
         r = {"shape": shape, "layers": n_layers, "width": cfg.width, "ff": cfg.layers[0].mlp.ff, "heads": a.heads, "window": window,
-             "head_dims": [a.dim, a.rot_dim, a.vdim], "ranks": [a.q_rank, a.kv_rank], "latent": loop_times(m)}
+             "head_dims": [a.dim, a.rot_dim, a.vdim], "ranks": [a.q_rank, a.kv_rank], "latent": self.loop_times(m)}
         wb = lambda *names: sum(x[n].w.numel() * 2 for x in m.layers for n in names)
         up = [(x["ukv"].ld * 2 * c.attn.heads * c.attn.dim, x["ukv"].ld * 2 * c.attn.heads * c.attn.vdim) for x, c in zip(m.layers, cfg.layers)]
-        r["latent"]["token_step"] = phases(m, {"projections": wb("dq_dkv", "uq", "o", "gate_up", "down"), "latent_query": sum(u for u, _ in up),
+        r["latent"]["token_step"] = self.phases(m, {"projections": wb("dq_dkv", "uq", "o", "gate_up", "down"), "latent_query": sum(u for u, _ in up),
                                                "attention": sum(min(window, x.slots) * x.ld * 2 for x in m.rings), "latent_value": sum(v for _, v in up),
                                                "head": m.embed.w.numel() * 2})
         # kernels of one prompt portion: 2048 queries behind a full window
@@ -860,19 +858,19 @@ def run_latent(args):
             s = sets[k % 3]
             check(lib.llvq_dn_latent_rows(C.byref(lat), s["yd"].data_ptr(), s["yd"].shape[1], a.q_rank, L["dq_norm"].data_ptr(), s["cq"].data_ptr(), 0, n, 1, st()))
         pk = {}
-        ms = event_ms(attend, 12)
+        ms = self.event_ms(attend, 12)
         fl = 2.0 * pairs * a.heads * (a.dim + a.rot_dim + a.vdim)
         pk["attention"] = {"us": round(ms * 1e3, 1), "TFLOPs": round(fl / ms / 1e9, 1), "frac": round(fl / ms / 1e9 / tflops, 4)}
         for name, fn, b in (("add_norm", norm, n * cfg.width * 12), ("gated_unit", glu, n * cfg.layers[0].mlp.ff * 6),
                             ("latent_rows", rows, 2 * n * (2 * a.q_rank + 2 * a.kv_rank + 2 * a.rot_dim))):
-            ms = event_ms(fn, 24)
+            ms = self.event_ms(fn, 24)
             pk[name] = {"us": round(ms * 1e3, 1), "GBps": round(b / ms / 1e6, 1), "frac": round(b / ms / 1e6 / peak, 4)}
 
         def products(k):
             s = sets[k % 3]
             for x, w in ((s["xt"], L["dq_dkv"]), (s["cq"], L["uq"]), (s["out"], L["o"]), (s["xt"], L["gate_up"]), (s["act"], L["down"])):
                 m._mm(x, w.rows(0))
-        ms = event_ms(products, 12)
+        ms = self.event_ms(products, 12)
         fl = 2.0 * n * sum(L[k].n * L[k].k for k in ("dq_dkv", "uq", "o", "gate_up", "down"))
         pk["library products"] = {"us": round(ms * 1e3, 1), "TFLOPs": round(fl / ms / 1e9, 1), "frac": round(fl / ms / 1e9 / tflops, 4)}
         r["latent"]["prompt_kernels"] = pk
@@ -882,27 +880,50 @@ def run_latent(args):
         del m, sets, L, lat
         gc.collect()
         torch.cuda.empty_cache()
+        return r
+
+
+def run_latent(args):
+    """--latent: prefill and greedy decode of latent-attention models (bf16, random weights) at the layer sizes of
+    qwen3-4b / 8b / 14b, beside the archive-code Qwen3 model of the same size on the same tokens, with the time of each
+    kernel against its roofline: bytes over the measured copy bandwidth, for the prompt attention and the matrix
+    products FLOPs over the measured bf16 throughput. Token-step phases are replayed apart (all layers; the weights of a
+    phase exceed L2 where `l2` says so); prompt kernels rotate over operand sets larger than L2. Device-timed."""
+    import gc
+    import torch
+    from llvq_b200 import FusedRuntime
+    from llvq_b200.model import Qwen3Config, synthetic_model
+    B = LayerBench(args)
+    n_layers, window, prompt_len, new_tokens, peak, tflops = B.n_layers, B.window, B.prompt_len, B.new_tokens, B.peak, B.tflops
+    torch.cuda.set_device(0)
+    sampler = ClockSampler(0)
+    sampler.start()
+
+    results, T = [], prompt_len + window - 1
+    n = prompt_len
+    for shape in args.latent_shapes.split(","):
+        r = B.latent(shape)
 
         # the archive-code model of the same size
         rt = FusedRuntime(0)
         qc = Qwen3Config.named(shape)
         q, _ = synthetic_model(rt, qc, config_id=2, capacity=prompt_len + 128, layers=n_layers, keep_host=False, device_codes=True)
-        r["qwen3"] = loop_times(q)
+        r["qwen3"] = B.loop_times(q)
         pb = sum(blk[k].algorithmic_bytes(2, 2) for blk in q.blocks for k in ("qkv", "o", "gate_up", "down"))
-        r["qwen3"]["token_step"] = phases(q, {"projections": pb, "attention": sum(c.bytes_per_position() * window for c in q.caches),
+        r["qwen3"]["token_step"] = B.phases(q, {"projections": pb, "attention": sum(c.bytes_per_position() * window for c in q.caches),
                                               "head": qc.vocab * qc.hidden * 2})
         # its prompt attention over as many keys (full causal, through the library), and its norm and gated unit
         half = lambda *s: torch.randn(*s, device="cuda").half()
         q.positions = torch.arange(T, device="cuda")
         qs = [(half(n, qc.n_heads, qc.head_dim), half(T, qc.n_kv, qc.head_dim), half(T, qc.n_kv, qc.head_dim)) for _ in range(3)]
         xs = [(half(n, qc.hidden), half(n, qc.hidden), half(n, 2 * qc.inter)) for _ in range(3)]
-        ms = event_ms(lambda k: q._attend(*qs[k % 3], q.positions[T - n:], T), 6)
+        ms = B.event_ms(lambda k: q._attend(*qs[k % 3], q.positions[T - n:], T), 6)
         fl = 4.0 * (n * (T - n) + n * (n + 1) / 2) * qc.n_heads * qc.head_dim
         pk = {"attention": {"us": round(ms * 1e3, 1), "TFLOPs": round(fl / ms / 1e9, 1), "frac": round(fl / ms / 1e9 / tflops, 4)}}
         from llvq_b200.model import _silu
-        ms = event_ms(lambda k: q._rms(xs[k % 3][0] + xs[k % 3][1], q.final_norm), 24)
+        ms = B.event_ms(lambda k: q._rms(xs[k % 3][0] + xs[k % 3][1], q.final_norm), 24)
         pk["add_norm"] = {"us": round(ms * 1e3, 1), "frac": round(n * qc.hidden * 8 / ms / 1e6 / peak, 4)}
-        ms = event_ms(lambda k: (_silu(xs[k % 3][2][:, :qc.inter].float()) * xs[k % 3][2][:, qc.inter:].float()).half(), 24)
+        ms = B.event_ms(lambda k: (_silu(xs[k % 3][2][:, :qc.inter].float()) * xs[k % 3][2][:, qc.inter:].float()).half(), 24)
         pk["gated_unit"] = {"us": round(ms * 1e3, 1), "frac": round(n * qc.inter * 6 / ms / 1e6 / peak, 4)}
         r["qwen3"]["prompt_kernels"] = pk
         results.append(r)
@@ -915,6 +936,180 @@ def run_latent(args):
           "warmup": 3, "ms_per_step": results[0]["latent"]["decode_ms_per_token"], "higher_is_better": True, "vs_baseline": None, "dtype": "bf16",
           "data": "synthetic (random weights and tokens)", "clocks": clocks, "peaks": {"hbm_gbs": peak, "bf16_tflops": tflops},
           "config": {"prompt_tokens": prompt_len, "window": window, "layers": n_layers}, "results": results})
+
+
+def hybrid_config(shape: str, layers: int, window: int, routed: bool):
+    """A hybrid model of the named model's width, heads, feed-forward and vocabulary: attention beside recurrence and the
+    delta rule by turns. `routed`: 32 experts of a quarter of the feed-forward, four of them per token."""
+    from llvq_b200 import hybrid, synth
+    h, inter, qh, kvh, hd, _, vocab = synth.MODEL_SHAPES[shape]
+    mlp = hybrid.MlpConfig(inter // 4, 32, 4) if routed else hybrid.MlpConfig(inter)
+
+    def layer(i):
+        if i % 2:
+            return hybrid.HybridLayerConfig(hybrid.DeltaConfig(qh, qh // 2, hd, hd, 4), mlp)
+        return hybrid.HybridLayerConfig(hybrid.ParallelConfig(hybrid.AttentionConfig(qh, kvh, hd, hd, hd ** -0.5, window),
+                                                              hybrid.RecurrenceConfig(h, h // 256, 4), 0.7, 0.7), mlp)
+    return hybrid.HybridConfig(vocab, h, 1e-5, [layer(i) for i in range(layers)], tuple(range(layers)))
+
+
+def hybrid_model(torch, cfg, capacity, seed=1):
+    """Random bf16 weights drawn on the device, fan-in scaled."""
+    from llvq_b200 import hybrid
+    g = torch.Generator(device="cuda").manual_seed(seed)
+    shapes = {"embed": (cfg.vocab, cfg.width), "head": (cfg.vocab, cfg.width), "final.norm": (cfg.width,)}
+    D = cfg.width
+    for i, l in enumerate(cfg.layers):
+        c, p, m = l.mixer, f"l{i}.mix", f"l{i}.mlp"
+        shapes.update({f"l{i}.norm1": (D,), f"l{i}.norm2": (D,)})
+        if isinstance(c, hybrid.DeltaConfig):
+            qk, v = c.kv_heads * c.dim, c.heads * c.vdim
+            shapes.update({p + ".q": (qk, D), p + ".k": (qk, D), p + ".v": (v, D), p + ".g": (v, D), p + ".b": (c.heads, D), p + ".a": (c.heads, D),
+                           p + ".q.conv": (qk, c.taps), p + ".k.conv": (qk, c.taps), p + ".v.conv": (v, c.taps), p + ".A_log": (c.heads,),
+                           p + ".dt_bias": (c.heads,), p + ".norm": (c.vdim,), p + ".o": (D, v)})
+        else:
+            a, r = c.left, c.right
+            n = r.width // r.blocks
+            shapes.update({p + ".left.q": (a.heads * a.dim, D), p + ".left.k": (a.kv_heads * a.dim, D), p + ".left.v": (a.kv_heads * a.vdim, D),
+                           p + ".left.g": (a.heads * a.vdim, D), p + ".left.q.norm": (a.dim,), p + ".left.k.norm": (a.dim,),
+                           p + ".left.o": (D, a.heads * a.vdim), p + ".right.conv": (r.width, r.taps), p + ".right.conv.b": (r.width,),
+                           p + ".right.lam": (r.width,), p + ".right.o": (D, r.width)})
+            for k in ("x", "y"):
+                shapes.update({f"{p}.right.{k}": (r.width, D), f"{p}.right.{k}.b": (r.width,)})
+            for k in ("ra", "ri"):
+                shapes.update({f"{p}.right.{k}": (r.blocks, n, n), f"{p}.right.{k}.b": (r.blocks, n)})
+        for u in [m] if not l.mlp.experts else [f"{m}.e{e}" for e in range(l.mlp.experts)]:
+            shapes.update({u + ".gate": (l.mlp.ff, D), u + ".up": (l.mlp.ff, D), u + ".down": (D, l.mlp.ff)})
+        if l.mlp.experts:
+            shapes[m + ".table"] = (cfg.vocab, l.mlp.top)
+
+    def tensor(name):
+        s = shapes[name]
+        if name.endswith(".table"):
+            experts = cfg.layers[int(name[1:name.index(".")])].mlp.experts
+            return torch.rand(s[0], experts, generator=g, device="cuda").argsort(1)[:, :s[1]].int()
+        w = torch.randn(*s, generator=g, device="cuda", dtype=torch.float32)
+        if name.endswith((".lam", ".A_log")):
+            return (w - 3).bfloat16()
+        return (w * s[-1] ** -0.5 if len(s) > 1 else 1 + 0.02 * w if "norm" in name else 0.02 * w).bfloat16()
+    return hybrid.HybridLM(cfg, tensor, "bfloat16", capacity, torch.device("cuda"))
+
+
+def run_hybrid(args):
+    """--hybrid: prefill and greedy decode of hybrid models (bf16, random weights; attention beside a linear recurrence and
+    the delta rule by turns, dense and routed feed-forwards) at the layer sizes of the named models, beside the
+    latent-attention model of the same size on the same tokens, with the time of each kernel against its roofline as
+    --latent takes it. The delta rule's scan is f32 arithmetic in registers: its roofline is the f32 rate of the CUDA cores
+    at the sampled clock (2 x 128 lanes per SM)."""
+    import gc
+    import torch
+    from llvq_b200.hybrid import DeltaConfig
+    B = LayerBench(args)
+    torch.cuda.set_device(0)
+    sampler = ClockSampler(0)
+    sampler.start()
+    n, window, peak, tflops = B.prompt_len, B.window, B.peak, B.tflops
+    sms = torch.cuda.get_device_properties(0).multi_processor_count
+    results = []
+    for shape in args.latent_shapes.split(","):
+        r = {"shape": shape, "layers": B.n_layers, "window": window}
+        for kind in ("dense", "routed"):
+            cfg = hybrid_config(shape, B.n_layers, window, kind == "routed")
+            m = hybrid_model(torch, cfg, n + 128)
+            lib = m.lib
+            launches = lib.llvq_dn_launch_count()
+            e = r["hybrid " + kind] = B.loop_times(m)
+            size = lambda t: t.numel() * t.element_size()
+            pairs = [(L, c, s) for L, c, s in zip(m.layers, cfg.layers, m.states)]
+            used = lambda L, c, k: c.mlp.top * size(L[k]) // c.mlp.experts
+            proj = sum(size(L["in"].w) + (used(L, c, "experts_up") if c.mlp.experts else size(L["gate_up"].w)) for L, c, _ in pairs)
+            outp = sum(size(L["out"].w) + (used(L, c, "experts_down") if c.mlp.experts else size(L["down"].w) if L["down"] is not None else 0) for L, c, _ in pairs)
+            att = sum(min(window, s["ring"].slots) * s["ring"].ld * 2 + size(L["gates"]) for L, _, s in pairs if "ring" in s)
+            dl = sum(size(s["state"].halves) for _, c, s in pairs if isinstance(c.mixer, DeltaConfig))  # one half read, one written
+            e["token_step"] = B.phases(m, {"projections": proj, "output": outp, "mixer": att, "delta": dl, "head": size(m.head.w)},
+                                       {"mixer": (B.n_layers + 1) // 2, "delta": B.n_layers // 2})
+            if kind == "dense":
+                e["prompt_kernels"] = hybrid_prompt_kernels(torch, B, m, cfg, sms)
+            e["launches"] = int(lib.llvq_dn_launch_count() - launches)
+            e["state_bytes"] = m.cache_bytes()
+            del m, pairs, lib
+            gc.collect()
+            torch.cuda.empty_cache()
+        r["latent"] = B.latent(shape)["latent"]
+        gc.collect()
+        torch.cuda.empty_cache()
+        results.append(r)
+    clocks = sampler.stop()
+    first = results[0]["hybrid dense"]
+    emit({"metric": "hybrid_decode_tok_per_s", "value": first["decode_tok_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": B.new_tokens - 8, "warmup": 3,
+          "ms_per_step": first["decode_ms_per_token"], "higher_is_better": True, "vs_baseline": None, "dtype": "bf16",
+          "data": "synthetic (random weights and tokens)", "clocks": clocks, "peaks": {"hbm_gbs": peak, "bf16_tflops": tflops},
+          "config": {"prompt_tokens": n, "window": window, "layers": B.n_layers}, "results": results})
+
+
+def hybrid_prompt_kernels(torch, B, m, cfg, sms):
+    """Kernels of one prompt portion behind a full window, rotating over three operand sets."""
+    import ctypes as C
+    from llvq_b200 import _lib
+    lib, check, st, n, window = m.lib, _lib.check_dense, m._cuda_stream, B.prompt_len, B.window
+    p, d = cfg.layers[0].mixer, cfg.layers[1].mixer
+    a, r, L, Ld, (g, u), dd, ring = p.left, p.right, m.layers[0], m.layers[1], m._mix[0], m._mix[1], m.states[0]["ring"]
+    D, ff, T = cfg.width, cfg.layers[0].mlp.ff, B.prompt_len + B.window - 1
+    new = lambda *s: torch.randn(*s, device="cuda").bfloat16()
+    floats = C.c_size_t()
+    check(lib.llvq_dn_delta_scratch(C.byref(dd), n, C.byref(floats)))
+    hv, v = d.heads * d.vdim, d.channels + d.heads * d.vdim
+    k = r.width // r.blocks
+    sets = [dict(y=new(n, L["in"].n), yd=new(n, v), ba=torch.randn(n, 2 * d.heads, device="cuda"), qn=new(n, a.heads * a.dim), rows=new(T, ring.ld),
+                 vt=new(a.kv_heads * a.vdim, -(-T // 8) * 8), ctx=new(n, a.heads * a.vdim), act=new(n, L["out"].ld), u=new(n, r.width),
+                 z=torch.randn(r.blocks, n, 2 * k, device="cuda"), scratch=torch.empty(floats.value, device="cuda"), x=torch.randn(n, D, device="cuda"),
+                 o=new(n, D), h1=new(n, D), h2=new(n, D), gu=new(n, 2 * ff)) for _ in range(3)]
+    at = lambda s, name: s["y"].data_ptr() + 2 * L["at"][name]
+    ldy = L["in"].n
+    P = lambda t: t.data_ptr()
+    ring_conv = P(m.states[0]["conv"].rows)
+    calls = {
+        "attention": lambda s: lib.llvq_dn_gqa_prefill(C.byref(g), P(s["qn"]), P(s["rows"]), P(s["vt"]), s["vt"].shape[1], n, T, window - 1, 0, P(s["ctx"]), 0, st()),
+        "query norms and cache rows": lambda s: lib.llvq_dn_gqa_rows(C.byref(g), at(s, "q"), at(s, "k"), at(s, "v"), ldy, P(s["qn"]), 0, n, st()),
+        "output gate": lambda s: lib.llvq_dn_gate_rows(m.dt, P(s["ctx"]), hv, at(s, "g"), ldy, P(s["act"]), L["out"].ld, n, hv, 0.7, st()),
+        "convolution": lambda s: lib.llvq_dn_conv_rows(m.dt, at(s, "x"), ldy, P(L["x_b"]), P(L["conv"]), P(L["conv_b"]), ring_conv, P(s["u"]), r.width, r.taps, 0, n, st()),
+        "linear recurrence": lambda s: lib.llvq_dn_lru_rows(C.byref(u), P(s["u"]), P(s["z"]), at(s, "y"), ldy, P(L["y_b"]), P(s["act"]), L["out"].ld, 0, n, st()),
+        "delta rule (convolution to gate)": lambda s: lib.llvq_dn_delta_rows(C.byref(dd), P(s["yd"]), v, P(s["ba"]), P(s["yd"]) + 2 * d.channels, v, P(s["scratch"]),
+                                                                             P(s["act"]), L["out"].ld, 0, n, st()),
+        "sum and two norms": lambda s: lib.llvq_dn_add_norms_rows(m.dt, P(s["x"]), P(s["o"]), None, None, 0, P(L["norm1"]), P(s["h1"]), P(L["norm2"]), P(s["h2"]), 1e-5, n, D, st()),
+        "gated unit": lambda s: lib.llvq_dn_gated_rows(m.dt, P(s["gu"]), None, P(s["act"]), L["out"].ld, n, ff, float("inf"), 1.0, 0.0, 1.0, st())
+        if L["out"].ld >= ff else 0,
+    }
+    bytes_ = {"query norms and cache rows": 2 * 2 * n * (a.heads * a.dim + a.kv_heads * (a.dim + a.vdim)), "output gate": 2 * 3 * n * hv, "convolution": 2 * 2 * n * r.width,
+              "linear recurrence": n * r.width * (8 + 2 * 3), "sum and two norms": n * D * (8 + 6), "gated unit": n * ff * 6,
+              "delta rule (convolution to gate)": 2 * n * (v + hv)}
+    out = {}
+    for name, fn in calls.items():
+        ms = B.event_ms(lambda k: check(fn(sets[k % 3])), 12)
+        e = out[name] = {"us": round(ms * 1e3, 1)}
+        if name in bytes_:
+            e.update(GBps=round(bytes_[name] / ms / 1e6, 1), frac=round(bytes_[name] / ms / 1e6 / B.peak, 4))
+        if name == "attention":
+            fl = 2.0 * n * window * a.heads * (a.dim + a.vdim)
+            e.update(TFLOPs=round(fl / ms / 1e9, 1), frac=round(fl / ms / 1e9 / B.tflops, 4))
+        if name.startswith("delta"):
+            fl = 8.0 * n * d.heads * d.dim * d.vdim
+            e.update(f32_TFLOPs=round(fl / ms / 1e9, 1), f32_frac=round(fl / ms / 1e9 / (sms * 256 * 1.965e-3), 4))
+
+    def gates(i):
+        m._bmm(sets[i % 3]["u"].view(n, r.blocks, k).transpose(0, 1), L["gates"][:, :, :k], torch.float32)
+
+    def products(i):
+        s = sets[i % 3]
+        for x, w in ((s["h1"], L["in"]), (s["h2"], L["gate_up"]), (s["h1"], Ld["in"]), (s["h2"], Ld["gate_up"])):
+            m._mm(x, w.rows(0))
+        for w in (L["out"], Ld["out"]):
+            m._mm(s["act"][:, :w.k], w.rows(0))
+    for name, fn, fl in (("gate matrices", gates, 4.0 * n * r.width * k),
+                         ("library products (two layers)", products, 2.0 * n * sum(x[w].n * x[w].k for x in (L, Ld) for w in ("in", "gate_up", "out")))):
+        ms = B.event_ms(fn, 12)
+        out[name] = {"us": round(ms * 1e3, 1), "TFLOPs": round(fl / ms / 1e9, 1), "frac": round(fl / ms / 1e9 / B.tflops, 4)}
+    return out
 
 
 _RESULT_FD = None
@@ -972,12 +1167,16 @@ def main():
                     help="launch q, k, v and gate, up separately instead of row-concatenated")
     ap.add_argument("--latent", action="store_true",
                     help="instead of the headline workload: latent-attention models beside the Qwen3 model of equal size")
-    ap.add_argument("--latent-shapes", default="qwen3-4b,qwen3-8b,qwen3-14b", help="--latent: layer sizes, by model name")
-    ap.add_argument("--latent-layers", type=int, default=8, help="--latent: layers of both models")
-    ap.add_argument("--window", type=int, default=1024, help="--latent: sliding window of the latent layers")
+    ap.add_argument("--hybrid", action="store_true",
+                    help="instead of the headline workload: hybrid models beside the latent-attention model of equal size")
+    ap.add_argument("--latent-shapes", default="qwen3-4b,qwen3-8b,qwen3-14b", help="--latent, --hybrid: layer sizes, by model name")
+    ap.add_argument("--latent-layers", type=int, default=8, help="--latent, --hybrid: layers of every model")
+    ap.add_argument("--window", type=int, default=1024, help="--latent, --hybrid: sliding window of the attention layers")
     args = ap.parse_args()
     if args.latent:
         return run_latent(args)
+    if args.hybrid:
+        return run_hybrid(args)
     if args.impl == "reference":
         return run_reference(args)
     if args.tp_decode:
