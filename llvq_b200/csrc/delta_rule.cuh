@@ -10,9 +10,9 @@
 //
 //   delta_token_kernel  a CTA takes 32 value columns of a head; the head's last CTA to arrive norms and gates its
 //                       output: no CTA waits for another.
-//   delta_prep_kernel   a portion's convolutions, unit vectors, k q, decays and step sizes.
+//   delta_prep_kernel   a portion's convolutions, and the scalars of every four tokens.
 //   delta_scan_kernel   the recurrence of a portion: a CTA keeps 32 columns of a head's state in registers, LANES lanes
-//                       per column, and walks the tokens; keys and queries come in double-buffered tiles.
+//                       per four columns, and walks the tokens; keys and queries come in double-buffered tiles.
 //   head_gate_rows_kernel  per head: o / rms(o) * w * silu(gate).
 #pragma once
 #include "linear_recurrence.cuh"
@@ -156,13 +156,26 @@ delta_token_kernel(DeltaArgs A) {
 }
 
 // ---- prompt portions ----
+//
+// Tokens go four at a time. With G_i the decay from the group's start through token i, R_im = G_i / G_m (k_m k_i) and
+// P_im = G_i / G_m (k_m q_i), the four steps from a state S are
+//
+//   u_i = beta_i (v_i - G_i S^T k_i - sum_{m<i} R_im u_m),  o_i = G_i S^T q_i + sum_{m<=i} P_im u_m,
+//   S <- G_3 S + sum_i (G_3 / G_i) k_i u_i^T:
+//
+// one reduction over dim and one update of the state for four tokens. Keys and queries stay as the convolution left them;
+// their scales to unit vectors go with the group's scalars.
+
+constexpr int kDeltaGroup = 4;
+constexpr int kDeltaScalars = 40;  // beta[4], G - 1 [4], key scales [4], query scales [4], G_3 / G_i key scale [4], R [6], P [10]
 
 // Lanes of a column and rows of a lane (in fours) of the scan; dims beyond 1024 are not served.
-__host__ __device__ inline int delta_lanes(int dim) { return dim <= 256 ? 8 : 32; }
+__host__ __device__ inline int delta_lanes(int dim) { return dim <= 256 ? 16 : 32; }
 __host__ __device__ inline int delta_fours(int dim) { return (dim + 4 * delta_lanes(dim) - 1) / (4 * delta_lanes(dim)); }
-// Row length of the unit vectors of a portion: what the lanes of a column hold, zeros beyond dim.
+// Row length of the keys and queries of a portion: what the lanes of a column hold, zeros beyond dim.
 __host__ __device__ inline int delta_padded(int dim) { return delta_fours(dim) * 4 * delta_lanes(dim); }
 __host__ __device__ inline int delta_tile(int dim) { return dim <= 128 ? 32 : dim <= 256 ? 16 : 4; }  // tokens of a staged tile
+__host__ __device__ inline int delta_groups(int n) { return (n + kDeltaGroup - 1) / kDeltaGroup; }
 
 struct DeltaPrepArgs {
     const void* x;   // rows of one product, stride ldx: [q | k | v] channels
@@ -171,51 +184,127 @@ struct DeltaPrepArgs {
     const float* conv;
     const float* decay;
     const float* dt_bias;
-    float* qk;       // [n, kv_heads, 2, dp]: unit key, unit query / sqrt(dim)
+    float* qk;       // [groups * 4, kv_heads, 2, dp]: key, query
     float* v;        // [n, heads, vdim]
-    float* sc;       // [n, heads, 4]: g - 1, beta, k q, 0
+    float* sc;       // [groups, heads, 40]
     long long pos0;
-    int ldx, heads, kv_heads, dim, vdim, taps, dp;
+    int n, ldx, heads, kv_heads, dim, vdim, taps, dp;
 };
 
-// grid = n, 256 threads. Dynamic shared memory: kv_heads floats.
+// silu of the convolution of channel c at places t0 .. t0 + 3.
+template <typename T>
+__device__ __forceinline__ void delta_conv4(const DeltaPrepArgs& A, int channels, int t0, int c, float (&out)[kDeltaGroup]) {
+    const T* X = reinterpret_cast<const T*>(A.x);
+    if (A.taps == 4) {
+        const float4 w = *reinterpret_cast<const float4*>(A.conv_w + (size_t)c * 4);
+        float in[kDeltaGroup + 3];
+        if (t0 >= 3 && t0 + kDeltaGroup <= A.n) {
+            const T* p = X + (size_t)(t0 - 3) * A.ldx + c;
+#pragma unroll
+            for (int k = 0; k < kDeltaGroup + 3; ++k) in[k] = to_f32(p[(size_t)k * A.ldx]);
+        } else {
+#pragma unroll
+            for (int k = 0; k < kDeltaGroup + 3; ++k) in[k] = conv_input(X, A.ldx, 0.0f, A.conv, channels, 4, A.pos0, min(t0 + k - 3, A.n - 1), c);
+        }
+#pragma unroll
+        for (int i = 0; i < kDeltaGroup; ++i) out[i] = silu_f(fmaf(w.x, in[i], fmaf(w.y, in[i + 1], fmaf(w.z, in[i + 2], w.w * in[i + 3]))));
+        return;
+    }
+    const float* w = A.conv_w + (size_t)c * A.taps;
+#pragma unroll
+    for (int i = 0; i < kDeltaGroup; ++i) {
+        float u = 0.0f;
+        for (int k = 0; k < A.taps; ++k) u = fmaf(w[A.taps - 1 - k], conv_input(X, A.ldx, 0.0f, A.conv, channels, A.taps, A.pos0, min(t0 + i - k, A.n - 1), c), u);
+        out[i] = silu_f(u);
+    }
+}
+
+// grid = groups, 256 threads: a warp takes a key head at a time, then all share the values.
 template <typename T>
 __global__ void __launch_bounds__(256)
 delta_prep_kernel(DeltaPrepArgs A) {
-    extern __shared__ float kq_s[];
     llvq_dependent_enter();
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, t = blockIdx.x;
-    const int channels = 2 * A.kv_heads * A.dim + A.heads * A.vdim;
-    const T* X = reinterpret_cast<const T*>(A.x);
-    auto conv = [&](int c) {
-        const float* w = A.conv_w + (size_t)c * A.taps;
-        float u = 0.0f;
-        for (int k = 0; k < A.taps; ++k) u = fmaf(w[A.taps - 1 - k], conv_input(X, A.ldx, 0.0f, A.conv, channels, A.taps, A.pos0, t - k, c), u);
-        return silu_f(u);
-    };
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, t0 = blockIdx.x * kDeltaGroup, here = min(kDeltaGroup, A.n - t0);
+    const int channels = 2 * A.kv_heads * A.dim + A.heads * A.vdim, rep = A.heads / A.kv_heads;
     for (int g = warp; g < A.kv_heads; g += 8) {
-        float* kd = A.qk + ((size_t)t * A.kv_heads + g) * 2 * A.dp;
-        float* qd = kd + A.dp;
-        float qq = 0.0f, kk = 0.0f, kq = 0.0f;
-        for (int i = lane; i < A.dp; i += 32) {
-            float q = 0.0f, k = 0.0f;
-            if (i < A.dim) q = conv(g * A.dim + i), k = conv((A.kv_heads + g) * A.dim + i);
-            kd[i] = k;
-            qd[i] = q;
-            qq = fmaf(q, q, qq), kk = fmaf(k, k, kk), kq = fmaf(k, q, kq);
+        float kk[kDeltaGroup][kDeltaGroup], kq[kDeltaGroup][kDeltaGroup], qq[kDeltaGroup];  // [i][m], m <= i
+#pragma unroll
+        for (int i = 0; i < kDeltaGroup; ++i) {
+            qq[i] = 0.0f;
+#pragma unroll
+            for (int m = 0; m <= i; ++m) kk[i][m] = kq[i][m] = 0.0f;
         }
-        const float fq = 1.0f / sqrtf(warp_sum_f(qq) + kUnitEps) / sqrtf((float)A.dim), fk = 1.0f / sqrtf(warp_sum_f(kk) + kUnitEps);
-        kq = warp_sum_f(kq) * fq * fk;
-        for (int i = lane; i < A.dp; i += 32) kd[i] *= fk, qd[i] *= fq;  // what this lane wrote
-        if (lane == 0) kq_s[g] = kq;
+        for (int e = lane; e < A.dp; e += 32) {
+            float q[kDeltaGroup] = {0.0f, 0.0f, 0.0f, 0.0f}, k[kDeltaGroup] = {0.0f, 0.0f, 0.0f, 0.0f};
+            if (e < A.dim) {
+                delta_conv4<T>(A, channels, t0, g * A.dim + e, q);
+                delta_conv4<T>(A, channels, t0, (A.kv_heads + g) * A.dim + e, k);
+            }
+#pragma unroll
+            for (int i = 0; i < kDeltaGroup; ++i) {
+                if (i >= here) q[i] = k[i] = 0.0f;
+                float* dst = A.qk + ((size_t)(t0 + i) * A.kv_heads + g) * 2 * A.dp + e;
+                dst[0] = k[i];
+                dst[A.dp] = q[i];
+                qq[i] = fmaf(q[i], q[i], qq[i]);
+#pragma unroll
+                for (int m = 0; m <= i; ++m) {
+                    kk[i][m] = fmaf(k[m], k[i], kk[i][m]);
+                    kq[i][m] = fmaf(k[m], q[i], kq[i][m]);
+                }
+            }
+        }
+        float fk[kDeltaGroup], fq[kDeltaGroup];
+        const float root = 1.0f / sqrtf((float)A.dim);
+#pragma unroll
+        for (int i = 0; i < kDeltaGroup; ++i) {
+#pragma unroll
+            for (int m = 0; m <= i; ++m) {
+                kk[i][m] = warp_sum_f(kk[i][m]);
+                kq[i][m] = warp_sum_f(kq[i][m]);
+            }
+            fk[i] = 1.0f / sqrtf(kk[i][i] + kUnitEps);
+            fq[i] = root / sqrtf(warp_sum_f(qq[i]) + kUnitEps);
+        }
+        for (int r = lane; r < rep; r += 32) {
+            const int h = g * rep + r;
+            float sc[kDeltaScalars], lg[kDeltaGroup];
+#pragma unroll
+            for (int i = 0; i < kDeltaScalars; ++i) sc[i] = 0.0f;
+            float sum = 0.0f;
+#pragma unroll
+            for (int i = 0; i < kDeltaGroup; ++i) {
+                const float* ba = A.ba + (size_t)min(t0 + i, A.n - 1) * 2 * A.heads;
+                lg[i] = i < here ? -A.decay[h] * softplus_f(ba[A.heads + h] + A.dt_bias[h]) : 0.0f;
+                sum += lg[i];
+                sc[i] = i < here ? sigmoid_f(ba[h]) : 0.0f;
+                sc[4 + i] = expm1f(sum);
+                sc[8 + i] = fk[i];
+                sc[12 + i] = fq[i];
+            }
+#pragma unroll
+            for (int m = 0; m < kDeltaGroup; ++m) {
+                float from = 0.0f;  // log of the decay from token m on
+#pragma unroll
+                for (int i = m; i < kDeltaGroup; ++i) {
+                    if (i > m) from += lg[i];
+                    const float f = i > m ? expf(from) : 1.0f;
+                    sc[26 + i * (i + 1) / 2 + m] = f * kq[i][m] * fk[m] * fq[i];
+                    if (i > m) sc[20 + i * (i - 1) / 2 + m] = f * kk[i][m] * fk[m] * fk[i];
+                    if (i == kDeltaGroup - 1) sc[16 + m] = f * fk[m];
+                }
+            }
+            float4* dst = reinterpret_cast<float4*>(A.sc + ((size_t)blockIdx.x * A.heads + h) * kDeltaScalars);
+#pragma unroll
+            for (int i = 0; i < kDeltaScalars / 4; ++i) dst[i] = make_float4(sc[4 * i], sc[4 * i + 1], sc[4 * i + 2], sc[4 * i + 3]);
+        }
     }
-    for (int c = threadIdx.x; c < A.heads * A.vdim; c += 256) A.v[(size_t)t * A.heads * A.vdim + c] = conv(2 * A.kv_heads * A.dim + c);
-    __syncthreads();
-    const int rep = A.heads / A.kv_heads;
-    for (int h = threadIdx.x; h < A.heads; h += 256) {
-        const float* ba = A.ba + (size_t)t * 2 * A.heads;
-        reinterpret_cast<float4*>(A.sc)[(size_t)t * A.heads + h] =
-            make_float4(expm1f(-A.decay[h] * softplus_f(ba[A.heads + h] + A.dt_bias[h])), sigmoid_f(ba[h]), kq_s[h / rep], 0.0f);
+    for (int c = threadIdx.x; c < A.heads * A.vdim; c += 256) {
+        float v[kDeltaGroup];
+        delta_conv4<T>(A, channels, t0, 2 * A.kv_heads * A.dim + c, v);
+#pragma unroll
+        for (int i = 0; i < kDeltaGroup; ++i)
+            if (i < here) A.v[(size_t)(t0 + i) * A.heads * A.vdim + c] = v[i];
     }
 }
 
@@ -230,7 +319,7 @@ struct DeltaScanArgs {
 };
 
 inline size_t delta_scan_smem(int dim) {  // two tiles of keys, queries, values and scalars; one of outputs
-    return (size_t)delta_tile(dim) * (2 * (2 * delta_padded(dim) + kDtCols + 4) + kDtCols) * sizeof(float);
+    return (size_t)delta_tile(dim) * (2 * (2 * delta_padded(dim) + kDtCols + kDeltaScalars / kDeltaGroup) + kDtCols) * sizeof(float);
 }
 
 // Two f32 at a time.
@@ -251,108 +340,180 @@ __device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
     return r;
 }
 
-// grid = (ceil(vdim / 32), heads), 32 * LANES threads: lane l of a column holds rows 4 (l + LANES m) .. + 3, m < FOURS.
+constexpr int kDsCols = 4;  // columns of a thread
+
+// grid = (ceil(vdim / 32), heads), 8 * LANES threads: lane l of a group of four columns holds rows 4 (l + LANES m) .. + 3,
+// m < FOURS, of each.
 template <int LANES, int FOURS>
-__global__ void __launch_bounds__(kDtCols * LANES)
+__global__ void __launch_bounds__(kDtCols / kDsCols * LANES)
 delta_scan_kernel(DeltaScanArgs A) {
-    constexpr int kThreads = kDtCols * LANES, dp = 4 * LANES * FOURS;
+    constexpr int kThreads = kDtCols / kDsCols * LANES, dp = 4 * LANES * FOURS, G = kDeltaGroup, NC = kDsCols;
     extern __shared__ __align__(16) float ds_smem[];
-    const int TT = delta_tile(A.dim), tid = threadIdx.x, l = tid % LANES, col = tid / LANES;
-    const int h = blockIdx.y, g = h / (A.heads / A.kv_heads), j = blockIdx.x * kDtCols + col;
-    float* qk_s = ds_smem;                          // [2][TT][2 dp]
-    float* sc_s = qk_s + 2 * TT * 2 * dp;           // [2][TT][4]
-    float* v_s = sc_s + 2 * TT * 4;                 // [2][TT][32]
-    float* o_s = v_s + 2 * TT * kDtCols;            // [TT][32]
+    const int TT = delta_tile(A.dim), tid = threadIdx.x, l = tid % LANES, cg = tid / LANES;
+    const int h = blockIdx.y, g = h / (A.heads / A.kv_heads), c0 = blockIdx.x * kDtCols, cols = min(kDtCols, A.vdim - c0);
+    float* qk_s = ds_smem;                                  // [2][TT][2 dp]
+    float* sc_s = qk_s + 2 * TT * 2 * dp;                   // [2][TT / 4][40]
+    float* v_s = sc_s + 2 * (TT / G) * kDeltaScalars;       // [2][TT][32]
+    float* o_s = v_s + 2 * TT * kDtCols;                    // [TT][32]
     llvq_dependent_enter();
     auto copy16 = [](float* dst, const float* src) {
         asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((unsigned int)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
     };
-    const int c0 = blockIdx.x * kDtCols, cols = min(kDtCols, A.vdim - c0);
+    const int whole = delta_groups(A.n) * G;  // rows of qk
     auto stage = [&](int t0, int buf) {
-        const int here = min(TT, A.n - t0);
+        const int here = min(TT, whole - t0);
         constexpr int per = 2 * dp / 4;
         for (int i = tid; i < here * per; i += kThreads) {
             const int t = i / per, c = i - t * per;
             copy16(qk_s + (size_t)(buf * TT + t) * 2 * dp + 4 * c, A.qk + ((size_t)(t0 + t) * A.kv_heads + g) * 2 * dp + 4 * c);
         }
-        for (int t = tid; t < here; t += kThreads) copy16(sc_s + (buf * TT + t) * 4, A.sc + ((size_t)(t0 + t) * A.heads + h) * 4);
+        constexpr int ps = kDeltaScalars / 4;
+        for (int i = tid; i < here / G * ps; i += kThreads) {
+            const int t = i / ps, c = i - t * ps;
+            copy16(sc_s + (size_t)(buf * (TT / G) + t) * kDeltaScalars + 4 * c, A.sc + ((size_t)(t0 / G + t) * A.heads + h) * kDeltaScalars + 4 * c);
+        }
         for (int i = tid; i < here * kDtCols; i += kThreads) {
             const int t = i / kDtCols, c = i - t * kDtCols;
-            if (c < cols)
-                asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((unsigned int)__cvta_generic_to_shared(v_s + buf * TT * kDtCols + i)),
+            float* dst = v_s + buf * TT * kDtCols + i;
+            if (c < cols && t0 + t < A.n)
+                asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((unsigned int)__cvta_generic_to_shared(dst)),
                              "l"(A.v + ((size_t)(t0 + t) * A.heads + h) * A.vdim + c0 + c)
                              : "memory");
+            else
+                *dst = 0.0f;
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     stage(0, 0);
-    f32x2 S[FOURS][2];
-    const size_t half = (size_t)A.heads * A.dim * A.vp, base = (size_t)h * A.dim * A.vp + j;
+    f32x2 S[NC][FOURS][2];
+    const size_t half = (size_t)A.heads * A.dim * A.vp, base = (size_t)h * A.dim * A.vp + c0 + cg * NC;
+    const bool in = c0 + cg * NC < A.vp;  // vp is a multiple of four
     const float* S0 = A.state + (A.pos0 & 1) * half + base;
 #pragma unroll
     for (int m = 0; m < FOURS; ++m) {
-        float e[4];
+        float4 e[4];
 #pragma unroll
         for (int r = 0; r < 4; ++r) {
             const int i = 4 * (l + LANES * m) + r;
-            e[r] = A.pos0 > 0 && i < A.dim && j < A.vdim ? S0[(size_t)i * A.vp] : 0.0f;
+            e[r] = A.pos0 > 0 && in && i < A.dim ? *reinterpret_cast<const float4*>(S0 + (size_t)i * A.vp) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
         }
-        S[m][0] = pack2(e[0], e[1]);
-        S[m][1] = pack2(e[2], e[3]);
+        S[0][m][0] = pack2(e[0].x, e[1].x), S[0][m][1] = pack2(e[2].x, e[3].x);
+        S[1][m][0] = pack2(e[0].y, e[1].y), S[1][m][1] = pack2(e[2].y, e[3].y);
+        S[2][m][0] = pack2(e[0].z, e[1].z), S[2][m][1] = pack2(e[2].z, e[3].z);
+        S[3][m][0] = pack2(e[0].w, e[1].w), S[3][m][1] = pack2(e[2].w, e[3].w);
     }
+    const bool hi = l & (LANES / 2), hi2 = l & (LANES / 4);
+    const int mine = (hi ? 2 : 0) + (hi2 ? 1 : 0);  // the column whose sums end up in this lane
     for (int t0 = 0, buf = 0; t0 < A.n; t0 += TT, buf ^= 1) {
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();  // the tile is staged, the outputs before are stored and the other buffer is read
         if (t0 + TT < A.n) stage(t0 + TT, buf ^ 1);
-        const int here = min(TT, A.n - t0);
-        for (int t = 0; t < here; ++t) {
+        const int here = min(TT, whole - t0);
+        for (int t = 0; t < here; t += G) {
             const float* kr = qk_s + (size_t)(buf * TT + t) * 2 * dp + 4 * l;
-            const float4 sc = *reinterpret_cast<const float4*>(sc_s + (buf * TT + t) * 4);
-            const float v = v_s[(buf * TT + t) * kDtCols + col];
-            f32x2 k[FOURS][2], sk[2] = {0ull, 0ull}, sq[2] = {0ull, 0ull};
+            float sc[36];
 #pragma unroll
-            for (int m = 0; m < FOURS; ++m) {
-                const ulonglong2 kk = *reinterpret_cast<const ulonglong2*>(kr + 4 * LANES * m), qq = *reinterpret_cast<const ulonglong2*>(kr + dp + 4 * LANES * m);
-                k[m][0] = kk.x, k[m][1] = kk.y;
-                sk[0] = fma2(S[m][0], kk.x, sk[0]);
-                sk[1] = fma2(S[m][1], kk.y, sk[1]);
-                sq[0] = fma2(S[m][0], qq.x, sq[0]);
-                sq[1] = fma2(S[m][1], qq.y, sq[1]);
+            for (int i = 0; i < 9; ++i) {
+                const float4 q = *reinterpret_cast<const float4*>(sc_s + (size_t)(buf * (TT / G) + t / G) * kDeltaScalars + 4 * i);
+                sc[4 * i] = q.x, sc[4 * i + 1] = q.y, sc[4 * i + 2] = q.z, sc[4 * i + 3] = q.w;
             }
-            const float2 k0 = unpack2(sk[0]), k1 = unpack2(sk[1]), q0 = unpack2(sq[0]), q1 = unpack2(sq[1]);
-            float tk = (k0.x + k0.y) + (k1.x + k1.y), tq = (q0.x + q0.y) + (q1.x + q1.y);
+            f32x2 k[G][FOURS][2];
+            float val[NC][2 * G];
 #pragma unroll
-            for (int o = LANES / 2; o > 0; o >>= 1) {
-                tk += __shfl_xor_sync(0xffffffffu, tk, o);
-                tq += __shfl_xor_sync(0xffffffffu, tq, o);
-            }
-            const float u = sc.y * (v - carry(sc.x, tk, 0.0f));
-            const f32x2 g2 = pack2(sc.x, sc.x), u2 = pack2(u, u);
+            for (int i = 0; i < G; ++i) {
+                f32x2 ak[NC], aq[NC];
 #pragma unroll
-            for (int m = 0; m < FOURS; ++m) {
-                S[m][0] = fma2(k[m][0], u2, fma2(g2, S[m][0], S[m][0]));
-                S[m][1] = fma2(k[m][1], u2, fma2(g2, S[m][1], S[m][1]));
+                for (int c = 0; c < NC; ++c) ak[c] = aq[c] = 0ull;
+#pragma unroll
+                for (int m = 0; m < FOURS; ++m) {
+                    const ulonglong2 kk = *reinterpret_cast<const ulonglong2*>(kr + (size_t)i * 2 * dp + 4 * LANES * m);
+                    const ulonglong2 qq = *reinterpret_cast<const ulonglong2*>(kr + (size_t)i * 2 * dp + dp + 4 * LANES * m);
+                    k[i][m][0] = kk.x, k[i][m][1] = kk.y;
+#pragma unroll
+                    for (int c = 0; c < NC; ++c) {
+                        ak[c] = fma2(S[c][m][0], kk.x, ak[c]);
+                        aq[c] = fma2(S[c][m][0], qq.x, aq[c]);
+                        ak[c] = fma2(S[c][m][1], kk.y, ak[c]);
+                        aq[c] = fma2(S[c][m][1], qq.y, aq[c]);
+                    }
+                }
+#pragma unroll
+                for (int c = 0; c < NC; ++c) {
+                    const float2 a = unpack2(ak[c]), b = unpack2(aq[c]);
+                    val[c][i] = a.x + a.y;
+                    val[c][G + i] = b.x + b.y;
+                }
             }
-            if (l == 0) o_s[t * kDtCols + col] = fmaf(sc.z, u, carry(sc.x, tq, 0.0f));
+            // the sums over dim: two exchanges leave a column to a lane, the rest adds up among the lanes that share it
+            float two[2][2 * G], s[2 * G];
+#pragma unroll
+            for (int e = 0; e < 2 * G; ++e)
+#pragma unroll
+                for (int c = 0; c < 2; ++c)
+                    two[c][e] = (hi ? val[2 + c][e] : val[c][e]) + __shfl_xor_sync(0xffffffffu, hi ? val[c][e] : val[2 + c][e], LANES / 2);
+#pragma unroll
+            for (int e = 0; e < 2 * G; ++e) {
+                s[e] = (hi2 ? two[1][e] : two[0][e]) + __shfl_xor_sync(0xffffffffu, hi2 ? two[0][e] : two[1][e], LANES / 4);
+#pragma unroll
+                for (int o = LANES / 8; o > 0; o >>= 1) s[e] += __shfl_xor_sync(0xffffffffu, s[e], o);
+            }
+            float u[G], w[NC][G], out = 0.0f;
+#pragma unroll
+            for (int i = 0; i < G; ++i) {
+                const float tk = s[i] * sc[8 + i], tq = s[G + i] * sc[12 + i];
+                float x = v_s[(buf * TT + t + i) * kDtCols + cg * NC + mine] - carry(sc[4 + i], tk, 0.0f);
+                float y = carry(sc[4 + i], tq, 0.0f);
+#pragma unroll
+                for (int m = 0; m < i; ++m) {
+                    x = fmaf(-sc[20 + i * (i - 1) / 2 + m], u[m], x);
+                    y = fmaf(sc[26 + i * (i + 1) / 2 + m], u[m], y);
+                }
+                u[i] = sc[i] * x;
+                y = fmaf(sc[26 + i * (i + 1) / 2 + i], u[i], y);
+                if ((l & 3) == i) out = y;
+            }
+            if (l % (LANES / 4) < G) o_s[(t + (l & 3)) * kDtCols + cg * NC + mine] = out;
+#pragma unroll
+            for (int i = 0; i < G; ++i) {
+                const float own = u[i] * sc[16 + i], next = __shfl_xor_sync(0xffffffffu, own, LANES / 4);
+                const float a = hi2 ? next : own, b = hi2 ? own : next;
+                const float c = __shfl_xor_sync(0xffffffffu, a, LANES / 2), d = __shfl_xor_sync(0xffffffffu, b, LANES / 2);
+                w[0][i] = hi ? c : a, w[1][i] = hi ? d : b, w[2][i] = hi ? a : c, w[3][i] = hi ? b : d;
+            }
+            const f32x2 g2 = pack2(sc[7], sc[7]);
+#pragma unroll
+            for (int c = 0; c < NC; ++c) {
+#pragma unroll
+                for (int m = 0; m < FOURS; ++m)
+#pragma unroll
+                    for (int p = 0; p < 2; ++p) S[c][m][p] = fma2(g2, S[c][m][p], S[c][m][p]);
+#pragma unroll
+                for (int i = 0; i < G; ++i) {
+                    const f32x2 w2 = pack2(w[c][i], w[c][i]);
+#pragma unroll
+                    for (int m = 0; m < FOURS; ++m)
+#pragma unroll
+                        for (int p = 0; p < 2; ++p) S[c][m][p] = fma2(k[i][m][p], w2, S[c][m][p]);
+                }
+            }
         }
         __syncthreads();
-        for (int i = tid; i < here * kDtCols; i += kThreads) {
+        for (int i = tid; i < min(TT, A.n - t0) * kDtCols; i += kThreads) {
             const int t = i / kDtCols, c = i - t * kDtCols;
             if (c < cols) A.o[((size_t)(t0 + t) * A.heads + h) * A.vdim + c0 + c] = o_s[i];
         }
     }
-    if (j >= A.vdim) return;
+    if (!in) return;
     float* Sn = A.state + ((A.pos0 + A.n) & 1) * half + base;
 #pragma unroll
-    for (int m = 0; m < FOURS; ++m) {
-        const float2 a = unpack2(S[m][0]), b = unpack2(S[m][1]);
-        const float e[4] = {a.x, a.y, b.x, b.y};
+    for (int m = 0; m < FOURS; ++m)
 #pragma unroll
-        for (int r = 0; r < 4; ++r) {
-            const int i = 4 * (l + LANES * m) + r;
-            if (i < A.dim) Sn[(size_t)i * A.vp] = e[r];
+        for (int p = 0; p < 2; ++p) {
+            const float2 a = unpack2(S[0][m][p]), b = unpack2(S[1][m][p]), c = unpack2(S[2][m][p]), d = unpack2(S[3][m][p]);
+            const int i = 4 * (l + LANES * m) + 2 * p;
+            if (i < A.dim) *reinterpret_cast<float4*>(Sn + (size_t)i * A.vp) = make_float4(a.x, b.x, c.x, d.x);
+            if (i + 1 < A.dim) *reinterpret_cast<float4*>(Sn + (size_t)(i + 1) * A.vp) = make_float4(a.y, b.y, c.y, d.y);
         }
-    }
 }
 
 // out[t, h, :] = o / sqrt(mean(o^2) + eps) * w * silu(gate); grid = rows, 256 threads: a warp takes a head at a time.

@@ -115,7 +115,7 @@ bool plan_stream(DenseGemvArgs& a, int* grid, size_t* smem) {
     if (a.w_r) {  // segments of one length for the matrix and for each routed one
         const int vecs_r = a.ld_r / 8, total = vecs + a.top * vecs_r;
         bool found = false;
-        for (int n = (total + 6 * 32 - 1) / (6 * 32); n <= kGvWarps && !found; ++n) {
+        for (int n = std::min(kGvWarps, (total + 6 * 32 - 1) / (6 * 32)); n <= kGvWarps && !found; ++n) {
             a.segv = (total + n - 1) / n - 1;
             while (!found && ++a.segv <= kGsMaxVpl * 32) {
                 a.seg_r = (vecs_r + a.segv - 1) / a.segv;

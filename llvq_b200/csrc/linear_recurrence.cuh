@@ -14,8 +14,8 @@
 //   lru_token            the token step: a CTA takes 32 channels of a block: the block's u, two rows of the gate matrix
 //                        per channel, the recurrence, the gate branch.
 //   conv_rows_kernel     u of a prompt portion; conv_keep_kernel then stores the inputs the next step reads.
-//   lru_scan_kernel      the recurrence of a portion, one pass: a CTA owns 32 channels, a warp 32 tokens at a time in
-//                        registers; the warps' products and sums meet in shared memory, 512 tokens a turn.
+//   lru_scan_kernel      the recurrence of a portion, one pass: a CTA owns 16 channels, a thread 16 tokens at a time in
+//                        registers; their products and sums meet in shared memory, 512 tokens a turn.
 #pragma once
 #include "gqa_attn.cuh"
 
@@ -197,62 +197,75 @@ struct LruScanArgs {
     float out_scale;
 };
 
-constexpr int kScanTok = 32, kScanWarps = 16;
+constexpr int kScanTok = 16, kScanWarps = 16, kScanCh = 16, kScanTurn = 2 * kScanTok * kScanWarps;
 
-// grid = ceil(width / 32), 512 threads: lane = channel, warp = 32 tokens of the turn's 512.
+// sigmoid and gelu for results that are rounded to T: in bf16 the fast exponential and division are far inside the rounding.
+template <typename T>
+__device__ __forceinline__ float sigmoid_t(float x) {
+    if constexpr (sizeof(T) == 2) return __fdividef(1.0f, 1.0f + __expf(-x));
+    return sigmoid_f(x);
+}
+template <typename T>
+__device__ __forceinline__ float gelu_tanh_t(float z) {
+    if constexpr (sizeof(T) == 2) return z * sigmoid_t<T>(1.5957691216057308f * (z + 0.044715f * z * z * z));
+    return gelu_tanh_f(z);
+}
+
+// grid = ceil(width / 16), 512 threads: a warp's halves take 16 channels over 16 tokens each, a turn is 512 tokens.
 template <typename T>
 __global__ void __launch_bounds__(kScanWarps * 32)
 lru_scan_kernel(LruScanArgs A) {
-    __shared__ float prod_s[kScanWarps][32], sum_s[kScanWarps][32], carry_s[32];
+    __shared__ float2 part_s[2][kScanWarps][kScanCh];  // decay product and sum of a warp's 32 tokens; two turns' worth
     llvq_dependent_enter();
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, width = A.blocks * A.n;
-    const int ch = blockIdx.x * 32 + lane, cc = min(ch, width - 1), blk = cc / A.n, c = cc - blk * A.n;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, width = A.blocks * A.n, lc = lane & (kScanCh - 1), upper = lane / kScanCh;
+    const int ch = blockIdx.x * kScanCh + lc, cc = min(ch, width - 1), blk = cc / A.n, c = cc - blk * A.n;
     const float br = A.b[(size_t)blk * 2 * A.n + c], bi = A.b[(size_t)blk * 2 * A.n + A.n + c], lam = A.lam[cc], yb = A.y_bias[cc];
     const float* z = A.z + (size_t)blk * A.n_tok * 2 * A.n + c;
     const T* U = reinterpret_cast<const T*>(A.u) + cc;
     const T* Y = reinterpret_cast<const T*>(A.y) + cc;
     T* O = reinterpret_cast<T*>(A.out) + cc;
-    if (warp == 0) carry_s[lane] = A.pos0 > 0 ? A.state[(size_t)(A.pos0 & 1) * width + cc] : 0.0f;
-    for (int t0 = 0; t0 < A.n_tok; t0 += kScanWarps * kScanTok) {
-        const int tw = t0 + warp * kScanTok;
-        float a[kScanTok], x[kScanTok];
+    float state = A.pos0 > 0 ? A.state[(size_t)(A.pos0 & 1) * width + cc] : 0.0f;  // before the turn, the same in every thread of a channel
+    for (int t0 = 0, turn = 0; t0 < A.n_tok; t0 += kScanTurn, ++turn) {
+        const int tw = t0 + (2 * warp + upper) * kScanTok;
+        float a[kScanTok], x[kScanTok], u[kScanTok], y[kScanTok];
 #pragma unroll
         for (int k = 0; k < kScanTok; ++k) {
             const int t = min(tw + k, A.n_tok - 1);
             a[k] = z[(size_t)t * 2 * A.n];
             x[k] = z[(size_t)t * 2 * A.n + A.n];
+            u[k] = to_f32(U[(size_t)t * width]);
+            y[k] = to_f32(Y[(size_t)t * A.ldy]);
         }
         float prod = 1.0f, sum = 0.0f;  // a[] holds decays less one from here on
 #pragma unroll
         for (int k = 0; k < kScanTok; ++k) {
-            const int t = tw + k;
-            if (t < A.n_tok) {
-                a[k] = lru_decay(sigmoid_f(a[k] + br), lam);
-                x[k] = lru_input(a[k], sigmoid_f(x[k] + bi), to_f32(U[(size_t)t * width]));
-            } else {
-                a[k] = 0.0f;
-                x[k] = 0.0f;
-            }
+            const bool in = tw + k < A.n_tok;
+            a[k] = in ? lru_decay(sigmoid_f(a[k] + br), lam) : 0.0f;
+            x[k] = in ? lru_input(a[k], sigmoid_t<T>(x[k] + bi), u[k]) : 0.0f;
+            y[k] = gelu_tanh_t<T>(y[k] + yb) * A.out_scale;
             prod = carry(a[k], prod, 0.0f);
             sum = carry(a[k], sum, x[k]);
         }
-        prod_s[warp][lane] = prod;
-        sum_s[warp][lane] = sum;
+        // the lower half's tokens come first
+        const float lp = __shfl_sync(0xffffffffu, prod, lc), ls = __shfl_sync(0xffffffffu, sum, lc);
+        if (upper) part_s[turn & 1][warp][lc] = make_float2(prod * lp, fmaf(prod, ls, sum));
         __syncthreads();
-        float s = carry_s[lane];
-        for (int w = 0; w < warp; ++w) s = fmaf(prod_s[w][lane], s, sum_s[w][lane]);
-        __syncthreads();  // the carry and the warps' sums are read
-        if (warp == kScanWarps - 1) carry_s[lane] = fmaf(prod, s, sum);
+        float s = state, all = state;
+#pragma unroll
+        for (int w = 0; w < kScanWarps; ++w) {
+            const float2 p = part_s[turn & 1][w][lc];
+            all = fmaf(p.x, all, p.y);
+            if (w + 1 == warp) s = all;
+        }
+        state = all;
+        if (upper) s = fmaf(lp, s, ls);
 #pragma unroll
         for (int k = 0; k < kScanTok; ++k) {
-            const int t = tw + k;
             s = carry(a[k], s, x[k]);
-            if (t < A.n_tok && ch < width)
-                O[(size_t)t * A.ldo] = from_f32<T>(s * gelu_tanh_f(to_f32(Y[(size_t)t * A.ldy]) + yb) * A.out_scale);
+            if (tw + k < A.n_tok && ch < width) O[(size_t)(tw + k) * A.ldo] = from_f32<T>(s * y[k]);
         }
     }
-    __syncthreads();
-    if (warp == 0 && ch < width) A.state[(size_t)((A.pos0 + A.n_tok) & 1) * width + ch] = carry_s[lane];
+    if (warp == 0 && !upper && ch < width) A.state[(size_t)((A.pos0 + A.n_tok) & 1) * width + ch] = state;
 }
 
 }  // namespace llvq

@@ -65,22 +65,18 @@ int delta_scan_t(const DeltaScanArgs& k, cudaStream_t s) {
     const size_t smem = delta_scan_smem(k.dim);
     const int st = ensure_dyn_smem((const void*)delta_scan_kernel<LANES, FOURS>, smem);
     if (st) return st;
-    CUDA_TRY(launch_dep(delta_scan_kernel<LANES, FOURS>, dim3((k.vdim + kDtCols - 1) / kDtCols, k.heads), dim3(kDtCols * LANES), smem, s, k));
+    CUDA_TRY(launch_dep(delta_scan_kernel<LANES, FOURS>, dim3((k.vdim + kDtCols - 1) / kDtCols, k.heads), dim3(kDtCols / kDsCols * LANES), smem, s, k));
     g_launches++;
     return kStatusOk;
 }
 
 int delta_scan(const DeltaScanArgs& k, cudaStream_t s) {
     const int fours = delta_fours(k.dim);
-    if (delta_lanes(k.dim) == 8) switch (fours) {
-        case 1: return delta_scan_t<8, 1>(k, s);
-        case 2: return delta_scan_t<8, 2>(k, s);
-        case 3: return delta_scan_t<8, 3>(k, s);
-        case 4: return delta_scan_t<8, 4>(k, s);
-        case 5: return delta_scan_t<8, 5>(k, s);
-        case 6: return delta_scan_t<8, 6>(k, s);
-        case 7: return delta_scan_t<8, 7>(k, s);
-        default: return delta_scan_t<8, 8>(k, s);
+    if (delta_lanes(k.dim) == 16) switch (fours) {
+        case 1: return delta_scan_t<16, 1>(k, s);
+        case 2: return delta_scan_t<16, 2>(k, s);
+        case 3: return delta_scan_t<16, 3>(k, s);
+        default: return delta_scan_t<16, 4>(k, s);
     }
     switch (fours) {
         case 3: return delta_scan_t<32, 3>(k, s);
@@ -198,9 +194,9 @@ int llvq_dn_lru_rows(const llvq_dn_lru* a, const void* u, const float* z, const 
     if (!u || !z || !y || !y_bias || !out || ldy < width || ldo < width || pos0 < 0 || rows <= 0) return fail(kStatusInvalid, "dn_lru_rows: bad argument");
     LruScanArgs k{u, z, a->b, a->lam, y, y_bias, a->state, out, pos0, rows, a->blocks, a->n, ldy, ldo, a->out_scale};
     if (a->dtype == LLVQ_DN_BF16)
-        CUDA_TRY(launch_dep(lru_scan_kernel<bf16>, dim3((width + 31) / 32), dim3(kScanWarps * 32), 0, (cudaStream_t)stream, k));
+        CUDA_TRY(launch_dep(lru_scan_kernel<bf16>, dim3((width + kScanCh - 1) / kScanCh), dim3(kScanWarps * 32), 0, (cudaStream_t)stream, k));
     else
-        CUDA_TRY(launch_dep(lru_scan_kernel<float>, dim3((width + 31) / 32), dim3(kScanWarps * 32), 0, (cudaStream_t)stream, k));
+        CUDA_TRY(launch_dep(lru_scan_kernel<float>, dim3((width + kScanCh - 1) / kScanCh), dim3(kScanWarps * 32), 0, (cudaStream_t)stream, k));
     g_launches++;
     return kStatusOk;
 }
@@ -224,7 +220,8 @@ int llvq_dn_delta_scratch(const llvq_dn_delta* a, int32_t rows, size_t* floats) 
     const int st = check_delta(a, "dn_delta_scratch");
     if (st) return st;
     if (rows <= 0 || !floats) return fail(kStatusInvalid, "dn_delta_scratch: bad argument");
-    *floats = (size_t)rows * ((size_t)2 * a->kv_heads * delta_padded(a->dim) + (size_t)a->heads * 4 + (size_t)2 * a->heads * a->vdim);
+    const size_t groups = delta_groups(rows);
+    *floats = groups * (kDeltaGroup * (size_t)2 * a->kv_heads * delta_padded(a->dim) + (size_t)a->heads * kDeltaScalars) + (size_t)2 * rows * a->heads * a->vdim;
     return kStatusOk;
 }
 
@@ -238,16 +235,15 @@ int llvq_dn_delta_rows(const llvq_dn_delta* a, const void* x, int32_t ldx, const
     cudaStream_t s = (cudaStream_t)stream;
     const int dp = delta_padded(a->dim);
     float* qk = scratch;
-    float* sc = qk + (size_t)rows * 2 * a->kv_heads * dp;
-    float* v = sc + (size_t)rows * a->heads * 4;
+    float* sc = qk + (size_t)delta_groups(rows) * kDeltaGroup * 2 * a->kv_heads * dp;
+    float* v = sc + (size_t)delta_groups(rows) * a->heads * kDeltaScalars;
     float* o = v + (size_t)rows * hv;
-    DeltaPrepArgs p{x, ba, a->conv_w, a->conv, a->decay, a->dt_bias, qk, v, sc, pos0, ldx, a->heads, a->kv_heads, a->dim, a->vdim, a->taps, dp};
-    const size_t smem = (size_t)a->kv_heads * sizeof(float);
-    if (smem > 40 * 1024) return fail(kStatusUnsupported, "dn_delta_rows: %d key heads", a->kv_heads);
+    DeltaPrepArgs p{x, ba, a->conv_w, a->conv, a->decay, a->dt_bias, qk, v, sc, pos0, rows, ldx, a->heads, a->kv_heads, a->dim, a->vdim, a->taps, dp};
+    if (a->taps == 4 && ((uintptr_t)a->conv_w & 15)) return fail(kStatusInvalid, "dn_delta_rows: convolution weights not on 16 bytes");
     if (a->dtype == LLVQ_DN_BF16)
-        CUDA_TRY(launch_dep(delta_prep_kernel<bf16>, dim3(rows), dim3(256), smem, s, p));
+        CUDA_TRY(launch_dep(delta_prep_kernel<bf16>, dim3(delta_groups(rows)), dim3(256), 0, s, p));
     else
-        CUDA_TRY(launch_dep(delta_prep_kernel<float>, dim3(rows), dim3(256), smem, s, p));
+        CUDA_TRY(launch_dep(delta_prep_kernel<float>, dim3(delta_groups(rows)), dim3(256), 0, s, p));
     g_launches++;
     int st2 = llvq_dn_conv_keep(a->dtype, x, ldx, nullptr, a->conv, channels, a->taps, pos0, rows, stream);
     if (st2) return st2;
