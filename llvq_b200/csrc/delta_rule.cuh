@@ -207,7 +207,7 @@ __device__ __forceinline__ void delta_conv4(const DeltaPrepArgs& A, int channels
             for (int k = 0; k < kDeltaGroup + 3; ++k) in[k] = conv_input(X, A.ldx, 0.0f, A.conv, channels, 4, A.pos0, min(t0 + k - 3, A.n - 1), c);
         }
 #pragma unroll
-        for (int i = 0; i < kDeltaGroup; ++i) out[i] = silu_f(fmaf(w.x, in[i], fmaf(w.y, in[i + 1], fmaf(w.z, in[i + 2], w.w * in[i + 3]))));
+        for (int i = 0; i < kDeltaGroup; ++i) out[i] = silu_t<T>(fmaf(w.x, in[i], fmaf(w.y, in[i + 1], fmaf(w.z, in[i + 2], w.w * in[i + 3]))));
         return;
     }
     const float* w = A.conv_w + (size_t)c * A.taps;
@@ -215,7 +215,7 @@ __device__ __forceinline__ void delta_conv4(const DeltaPrepArgs& A, int channels
     for (int i = 0; i < kDeltaGroup; ++i) {
         float u = 0.0f;
         for (int k = 0; k < A.taps; ++k) u = fmaf(w[A.taps - 1 - k], conv_input(X, A.ldx, 0.0f, A.conv, channels, A.taps, A.pos0, min(t0 + i - k, A.n - 1), c), u);
-        out[i] = silu_f(u);
+        out[i] = silu_t<T>(u);
     }
 }
 
@@ -516,19 +516,61 @@ delta_scan_kernel(DeltaScanArgs A) {
         }
 }
 
-// out[t, h, :] = o / sqrt(mean(o^2) + eps) * w * silu(gate); grid = rows, 256 threads: a warp takes a head at a time.
+// out[t, h, :] = o / sqrt(mean(o^2) + eps) * w * silu(gate); grid = rows, 256 threads: a warp takes a head at a time, or (vec:
+// whole vectors of 8 on 16-byte boundaries, vdim <= 256) each of its halves one.
 template <typename T>
 __global__ void __launch_bounds__(256)
 head_gate_rows_kernel(const float* __restrict__ o, const float* __restrict__ w, const T* __restrict__ gate, int ldg, T* __restrict__ out, int ldo,
-                      int heads, int vdim, float eps) {
+                      int heads, int vdim, float eps, int vec) {
     llvq_dependent_enter();
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const size_t t = blockIdx.x;
+    if (vec) {
+        const int lane = threadIdx.x & 15;
+        const unsigned int mask = 0xffffu << (threadIdx.x & 16);
+        for (int h = threadIdx.x >> 4; h < heads; h += 16) {
+            const float* src = o + (t * heads + h) * vdim;
+            float f[2][8], g[2][8], ss = 0.0f;
+#pragma unroll
+            for (int k = 0; k < 2; ++k) {
+                const int i = (lane + 16 * k) * 8;
+                if (i >= vdim) break;
+                float4 a = *reinterpret_cast<const float4*>(src + i), b = *reinterpret_cast<const float4*>(src + i + 4);
+                f[k][0] = a.x, f[k][1] = a.y, f[k][2] = a.z, f[k][3] = a.w, f[k][4] = b.x, f[k][5] = b.y, f[k][6] = b.z, f[k][7] = b.w;
+#pragma unroll
+                for (int j = 0; j < 8; ++j) g[k][j] = 0.0f, ss = fmaf(f[k][j], f[k][j], ss);
+                const T* gp = gate + t * ldg + (size_t)h * vdim + i;
+#pragma unroll
+                for (int e = 0; e < 8; e += Vec16<T>::N) {
+                    float v[Vec16<T>::N];
+                    load_vec(gp + e, v);
+#pragma unroll
+                    for (int j = 0; j < Vec16<T>::N; ++j) g[k][e + j] = v[j];
+                }
+            }
+#pragma unroll
+            for (int s = 8; s > 0; s >>= 1) ss += __shfl_xor_sync(mask, ss, s);
+            const float r = 1.0f / sqrtf(ss / (float)vdim + eps);
+#pragma unroll
+            for (int k = 0; k < 2; ++k) {
+                const int i = (lane + 16 * k) * 8;
+                if (i >= vdim) break;
+#pragma unroll
+                for (int e = 0; e < 8; e += Vec16<T>::N) {
+                    float v[Vec16<T>::N];
+#pragma unroll
+                    for (int j = 0; j < Vec16<T>::N; ++j) v[j] = f[k][e + j] * r * w[i + e + j] * silu_t<T>(g[k][e + j]);
+                    store_vec(out + t * ldo + (size_t)h * vdim + i + e, v);
+                }
+            }
+        }
+        return;
+    }
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     for (int h = warp; h < heads; h += 8) {
         const float* src = o + (t * heads + h) * vdim;
         const float f = warp_inv_rms(src, vdim, eps);
         for (int i = lane; i < vdim; i += 32)
-            out[t * ldo + (size_t)h * vdim + i] = from_f32<T>(src[i] * f * w[i] * silu_f(to_f32(gate[t * ldg + (size_t)h * vdim + i])));
+            out[t * ldo + (size_t)h * vdim + i] = from_f32<T>(src[i] * f * w[i] * silu_t<T>(to_f32(gate[t * ldg + (size_t)h * vdim + i])));
     }
 }
 

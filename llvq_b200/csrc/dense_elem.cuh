@@ -34,6 +34,15 @@ struct Vec16<bf16> {
             f[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
         }
     }
+    static __device__ __forceinline__ uint4 narrow(const float (&f)[8]) {
+        unsigned int w[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const __nv_bfloat162 v = __floats2bfloat162_rn(f[2 * i], f[2 * i + 1]);
+            w[i] = *reinterpret_cast<const unsigned int*>(&v);
+        }
+        return make_uint4(w[0], w[1], w[2], w[3]);
+    }
 };
 template <>
 struct Vec16<float> {
@@ -41,7 +50,15 @@ struct Vec16<float> {
     static __device__ __forceinline__ void widen(const uint4& u, float (&f)[4]) {
         f[0] = __uint_as_float(u.x), f[1] = __uint_as_float(u.y), f[2] = __uint_as_float(u.z), f[3] = __uint_as_float(u.w);
     }
+    static __device__ __forceinline__ uint4 narrow(const float (&f)[4]) {
+        return make_uint4(__float_as_uint(f[0]), __float_as_uint(f[1]), __float_as_uint(f[2]), __float_as_uint(f[3]));
+    }
 };
+// A vector at p (16-byte aligned), widened, and back.
+template <typename T>
+__device__ __forceinline__ void load_vec(const T* p, float (&f)[Vec16<T>::N]) { Vec16<T>::widen(*reinterpret_cast<const uint4*>(p), f); }
+template <typename T>
+__device__ __forceinline__ void store_vec(T* p, const float (&f)[Vec16<T>::N]) { *reinterpret_cast<uint4*>(p) = Vec16<T>::narrow(f); }
 
 // Sum over the CTA, the same value in every thread. `red` holds one float per warp; two barriers.
 __device__ __forceinline__ float block_sum_f(float v, float* red) {

@@ -52,6 +52,15 @@ inline size_t gqa_token_smem(int kd, int vd) {
 
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
 
+// sigmoid, silu and gelu for results that are rounded to T: in bf16 the fast exponential and division are far inside the rounding.
+template <typename T>
+__device__ __forceinline__ float sigmoid_t(float x) {
+    if constexpr (sizeof(T) == 2) return __fdividef(1.0f, 1.0f + __expf(-x));
+    return sigmoid_f(x);
+}
+template <typename T>
+__device__ __forceinline__ float silu_t(float x) { return x * sigmoid_t<T>(x); }
+
 // 1 / rms of a row by one warp, the same value in every lane.
 template <typename X>
 __device__ __forceinline__ float warp_inv_rms(const X* x, int n, float eps) {
@@ -270,46 +279,105 @@ struct GqaRowsArgs {
     long long pos0;
     int ldy, heads, kv_heads, dim, vdim;
     float eps;
+    int vec;        // heads and rows are whole 16-byte vectors on 16-byte boundaries
 };
 
-// grid = rows, 256 threads: a warp takes a head at a time.
+// out = x / rms(x) * w of n values by half a warp (lanes 0 .. 15 of it), in whole vectors.
+template <typename T>
+__device__ __forceinline__ void half_warp_norm(const T* x, const float* w, T* out, int n, float eps) {
+    constexpr int VN = Vec16<T>::N;
+    const int lane = threadIdx.x & 15;
+    const unsigned int mask = 0xffffu << (threadIdx.x & 16);
+    float ss = 0.0f, f[VN];
+    for (int i = lane * VN; i < n; i += 16 * VN) {
+        load_vec(x + i, f);
+#pragma unroll
+        for (int j = 0; j < VN; ++j) ss = fmaf(f[j], f[j], ss);
+    }
+#pragma unroll
+    for (int o = 8; o > 0; o >>= 1) ss += __shfl_xor_sync(mask, ss, o);
+    const float r = 1.0f / sqrtf(ss / (float)n + eps);
+    for (int i = lane * VN; i < n; i += 16 * VN) {
+        if (n > 16 * VN) load_vec(x + i, f);  // else it is still there
+#pragma unroll
+        for (int j = 0; j < VN; ++j) f[j] *= r * w[i + j];
+        store_vec(out + i, f);
+    }
+}
+
+// grid = rows, 256 threads: a warp takes a head at a time, or each of its halves one.
 template <typename T>
 __global__ void __launch_bounds__(256)
 gqa_rows_kernel(GqaRowsArgs A) {
     llvq_dependent_enter();
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const size_t o = (size_t)blockIdx.x * A.ldy;
     const long long pos = A.pos0 + blockIdx.x;
     T* row = reinterpret_cast<T*>(A.ring.rows) + (size_t)(pos % A.ring.slots) * A.ring.ld;
+    const T* Q = reinterpret_cast<const T*>(A.q) + o;
+    const T* K = reinterpret_cast<const T*>(A.k) + o;
+    const T* V = reinterpret_cast<const T*>(A.v) + o;
+    T* QN = reinterpret_cast<T*>(A.qn) + (size_t)blockIdx.x * A.heads * A.dim;
+    T* rv = row + (size_t)A.kv_heads * A.ring.kd;
+    if (A.vec) {
+        constexpr int VN = Vec16<T>::N;
+        const int lane = threadIdx.x & 15;
+        for (int u = threadIdx.x >> 4; u < A.heads + 2 * A.kv_heads; u += 16) {
+            if (u < A.heads) {
+                half_warp_norm(Q + (size_t)u * A.dim, A.q_norm, QN + (size_t)u * A.dim, A.dim, A.eps);
+            } else if (u < A.heads + A.kv_heads) {
+                half_warp_norm(K + (size_t)(u - A.heads) * A.dim, A.k_norm, row + (size_t)(u - A.heads) * A.ring.kd, A.dim, A.eps);
+            } else {
+                const int g = u - A.heads - A.kv_heads;
+                for (int i = lane * VN; i < A.vdim; i += 16 * VN)
+                    *reinterpret_cast<uint4*>(rv + (size_t)g * A.ring.vd + i) = *reinterpret_cast<const uint4*>(V + (size_t)g * A.vdim + i);
+            }
+        }
+        return;
+    }
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     for (int u = warp; u < A.heads + 2 * A.kv_heads; u += 8) {
         if (u < A.heads) {
-            const T* q = reinterpret_cast<const T*>(A.q) + o + (size_t)u * A.dim;
-            T* dst = reinterpret_cast<T*>(A.qn) + ((size_t)blockIdx.x * A.heads + u) * A.dim;
+            const T* q = Q + (size_t)u * A.dim;
             const float f = warp_inv_rms(q, A.dim, A.eps);
-            for (int i = lane; i < A.dim; i += 32) dst[i] = from_f32<T>(to_f32(q[i]) * f * A.q_norm[i]);
+            for (int i = lane; i < A.dim; i += 32) QN[(size_t)u * A.dim + i] = from_f32<T>(to_f32(q[i]) * f * A.q_norm[i]);
         } else if (u < A.heads + A.kv_heads) {
             const int g = u - A.heads;
-            const T* k = reinterpret_cast<const T*>(A.k) + o + (size_t)g * A.dim;
+            const T* k = K + (size_t)g * A.dim;
             const float f = warp_inv_rms(k, A.dim, A.eps);
             for (int i = lane; i < A.dim; i += 32) row[(size_t)g * A.ring.kd + i] = from_f32<T>(to_f32(k[i]) * f * A.k_norm[i]);
         } else {
             const int g = u - A.heads - A.kv_heads;
-            const T* v = reinterpret_cast<const T*>(A.v) + o + (size_t)g * A.vdim;
-            for (int i = lane; i < A.vdim; i += 32) row[(size_t)A.kv_heads * A.ring.kd + (size_t)g * A.ring.vd + i] = v[i];
+            for (int i = lane; i < A.vdim; i += 32) rv[(size_t)g * A.ring.vd + i] = V[(size_t)g * A.vdim + i];
         }
     }
 }
 
-// out[r, c] = x[r, c] * sigmoid(gate[r, c]) * scale; grid = (rows, ceil(n / 1024)).
+// out[r, c] = x[r, c] * sigmoid(gate[r, c]) * scale; grid = (rows, ceil(n / (1024, or with vec 2048))). vec: whole 16-byte
+// vectors on 16-byte boundaries.
 template <typename T>
 __global__ void __launch_bounds__(256)
-gate_rows_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ gate, int ldg, T* __restrict__ out, int ldo, int n, float scale) {
+gate_rows_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ gate, int ldg, T* __restrict__ out, int ldo, int n, float scale, int vec) {
     llvq_dependent_enter();
     const size_t r = blockIdx.x;
+    if (vec) {
+        constexpr int VN = Vec16<T>::N, K = 8 / VN;
+#pragma unroll
+        for (int k = 0; k < K; ++k) {
+            const int c = ((blockIdx.y * K + k) * 256 + threadIdx.x) * VN;
+            if (c >= n) break;
+            float f[VN], g[VN];
+            load_vec(x + r * ldx + c, f);
+            load_vec(gate + r * ldg + c, g);
+#pragma unroll
+            for (int j = 0; j < VN; ++j) f[j] *= scale * sigmoid_t<T>(g[j]);
+            store_vec(out + r * ldo + c, f);
+        }
+        return;
+    }
 #pragma unroll
     for (int k = 0; k < 4; ++k) {
         const int c = (blockIdx.y * 4 + k) * 256 + threadIdx.x;
-        if (c < n) out[r * ldo + c] = from_f32<T>(to_f32(x[r * ldx + c]) * scale * sigmoid_f(to_f32(gate[r * ldg + c])));
+        if (c < n) out[r * ldo + c] = from_f32<T>(to_f32(x[r * ldx + c]) * scale * sigmoid_t<T>(to_f32(gate[r * ldg + c])));
     }
 }
 

@@ -199,12 +199,6 @@ struct LruScanArgs {
 
 constexpr int kScanTok = 16, kScanWarps = 16, kScanCh = 16, kScanTurn = 2 * kScanTok * kScanWarps;
 
-// sigmoid and gelu for results that are rounded to T: in bf16 the fast exponential and division are far inside the rounding.
-template <typename T>
-__device__ __forceinline__ float sigmoid_t(float x) {
-    if constexpr (sizeof(T) == 2) return __fdividef(1.0f, 1.0f + __expf(-x));
-    return sigmoid_f(x);
-}
 template <typename T>
 __device__ __forceinline__ float gelu_tanh_t(float z) {
     if constexpr (sizeof(T) == 2) return z * sigmoid_t<T>(1.5957691216057308f * (z + 0.044715f * z * z * z));

@@ -2,7 +2,18 @@
 // delta rule. Included by dense_api.cu, whose helpers it uses.
 #pragma once
 
+#include <initializer_list>
+
 namespace {
+
+// Sizes are whole 16-byte vectors and pointers on 16-byte boundaries.
+int whole_vectors(int dtype, std::initializer_list<int> sizes, std::initializer_list<const void*> pointers) {
+    for (const int n : sizes)
+        if (n % (16 / elem_size(dtype))) return 0;
+    for (const void* p : pointers)
+        if ((uintptr_t)p & 15) return 0;
+    return 1;
+}
 
 GqaRing ring_of(const llvq_dn_gqa* a) { return GqaRing{a->ring, a->slots, a->ld, a->kd, a->vd}; }
 
@@ -117,7 +128,8 @@ int llvq_dn_gqa_rows(const llvq_dn_gqa* a, const void* q, const void* k, const v
     if (st) return st;
     if (!q || !k || !v || !qn || !a->q_norm || !a->k_norm || ldy <= 0 || pos0 < 0 || rows <= 0 || rows > a->slots)
         return fail(kStatusInvalid, "dn_gqa_rows: null argument, or %d rows into %d slots", rows, a->slots);
-    GqaRowsArgs p{q, k, v, qn, a->q_norm, a->k_norm, ring_of(a), pos0, ldy, a->heads, a->kv_heads, a->dim, a->vdim, a->eps};
+    GqaRowsArgs p{q, k, v, qn, a->q_norm, a->k_norm, ring_of(a), pos0, ldy, a->heads, a->kv_heads, a->dim, a->vdim, a->eps, 0};
+    p.vec = whole_vectors(a->dtype, {a->dim, a->vdim, ldy}, {q, k, v, qn});
     if (a->dtype == LLVQ_DN_BF16)
         CUDA_TRY(launch_dep(gqa_rows_kernel<bf16>, dim3(rows), dim3(256), 0, (cudaStream_t)stream, p));
     else
@@ -150,11 +162,12 @@ int llvq_dn_gqa_prefill(const llvq_dn_gqa* a, const void* qn, const void* rows, 
 int llvq_dn_gate_rows(int32_t dtype, const void* x, int32_t ldx, const void* gate, int32_t ldg, void* out, int32_t ldo, int32_t rows, int32_t n, float scale,
                       llvq_dn_stream stream) {
     if (bad_dtype(dtype) || !x || !gate || !out || rows <= 0 || n <= 0 || ldx < n || ldg < n || ldo < n) return fail(kStatusInvalid, "dn_gate_rows: bad argument");
-    const dim3 grid(rows, (n + 1023) / 1024);
+    const int vec = whole_vectors(dtype, {n, ldx, ldg, ldo}, {x, gate, out});
+    const dim3 grid(rows, vec ? (n + 2047) / 2048 : (n + 1023) / 1024);
     if (dtype == LLVQ_DN_BF16)
-        CUDA_TRY(launch_dep(gate_rows_kernel<bf16>, grid, dim3(256), 0, (cudaStream_t)stream, (const bf16*)x, ldx, (const bf16*)gate, ldg, (bf16*)out, ldo, n, scale));
+        CUDA_TRY(launch_dep(gate_rows_kernel<bf16>, grid, dim3(256), 0, (cudaStream_t)stream, (const bf16*)x, ldx, (const bf16*)gate, ldg, (bf16*)out, ldo, n, scale, vec));
     else
-        CUDA_TRY(launch_dep(gate_rows_kernel<float>, grid, dim3(256), 0, (cudaStream_t)stream, (const float*)x, ldx, (const float*)gate, ldg, (float*)out, ldo, n, scale));
+        CUDA_TRY(launch_dep(gate_rows_kernel<float>, grid, dim3(256), 0, (cudaStream_t)stream, (const float*)x, ldx, (const float*)gate, ldg, (float*)out, ldo, n, scale, vec));
     g_launches++;
     return kStatusOk;
 }
@@ -247,12 +260,13 @@ int llvq_dn_delta_rows(const llvq_dn_delta* a, const void* x, int32_t ldx, const
     g_launches++;
     int st2 = llvq_dn_conv_keep(a->dtype, x, ldx, nullptr, a->conv, channels, a->taps, pos0, rows, stream);
     if (st2) return st2;
+    const int vec = a->vdim <= 256 && a->vdim % 8 == 0 && whole_vectors(a->dtype, {a->vdim, ldg, ldo}, {gate, out, o});
     st2 = delta_scan(DeltaScanArgs{qk, v, sc, a->state, o, pos0, rows, a->heads, a->kv_heads, a->dim, a->vdim, a->vp}, s);
     if (st2) return st2;
     if (a->dtype == LLVQ_DN_BF16)
-        CUDA_TRY(launch_dep(head_gate_rows_kernel<bf16>, dim3(rows), dim3(256), 0, s, (const float*)o, a->norm, (const bf16*)gate, ldg, (bf16*)out, ldo, a->heads, a->vdim, a->eps));
+        CUDA_TRY(launch_dep(head_gate_rows_kernel<bf16>, dim3(rows), dim3(256), 0, s, (const float*)o, a->norm, (const bf16*)gate, ldg, (bf16*)out, ldo, a->heads, a->vdim, a->eps, vec));
     else
-        CUDA_TRY(launch_dep(head_gate_rows_kernel<float>, dim3(rows), dim3(256), 0, s, (const float*)o, a->norm, (const float*)gate, ldg, (float*)out, ldo, a->heads, a->vdim, a->eps));
+        CUDA_TRY(launch_dep(head_gate_rows_kernel<float>, dim3(rows), dim3(256), 0, s, (const float*)o, a->norm, (const float*)gate, ldg, (float*)out, ldo, a->heads, a->vdim, a->eps, vec));
     g_launches++;
     return kStatusOk;
 }
