@@ -219,45 +219,81 @@ __device__ __forceinline__ void delta_conv4(const DeltaPrepArgs& A, int channels
     }
 }
 
-// grid = groups, 256 threads: a warp takes a key head at a time, then all share the values.
-template <typename T>
+// The same for channels c .. c + CH - 1 (CH = 4: taps 4, dims, offsets and rows in fours, T vectors of four aligned).
+template <typename T, int CH>
+__device__ __forceinline__ void delta_conv(const DeltaPrepArgs& A, int channels, int t0, int c, float (&out)[CH][kDeltaGroup]) {
+    if constexpr (CH == 1) {
+        delta_conv4<T>(A, channels, t0, c, out[0]);
+    } else {
+        if (t0 < 3 || t0 + kDeltaGroup > A.n) {
+#pragma unroll
+            for (int j = 0; j < CH; ++j) delta_conv4<T>(A, channels, t0, c + j, out[j]);
+            return;
+        }
+        const T* p = reinterpret_cast<const T*>(A.x) + (size_t)(t0 - 3) * A.ldx + c;
+        float4 in[kDeltaGroup + 3];
+#pragma unroll
+        for (int k = 0; k < kDeltaGroup + 3; ++k) in[k] = load4(p + (size_t)k * A.ldx);
+#pragma unroll
+        for (int j = 0; j < CH; ++j) {
+            const float4 w = *reinterpret_cast<const float4*>(A.conv_w + (size_t)(c + j) * 4);
+            auto at = [&](int k) { return j == 0 ? in[k].x : j == 1 ? in[k].y : j == 2 ? in[k].z : in[k].w; };
+#pragma unroll
+            for (int i = 0; i < kDeltaGroup; ++i) out[j][i] = silu_t<T>(fmaf(w.x, at(i), fmaf(w.y, at(i + 1), fmaf(w.z, at(i + 2), w.w * at(i + 3)))));
+        }
+    }
+}
+
+// grid = groups, 256 threads: a warp takes a key head at a time, then all share the values. A thread takes CH channels.
+template <typename T, int CH>
 __global__ void __launch_bounds__(256)
 delta_prep_kernel(DeltaPrepArgs A) {
     llvq_dependent_enter();
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, t0 = blockIdx.x * kDeltaGroup, here = min(kDeltaGroup, A.n - t0);
+    constexpr int G = kDeltaGroup;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, t0 = blockIdx.x * G, here = min(G, A.n - t0);
     const int channels = 2 * A.kv_heads * A.dim + A.heads * A.vdim, rep = A.heads / A.kv_heads;
     for (int g = warp; g < A.kv_heads; g += 8) {
-        float kk[kDeltaGroup][kDeltaGroup], kq[kDeltaGroup][kDeltaGroup], qq[kDeltaGroup];  // [i][m], m <= i
+        float kk[G][G], kq[G][G], qq[G];  // [i][m], m <= i
 #pragma unroll
-        for (int i = 0; i < kDeltaGroup; ++i) {
+        for (int i = 0; i < G; ++i) {
             qq[i] = 0.0f;
 #pragma unroll
             for (int m = 0; m <= i; ++m) kk[i][m] = kq[i][m] = 0.0f;
         }
-        for (int e = lane; e < A.dp; e += 32) {
-            float q[kDeltaGroup] = {0.0f, 0.0f, 0.0f, 0.0f}, k[kDeltaGroup] = {0.0f, 0.0f, 0.0f, 0.0f};
+        for (int e = lane * CH; e < A.dp; e += 32 * CH) {
+            float q[CH][G], k[CH][G];
             if (e < A.dim) {
-                delta_conv4<T>(A, channels, t0, g * A.dim + e, q);
-                delta_conv4<T>(A, channels, t0, (A.kv_heads + g) * A.dim + e, k);
+                delta_conv<T, CH>(A, channels, t0, g * A.dim + e, q);
+                delta_conv<T, CH>(A, channels, t0, (A.kv_heads + g) * A.dim + e, k);
             }
 #pragma unroll
-            for (int i = 0; i < kDeltaGroup; ++i) {
-                if (i >= here) q[i] = k[i] = 0.0f;
-                float* dst = A.qk + ((size_t)(t0 + i) * A.kv_heads + g) * 2 * A.dp + e;
-                dst[0] = k[i];
-                dst[A.dp] = q[i];
-                qq[i] = fmaf(q[i], q[i], qq[i]);
+            for (int i = 0; i < G; ++i) {
 #pragma unroll
-                for (int m = 0; m <= i; ++m) {
-                    kk[i][m] = fmaf(k[m], k[i], kk[i][m]);
-                    kq[i][m] = fmaf(k[m], q[i], kq[i][m]);
+                for (int j = 0; j < CH; ++j)
+                    if (i >= here || e >= A.dim) q[j][i] = k[j][i] = 0.0f;
+                float* dst = A.qk + ((size_t)(t0 + i) * A.kv_heads + g) * 2 * A.dp + e;
+                if constexpr (CH == 4) {
+                    *reinterpret_cast<float4*>(dst) = make_float4(k[0][i], k[1][i], k[2][i], k[3][i]);
+                    *reinterpret_cast<float4*>(dst + A.dp) = make_float4(q[0][i], q[1][i], q[2][i], q[3][i]);
+                } else {
+                    dst[0] = k[0][i];
+                    dst[A.dp] = q[0][i];
+                }
+#pragma unroll
+                for (int j = 0; j < CH; ++j) {
+                    qq[i] = fmaf(q[j][i], q[j][i], qq[i]);
+#pragma unroll
+                    for (int m = 0; m <= i; ++m) {
+                        kk[i][m] = fmaf(k[j][m], k[j][i], kk[i][m]);
+                        kq[i][m] = fmaf(k[j][m], q[j][i], kq[i][m]);
+                    }
                 }
             }
         }
-        float fk[kDeltaGroup], fq[kDeltaGroup];
+        float fk[G], fq[G];
         const float root = 1.0f / sqrtf((float)A.dim);
 #pragma unroll
-        for (int i = 0; i < kDeltaGroup; ++i) {
+        for (int i = 0; i < G; ++i) {
 #pragma unroll
             for (int m = 0; m <= i; ++m) {
                 kk[i][m] = warp_sum_f(kk[i][m]);
@@ -268,12 +304,12 @@ delta_prep_kernel(DeltaPrepArgs A) {
         }
         for (int r = lane; r < rep; r += 32) {
             const int h = g * rep + r;
-            float sc[kDeltaScalars], lg[kDeltaGroup];
+            float sc[kDeltaScalars], lg[G];
 #pragma unroll
             for (int i = 0; i < kDeltaScalars; ++i) sc[i] = 0.0f;
             float sum = 0.0f;
 #pragma unroll
-            for (int i = 0; i < kDeltaGroup; ++i) {
+            for (int i = 0; i < G; ++i) {
                 const float* ba = A.ba + (size_t)min(t0 + i, A.n - 1) * 2 * A.heads;
                 lg[i] = i < here ? -A.decay[h] * softplus_f(ba[A.heads + h] + A.dt_bias[h]) : 0.0f;
                 sum += lg[i];
@@ -283,15 +319,15 @@ delta_prep_kernel(DeltaPrepArgs A) {
                 sc[12 + i] = fq[i];
             }
 #pragma unroll
-            for (int m = 0; m < kDeltaGroup; ++m) {
+            for (int m = 0; m < G; ++m) {
                 float from = 0.0f;  // log of the decay from token m on
 #pragma unroll
-                for (int i = m; i < kDeltaGroup; ++i) {
+                for (int i = m; i < G; ++i) {
                     if (i > m) from += lg[i];
                     const float f = i > m ? expf(from) : 1.0f;
                     sc[26 + i * (i + 1) / 2 + m] = f * kq[i][m] * fk[m] * fq[i];
                     if (i > m) sc[20 + i * (i - 1) / 2 + m] = f * kk[i][m] * fk[m] * fk[i];
-                    if (i == kDeltaGroup - 1) sc[16 + m] = f * fk[m];
+                    if (i == G - 1) sc[16 + m] = f * fk[m];
                 }
             }
             float4* dst = reinterpret_cast<float4*>(A.sc + ((size_t)blockIdx.x * A.heads + h) * kDeltaScalars);
@@ -299,12 +335,18 @@ delta_prep_kernel(DeltaPrepArgs A) {
             for (int i = 0; i < kDeltaScalars / 4; ++i) dst[i] = make_float4(sc[4 * i], sc[4 * i + 1], sc[4 * i + 2], sc[4 * i + 3]);
         }
     }
-    for (int c = threadIdx.x; c < A.heads * A.vdim; c += 256) {
-        float v[kDeltaGroup];
-        delta_conv4<T>(A, channels, t0, 2 * A.kv_heads * A.dim + c, v);
+    for (int c = threadIdx.x * CH; c < A.heads * A.vdim; c += 256 * CH) {
+        float v[CH][G];
+        delta_conv<T, CH>(A, channels, t0, 2 * A.kv_heads * A.dim + c, v);
 #pragma unroll
-        for (int i = 0; i < kDeltaGroup; ++i)
-            if (i < here) A.v[(size_t)(t0 + i) * A.heads * A.vdim + c] = v[i];
+        for (int i = 0; i < G; ++i) {
+            if (i >= here) break;
+            float* dst = A.v + (size_t)(t0 + i) * A.heads * A.vdim + c;
+            if constexpr (CH == 4)
+                *reinterpret_cast<float4*>(dst) = make_float4(v[0][i], v[1][i], v[2][i], v[3][i]);
+            else
+                dst[0] = v[0][i];
+        }
     }
 }
 
@@ -340,10 +382,17 @@ __device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
     return r;
 }
 
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+    f32x2 r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+
 constexpr int kDsCols = 4;  // columns of a thread
 
 // grid = (ceil(vdim / 32), heads), 8 * LANES threads: lane l of a group of four columns holds rows 4 (l + LANES m) .. + 3,
-// m < FOURS, of each.
+// m < FOURS, of each. A lane numbers its columns by its own two highest bits (number c is column c ^ mine), so that the
+// exchanges below always send numbers 2, 3 and then 1, and number 0 is the column whose sums end up in this lane.
 template <int LANES, int FOURS>
 __global__ void __launch_bounds__(kDtCols / kDsCols * LANES)
 delta_scan_kernel(DeltaScanArgs A) {
@@ -385,6 +434,11 @@ delta_scan_kernel(DeltaScanArgs A) {
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     stage(0, 0);
+    const int mine = l / (LANES / 4);
+    auto own_order = [&](float4 v) {
+        if (mine & 2) v = make_float4(v.z, v.w, v.x, v.y);
+        return mine & 1 ? make_float4(v.y, v.x, v.w, v.z) : v;
+    };
     f32x2 S[NC][FOURS][2];
     const size_t half = (size_t)A.heads * A.dim * A.vp, base = (size_t)h * A.dim * A.vp + c0 + cg * NC;
     const bool in = c0 + cg * NC < A.vp;  // vp is a multiple of four
@@ -397,13 +451,12 @@ delta_scan_kernel(DeltaScanArgs A) {
             const int i = 4 * (l + LANES * m) + r;
             e[r] = A.pos0 > 0 && in && i < A.dim ? *reinterpret_cast<const float4*>(S0 + (size_t)i * A.vp) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
         }
-        S[0][m][0] = pack2(e[0].x, e[1].x), S[0][m][1] = pack2(e[2].x, e[3].x);
-        S[1][m][0] = pack2(e[0].y, e[1].y), S[1][m][1] = pack2(e[2].y, e[3].y);
-        S[2][m][0] = pack2(e[0].z, e[1].z), S[2][m][1] = pack2(e[2].z, e[3].z);
-        S[3][m][0] = pack2(e[0].w, e[1].w), S[3][m][1] = pack2(e[2].w, e[3].w);
+        const float4 f[4] = {own_order(e[0]), own_order(e[1]), own_order(e[2]), own_order(e[3])};
+        S[0][m][0] = pack2(f[0].x, f[1].x), S[0][m][1] = pack2(f[2].x, f[3].x);
+        S[1][m][0] = pack2(f[0].y, f[1].y), S[1][m][1] = pack2(f[2].y, f[3].y);
+        S[2][m][0] = pack2(f[0].z, f[1].z), S[2][m][1] = pack2(f[2].z, f[3].z);
+        S[3][m][0] = pack2(f[0].w, f[1].w), S[3][m][1] = pack2(f[2].w, f[3].w);
     }
-    const bool hi = l & (LANES / 2), hi2 = l & (LANES / 4);
-    const int mine = (hi ? 2 : 0) + (hi2 ? 1 : 0);  // the column whose sums end up in this lane
     for (int t0 = 0, buf = 0; t0 < A.n; t0 += TT, buf ^= 1) {
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();  // the tile is staged, the outputs before are stored and the other buffer is read
@@ -423,16 +476,14 @@ delta_scan_kernel(DeltaScanArgs A) {
             for (int i = 0; i < G; ++i) {
                 f32x2 ak[NC], aq[NC];
 #pragma unroll
-                for (int c = 0; c < NC; ++c) ak[c] = aq[c] = 0ull;
-#pragma unroll
                 for (int m = 0; m < FOURS; ++m) {
                     const ulonglong2 kk = *reinterpret_cast<const ulonglong2*>(kr + (size_t)i * 2 * dp + 4 * LANES * m);
                     const ulonglong2 qq = *reinterpret_cast<const ulonglong2*>(kr + (size_t)i * 2 * dp + dp + 4 * LANES * m);
                     k[i][m][0] = kk.x, k[i][m][1] = kk.y;
 #pragma unroll
                     for (int c = 0; c < NC; ++c) {
-                        ak[c] = fma2(S[c][m][0], kk.x, ak[c]);
-                        aq[c] = fma2(S[c][m][0], qq.x, aq[c]);
+                        ak[c] = m ? fma2(S[c][m][0], kk.x, ak[c]) : mul2(S[c][m][0], kk.x);
+                        aq[c] = m ? fma2(S[c][m][0], qq.x, aq[c]) : mul2(S[c][m][0], qq.x);
                         ak[c] = fma2(S[c][m][1], kk.y, ak[c]);
                         aq[c] = fma2(S[c][m][1], qq.y, aq[c]);
                     }
@@ -449,11 +500,10 @@ delta_scan_kernel(DeltaScanArgs A) {
 #pragma unroll
             for (int e = 0; e < 2 * G; ++e)
 #pragma unroll
-                for (int c = 0; c < 2; ++c)
-                    two[c][e] = (hi ? val[2 + c][e] : val[c][e]) + __shfl_xor_sync(0xffffffffu, hi ? val[c][e] : val[2 + c][e], LANES / 2);
+                for (int c = 0; c < 2; ++c) two[c][e] = val[c][e] + __shfl_xor_sync(0xffffffffu, val[2 + c][e], LANES / 2);
 #pragma unroll
             for (int e = 0; e < 2 * G; ++e) {
-                s[e] = (hi2 ? two[1][e] : two[0][e]) + __shfl_xor_sync(0xffffffffu, hi2 ? two[0][e] : two[1][e], LANES / 4);
+                s[e] = two[0][e] + __shfl_xor_sync(0xffffffffu, two[1][e], LANES / 4);
 #pragma unroll
                 for (int o = LANES / 8; o > 0; o >>= 1) s[e] += __shfl_xor_sync(0xffffffffu, s[e], o);
             }
@@ -475,10 +525,10 @@ delta_scan_kernel(DeltaScanArgs A) {
             if (l % (LANES / 4) < G) o_s[(t + (l & 3)) * kDtCols + cg * NC + mine] = out;
 #pragma unroll
             for (int i = 0; i < G; ++i) {
-                const float own = u[i] * sc[16 + i], next = __shfl_xor_sync(0xffffffffu, own, LANES / 4);
-                const float a = hi2 ? next : own, b = hi2 ? own : next;
-                const float c = __shfl_xor_sync(0xffffffffu, a, LANES / 2), d = __shfl_xor_sync(0xffffffffu, b, LANES / 2);
-                w[0][i] = hi ? c : a, w[1][i] = hi ? d : b, w[2][i] = hi ? a : c, w[3][i] = hi ? b : d;
+                w[0][i] = u[i] * sc[16 + i];
+                w[1][i] = __shfl_xor_sync(0xffffffffu, w[0][i], LANES / 4);
+                w[2][i] = __shfl_xor_sync(0xffffffffu, w[0][i], LANES / 2);
+                w[3][i] = __shfl_xor_sync(0xffffffffu, w[1][i], LANES / 2);
             }
             const f32x2 g2 = pack2(sc[7], sc[7]);
 #pragma unroll
@@ -511,8 +561,8 @@ delta_scan_kernel(DeltaScanArgs A) {
         for (int p = 0; p < 2; ++p) {
             const float2 a = unpack2(S[0][m][p]), b = unpack2(S[1][m][p]), c = unpack2(S[2][m][p]), d = unpack2(S[3][m][p]);
             const int i = 4 * (l + LANES * m) + 2 * p;
-            if (i < A.dim) *reinterpret_cast<float4*>(Sn + (size_t)i * A.vp) = make_float4(a.x, b.x, c.x, d.x);
-            if (i + 1 < A.dim) *reinterpret_cast<float4*>(Sn + (size_t)(i + 1) * A.vp) = make_float4(a.y, b.y, c.y, d.y);
+            if (i < A.dim) *reinterpret_cast<float4*>(Sn + (size_t)i * A.vp) = own_order(make_float4(a.x, b.x, c.x, d.x));
+            if (i + 1 < A.dim) *reinterpret_cast<float4*>(Sn + (size_t)(i + 1) * A.vp) = own_order(make_float4(a.y, b.y, c.y, d.y));
         }
 }
 

@@ -60,6 +60,26 @@ __device__ __forceinline__ void load_vec(const T* p, float (&f)[Vec16<T>::N]) { 
 template <typename T>
 __device__ __forceinline__ void store_vec(T* p, const float (&f)[Vec16<T>::N]) { *reinterpret_cast<uint4*>(p) = Vec16<T>::narrow(f); }
 
+// Four consecutive values as f32 and back.
+template <typename T>
+__device__ __forceinline__ float4 load4(const T* p) {
+    if constexpr (sizeof(T) == 4) {
+        return *reinterpret_cast<const float4*>(p);
+    } else {
+        const uint2 u = *reinterpret_cast<const uint2*>(p);
+        return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xffff0000u));
+    }
+}
+template <typename T>
+__device__ __forceinline__ void store4(T* p, float4 v) {
+    if constexpr (sizeof(T) == 4) {
+        *reinterpret_cast<float4*>(p) = v;
+    } else {
+        __align__(16) const T r[4] = {from_f32<T>(v.x), from_f32<T>(v.y), from_f32<T>(v.z), from_f32<T>(v.w)};
+        *reinterpret_cast<uint2*>(p) = *reinterpret_cast<const uint2*>(r);
+    }
+}
+
 // Sum over the CTA, the same value in every thread. `red` holds one float per warp; two barriers.
 __device__ __forceinline__ float block_sum_f(float v, float* red) {
     v = warp_sum_f(v);

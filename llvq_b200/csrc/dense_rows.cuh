@@ -30,26 +30,6 @@ embed_rows_kernel(const T* __restrict__ table, int ld, int table_rows, const lon
     }
 }
 
-// Four consecutive values as f32 and back.
-template <typename T>
-__device__ __forceinline__ float4 load4(const T* p) {
-    if constexpr (sizeof(T) == 4) {
-        return *reinterpret_cast<const float4*>(p);
-    } else {
-        const uint2 u = *reinterpret_cast<const uint2*>(p);
-        return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xffff0000u));
-    }
-}
-template <typename T>
-__device__ __forceinline__ void store4(T* p, float4 v) {
-    if constexpr (sizeof(T) == 4) {
-        *reinterpret_cast<float4*>(p) = v;
-    } else {
-        __align__(16) const T r[4] = {from_f32<T>(v.x), from_f32<T>(v.y), from_f32<T>(v.z), from_f32<T>(v.w)};
-        *reinterpret_cast<uint2*>(p) = *reinterpret_cast<const uint2*>(r);
-    }
-}
-
 // Dynamic shared memory: n floats. out may be x: a CTA has read its row before it writes; y may be null (alpha = 1: a
 // plain norm). vec: n % 4 == 0 and every row on a 16-byte boundary.
 template <typename T>

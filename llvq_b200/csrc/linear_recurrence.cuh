@@ -14,8 +14,8 @@
 //   lru_token            the token step: a CTA takes 32 channels of a block: the block's u, two rows of the gate matrix
 //                        per channel, the recurrence, the gate branch.
 //   conv_rows_kernel     u of a prompt portion; conv_keep_kernel then stores the inputs the next step reads.
-//   lru_scan_kernel      the recurrence of a portion, one pass: a CTA owns 16 channels, a thread 16 tokens at a time in
-//                        registers; their products and sums meet in shared memory, 512 tokens a turn.
+//   lru_scan_kernel      the recurrence of a portion, one pass: a CTA owns 16 channels, a thread 8 tokens at a time in
+//                        registers; their products and sums meet in shared memory, 256 tokens a turn.
 #pragma once
 #include "gqa_attn.cuh"
 
@@ -197,7 +197,7 @@ struct LruScanArgs {
     float out_scale;
 };
 
-constexpr int kScanTok = 16, kScanWarps = 16, kScanCh = 16, kScanTurn = 2 * kScanTok * kScanWarps;
+constexpr int kScanTok = 8, kScanWarps = 16, kScanCh = 16, kScanTurn = 2 * kScanTok * kScanWarps;
 
 template <typename T>
 __device__ __forceinline__ float gelu_tanh_t(float z) {
@@ -205,11 +205,11 @@ __device__ __forceinline__ float gelu_tanh_t(float z) {
     return gelu_tanh_f(z);
 }
 
-// grid = ceil(width / 16), 512 threads: a warp's halves take 16 channels over 16 tokens each, a turn is 512 tokens.
+// grid = ceil(width / 16), 512 threads: a warp's halves take 16 channels over 8 tokens each, a turn is 256 tokens.
 template <typename T>
-__global__ void __launch_bounds__(kScanWarps * 32)
+__global__ void __launch_bounds__(kScanWarps * 32, 2)
 lru_scan_kernel(LruScanArgs A) {
-    __shared__ float2 part_s[2][kScanWarps][kScanCh];  // decay product and sum of a warp's 32 tokens; two turns' worth
+    __shared__ float2 part_s[2][kScanWarps][kScanCh];  // decay product and sum of a warp's 16 tokens; two turns' worth
     llvq_dependent_enter();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, width = A.blocks * A.n, lc = lane & (kScanCh - 1), upper = lane / kScanCh;
     const int ch = blockIdx.x * kScanCh + lc, cc = min(ch, width - 1), blk = cc / A.n, c = cc - blk * A.n;

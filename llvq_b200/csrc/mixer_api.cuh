@@ -253,10 +253,11 @@ int llvq_dn_delta_rows(const llvq_dn_delta* a, const void* x, int32_t ldx, const
     float* o = v + (size_t)rows * hv;
     DeltaPrepArgs p{x, ba, a->conv_w, a->conv, a->decay, a->dt_bias, qk, v, sc, pos0, rows, ldx, a->heads, a->kv_heads, a->dim, a->vdim, a->taps, dp};
     if (a->taps == 4 && ((uintptr_t)a->conv_w & 15)) return fail(kStatusInvalid, "dn_delta_rows: convolution weights not on 16 bytes");
-    if (a->dtype == LLVQ_DN_BF16)
-        CUDA_TRY(launch_dep(delta_prep_kernel<bf16>, dim3(delta_groups(rows)), dim3(256), 0, s, p));
-    else
-        CUDA_TRY(launch_dep(delta_prep_kernel<float>, dim3(delta_groups(rows)), dim3(256), 0, s, p));
+    const int elem = elem_size(a->dtype);
+    const bool fours = a->taps == 4 && !((a->dim | a->vdim | ldx) & 3) && !((uintptr_t)x & (4 * elem - 1));
+    const auto prep = a->dtype == LLVQ_DN_BF16 ? (fours ? delta_prep_kernel<bf16, 4> : delta_prep_kernel<bf16, 1>)
+                                                : (fours ? delta_prep_kernel<float, 4> : delta_prep_kernel<float, 1>);
+    CUDA_TRY(launch_dep(prep, dim3(delta_groups(rows)), dim3(256), 0, s, p));
     g_launches++;
     int st2 = llvq_dn_conv_keep(a->dtype, x, ldx, nullptr, a->conv, channels, a->taps, pos0, rows, stream);
     if (st2) return st2;
