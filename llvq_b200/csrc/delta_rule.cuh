@@ -388,15 +388,14 @@ __device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
     return r;
 }
 
-constexpr int kDsCols = 4;  // columns of a thread
-
-// grid = (ceil(vdim / 32), heads), 8 * LANES threads: lane l of a group of four columns holds rows 4 (l + LANES m) .. + 3,
-// m < FOURS, of each. A lane numbers its columns by its own two highest bits (number c is column c ^ mine), so that the
-// exchanges below always send numbers 2, 3 and then 1, and number 0 is the column whose sums end up in this lane.
-template <int LANES, int FOURS>
-__global__ void __launch_bounds__(kDtCols / kDsCols * LANES)
+// grid = (ceil(vdim / 32), heads), 32 / NC * LANES threads: lane l of a group of NC (4 or 2) columns holds rows
+// 4 (l + LANES m) .. + 3, m < FOURS, of each. A lane numbers its columns by its own highest bits (number c is column
+// c ^ mine), so that the exchanges below always send the upper numbers, and number 0 is the column whose sums end up in
+// this lane.
+template <int LANES, int FOURS, int NC>
+__global__ void __launch_bounds__(kDtCols / NC * LANES)
 delta_scan_kernel(DeltaScanArgs A) {
-    constexpr int kThreads = kDtCols / kDsCols * LANES, dp = 4 * LANES * FOURS, G = kDeltaGroup, NC = kDsCols;
+    constexpr int kThreads = kDtCols / NC * LANES, dp = 4 * LANES * FOURS, G = kDeltaGroup;
     extern __shared__ __align__(16) float ds_smem[];
     const int TT = delta_tile(A.dim), tid = threadIdx.x, l = tid % LANES, cg = tid / LANES;
     const int h = blockIdx.y, g = h / (A.heads / A.kv_heads), c0 = blockIdx.x * kDtCols, cols = min(kDtCols, A.vdim - c0);
@@ -434,28 +433,24 @@ delta_scan_kernel(DeltaScanArgs A) {
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     stage(0, 0);
-    const int mine = l / (LANES / 4);
-    auto own_order = [&](float4 v) {
-        if (mine & 2) v = make_float4(v.z, v.w, v.x, v.y);
-        return mine & 1 ? make_float4(v.y, v.x, v.w, v.z) : v;
-    };
+    const int mine = l / (LANES / NC);
     f32x2 S[NC][FOURS][2];
     const size_t half = (size_t)A.heads * A.dim * A.vp, base = (size_t)h * A.dim * A.vp + c0 + cg * NC;
     const bool in = c0 + cg * NC < A.vp;  // vp is a multiple of four
     const float* S0 = A.state + (A.pos0 & 1) * half + base;
 #pragma unroll
     for (int m = 0; m < FOURS; ++m) {
-        float4 e[4];
 #pragma unroll
-        for (int r = 0; r < 4; ++r) {
-            const int i = 4 * (l + LANES * m) + r;
-            e[r] = A.pos0 > 0 && in && i < A.dim ? *reinterpret_cast<const float4*>(S0 + (size_t)i * A.vp) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        for (int c = 0; c < NC; ++c) {
+            float e[4];
+#pragma unroll
+            for (int r = 0; r < 4; ++r) {
+                const int i = 4 * (l + LANES * m) + r;
+                e[r] = A.pos0 > 0 && in && i < A.dim ? S0[(size_t)i * A.vp + (c ^ mine)] : 0.0f;
+            }
+            S[c][m][0] = pack2(e[0], e[1]);
+            S[c][m][1] = pack2(e[2], e[3]);
         }
-        const float4 f[4] = {own_order(e[0]), own_order(e[1]), own_order(e[2]), own_order(e[3])};
-        S[0][m][0] = pack2(f[0].x, f[1].x), S[0][m][1] = pack2(f[2].x, f[3].x);
-        S[1][m][0] = pack2(f[0].y, f[1].y), S[1][m][1] = pack2(f[2].y, f[3].y);
-        S[2][m][0] = pack2(f[0].z, f[1].z), S[2][m][1] = pack2(f[2].z, f[3].z);
-        S[3][m][0] = pack2(f[0].w, f[1].w), S[3][m][1] = pack2(f[2].w, f[3].w);
     }
     for (int t0 = 0, buf = 0; t0 < A.n; t0 += TT, buf ^= 1) {
         asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -495,18 +490,24 @@ delta_scan_kernel(DeltaScanArgs A) {
                     val[c][G + i] = b.x + b.y;
                 }
             }
-            // the sums over dim: two exchanges leave a column to a lane, the rest adds up among the lanes that share it
-            float two[2][2 * G], s[2 * G];
+            // the sums over dim: exchanges leave a column to a lane, the rest adds up among the lanes that share it
+            float s[2 * G];
+            if constexpr (NC == 4) {
+                float two[2][2 * G];
 #pragma unroll
-            for (int e = 0; e < 2 * G; ++e)
+                for (int e = 0; e < 2 * G; ++e)
 #pragma unroll
-                for (int c = 0; c < 2; ++c) two[c][e] = val[c][e] + __shfl_xor_sync(0xffffffffu, val[2 + c][e], LANES / 2);
+                    for (int c = 0; c < 2; ++c) two[c][e] = val[c][e] + __shfl_xor_sync(0xffffffffu, val[2 + c][e], LANES / 2);
 #pragma unroll
-            for (int e = 0; e < 2 * G; ++e) {
-                s[e] = two[0][e] + __shfl_xor_sync(0xffffffffu, two[1][e], LANES / 4);
+                for (int e = 0; e < 2 * G; ++e) s[e] = two[0][e] + __shfl_xor_sync(0xffffffffu, two[1][e], LANES / 4);
+            } else {
 #pragma unroll
-                for (int o = LANES / 8; o > 0; o >>= 1) s[e] += __shfl_xor_sync(0xffffffffu, s[e], o);
+                for (int e = 0; e < 2 * G; ++e) s[e] = val[0][e] + __shfl_xor_sync(0xffffffffu, val[1][e], LANES / 2);
             }
+#pragma unroll
+            for (int o = LANES / (2 * NC); o > 0; o >>= 1)
+#pragma unroll
+                for (int e = 0; e < 2 * G; ++e) s[e] += __shfl_xor_sync(0xffffffffu, s[e], o);
             float u[G], w[NC][G], out = 0.0f;
 #pragma unroll
             for (int i = 0; i < G; ++i) {
@@ -522,13 +523,15 @@ delta_scan_kernel(DeltaScanArgs A) {
                 y = fmaf(sc[26 + i * (i + 1) / 2 + i], u[i], y);
                 if ((l & 3) == i) out = y;
             }
-            if (l % (LANES / 4) < G) o_s[(t + (l & 3)) * kDtCols + cg * NC + mine] = out;
+            if (l % (LANES / NC) < G) o_s[(t + (l & 3)) * kDtCols + cg * NC + mine] = out;
 #pragma unroll
             for (int i = 0; i < G; ++i) {
                 w[0][i] = u[i] * sc[16 + i];
-                w[1][i] = __shfl_xor_sync(0xffffffffu, w[0][i], LANES / 4);
-                w[2][i] = __shfl_xor_sync(0xffffffffu, w[0][i], LANES / 2);
-                w[3][i] = __shfl_xor_sync(0xffffffffu, w[1][i], LANES / 2);
+                w[1][i] = __shfl_xor_sync(0xffffffffu, w[0][i], LANES / NC);
+                if constexpr (NC == 4) {
+                    w[2][i] = __shfl_xor_sync(0xffffffffu, w[0][i], LANES / 2);
+                    w[3][i] = __shfl_xor_sync(0xffffffffu, w[1][i], LANES / 2);
+                }
             }
             const f32x2 g2 = pack2(sc[7], sc[7]);
 #pragma unroll
@@ -558,12 +561,14 @@ delta_scan_kernel(DeltaScanArgs A) {
 #pragma unroll
     for (int m = 0; m < FOURS; ++m)
 #pragma unroll
-        for (int p = 0; p < 2; ++p) {
-            const float2 a = unpack2(S[0][m][p]), b = unpack2(S[1][m][p]), c = unpack2(S[2][m][p]), d = unpack2(S[3][m][p]);
-            const int i = 4 * (l + LANES * m) + 2 * p;
-            if (i < A.dim) *reinterpret_cast<float4*>(Sn + (size_t)i * A.vp) = own_order(make_float4(a.x, b.x, c.x, d.x));
-            if (i + 1 < A.dim) *reinterpret_cast<float4*>(Sn + (size_t)(i + 1) * A.vp) = own_order(make_float4(a.y, b.y, c.y, d.y));
-        }
+        for (int p = 0; p < 2; ++p)
+#pragma unroll
+            for (int c = 0; c < NC; ++c) {
+                const float2 a = unpack2(S[c][m][p]);
+                const int i = 4 * (l + LANES * m) + 2 * p;
+                if (i < A.dim) Sn[(size_t)i * A.vp + (c ^ mine)] = a.x;
+                if (i + 1 < A.dim) Sn[(size_t)(i + 1) * A.vp + (c ^ mine)] = a.y;
+            }
 }
 
 // out[t, h, :] = o / sqrt(mean(o^2) + eps) * w * silu(gate); grid = rows, 256 threads: a warp takes a head at a time, or (vec:

@@ -71,12 +71,12 @@ int mixer_token_t(const llvq_dn_gqa* a, const llvq_dn_lru* r, const int64_t* pos
     return kStatusOk;
 }
 
-template <int LANES, int FOURS>
+template <int LANES, int FOURS, int NC>
 int delta_scan_t(const DeltaScanArgs& k, cudaStream_t s) {
     const size_t smem = delta_scan_smem(k.dim);
-    const int st = ensure_dyn_smem((const void*)delta_scan_kernel<LANES, FOURS>, smem);
+    const int st = ensure_dyn_smem((const void*)delta_scan_kernel<LANES, FOURS, NC>, smem);
     if (st) return st;
-    CUDA_TRY(launch_dep(delta_scan_kernel<LANES, FOURS>, dim3((k.vdim + kDtCols - 1) / kDtCols, k.heads), dim3(kDtCols / kDsCols * LANES), smem, s, k));
+    CUDA_TRY(launch_dep(delta_scan_kernel<LANES, FOURS, NC>, dim3((k.vdim + kDtCols - 1) / kDtCols, k.heads), dim3(kDtCols / NC * LANES), smem, s, k));
     g_launches++;
     return kStatusOk;
 }
@@ -84,18 +84,18 @@ int delta_scan_t(const DeltaScanArgs& k, cudaStream_t s) {
 int delta_scan(const DeltaScanArgs& k, cudaStream_t s) {
     const int fours = delta_fours(k.dim);
     if (delta_lanes(k.dim) == 16) switch (fours) {
-        case 1: return delta_scan_t<16, 1>(k, s);
-        case 2: return delta_scan_t<16, 2>(k, s);
-        case 3: return delta_scan_t<16, 3>(k, s);
-        default: return delta_scan_t<16, 4>(k, s);
+        case 1: return delta_scan_t<16, 1, 4>(k, s);
+        case 2: return delta_scan_t<16, 2, 4>(k, s);
+        case 3: return delta_scan_t<16, 3, 4>(k, s);
+        default: return delta_scan_t<16, 4, 4>(k, s);
     }
     switch (fours) {
-        case 3: return delta_scan_t<32, 3>(k, s);
-        case 4: return delta_scan_t<32, 4>(k, s);
-        case 5: return delta_scan_t<32, 5>(k, s);
-        case 6: return delta_scan_t<32, 6>(k, s);
-        case 7: return delta_scan_t<32, 7>(k, s);
-        case 8: return delta_scan_t<32, 8>(k, s);
+        case 3: return delta_scan_t<32, 3, 4>(k, s);
+        case 4: return delta_scan_t<32, 4, 4>(k, s);
+        case 5: return delta_scan_t<32, 5, 4>(k, s);
+        case 6: return delta_scan_t<32, 6, 4>(k, s);
+        case 7: return delta_scan_t<32, 7, 4>(k, s);
+        case 8: return delta_scan_t<32, 8, 4>(k, s);
         default: return fail(kStatusUnsupported, "dn_delta_rows: keys of %d (at most 1024)", k.dim);
     }
 }
