@@ -1,8 +1,7 @@
 """Small random models of the hybrid design for the tests: sizes that are not multiples of anything, layers that differ
 from one another, loops, windows of one, one tap, one head, several experts per token, no feed-forward."""
-import torch
-
 from latent_cases import write_folder  # noqa: F401
+from oracle.hybrid_lm import random_model  # noqa: F401
 
 
 def attention(heads, kv_heads, dim, vdim, window, scale=None):
@@ -61,65 +60,3 @@ LARGE = config(256, 300, [
 ], loop={"start": 2, "stop": 3, "times": 3})
 
 ALL = {"uneven": UNEVEN, "even": EVEN, "large": LARGE}
-
-
-def random_model(cfg, seed=0):
-    """Seeded bf16 weights (tables int32): fan-in scaled matrices, norm weights, biases and decays away from neutral
-    values, so that leaving one out shows; decays slow enough that far tokens count."""
-    g = torch.Generator().manual_seed(seed)
-    D, w = cfg["width"], {}
-
-    def mat(name, *shape, gain=1.0):
-        w[name] = (torch.randn(*shape, generator=g) * (gain / shape[-1] ** 0.5)).bfloat16()
-
-    def vec(name, *shape, mean=0.0, std=0.3):
-        w[name] = (mean + std * torch.randn(*shape, generator=g)).bfloat16()
-
-    mat("embed", cfg["vocab"], D, gain=D ** 0.5)
-    mat("head", cfg["vocab"], D)
-    vec("final.norm", D, mean=1.0)
-    for i, layer in enumerate(cfg["layers"]):
-        mx, p, mlp = layer["mixer"], f"l{i}.mix", layer.get("mlp")
-        vec(f"l{i}.norm1", D, mean=1.0)
-        if layer["type"] == "delta":
-            H, G, dim, vdim, taps = mx["heads"], mx["kv_heads"], mx["dim"], mx["vdim"], mx["conv"]
-            for name, n in (("q", G * dim), ("k", G * dim), ("v", H * vdim)):
-                mat(f"{p}.{name}", n, D)
-                mat(f"{p}.{name}.conv", n, taps, gain=1.5)
-            mat(p + ".b", H, D)
-            mat(p + ".a", H, D)
-            vec(p + ".A_log", H, mean=-2.0, std=1.0)
-            vec(p + ".dt_bias", H, mean=-1.0, std=1.0)
-            vec(p + ".norm", vdim, mean=1.0)
-            mat(p + ".g", H * vdim, D)
-            mat(p + ".o", D, H * vdim, gain=2.0)
-        else:
-            a, r = mx["left"], mx["right"]
-            for name, n in (("q", a["heads"] * a["dim"]), ("k", a["kv_heads"] * a["dim"]), ("v", a["kv_heads"] * a["vdim"]), ("g", a["heads"] * a["vdim"])):
-                mat(f"{p}.left.{name}", n, D)
-            vec(p + ".left.q.norm", a["dim"], mean=1.0)
-            vec(p + ".left.k.norm", a["dim"], mean=1.0)
-            mat(p + ".left.o", D, a["heads"] * a["vdim"], gain=2.0)
-            W, B = r["width"], r["blocks"]
-            for name in ("y", "x"):
-                mat(f"{p}.right.{name}", W, D)
-                vec(f"{p}.right.{name}.b", W)
-            mat(p + ".right.conv", W, r["conv"], gain=1.5)
-            vec(p + ".right.conv.b", W)
-            for name in ("ra", "ri"):
-                mat(f"{p}.right.{name}", B, W // B, W // B)
-                vec(f"{p}.right.{name}.b", B, W // B)
-            vec(p + ".right.lam", W, mean=-4.0, std=1.5)
-            mat(p + ".right.o", D, W, gain=2.0)
-        if mlp is None:
-            continue
-        vec(f"l{i}.norm2", D, mean=1.0)
-        units = [(f"l{i}.mlp", mlp["ff"])] if mlp["kind"] == "dense" else [(f"l{i}.mlp.e{e}", mlp["expert"]["ff"]) for e in range(mlp["router"]["experts"])]
-        for m, ff in units:
-            mat(m + ".gate", ff, D, gain=1.5)
-            mat(m + ".up", ff, D, gain=1.5)
-            mat(m + ".down", D, ff, gain=1.5)
-        if mlp["kind"] == "moe":
-            E, top = mlp["router"]["experts"], mlp["router"]["top"]
-            w[f"l{i}.mlp.table"] = torch.stack([torch.randperm(E, generator=g)[:top] for _ in range(cfg["vocab"])]).int()
-    return w
