@@ -186,6 +186,11 @@ int llvq_dn_conv_keep(int32_t dtype, const void* x, int32_t ldx, const float* x_
 int llvq_dn_lru_rows(const llvq_dn_lru* a, const void* u, const float* z, const void* y, int32_t ldy, const float* y_bias, void* out, int32_t ldo, int64_t pos0,
                      int32_t rows, llvq_dn_stream stream);
 
+/* A portion's rows by expert: table [table_rows, top] names each token's. Place i of the sorted list (by expert, then by row) belongs to
+ * row source[i]; places[row * top + j] is where choice j of a row sits; ends[e] is the end of expert e's places. */
+int llvq_dn_route_rows(const int32_t* table, int32_t table_rows, int32_t top, int32_t experts, const int64_t* tokens, int32_t rows, int32_t* source,
+                       int32_t* places, int32_t* ends, llvq_dn_stream stream);
+
 /* ---- gated delta rule ---- */
 typedef struct {
     int32_t dtype;

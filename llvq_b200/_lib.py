@@ -187,6 +187,7 @@ _DENSE_SIGNATURES = {
     "llvq_dn_conv_rows": (C.c_int, [C.c_int32, C.c_void_p, C.c_int32] + [C.c_void_p] * 5 + [C.c_int32] * 2 + [C.c_int64, C.c_int32, C.c_void_p]),
     "llvq_dn_conv_keep": (C.c_int, [C.c_int32, C.c_void_p, C.c_int32] + [C.c_void_p] * 2 + [C.c_int32] * 2 + [C.c_int64, C.c_int32, C.c_void_p]),
     "llvq_dn_lru_rows": (C.c_int, [C.POINTER(DenseLru)] + [C.c_void_p] * 3 + [C.c_int32, C.c_void_p, C.c_void_p, C.c_int32, C.c_int64, C.c_int32, C.c_void_p]),
+    "llvq_dn_route_rows": (C.c_int, [C.c_void_p] + [C.c_int32] * 3 + [C.c_void_p, C.c_int32] + [C.c_void_p] * 4),
     "llvq_dn_delta_token": (C.c_int, [C.POINTER(DenseDelta)] + [C.c_void_p] * 2),
     "llvq_dn_delta_scratch": (C.c_int, [C.POINTER(DenseDelta), C.c_int32, C.POINTER(C.c_size_t)]),
     "llvq_dn_delta_rows": (C.c_int, [C.POINTER(DenseDelta), C.c_void_p, C.c_int32, C.c_void_p, C.c_void_p, C.c_int32, C.c_void_p, C.c_void_p, C.c_int32, C.c_int64,

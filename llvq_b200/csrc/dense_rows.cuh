@@ -5,6 +5,7 @@
 //   latent_rows_kernel  the down projections of a latent-attention layer: the query latent normed into cq, the
 //                       token's cache row normed, rotated and stored into the ring
 //   add_norms_rows_kernel  x += y (+ the token's rows of a routed product); two norms of the sum for two sublayers
+//   route_rows_kernel   a portion's rows sorted by the expert their tokens name
 //   glu_rows_kernel     clamped gated unit of (gate, up) pairs with their biases
 //   softcap_kernel      logits <- cap * tanh(logits / cap)
 #pragma once
@@ -155,6 +156,60 @@ add_norms_rows_kernel(AddNormsArgs A) {
         } else {
             for (int i = threadIdx.x; i < A.n; i += kRowThreads) h[o + i] = from_f32<T>(row_s[i] * r * w[i]);
         }
+    }
+}
+
+constexpr int kRouteThreads = 1024;
+
+// One CTA. Counts, ends, then a warp per expert walks all choices in order and hands out the expert's places. Dynamic shared
+// memory: experts + 1 ints.
+__global__ void __launch_bounds__(kRouteThreads)
+route_rows_kernel(const int* __restrict__ table, int table_rows, int top, int experts, const long long* __restrict__ tokens, int rows,
+                  int* __restrict__ source, int* places, int* __restrict__ ends) {
+    extern __shared__ int start_s[];
+    llvq_dependent_enter();
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, n = rows * top;
+    for (int e = tid; e <= experts; e += kRouteThreads) start_s[e] = 0;
+    __syncthreads();
+    for (int i = tid; i < n; i += kRouteThreads) {
+        const int r = i / top;
+        long long t = tokens[r];
+        if (t < 0 || t >= table_rows) t = 0;
+        const int e = min(max(table[t * top + (i - r * top)], 0), experts - 1);
+        places[i] = e;  // the expert for now
+        atomicAdd(start_s + e + 1, 1);
+    }
+    __syncthreads();
+    if (warp == 0) {
+        int sum = 0;
+        for (int lo = 0; lo < experts; lo += 32) {
+            int c = lo + lane < experts ? start_s[lo + lane + 1] : 0;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const int v = __shfl_up_sync(0xffffffffu, c, o);
+                if (lane >= o) c += v;
+            }
+            if (lo + lane < experts) ends[lo + lane] = start_s[lo + lane + 1] = sum + c;
+            sum += __shfl_sync(0xffffffffu, c, 31);
+        }
+    }
+    __syncthreads();
+    for (int e = warp; e < experts; e += kRouteThreads / 32) {
+        int at = start_s[e];
+        const int end = start_s[e + 1];
+        for (int lo = 0; lo < n && at < end; lo += 32) {
+            const int i = lo + lane;
+            const bool mine = i < n && places[i] == e;
+            const unsigned int votes = __ballot_sync(0xffffffffu, mine);
+            if (mine) source[at + __popc(votes & ((1u << lane) - 1u))] = i;
+            at += __popc(votes);
+        }
+    }
+    __syncthreads();
+    for (int p = tid; p < n; p += kRouteThreads) {
+        const int i = source[p];
+        places[i] = p;
+        source[p] = i / top;
     }
 }
 

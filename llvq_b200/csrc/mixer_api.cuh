@@ -73,10 +73,13 @@ int mixer_token_t(const llvq_dn_gqa* a, const llvq_dn_lru* r, const int64_t* pos
 
 template <int LANES, int FOURS, int NC>
 int delta_scan_t(const DeltaScanArgs& k, cudaStream_t s) {
-    const size_t smem = delta_scan_smem(k.dim);
+    const dim3 grid((k.vdim + kDtCols - 1) / kDtCols, k.heads);
+    // A CTA is bound by its own chain of tokens: two on one SM slow each other down. Where every CTA can have an SM, it
+    // asks for more than half of the shared memory (CTAs launched into the tail of the kernel before would pile up).
+    const size_t smem = std::max(delta_scan_smem(k.dim), (int)(grid.x * grid.y) <= sm_count() ? kMaxSmem / 2 + 1024 : 0);
     const int st = ensure_dyn_smem((const void*)delta_scan_kernel<LANES, FOURS, NC>, smem);
     if (st) return st;
-    CUDA_TRY(launch_dep(delta_scan_kernel<LANES, FOURS, NC>, dim3((k.vdim + kDtCols - 1) / kDtCols, k.heads), dim3(kDtCols / NC * LANES), smem, s, k));
+    CUDA_TRY(launch_dep(delta_scan_kernel<LANES, FOURS, NC>, grid, dim3(kDtCols / NC * LANES), smem, s, k));
     g_launches++;
     return kStatusOk;
 }
@@ -210,6 +213,18 @@ int llvq_dn_lru_rows(const llvq_dn_lru* a, const void* u, const float* z, const 
         CUDA_TRY(launch_dep(lru_scan_kernel<bf16>, dim3((width + kScanCh - 1) / kScanCh), dim3(kScanWarps * 32), 0, (cudaStream_t)stream, k));
     else
         CUDA_TRY(launch_dep(lru_scan_kernel<float>, dim3((width + kScanCh - 1) / kScanCh), dim3(kScanWarps * 32), 0, (cudaStream_t)stream, k));
+    g_launches++;
+    return kStatusOk;
+}
+
+int llvq_dn_route_rows(const int32_t* table, int32_t table_rows, int32_t top, int32_t experts, const int64_t* tokens, int32_t rows, int32_t* source,
+                       int32_t* places, int32_t* ends, llvq_dn_stream stream) {
+    if (!table || !tokens || !source || !places || !ends || table_rows <= 0 || top <= 0 || experts <= 0 || rows <= 0 || (long long)rows * top > INT32_MAX)
+        return fail(kStatusInvalid, "dn_route_rows: bad argument");
+    const size_t smem = ((size_t)experts + 1) * sizeof(int);
+    if (smem > 40 * 1024) return fail(kStatusUnsupported, "dn_route_rows: %d experts", experts);
+    CUDA_TRY(launch_dep(route_rows_kernel, dim3(1), dim3(kRouteThreads), smem, (cudaStream_t)stream, table, table_rows, top, experts, (const long long*)tokens, rows,
+                        source, places, ends));
     g_launches++;
     return kStatusOk;
 }

@@ -164,26 +164,18 @@ class HybridConfig:
 class _Route:
     """Which rows of a portion go to which expert: rows sorted by expert, where each row's results end up."""
 
-    def __init__(self, table, tokens):
+    def __init__(self, lib, table, experts: int, tokens, stream):
         import torch
-        self.top = table.shape[1]
-        ids = table[tokens.clamp(0, table.shape[0] - 1)].flatten()
-        experts, order = torch.sort(ids, stable=True)
-        self.source = order // self.top                       # the row behind each sorted place
-        self.places = torch.empty_like(ids)
-        self.places[order] = torch.arange(ids.numel(), dtype=ids.dtype, device=ids.device)
-        self._experts, self._ends, self._host = experts, None, None
+        n, self.top = tokens.numel(), table.shape[1]
+        new = lambda k: torch.empty(k, dtype=torch.int32, device=table.device)
+        self.source, self.places, self.ends = new(n * self.top), new(n * self.top), new(experts)
+        _lib.check_dense(lib.llvq_dn_route_rows(table.data_ptr(), table.shape[0], self.top, experts, tokens.data_ptr(), n, self.source.data_ptr(),
+                                                self.places.data_ptr(), self.ends.data_ptr(), stream))
+        self._host = None
 
-    def ends(self, experts: int):
-        """End of each expert's rows, on the device."""
-        import torch
-        if self._ends is None:
-            self._ends = torch.searchsorted(self._experts, torch.arange(experts, dtype=self._experts.dtype, device=self._experts.device), right=True).int()
-        return self._ends
-
-    def host_ends(self, experts: int) -> List[int]:
+    def host_ends(self) -> List[int]:
         if self._host is None:
-            self._host = self.ends(experts).tolist()
+            self._host = self.ends.tolist()
         return self._host
 
 
@@ -400,14 +392,14 @@ class HybridLM(DenseLM):
         self._steps = steps
 
     # ---- prompt portions ---------------------------------------------------------
-    def _grouped(self, x, stack, route: _Route, experts: int):
+    def _grouped(self, x, stack, route: _Route):
         """Rows of x, sorted by expert, through their expert's matrix [experts, out, in]."""
         import torch
         if self.dtype == torch.bfloat16 and not (stack.shape[1] | stack.shape[2]) & 7:
-            return torch._grouped_mm(x, stack.transpose(1, 2), offs=route.ends(experts))
+            return torch._grouped_mm(x, stack.transpose(1, 2), offs=route.ends)
         y = torch.empty(x.shape[0], stack.shape[1], dtype=x.dtype, device=x.device)
         lo = 0
-        for e, hi in enumerate(route.host_ends(experts)):
+        for e, hi in enumerate(route.host_ends()):
             if hi > lo:
                 y[lo:hi] = self._mm(x[lo:hi], stack[e])
             lo = hi
@@ -485,12 +477,12 @@ class HybridLM(DenseLM):
                                                                                 scale, st))
             if mlp is not None and mlp.experts:
                 if i not in routes:
-                    routes[i] = _Route(L["table"], tokens)
+                    routes[i] = _Route(lib, L["table"], mlp.experts, tokens, st)
                 route, ff = routes[i], L["experts_down"].shape[2]
-                gu = self._grouped(h2[route.source], L["experts_up"][:, :, :D], route, mlp.experts)
+                gu = self._grouped(h2.index_select(0, route.source), L["experts_up"][:, :, :D], route)
                 e = new(gu.shape[0], ff)
                 gated(gu, e.data_ptr(), ff, ff, 1.0 / mlp.top)
-                routed, places, top = self._grouped(e, L["experts_down"], route, mlp.experts), route.places, mlp.top
+                routed, places, top = self._grouped(e, L["experts_down"], route), route.places, mlp.top
             elif mlp is not None:
                 gu = self._mm(h2, L["gate_up"].rows(0))
                 if L["down"] is None:

@@ -71,19 +71,6 @@ def test_matrices_side_by_side_are_one_product():
         ColumnMatrix([torch.randn(5, 3), torch.randn(4, 3)], torch.float32, "cpu")
 
 
-def test_route_sorts_rows_by_expert_and_finds_them_again():
-    from llvq_b200.hybrid import _Route
-    table = torch.tensor([[2, 0], [1, 2], [0, 3]], dtype=torch.int32)
-    toks = torch.tensor([1, 1, 0, 2, 0, 7])          # an id outside the table reads its last row
-    r = _Route(table, toks)
-    assert r.host_ends(5) == [4, 6, 10, 12, 12]
-    lo = 0
-    for e, hi in enumerate(r.host_ends(5)):
-        assert sorted(r.source[lo:hi].tolist()) == [i for i, t in enumerate(toks.clamp(max=2)) if e in table[t]]
-        lo = hi
-    assert torch.equal(r.source[r.places.long()].reshape(6, 2), torch.arange(6)[:, None].expand(6, 2))
-
-
 def test_key_value_rows_and_their_transposed_values():
     from llvq_b200.cache import KvRing
     r = KvRing(50, 7, 5, 2, 3, 5, torch.bfloat16, "cpu")
@@ -121,6 +108,7 @@ def test_bad_arguments_are_refused_without_a_gpu():
     assert L.llvq_dn_delta_token(C.byref(e), 16, None) == bad
     assert L.llvq_dn_conv_rows(_lib.DN_F32, 16, 3, None, 16, None, 16, 16, 4, 4, 0, 1, None) == bad
     assert L.llvq_dn_gated_rows(_lib.DN_F32, 16, None, 16, 3, 1, 4, 1.0, 1.0, 0.0, 1.0, None) == bad
+    assert L.llvq_dn_route_rows(16, 5, 0, 3, 16, 4, 16, 16, 16, None) == bad
     assert L.llvq_dn_add_norms_rows(_lib.DN_F32, 16, None, None, None, 0, 16, None, None, None, 1e-5, 1, 4, None) == bad
 
 

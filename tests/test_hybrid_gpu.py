@@ -145,6 +145,26 @@ def test_row_kernels(dtype, n):
     assert rel(act[:, :n], 1.5 * y.double() * torch.sigmoid(gu.double()[:, :n])) < tol and bool((act[:, n:] == 7.0).all())
 
 
+@pytest.mark.parametrize("vocab,experts,top,n", [(3, 4, 2, 6), (50, 1, 1, 33), (200, 70, 5, 700), (90, 256, 8, 2048), (7, 9, 9, 31)])
+def test_route_sorts_rows_by_expert_and_finds_them_again(vocab, experts, top, n):
+    from llvq_b200.hybrid import _Route
+    _, L = lib()
+    table = torch.stack([torch.randperm(experts, generator=gen(r))[:top] for r in range(vocab)]).int()
+    toks = torch.randint(0, vocab, (n,), generator=gen(1))
+    toks[n // 2] = vocab + 5                         # an id outside the table reads its first row
+    r = _Route(L, table.cuda(), experts, toks.cuda(), stream())
+    named = table[torch.where(toks < vocab, toks, 0)]
+    source, lo = r.source.cpu().long(), 0
+    for e, hi in enumerate(r.host_ends()):
+        assert source[lo:hi].tolist() == (named == e).any(1).nonzero()[:, 0].tolist()
+        lo = hi
+    assert lo == n * top
+    places = r.places.cpu().long().reshape(n, top)
+    assert torch.equal(source[places], torch.arange(n)[:, None].expand(n, top))
+    expert_of = torch.searchsorted(torch.tensor(r.host_ends()), places, right=True)
+    assert torch.equal(expert_of, named.long())
+
+
 # ---- windowed grouped-query attention ------------------------------------------------
 class Attention:
     """One layer's operands: raw queries, keys, values and output gates of n positions, and the descriptor."""
