@@ -48,7 +48,7 @@ inline size_t delta_token_smem(int dim) { return (size_t)2 * dim * sizeof(float)
 __global__ void __launch_bounds__(kDtThreads)
 delta_token_kernel(DeltaArgs A) {
     extern __shared__ __align__(16) float dt_smem[];
-    __shared__ float red[8], col_s[8][2][kDtCols], u_s[kDtCols];
+    __shared__ float red[8], red3[8][3], col_s[8][2][kDtCols], u_s[kDtCols];
     __shared__ int last_s;
     float* q_s = dt_smem;
     float* k_s = dt_smem + A.dim;
@@ -68,24 +68,35 @@ delta_token_kernel(DeltaArgs A) {
     for (int k = 0; k < kDtKeep; ++k) keep[k] = load(rg + 32 * k);
 
     // ---- the token's query, key and value ----
+    const int conv_row = (int)((unsigned int)pos % (unsigned int)A.taps), j = c0 + tid, cv = 2 * A.kv_heads * A.dim + h * A.vdim + j;
+    const bool own_col = tid < kDtCols && j < A.vdim;
+    float xv = 0.0f, v = 0.0f;
+    if (own_col) {
+        xv = A.x[cv];
+        v = silu_f(conv_token(A.conv_w + (size_t)cv * A.taps, A.taps, A.conv, channels, cv, pos, conv_row, xv));
+        A.conv[(size_t)conv_row * channels + cv] = xv;
+    }
     const bool owner = blockIdx.x == 0 && h == g * (A.heads / A.kv_heads);  // stores the inputs of the shared q and k
     float qq = 0.0f, kk = 0.0f, kq = 0.0f;
     for (int i = tid; i < A.dim; i += kDtThreads) {
         const int cq = g * A.dim + i, ck = (A.kv_heads + g) * A.dim + i;
         const float xq = A.x[cq], xk = A.x[ck];
-        const float q = silu_f(conv_token(A.conv_w + (size_t)cq * A.taps, A.taps, A.conv, channels, cq, pos, xq));
-        const float k = silu_f(conv_token(A.conv_w + (size_t)ck * A.taps, A.taps, A.conv, channels, ck, pos, xk));
+        const float q = silu_f(conv_token(A.conv_w + (size_t)cq * A.taps, A.taps, A.conv, channels, cq, pos, conv_row, xq));
+        const float k = silu_f(conv_token(A.conv_w + (size_t)ck * A.taps, A.taps, A.conv, channels, ck, pos, conv_row, xk));
         if (owner) {
-            A.conv[(size_t)(pos % A.taps) * channels + cq] = xq;
-            A.conv[(size_t)(pos % A.taps) * channels + ck] = xk;
+            A.conv[(size_t)conv_row * channels + cq] = xq;
+            A.conv[(size_t)conv_row * channels + ck] = xk;
         }
         q_s[i] = q;
         k_s[i] = k;
         qq = fmaf(q, q, qq), kk = fmaf(k, k, kk), kq = fmaf(k, q, kq);
     }
-    qq = block_sum_f(qq, red);  // also publishes q_s and k_s
-    kk = block_sum_f(kk, red);
-    kq = block_sum_f(kq, red);
+    qq = warp_sum_f(qq), kk = warp_sum_f(kk), kq = warp_sum_f(kq);
+    if (lane == 0) red3[warp][0] = qq, red3[warp][1] = kk, red3[warp][2] = kq;
+    __syncthreads();  // q_s and k_s are there as well
+    qq = kk = kq = 0.0f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) qq += red3[w][0], kk += red3[w][1], kq += red3[w][2];
     const float fq = 1.0f / sqrtf(qq + kUnitEps) / sqrtf((float)A.dim), fk = 1.0f / sqrtf(kk + kUnitEps);
     const float dec = expm1f(-A.decay[h] * softplus_f(A.a[h] + A.dt_bias[h]));  // g - 1
 
@@ -108,19 +119,11 @@ delta_token_kernel(DeltaArgs A) {
         if (lane < 8) col_s[warp][e >> 2][j4 + (e & 3)] = v8[e];
     }
     __syncthreads();
-    if (tid < kDtCols && c0 + tid < A.vp) {
-        const int j = c0 + tid;
+    if (tid < kDtCols && j < A.vp) {
         float tk = 0.0f, tq = 0.0f;
 #pragma unroll
         for (int w = 0; w < 8; ++w) tk += col_s[w][0][tid], tq += col_s[w][1][tid];
-        float u = 0.0f;
-        if (j < A.vdim) {
-            const int cv = 2 * A.kv_heads * A.dim + h * A.vdim + j;
-            const float xv = A.x[cv];
-            const float v = silu_f(conv_token(A.conv_w + (size_t)cv * A.taps, A.taps, A.conv, channels, cv, pos, xv));
-            A.conv[(size_t)(pos % A.taps) * channels + cv] = xv;
-            u = sigmoid_f(A.b[h]) * (v - fk * carry(dec, tk, 0.0f));
-        }
+        const float u = own_col ? sigmoid_f(A.b[h]) * (v - fk * carry(dec, tk, 0.0f)) : 0.0f;
         u_s[tid] = u * fk;  // the key is scaled where it is used
         A.o[(size_t)h * A.vp + j] = fq * (carry(dec, tq, 0.0f) + kq * fk * u);
     }

@@ -47,7 +47,7 @@ inline int gqa_ctas(int heads, int kv_heads, int splits) { return kv_heads * gqa
 template <typename T>
 inline size_t gqa_token_smem(int kd, int vd) {
     return (size_t)kGqHeads * kd * 4 + (size_t)(kd + vd) * sizeof(T) + (size_t)4 * kGqHeads * kGqTile * 4 + (size_t)kGqHeads * kGqTile * 4 +
-           (size_t)kGqHeads * kGqMaxSplits * 4 + (size_t)kGqThreads * Vec16<T>::N * 4 + 64;
+           (size_t)kGqHeads * kGqMaxSplits * 4 + (size_t)kGqHeads * kGqThreads * Vec16<T>::N * 4 + 64;
 }
 
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
@@ -79,8 +79,8 @@ __device__ __forceinline__ void gqa_token(const GqaArgs& A, int cta, unsigned ch
     __shared__ float corr_s[kGqHeads], inv_s[kGqHeads];
     __shared__ int last_s;
     const int kd = A.ring.kd, vd = A.ring.vd, kvecs = kd / VN, vvecs = vd / VN;
-    float* red = reinterpret_cast<float*>(smem);                                 // [256][VN]
-    float* q_s = red + kGqThreads * VN;                                          // [4][kd]
+    float* red = reinterpret_cast<float*>(smem);                                 // [rows][4][values], at most 4 * 256 * VN
+    float* q_s = red + kGqHeads * kGqThreads * VN;                               // [4][kd]
     T* k_new = reinterpret_cast<T*>(q_s + kGqHeads * kd);                        // [kd]
     T* v_new = k_new + kd;                                                       // [vd]
     float* s_s = reinterpret_cast<float*>(v_new + vd);                           // [quarter][4][64]
@@ -96,8 +96,9 @@ __device__ __forceinline__ void gqa_token(const GqaArgs& A, int cta, unsigned ch
     per = (per + kGqTile - 1) / kGqTile * kGqTile;
     const int t0 = split * per, t1 = min(n, t0 + per);
     const bool own = t0 < n && t1 == n;  // this split holds the token itself
-    const int slot0 = (int)((pos - n + 1) % A.ring.slots);  // n <= slots: at most one wrap below
-    T* row_new = reinterpret_cast<T*>(A.ring.rows) + (size_t)(pos % A.ring.slots) * A.ring.ld;
+    const int slot_new = (int)((unsigned int)pos % (unsigned int)A.ring.slots);
+    const int slot0 = slot_new - n + 1 + (slot_new < n - 1 ? A.ring.slots : 0);  // n <= slots: at most one wrap below
+    T* row_new = reinterpret_cast<T*>(A.ring.rows) + (size_t)slot_new * A.ring.ld;
 
     if (warp < nh && t0 < t1) {
         const float* q = A.q + (size_t)(head0 + warp) * A.dim;
@@ -214,18 +215,28 @@ __device__ __forceinline__ void gqa_token(const GqaArgs& A, int cta, unsigned ch
         ml[0] = m;  // -inf for a split beyond the visible positions
         ml[1] = l;
     }
-    for (int h = 0; h < nh && t0 < t1; ++h) {
-        __syncthreads();
+    if (t0 < t1) {
+        // the position groups' sums: those of a warp by shuffles, then the warps' (or, of values wider than a warp, the groups')
+        for (int o = vl; o < 32; o *= 2)
 #pragma unroll
-        for (int k = 0; k < kGqHeads; ++k)
-            if (k == h) {
+            for (int h = 0; h < kGqHeads; ++h)
 #pragma unroll
-                for (int j = 0; j < VN; ++j) red[(grp * vl + vi) * VN + j] = acc[k][j];
-            }
+                for (int j = 0; j < VN; ++j) acc[h][j] += __shfl_xor_sync(0xffffffffu, acc[h][j], o);
+        const int row = vl < 32 ? warp : grp, rows = vl < 32 ? kGqThreads / 32 : grps, width = vl * VN;
+        if (vl >= 32 || lane < vl) {
+#pragma unroll
+            for (int h = 0; h < kGqHeads; ++h)
+#pragma unroll
+                for (int j = 0; j < VN; j += 4)
+                    *reinterpret_cast<float4*>(red + ((size_t)row * kGqHeads + h) * width + vi * VN + j) =
+                        make_float4(acc[h][j], acc[h][j + 1], acc[h][j + 2], acc[h][j + 3]);
+        }
         __syncthreads();
-        for (int d = tid; d < A.vdim; d += kGqThreads) {
+        for (int e = tid; e < nh * width; e += kGqThreads) {
+            const int h = e / width, d = e - h * width;
+            if (d >= A.vdim) continue;
             float o = 0.0f;
-            for (int k = 0; k < grps; ++k) o += red[k * vl * VN + d];
+            for (int k = 0; k < rows; ++k) o += red[((size_t)k * kGqHeads + h) * width + d];
             A.part_o[((size_t)(head0 + h) * A.splits + split) * A.vdim + d] = o;
         }
     }

@@ -30,11 +30,19 @@ __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.0f) + l
 constexpr float kLruDecay = 8.0f;  // c
 constexpr int kLruRows = 32;       // channels of a CTA
 
-// Convolution of one channel at `pos` over inputs kept in a ring of `taps` rows; x is the token's own input.
-__device__ __forceinline__ float conv_token(const float* w, int taps, const float* ring, int channels, int ch, long long pos, float x) {
+// Convolution of one channel at position `pos`, whose input's row in the ring of `taps` rows is `row`; x is the token's own
+// input.
+__device__ __forceinline__ float conv_token(const float* w, int taps, const float* ring, int channels, int ch, long long pos, int row, float x) {
+    if (taps == 4 && pos >= 3) {
+        const int r1 = (row + 3) & 3, r2 = (row + 2) & 3, r3 = (row + 1) & 3;
+        const float x1 = ring[(size_t)r1 * channels + ch], x2 = ring[(size_t)r2 * channels + ch], x3 = ring[(size_t)r3 * channels + ch];
+        return fmaf(w[0], x3, fmaf(w[1], x2, fmaf(w[2], x1, w[3] * x)));
+    }
     float u = w[taps - 1] * x;
-    for (int k = 1; k < taps; ++k)
-        if (pos >= k) u = fmaf(w[taps - 1 - k], ring[(size_t)((pos - k) % taps) * channels + ch], u);
+    for (int k = 1; k < taps; ++k) {
+        const int r = row - k + (row < k ? taps : 0);
+        if (pos >= k) u = fmaf(w[taps - 1 - k], ring[(size_t)r * channels + ch], u);
+    }
     return u;
 }
 
@@ -78,9 +86,10 @@ __device__ __forceinline__ void lru_token(const LruArgs& A, int cta, float* u_s)
     }
     llvq_dependent_enter();
     const long long pos = *A.pos;
+    const int conv_row = (int)((unsigned int)pos % (unsigned int)A.taps);
     for (int c = tid; c < A.ldw; c += 256) {
         const int ch = blk * A.n + c;
-        u_s[c] = c < A.n ? A.conv_b[ch] + conv_token(A.conv_w + (size_t)ch * A.taps, A.taps, A.conv, width, ch, pos, A.x[ch]) : 0.0f;
+        u_s[c] = c < A.n ? A.conv_b[ch] + conv_token(A.conv_w + (size_t)ch * A.taps, A.taps, A.conv, width, ch, pos, conv_row, A.x[ch]) : 0.0f;
     }
     __syncthreads();
     if (c0 >= A.n) return;
@@ -112,7 +121,7 @@ __device__ __forceinline__ void lru_token(const LruArgs& A, int cta, float* u_s)
         const float s = pos > 0 ? A.state[(size_t)(pos & 1) * width + ch] : 0.0f;
         const float d = lru_decay(r, A.lam[ch]), t = carry(d, s, lru_input(d, i, u_s[c]));
         A.state[(size_t)((pos + 1) & 1) * width + ch] = t;
-        A.conv[(size_t)(pos % A.taps) * width + ch] = A.x[ch];
+        A.conv[(size_t)conv_row * width + ch] = A.x[ch];
         A.out[ch] = t * gelu_tanh_f(A.y[ch]) * A.out_scale;
     }
 }
