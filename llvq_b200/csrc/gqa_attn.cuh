@@ -43,11 +43,20 @@ struct GqaArgs {
 
 __host__ __device__ inline int gqa_chunks(int heads, int kv_heads) { return (heads / kv_heads + kGqHeads - 1) / kGqHeads; }
 inline int gqa_ctas(int heads, int kv_heads, int splits) { return kv_heads * gqa_chunks(heads, kv_heads) * splits; }
-// Shared memory of one CTA: queries, the token's own key and value, quarter scores, weights, split factors, sums.
+// Shared memory of one CTA: queries, quarter scores, weights, split factors, and the tile of keys and values, whose place the
+// sums take afterwards. A tile has fewer than 64 positions where the rows are long.
+template <typename T>
+__host__ __device__ inline int gqa_key_pitch(int kd) { return kd + (kd / Vec16<T>::N % 2 ? 0 : Vec16<T>::N); }  // an odd number of vectors
+template <typename T>
+__host__ __device__ inline int gqa_tile(int kd, int vd) {
+    int tile = kGqTile;
+    while (tile > 8 && (size_t)tile * (gqa_key_pitch<T>(kd) + vd) * sizeof(T) > 96 * 1024) tile /= 2;
+    return tile;
+}
 template <typename T>
 inline size_t gqa_token_smem(int kd, int vd) {
-    return (size_t)kGqHeads * kd * 4 + (size_t)(kd + vd) * sizeof(T) + (size_t)4 * kGqHeads * kGqTile * 4 + (size_t)kGqHeads * kGqTile * 4 +
-           (size_t)kGqHeads * kGqMaxSplits * 4 + (size_t)kGqHeads * kGqThreads * Vec16<T>::N * 4 + 64;
+    const size_t tile = (size_t)gqa_tile<T>(kd, vd) * (gqa_key_pitch<T>(kd) + vd) * sizeof(T), sums = (size_t)kGqHeads * kGqThreads * Vec16<T>::N * 4;
+    return (tile > sums ? tile : sums) + (size_t)kGqHeads * kd * 4 + (size_t)5 * kGqHeads * kGqTile * 4 + (size_t)kGqHeads * kGqMaxSplits * 4 + 64;
 }
 
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
@@ -78,14 +87,14 @@ __device__ __forceinline__ void gqa_token(const GqaArgs& A, int cta, unsigned ch
     constexpr int VN = Vec16<T>::N;
     __shared__ float corr_s[kGqHeads], inv_s[kGqHeads];
     __shared__ int last_s;
-    const int kd = A.ring.kd, vd = A.ring.vd, kvecs = kd / VN, vvecs = vd / VN;
-    float* red = reinterpret_cast<float*>(smem);                                 // [rows][4][values], at most 4 * 256 * VN
-    float* q_s = red + kGqHeads * kGqThreads * VN;                               // [4][kd]
-    T* k_new = reinterpret_cast<T*>(q_s + kGqHeads * kd);                        // [kd]
-    T* v_new = k_new + kd;                                                       // [vd]
-    float* s_s = reinterpret_cast<float*>(v_new + vd);                           // [quarter][4][64]
+    const int kd = A.ring.kd, vd = A.ring.vd, kvecs = kd / VN, vvecs = vd / VN, kp = gqa_key_pitch<T>(kd), tile = gqa_tile<T>(kd, vd);
+    float* q_s = reinterpret_cast<float*>(smem);                                 // [4][kd]
+    float* s_s = q_s + kGqHeads * kd;                                            // [quarter][4][64]
     float* p_s = s_s + 4 * kGqHeads * kGqTile;                                   // [4][64]
     float* f_s = p_s + kGqHeads * kGqTile;                                       // [4][splits]
+    T* k_s = reinterpret_cast<T*>(f_s + kGqHeads * kGqMaxSplits);                // [tile][kp]
+    T* v_s = k_s + (size_t)tile * kp;                                            // [tile][vd]
+    float* red = reinterpret_cast<float*>(k_s);                                  // [rows][4][values], at most 4 * 256 * VN
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int unit = cta / A.splits, split = cta - unit * A.splits, chunks = gqa_chunks(A.heads, A.kv_heads);
     const int g = unit / chunks, chunk = unit - g * chunks, rep = A.heads / A.kv_heads;
@@ -93,12 +102,36 @@ __device__ __forceinline__ void gqa_token(const GqaArgs& A, int cta, unsigned ch
     const long long pos = *A.pos;
     const int n = (int)min((long long)A.window, pos + 1);  // visible positions pos - n + 1 .. pos
     int per = (n + A.splits - 1) / A.splits;
-    per = (per + kGqTile - 1) / kGqTile * kGqTile;
+    per = (per + tile - 1) / tile * tile;
     const int t0 = split * per, t1 = min(n, t0 + per);
     const bool own = t0 < n && t1 == n;  // this split holds the token itself
     const int slot_new = (int)((unsigned int)pos % (unsigned int)A.ring.slots);
     const int slot0 = slot_new - n + 1 + (slot_new < n - 1 ? A.ring.slots : 0);  // n <= slots: at most one wrap below
     T* row_new = reinterpret_cast<T*>(A.ring.rows) + (size_t)slot_new * A.ring.ld;
+
+    // positions base .. of this split into the tile, the token's own row aside
+    auto stage = [&](int base) {
+        const int here = min(tile, t1 - base), per_row = kvecs + vvecs;
+        int r = tid / per_row, c = tid - r * per_row;
+        const int dr = kGqThreads / per_row, dc = kGqThreads - dr * per_row;
+#pragma unroll 1
+        while (r < here) {
+            int slot = slot0 + base + r;
+            if (slot >= A.ring.slots) slot -= A.ring.slots;
+            const T* src = reinterpret_cast<const T*>(A.ring.rows) + (size_t)slot * A.ring.ld;
+            src += c < kvecs ? (size_t)g * kd + c * VN : (size_t)A.kv_heads * kd + (size_t)g * vd + (c - kvecs) * VN;
+            T* dst = c < kvecs ? k_s + (size_t)r * kp + c * VN : v_s + (size_t)r * vd + (c - kvecs) * VN;
+            if (base + r != n - 1)
+                asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((unsigned int)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+            c += dc;
+            r += dr;
+            if (c >= per_row) c -= per_row, ++r;
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    if (t0 < t1) stage(t0);
+    T* k_new = k_s + (size_t)(max(n - 1 - t0, 0) % tile) * kp;  // the token's own place, where this split holds it
+    T* v_new = v_s + (size_t)(max(n - 1 - t0, 0) % tile) * vd;
 
     if (warp < nh && t0 < t1) {
         const float* q = A.q + (size_t)(head0 + warp) * A.dim;
@@ -106,46 +139,48 @@ __device__ __forceinline__ void gqa_token(const GqaArgs& A, int cta, unsigned ch
         for (int i = lane; i < kd; i += 32) q_s[warp * kd + i] = i < A.dim ? q[i] * f * A.q_norm[i] : 0.0f;
     } else if (warp < kGqHeads) {
         for (int i = lane; i < kd; i += 32) q_s[warp * kd + i] = 0.0f;
-    } else if (own && warp == kGqHeads) {
-        const float* k = A.k + (size_t)g * A.dim;
-        const float f = warp_inv_rms(k, A.dim, A.eps);
-        for (int i = lane; i < kd; i += 32) {
-            const T t = from_f32<T>(i < A.dim ? k[i] * f * A.k_norm[i] : 0.0f);
-            k_new[i] = t;
-            if (chunk == 0) row_new[(size_t)g * kd + i] = t;
-        }
-    } else if (own && warp == kGqHeads + 1) {
-        const float* v = A.v + (size_t)g * A.vdim;
-        for (int i = lane; i < vd; i += 32) {
-            const T t = from_f32<T>(i < A.vdim ? v[i] : 0.0f);
-            v_new[i] = t;
-            if (chunk == 0) row_new[(size_t)A.kv_heads * kd + (size_t)g * vd + i] = t;
-        }
     }
-    __syncthreads();
+    // its normed key and its value: stored once per group, and kept by every CTA whose split ends with it
+    auto own_row = [&]() {
+        if (warp == kGqHeads) {
+            const float* k = A.k + (size_t)g * A.dim;
+            const float f = warp_inv_rms(k, A.dim, A.eps);
+            for (int i = lane; i < kd; i += 32) {
+                const T t = from_f32<T>(i < A.dim ? k[i] * f * A.k_norm[i] : 0.0f);
+                k_new[i] = t;
+                if (chunk == 0) row_new[(size_t)g * kd + i] = t;
+            }
+        } else if (warp == kGqHeads + 1) {
+            const float* v = A.v + (size_t)g * A.vdim;
+            for (int i = lane; i < vd; i += 32) {
+                const T t = from_f32<T>(i < A.vdim ? v[i] : 0.0f);
+                v_new[i] = t;
+                if (chunk == 0) row_new[(size_t)A.kv_heads * kd + (size_t)g * vd + i] = t;
+            }
+        }
+    };
+    int vl = 1;  // threads along the value vectors
+    while (vl < vvecs) vl *= 2;
+    const int vi = tid & (vl - 1), grp = tid / vl, grps = kGqThreads / vl;
 
     float m = -INFINITY, l = 0.0f;  // of head `warp`, in warps below nh
-    int vl = 1;                     // threads along the value vectors
-    while (vl < vvecs) vl *= 2;
-    const int vi = tid % vl, grp = tid / vl, grps = kGqThreads / vl;
     float acc[kGqHeads][VN];
 #pragma unroll
     for (int h = 0; h < kGqHeads; ++h)
 #pragma unroll
         for (int j = 0; j < VN; ++j) acc[h][j] = 0.0f;
-    auto row_at = [&](int idx) {
-        int slot = slot0 + idx;
-        if (slot >= A.ring.slots) slot -= A.ring.slots;
-        return reinterpret_cast<const T*>(A.ring.rows) + (size_t)slot * A.ring.ld;
-    };
-    for (int base = t0; base < t1; base += kGqTile) {
-        const int here = min(kGqTile, t1 - base);
+#pragma unroll 1
+    for (int base = t0; base < t1; base += tile) {
+        const int here = min(tile, t1 - base);
+        if (own && base + here == n) own_row();
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();
         {  // scores: thread = (position, quarter of the key's vectors)
-            const int p = tid & (kGqTile - 1), quarter = tid / kGqTile, idx = base + p;
+            const int p = tid & (kGqTile - 1), quarter = tid / kGqTile;
             float s[kGqHeads] = {0.0f, 0.0f, 0.0f, 0.0f};
             if (p < here) {
-                const uint4* kr = reinterpret_cast<const uint4*>(idx == n - 1 ? k_new : row_at(idx) + (size_t)g * kd);
-#pragma unroll 4
+                const uint4* kr = reinterpret_cast<const uint4*>(k_s + (size_t)p * kp);
+#pragma unroll 1
                 for (int c = quarter; c < kvecs; c += 4) {
                     float f[VN];
                     Vec16<T>::widen(kr[c], f);
@@ -165,7 +200,7 @@ __device__ __forceinline__ void gqa_token(const GqaArgs& A, int cta, unsigned ch
             for (int h = 0; h < kGqHeads; ++h) s_s[(quarter * kGqHeads + h) * kGqTile + p] = s[h];
         }
         __syncthreads();
-        if (warp < nh) {
+        if (warp < kGqHeads) {
             float s[2];
 #pragma unroll
             for (int k = 0; k < 2; ++k) {
@@ -184,23 +219,19 @@ __device__ __forceinline__ void gqa_token(const GqaArgs& A, int cta, unsigned ch
             p_s[warp * kGqTile + lane] = e0;
             p_s[warp * kGqTile + lane + 32] = e1;
             if (lane == 0) corr_s[warp] = corr;
-        } else if (warp < kGqHeads) {
-            p_s[warp * kGqTile + lane] = 0.0f;
-            p_s[warp * kGqTile + lane + 32] = 0.0f;
-            if (lane == 0) corr_s[warp] = 1.0f;
         }
         __syncthreads();
+        if (base > t0) {
 #pragma unroll
-        for (int h = 0; h < kGqHeads; ++h)
+            for (int h = 0; h < kGqHeads; ++h)
 #pragma unroll
-            for (int j = 0; j < VN; ++j) acc[h][j] *= corr_s[h];
+                for (int j = 0; j < VN; ++j) acc[h][j] *= corr_s[h];
+        }
         if (vi < vvecs) {
-#pragma unroll 4
+#pragma unroll 1
             for (int p = grp; p < here; p += grps) {
-                const int idx = base + p;
-                const T* vr = idx == n - 1 ? v_new : row_at(idx) + (size_t)A.kv_heads * kd + (size_t)g * vd;
                 float f[VN];
-                Vec16<T>::widen(reinterpret_cast<const uint4*>(vr)[vi], f);
+                Vec16<T>::widen(reinterpret_cast<const uint4*>(v_s + (size_t)p * vd)[vi], f);
 #pragma unroll
                 for (int h = 0; h < kGqHeads; ++h) {
                     const float w = p_s[h * kGqTile + p];
@@ -209,6 +240,8 @@ __device__ __forceinline__ void gqa_token(const GqaArgs& A, int cta, unsigned ch
                 }
             }
         }
+        __syncthreads();  // the tile is read
+        if (base + tile < t1) stage(base + tile);
     }
     if (warp < nh && lane == 0) {
         float* ml = A.part_ml + ((size_t)(head0 + warp) * A.splits + split) * 2;
@@ -267,7 +300,7 @@ __device__ __forceinline__ void gqa_token(const GqaArgs& A, int cta, unsigned ch
         const size_t at = (size_t)(head0 + h) * A.vdim + d;
         const float* po = A.part_o + (size_t)(head0 + h) * A.splits * A.vdim + d;
         float o = 0.0f;
-#pragma unroll 8
+#pragma unroll 4
         for (int s = 0; s < A.splits; ++s) {
             const float f = f_s[h * kGqMaxSplits + s];
             if (f != 0.0f) o = fmaf(__ldcg(po + (size_t)s * A.vdim), f, o);  // the sums of an empty split are not written
