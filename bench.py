@@ -1063,7 +1063,7 @@ def hybrid_prompt_kernels(torch, B, m, cfg, sms):
     sets = [dict(y=new(n, L["in"].n), yd=new(n, v), ba=torch.randn(n, 2 * d.heads, device="cuda"), qn=new(n, a.heads * a.dim), rows=new(T, ring.ld),
                  vt=new(a.kv_heads * a.vdim, -(-T // 8) * 8), ctx=new(n, a.heads * a.vdim), act=new(n, L["out"].ld), u=new(n, r.width),
                  z=torch.randn(r.blocks, n, 2 * k, device="cuda"), scratch=torch.empty(floats.value, device="cuda"), x=torch.randn(n, D, device="cuda"),
-                 o=new(n, D), h1=new(n, D), h2=new(n, D), gu=new(n, 2 * ff)) for _ in range(3)]
+                 o=new(n, D), h1=new(n, D), h2=new(n, D), gu=new(n, 2 * ff), unit=new(n, ff)) for _ in range(3)]
     at = lambda s, name: s["y"].data_ptr() + 2 * L["at"][name]
     ldy = L["in"].n
     P = lambda t: t.data_ptr()
@@ -1077,8 +1077,7 @@ def hybrid_prompt_kernels(torch, B, m, cfg, sms):
         "delta rule (convolution to gate)": lambda s: lib.llvq_dn_delta_rows(C.byref(dd), P(s["yd"]), v, P(s["ba"]), P(s["yd"]) + 2 * d.channels, v, P(s["scratch"]),
                                                                              P(s["act"]), L["out"].ld, 0, n, st()),
         "sum and two norms": lambda s: lib.llvq_dn_add_norms_rows(m.dt, P(s["x"]), P(s["o"]), None, None, 0, P(L["norm1"]), P(s["h1"]), P(L["norm2"]), P(s["h2"]), 1e-5, n, D, st()),
-        "gated unit": lambda s: lib.llvq_dn_gated_rows(m.dt, P(s["gu"]), None, P(s["act"]), L["out"].ld, n, ff, float("inf"), 1.0, 0.0, 1.0, st())
-        if L["out"].ld >= ff else 0,
+        "gated unit": lambda s: lib.llvq_dn_gated_rows(m.dt, P(s["gu"]), None, P(s["unit"]), ff, n, ff, float("inf"), 1.0, 0.0, 1.0, st()),
     }
     bytes_ = {"query norms and cache rows": 2 * 2 * n * (a.heads * a.dim + a.kv_heads * (a.dim + a.vdim)), "output gate": 2 * 3 * n * hv, "convolution": 2 * 2 * n * r.width,
               "linear recurrence": n * r.width * (8 + 2 * 3), "sum and two norms": n * D * (8 + 6), "gated unit": n * ff * 6,

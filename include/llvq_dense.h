@@ -57,7 +57,8 @@ typedef struct {
     const void* w2;         /* routed: the stack [matrices, rows2 / top, ldw]: rows of matrix route[*token][j] follow one another */
     const float* norm_w2;
     float* y2;              /* [rows2], or [rows2 / 2] with glu2 */
-    const void* w_r;        /* [matrices, n_out, ld_r]: y += sum_j w_r[route[*token][j]] x_j, x_j the k_r values at x + ldw + j ld_r */
+    const void* w_r;        /* [matrices, n_out, ld_r]: y += sum_j w_r[route[*token][j]] x_j, x_j the k_r values at x + ldw + j ld_r;
+                               with it w may be NULL and k, ldw 0 */
     const int32_t* route;   /* [route_rows, top], or NULL: nothing is routed */
 } llvq_dn_gemv_desc;
 int llvq_dn_gemv(const llvq_dn_gemv_desc* d, llvq_dn_stream stream);

@@ -40,7 +40,8 @@ int sm_count() {
 int check_gemv(const llvq_dn_gemv_desc* d, const char* who) {
     if (!d || bad_dtype(d->dtype)) return fail(kStatusInvalid, "%s: null descriptor or element type", who);
     const int vn = 16 / elem_size(d->dtype);
-    if (!d->w || d->n_out <= 0 || d->k <= 0 || d->ldw < d->k || d->ldw % vn || ((uintptr_t)d->w & 15))
+    const bool routed_only = !d->w && d->w_r && d->k == 0 && d->ldw == 0;
+    if (d->n_out <= 0 || (!routed_only && (!d->w || d->k <= 0 || d->ldw < d->k || d->ldw % vn || ((uintptr_t)d->w & 15))))
         return fail(kStatusInvalid, "%s: matrix of %d x %d, row stride %d (a multiple of %d, 16-byte aligned)", who, d->n_out, d->k, d->ldw, vn);
     if (d->glu && d->n_out % 2) return fail(kStatusInvalid, "%s: %d rows are not (gate, up) pairs", who, d->n_out);
     switch (d->prologue) {

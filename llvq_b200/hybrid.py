@@ -181,8 +181,8 @@ class _Route:
 
 class HybridLM(DenseLM):
     PHASES = ("projections", "mixer", "delta", "output", "head")
-    # columns one token projection takes: beyond, mixer and feed-forward have an output projection each
-    JOINED_COLUMNS = {2: 20480, 4: 40000}
+    # columns one token projection takes, in bf16 as segments of a matrix each; beyond, mixer and feed-forward have one each
+    JOINED_SEGMENTS, SEGMENT, JOINED_COLUMNS_F32 = 8, 2560, 40000
 
     def __init__(self, cfg: HybridConfig, tensor, dtype: str, capacity: int, device, prefill_chunk: int = 2048):
         """`tensor(name)` gives a weight by its name (any device)."""
@@ -257,16 +257,22 @@ class HybridLM(DenseLM):
         token projection takes them all)."""
         import torch
         D, m = self.cfg.width, p + ".mlp"
-        most = self.JOINED_COLUMNS[self.dtype.itemsize]
         L["parts"] = len(outs)
+        own = sum(whole_vectors(o.shape[1], self.dtype) for o in outs)
+
+        def joined(columns, times):
+            """Whether the mixer's columns and `times` further matrices of so many go into one projection."""
+            if self.dtype == torch.float32:
+                return own + times * columns <= self.JOINED_COLUMNS_F32
+            return -(-own // self.SEGMENT) + times * -(-columns // self.SEGMENT) <= self.JOINED_SEGMENTS
         if c is not None:
             L["norm2"] = self._vec(p + ".norm2", D)
         if c is not None and not c.experts:
             L["gate_up"] = DenseMatrix([self._take(f"{m}.{k}", c.ff, D) for k in ("gate", "up")], self.dtype, self.device, interleave=True)
             down = self._take(m + ".down", D, c.ff)
-            joined = sum(whole_vectors(o.shape[1], self.dtype) for o in [*outs, down]) <= most
-            L["down"] = None if joined else DenseMatrix([down], self.dtype, self.device)
-            outs = [*outs, down] if joined else outs
+            both = joined(whole_vectors(c.ff, self.dtype), 1)
+            L["down"] = None if both else DenseMatrix([down], self.dtype, self.device)
+            outs = [*outs, down] if both else outs
         elif c is not None:
             ffp = whole_vectors(c.ff, self.dtype)
             up = torch.zeros(c.experts, ffp, 2, whole_vectors(D, self.dtype), dtype=self.dtype, device=self.device)  # (gate, up) pairs
@@ -275,7 +281,7 @@ class HybridLM(DenseLM):
                 up[e, :c.ff, 0, :D].copy_(self._take(f"{m}.e{e}.gate", c.ff, D))
                 up[e, :c.ff, 1, :D].copy_(self._take(f"{m}.e{e}.up", c.ff, D))
                 down[e, :, :c.ff].copy_(self._take(f"{m}.e{e}.down", D, c.ff))
-            L["experts_up"], L["experts_down"] = up.flatten(1, 2), down
+            L["experts_up"], L["experts_down"], L["routed_apart"] = up.flatten(1, 2), down, not joined(ffp, c.top)
             L["table"] = self._take(m + ".table", self.cfg.vocab, c.top).to(dtype=torch.int32, device=self.device).contiguous()
             if int(L["table"].min()) < 0 or int(L["table"].max()) >= c.experts:
                 raise ValueError(f"{m}.table names experts outside 0 .. {c.experts - 1}")
@@ -334,7 +340,8 @@ class HybridLM(DenseLM):
         tok, pos, steps = self._tok.data_ptr(), self._pos.data_ptr(), []
 
         def gemv(phase, m, **kw):
-            d = _lib.DenseGemv(dtype=self.dt, n_out=m.n, k=m.k, ldw=m.ld, w=m.ptr(), eps=self.eps, alpha=1.0, limit=math.inf, gain=1.0, **kw)
+            own = dict(n_out=m.n, k=m.k, ldw=m.ld, w=m.ptr()) if m is not None else dict(n_out=cfg.width)
+            d = _lib.DenseGemv(dtype=self.dt, eps=self.eps, alpha=1.0, limit=math.inf, gain=1.0, **own, **kw)
             steps.append((phase, lambda st: check(lib.llvq_dn_gemv(C.byref(d), st))))
 
         self._mix = []   # descriptors per layer run
@@ -384,10 +391,16 @@ class HybridLM(DenseLM):
             kw = dict(prologue=_lib.DN_PLAIN, y=ptr(self._x), residual=ptr(self._x))
             if route:
                 down = L["experts_down"]
-                kw.update(w_r=ptr(down), k_r=down.shape[2], ld_r=down.shape[2], **route)
-            gemv("output", out, x=ptr(self._act), **kw)
-            if L.get("down") is not None:
-                gemv("output", L["down"], prologue=_lib.DN_PLAIN, x=ptr(self._act, act_at), y=ptr(self._x), residual=ptr(self._x))
+                route.update(w_r=ptr(down), k_r=down.shape[2], ld_r=down.shape[2])
+                if L["routed_apart"]:
+                    gemv("output", out, x=ptr(self._act), **kw)
+                    gemv("output", None, x=ptr(self._act, act_at), **kw, **route)
+                else:
+                    gemv("output", out, x=ptr(self._act), **kw, **route)
+            else:
+                gemv("output", out, x=ptr(self._act), **kw)
+                if L.get("down") is not None:
+                    gemv("output", L["down"], x=ptr(self._act, act_at), **kw)
         steps.append(("head", lambda st: self._head(self._x, st)))
         self._steps = steps
 

@@ -111,7 +111,13 @@ def test_output_projection_adds_routed_columns_to_the_stream(dtype, n, cols, top
         t = torch.tensor([tok], device="cuda")
         d = _lib.DenseGemv(y=P(xg), residual=P(xg), w_r=P(dg), k_r=ffp, ld_r=ffp, route=P(tg), route_rows=3, top=top, matrices=experts, token=P(t), **kw)
         ok(L.llvq_dn_gemv(C.byref(d), stream()))
-        assert rel(xg, base + sum(down[int(k)].double() @ e[j].double() for j, k in enumerate(table[tok]))) < 3e-6, tok
+        routed = sum(down[int(k)].double() @ e[j].double() for j, k in enumerate(table[tok]))
+        assert rel(xg, base + routed) < 3e-6, tok
+        xg.copy_(x)  # the routed columns alone
+        d = _lib.DenseGemv(dtype=dn(dtype), prologue=_lib.DN_PLAIN, n_out=n, x=act[m.ld:].data_ptr(), y=P(xg), residual=P(xg), eps=1.0, w_r=P(dg), k_r=ffp, ld_r=ffp,
+                           route=P(tg), route_rows=3, top=top, matrices=experts, token=P(t))
+        ok(L.llvq_dn_gemv(C.byref(d), stream()))
+        assert rel(xg, x.double() + routed) < 3e-6, tok
     no_time_out()
 
 
@@ -601,16 +607,16 @@ def test_output_projections_apart_where_one_would_be_too_long():
     toks = tokens_of(cases.EVEN, 90, 3)
     w = cases.random_model(cases.EVEN, 21)
     want = plain.forward(cases.EVEN, w, toks)
-    held = HybridLM.JOINED_COLUMNS
+    held = HybridLM.JOINED_SEGMENTS, HybridLM.JOINED_COLUMNS_F32
     try:
-        HybridLM.JOINED_COLUMNS = {2: 700, 4: 700}
+        HybridLM.JOINED_SEGMENTS, HybridLM.JOINED_COLUMNS_F32 = 0, 0
         for dtype in DTYPES:
             m, _ = build(cases.EVEN, 21, dtype, 128, weights=w)
-            assert m.layers[0]["down"] is not None
+            assert m.layers[0]["down"] is not None and m.layers[1]["routed_apart"] and m.layers[3]["routed_apart"]
             for sizes in ([90], [1], [40, 1, 1, 2]):
                 assert rel(run(m, toks, sizes), want) < TOL[dtype], sizes
     finally:
-        HybridLM.JOINED_COLUMNS = held
+        HybridLM.JOINED_SEGMENTS, HybridLM.JOINED_COLUMNS_F32 = held
 
 
 @pytest.mark.parametrize("name", list(cases.ALL))
