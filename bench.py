@@ -1061,7 +1061,7 @@ def hybrid_prompt_kernels(torch, B, m, cfg, sms):
     hv, v = d.heads * d.vdim, d.channels + d.heads * d.vdim
     k = r.width // r.blocks
     sets = [dict(y=new(n, L["in"].n), yd=new(n, v), ba=torch.randn(n, 2 * d.heads, device="cuda"), qn=new(n, a.heads * a.dim), rows=new(T, ring.ld),
-                 vt=new(a.kv_heads * a.vdim, -(-T // 8) * 8), ctx=new(n, a.heads * a.vdim), act=new(n, L["out"].ld), u=new(n, r.width),
+                 vt=new(a.kv_heads * a.vdim, -(-T // 8) * 8), ctx=new(n, a.heads * a.vdim), act=new(n, max(L["out"].ld, Ld["out"].ld)), u=new(n, r.width),
                  z=torch.randn(r.blocks, n, 2 * k, device="cuda"), scratch=torch.empty(floats.value, device="cuda"), x=torch.randn(n, D, device="cuda"),
                  o=new(n, D), h1=new(n, D), h2=new(n, D), gu=new(n, 2 * ff), unit=new(n, ff)) for _ in range(3)]
     at = lambda s, name: s["y"].data_ptr() + 2 * L["at"][name]
@@ -1071,11 +1071,11 @@ def hybrid_prompt_kernels(torch, B, m, cfg, sms):
     calls = {
         "attention": lambda s: lib.llvq_dn_gqa_prefill(C.byref(g), P(s["qn"]), P(s["rows"]), P(s["vt"]), s["vt"].shape[1], n, T, window - 1, 0, P(s["ctx"]), 0, st()),
         "query norms and cache rows": lambda s: lib.llvq_dn_gqa_rows(C.byref(g), at(s, "q"), at(s, "k"), at(s, "v"), ldy, P(s["qn"]), 0, n, st()),
-        "output gate": lambda s: lib.llvq_dn_gate_rows(m.dt, P(s["ctx"]), hv, at(s, "g"), ldy, P(s["act"]), L["out"].ld, n, hv, 0.7, st()),
+        "output gate": lambda s: lib.llvq_dn_gate_rows(m.dt, P(s["ctx"]), hv, at(s, "g"), ldy, P(s["act"]), s["act"].shape[1], n, hv, 0.7, st()),
         "convolution": lambda s: lib.llvq_dn_conv_rows(m.dt, at(s, "x"), ldy, P(L["x_b"]), P(L["conv"]), P(L["conv_b"]), ring_conv, P(s["u"]), r.width, r.taps, 0, n, st()),
-        "linear recurrence": lambda s: lib.llvq_dn_lru_rows(C.byref(u), P(s["u"]), P(s["z"]), at(s, "y"), ldy, P(L["y_b"]), P(s["act"]), L["out"].ld, 0, n, st()),
+        "linear recurrence": lambda s: lib.llvq_dn_lru_rows(C.byref(u), P(s["u"]), P(s["z"]), at(s, "y"), ldy, P(L["y_b"]), P(s["act"]), s["act"].shape[1], 0, n, st()),
         "delta rule (convolution to gate)": lambda s: lib.llvq_dn_delta_rows(C.byref(dd), P(s["yd"]), v, P(s["ba"]), P(s["yd"]) + 2 * d.channels, v, P(s["scratch"]),
-                                                                             P(s["act"]), L["out"].ld, 0, n, st()),
+                                                                             P(s["act"]), s["act"].shape[1], 0, n, st()),
         "sum and two norms": lambda s: lib.llvq_dn_add_norms_rows(m.dt, P(s["x"]), P(s["o"]), None, None, 0, P(L["norm1"]), P(s["h1"]), P(L["norm2"]), P(s["h2"]), 1e-5, n, D, st()),
         "gated unit": lambda s: lib.llvq_dn_gated_rows(m.dt, P(s["gu"]), None, P(s["unit"]), ff, n, ff, float("inf"), 1.0, 0.0, 1.0, st()),
     }
@@ -1098,14 +1098,18 @@ def hybrid_prompt_kernels(torch, B, m, cfg, sms):
     def gates(i):
         m._bmm(sets[i % 3]["u"].view(n, r.blocks, k).transpose(0, 1), L["gates"][:, :, :k], torch.float32)
 
+    down = [x["down"] for x in (L, Ld) if x["down"] is not None]
+
     def products(i):
         s = sets[i % 3]
         for x, w in ((s["h1"], L["in"]), (s["h2"], L["gate_up"]), (s["h1"], Ld["in"]), (s["h2"], Ld["gate_up"])):
             m._mm(x, w.rows(0))
         for w in (L["out"], Ld["out"]):
             m._mm(s["act"][:, :w.k], w.rows(0))
+        for w in down:
+            m._mm(s["unit"], w.rows(0))
     for name, fn, fl in (("gate matrices", gates, 4.0 * n * r.width * k),
-                         ("library products (two layers)", products, 2.0 * n * sum(x[w].n * x[w].k for x in (L, Ld) for w in ("in", "gate_up", "out")))):
+                         ("library products (two layers)", products, 2.0 * n * sum(w.n * w.k for w in [x[k] for x in (L, Ld) for k in ("in", "gate_up", "out")] + down))):
         ms = B.event_ms(fn, 12)
         out[name] = {"us": round(ms * 1e3, 1), "TFLOPs": round(fl / ms / 1e9, 1), "frac": round(fl / ms / 1e9 / B.tflops, 4)}
     return out

@@ -260,17 +260,18 @@ class HybridLM(DenseLM):
         L["parts"] = len(outs)
         own = sum(whole_vectors(o.shape[1], self.dtype) for o in outs)
 
-        def joined(columns, times):
-            """Whether the mixer's columns and `times` further matrices of so many go into one projection."""
+        def joined(columns, routed):
+            """Whether the mixer's columns and so many more, or `routed` matrices of so many, go into one projection."""
             if self.dtype == torch.float32:
-                return own + times * columns <= self.JOINED_COLUMNS_F32
-            return -(-own // self.SEGMENT) + times * -(-columns // self.SEGMENT) <= self.JOINED_SEGMENTS
+                return own + max(routed, 1) * columns <= self.JOINED_COLUMNS_F32
+            segments = -(-own // self.SEGMENT) + routed * -(-columns // self.SEGMENT) if routed else -(-(own + columns) // self.SEGMENT)
+            return segments <= self.JOINED_SEGMENTS
         if c is not None:
             L["norm2"] = self._vec(p + ".norm2", D)
         if c is not None and not c.experts:
             L["gate_up"] = DenseMatrix([self._take(f"{m}.{k}", c.ff, D) for k in ("gate", "up")], self.dtype, self.device, interleave=True)
             down = self._take(m + ".down", D, c.ff)
-            both = joined(whole_vectors(c.ff, self.dtype), 1)
+            both = joined(whole_vectors(c.ff, self.dtype), 0)
             L["down"] = None if both else DenseMatrix([down], self.dtype, self.device)
             outs = [*outs, down] if both else outs
         elif c is not None:
